@@ -58,6 +58,9 @@ struct GemmEpilogueArgs {
   int ldc;
   bf16* const* row_ptrs; // EPI_SCATTER: destination of every output row (null = drop), N elements each
   uint32_t* done_counter;  // EPI_SCATTER: local counter for the "last CTA publishes the flags" step
+  float act_limit;           // EPI_CLIP_GLU
+  const bf16* gate;          // EPI_GATE: [M, ldg], indexed by the row of W like the bias
+  int ldg;
   // EPI_SPLITK_T (operands swapped: accumulator row = output column, accumulator column = token)
   float* ws;                 // [splitk][tokens][ldws] fp32 partial sums, one slab per K range
   uint32_t* tile_counters;   // one per 128 output columns, zero between launches
@@ -73,6 +76,9 @@ struct GemmGroupArgs {
   const int* mt_row_end;   // end (exclusive) of the expert's segment: rows beyond are not stored
   const int* num_mt;       // number of m-tiles (device scalar)
   int w_rows_per_expert;   // rows of W per expert (N of one expert's matrix)
+  // per-head mode (heads > 0, num_mt == nullptr): every head multiplies its own columns of A with its own N rows
+  // of W into its own columns of C
+  int heads, a_head, c_head;
 };
 
 // Fused collectives (tensor parallelism inside a pipeline stage). All pointers in the arrays
@@ -98,13 +104,24 @@ struct GemmCommArgs {
 
 struct TileCoord {
   int a_row, b_row, row_end, n_blk;
+  int a_col, c_col;  // per-head mode: first column of the head in A and C
 };
 
 template <int BN>
 __device__ __forceinline__ TileCoord tile_coord(int tile, int num_m, int num_n, int M,
                                                 const GemmGroupArgs& g, const GemmCommArgs& comm) {
   TileCoord c;
-  if (g.num_mt != nullptr) {
+  c.a_col = c.c_col = 0;
+  if (g.heads > 0) {
+    const int m_blk = tile % num_m, hn = tile / num_m;
+    const int head = hn / num_n;
+    c.n_blk = hn % num_n;
+    c.a_row = m_blk * BM;
+    c.row_end = M;
+    c.b_row = head * g.w_rows_per_expert + c.n_blk * BN;
+    c.a_col = head * g.a_head;
+    c.c_col = head * g.c_head;
+  } else if (g.num_mt != nullptr) {
     const int mt = tile / num_n;
     c.n_blk = tile % num_n;
     c.a_row = g.mt_row0[mt];
@@ -258,7 +275,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
 
   const int num_m = grp.num_mt != nullptr ? *grp.num_mt : ceil_div(M, BM);
   const int num_n = ceil_div(N, BN);
-  const int num_tiles = num_m * num_n;
+  const int num_tiles = num_m * num_n * (grp.heads > 0 ? grp.heads : 1);
   const int num_kb = ceil_div(K, BK);
   // split-K (small-M path only): work item = (tile, K range); every range holds at least one k-block
   constexpr bool kCluster = EPI == PXL_EPI_SPLITK_C || EPI == PXL_EPI_SPLITK_CN;
@@ -325,7 +342,8 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           if (!ok) break;
           const uint32_t fb = full0 + 8 * stage;
           mbar_arrive_expect_tx(fb, A_STAGE_BYTES + Cfg::B_STAGE_BYTES);
-          tma_load_2d(smem_u32(smem_a + stage * A_STAGE_BYTES), &tmap_a, fb, kb * BK, tc.a_row);
+          tma_load_2d(smem_u32(smem_a + stage * A_STAGE_BYTES), &tmap_a, fb, tc.a_col + kb * BK,
+                      tc.a_row);
           tma_load_2d(smem_u32(smem_b + stage * Cfg::B_STAGE_BYTES), &tmap_b, fb, kb * BK,
                       tc.b_row);
           if (++stage == STAGES) {
@@ -399,7 +417,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
       }
       const int row = tc.a_row + q * 32 + lane;
       const uint32_t t_row = tmem_base + acc * BN + (static_cast<uint32_t>(q * 32) << 16);
-      if constexpr (EPI == PXL_EPI_SILU_MUL) {
+      if constexpr (EPI == PXL_EPI_SILU_MUL || EPI == PXL_EPI_CLIP_GLU) {
         // W rows come in groups of 128: 64 gate rows then the 64 up rows of the same outputs
         const int n_out = N / 2;
 #pragma unroll 1
@@ -420,10 +438,20 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                 for (int j = 0; j < 4; ++j) {
                   float g0 = __uint_as_float(g[v * 8 + 2 * j]);
                   float g1 = __uint_as_float(g[v * 8 + 2 * j + 1]);
-                  const float u0 = __uint_as_float(u[v * 8 + 2 * j]);
-                  const float u1 = __uint_as_float(u[v * 8 + 2 * j + 1]);
-                  g0 = g0 / (1.f + __expf(-g0));
-                  g1 = g1 / (1.f + __expf(-g1));
+                  float u0 = __uint_as_float(u[v * 8 + 2 * j]);
+                  float u1 = __uint_as_float(u[v * 8 + 2 * j + 1]);
+                  if constexpr (EPI == PXL_EPI_CLIP_GLU) {
+                    const float lim = ep.act_limit;
+                    g0 = fminf(g0, lim);
+                    g1 = fminf(g1, lim);
+                    g0 = g0 / (1.f + __expf(-1.702f * g0));
+                    g1 = g1 / (1.f + __expf(-1.702f * g1));
+                    u0 = fminf(fmaxf(u0, -lim), lim) + 1.f;
+                    u1 = fminf(fmaxf(u1, -lim), lim) + 1.f;
+                  } else {
+                    g0 = g0 / (1.f + __expf(-g0));
+                    g1 = g1 / (1.f + __expf(-g1));
+                  }
                   o.u[j] = pack_bf16x2(g0 * u0, g1 * u1);
                 }
                 st_bf16x8(dst + v * 8, o);
@@ -499,7 +527,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           tmem_ld_32x32b_x32(t_row + c0, r);
           tmem_ld_wait();
           if (row < M_end) {
-            size_t off = static_cast<size_t>(row) * ep.ldc + col0 + c0;
+            size_t off = static_cast<size_t>(row) * ep.ldc + tc.c_col + col0 + c0;
             bf16* c_base = ep.C;
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
@@ -525,6 +553,17 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                     const float2 bb = unpack_bf16x2(rr.u[j]);
                     f[2 * j] += bb.x;
                     f[2 * j + 1] += bb.y;
+                  }
+                }
+                if constexpr (EPI == PXL_EPI_GATE) {
+                  if (ep.gate) {
+                    const bf16x8 gg = ld_bf16x8(ep.gate + static_cast<size_t>(row) * ep.ldg + tc.b_row + c0 + v * 8);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                      const float2 bb = unpack_bf16x2(gg.u[j]);
+                      f[2 * j] *= 1.f / (1.f + __expf(-bb.x));
+                      f[2 * j + 1] *= 1.f / (1.f + __expf(-bb.y));
+                    }
                   }
                 }
                 if constexpr (EPI == PXL_EPI_F32) {
@@ -982,7 +1021,7 @@ int launch_gemm_cluster(const CUtensorMap& ta, const CUtensorMap& tb, const Gemm
     *max_clusters = n;
     return PXL_OK;
   }
-  GemmGroupArgs grp{nullptr, nullptr, nullptr, nullptr, 0};
+  GemmGroupArgs grp{};
   GemmCommArgs comm{};
   if (cudaLaunchKernelEx(&cfg, kern, ta, tb, ep, grp, comm, M, N, K, status) != cudaSuccess) {
     cudaGetLastError();
@@ -1199,7 +1238,7 @@ int gemm_small_m(const void* A, const void* W, void* C, bool f32_out, const void
     }
   }
   if (!small_m_scratch(stream, &ep.ws, &ep.tile_counters)) return PXL_ERR_CUDA;
-  GemmGroupArgs grp{nullptr, nullptr, nullptr, nullptr, 0};
+  GemmGroupArgs grp{};
   switch (bn_tok) {
     case 32:
       return launch_gemm<32, PXL_EPI_SPLITK_T>(ta, tb, ep, grp, GemmCommArgs{}, items, N, M, K, status, stream);
@@ -1365,7 +1404,7 @@ PXL_EXPORT int pxl_gemm_bf16(const void* A, const void* W, void* C, const void* 
   ep.residual = static_cast<const pxl::bf16*>(residual);
   ep.bias = static_cast<const pxl::bf16*>(bias);
   ep.ldc = ldc;
-  GemmGroupArgs grp{nullptr, nullptr, nullptr, nullptr, 0};
+  GemmGroupArgs grp{};
   switch (bn) {
     case 256: return dispatch_epi<256>(epi, ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
     case 192:  // plain epilogues only: fills the last wave better when N / 256 leaves SMs idle
@@ -1381,6 +1420,71 @@ PXL_EXPORT int pxl_gemm_bf16(const void* A, const void* W, void* C, const void* 
     case 128: return dispatch_epi<128>(epi, ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
     case 64: return dispatch_epi<64>(epi, ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
     default: return PXL_ERR_INVALID_ARG;
+  }
+}
+
+// Clipped GLU epilogue (see pxl_api.h): tiles of 128 or 256 columns of W.
+PXL_EXPORT int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,
+                                 float limit, int bn, int* status, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return PXL_ERR_INVALID_ARG;
+  if ((K % 8) || (lda % 8) || (ldw % 8) || (ldc % 8) || (N % 128)) return PXL_ERR_INVALID_ARG;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C)) & 15)
+    return PXL_ERR_INVALID_ARG;
+  if (bn == 0) bn = pxl_gemm_bf16_pick_bn(M, N, PXL_EPI_SILU_MUL);
+  if ((bn != 128 && bn != 256) || (N % bn)) return PXL_ERR_INVALID_ARG;
+  CUtensorMap ta, tb;
+  if (!pxl_host::make_tmap_2d(&ta, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, M, K, lda, BM, BK) ||
+      !pxl_host::make_tmap_2d(&tb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, N, K, ldw, bn, BK))
+    return PXL_ERR_TENSORMAP;
+  GemmEpilogueArgs ep{};
+  ep.C = static_cast<pxl::bf16*>(C);
+  ep.ldc = ldc;
+  ep.act_limit = limit;
+  GemmGroupArgs grp{};
+  if (bn == 256)
+    return launch_gemm<256, PXL_EPI_CLIP_GLU>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+  return launch_gemm<128, PXL_EPI_CLIP_GLU>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+}
+
+// Per-head products (see pxl_api.h). K columns past a head's K meet zeros: the tensor map of W ends at K.
+PXL_EXPORT int pxl_gemm_bf16_heads(const void* A, const void* W, void* C, const void* gate, int M, int heads, int N, int K,
+                                   int lda, int a_head, int ldw, int ldc, int c_head, int ldg, int* status,
+                                   cudaStream_t stream) {
+  if (M <= 0 || heads <= 0 || N <= 0 || K <= 0) return PXL_ERR_INVALID_ARG;
+  if ((K % 8) || (N % 8) || (lda % 8) || (a_head % 8) || (ldw % 8) || (ldc % 8) || (c_head % 8) || (gate && (ldg % 8)))
+    return PXL_ERR_INVALID_ARG;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C) |
+       reinterpret_cast<uintptr_t>(gate)) & 15)
+    return PXL_ERR_INVALID_ARG;
+  // widest tile that wastes no more than the next narrower one and still gives every SM a tile
+  const int num_m = pxl::ceil_div(M, BM), sms = pxl_host::num_sms();
+  int bn = 64;
+  for (const int cand : {256, 128}) {
+    if (pxl::ceil_div(N, cand) * cand <= pxl::ceil_div(N, 64) * 64 && heads * num_m * pxl::ceil_div(N, cand) >= sms) {
+      bn = cand;
+      break;
+    }
+  }
+  CUtensorMap ta, tb;
+  if (!pxl_host::make_tmap_2d(&ta, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, M,
+                              static_cast<uint64_t>(heads - 1) * a_head + K, lda, BM, BK) ||
+      !pxl_host::make_tmap_2d(&tb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, static_cast<uint64_t>(heads) * N, K, ldw, bn, BK))
+    return PXL_ERR_TENSORMAP;
+  GemmEpilogueArgs ep{};
+  ep.C = static_cast<pxl::bf16*>(C);
+  ep.ldc = ldc;
+  ep.gate = static_cast<const pxl::bf16*>(gate);
+  ep.ldg = ldg;
+  GemmGroupArgs grp{};
+  grp.w_rows_per_expert = N;
+  grp.heads = heads;
+  grp.a_head = a_head;
+  grp.c_head = c_head;
+  const int tiles = heads * num_m * pxl::ceil_div(N, bn);
+  switch (bn) {
+    case 256: return launch_gemm<256, PXL_EPI_GATE>(ta, tb, ep, grp, GemmCommArgs{}, tiles, M, N, K, status, stream);
+    case 128: return launch_gemm<128, PXL_EPI_GATE>(ta, tb, ep, grp, GemmCommArgs{}, tiles, M, N, K, status, stream);
+    default: return launch_gemm<64, PXL_EPI_GATE>(ta, tb, ep, grp, GemmCommArgs{}, tiles, M, N, K, status, stream);
   }
 }
 
@@ -1411,7 +1515,7 @@ PXL_EXPORT int pxl_gemm_bf16_grouped(const void* A, const void* W, void* C, cons
   ep.residual = nullptr;
   ep.bias = static_cast<const pxl::bf16*>(bias);  // optional [E * N], applied with PXL_EPI_NONE / F32
   ep.ldc = ldc;
-  GemmGroupArgs grp{mt_expert, mt_row0, mt_row_end, num_mt, N};
+  GemmGroupArgs grp{mt_expert, mt_row0, mt_row_end, num_mt, N, 0, 0, 0};
   const int max_tiles = max_m_tiles * pxl::ceil_div(N, bn);
   switch (bn) {
     case 256: return dispatch_epi<256>(epi, ta, tb, ep, grp, GemmCommArgs{}, max_tiles, P, N, K, status, stream);
@@ -1450,7 +1554,7 @@ PXL_EXPORT int pxl_gemm_bf16_grouped_scatter(const void* A, const void* W, void*
   comm.rank = rank;
   comm.tp = ep_size;
   comm.epoch = epoch;
-  GemmGroupArgs grp{mt_expert, mt_row0, mt_row_end, num_mt, N};
+  GemmGroupArgs grp{mt_expert, mt_row0, mt_row_end, num_mt, N, 0, 0, 0};
   return dispatch_epi<128>(PXL_EPI_SCATTER, ta, tb, ep, grp, comm, max_m_tiles * (N / bn), P, N, K, status, stream);
 }
 
@@ -1500,7 +1604,7 @@ PXL_EXPORT int pxl_gemm_bf16_rs(const void* A, const void* W, void* out, const v
   comm.ldo = ldo;
   comm.first_shard = (rank + 1) % tp;  // own rows last: the partials of the peers arrive meanwhile
   comm.epoch = epoch;
-  GemmGroupArgs grp{nullptr, nullptr, nullptr, nullptr, 0};
+  GemmGroupArgs grp{};
   switch (bn) {
     case 256: return dispatch_epi<256>(PXL_EPI_RS, ta, tb, ep, grp, comm, 0, M, N, K, status, stream);
     case 128: return dispatch_epi<128>(PXL_EPI_RS, ta, tb, ep, grp, comm, 0, M, N, K, status, stream);
@@ -1560,7 +1664,7 @@ PXL_EXPORT int pxl_gemm_bf16_ag(void* const* x_ptrs, void* const* ready_ptrs, vo
   comm.ag_ncopy = ncopy;
   comm.first_shard = rank;  // local rows first
   comm.epoch = epoch;
-  GemmGroupArgs grp{nullptr, nullptr, nullptr, nullptr, 0};
+  GemmGroupArgs grp{};
   switch (bn) {
     case 256: return dispatch_epi<256>(epi, ta, tb, ep, grp, comm, 0, M, N, K, status, stream);
     case 128: return dispatch_epi<128>(epi, ta, tb, ep, grp, comm, 0, M, N, K, status, stream);

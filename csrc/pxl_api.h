@@ -27,6 +27,11 @@ typedef struct CUstream_st* pxl_stream_t;
 #define PXL_EPI_SPLITK_T 6  // internal: small-M path (operands swapped, split along K, fp32 slabs + last-CTA finish)
 #define PXL_EPI_SPLITK_C 7  // internal: small-M path, the K ranges of a tile form a cluster and reduce over DSMEM
 #define PXL_EPI_SPLITK_CN 8 // internal: mid-M path (operands not swapped), K ranges of a tile reduce inside a cluster
+#define PXL_EPI_GATE 9      // internal: C = (A W^T) * sigmoid(gate)      bf16 out (pxl_gemm_bf16_heads)
+#define PXL_EPI_CLIP_GLU 10 // clipped GLU of gate / up groups arranged as for PXL_EPI_SILU_MUL (pxl_gemm_bf16_glu)
+
+#define PXL_NORM_LAYER 0    // (x - mean) / sqrt(variance + eps)
+#define PXL_NORM_RMS 1      // x / sqrt(mean(x^2) + eps)
 
 // ---- gemm_tcgen05.cu -------------------------------------------------------
 // C[M,N] = A[M,K] * W[N,K]^T. lda/ldw/ldc in elements. `bn` = tile width (64/128/256)
@@ -47,6 +52,16 @@ int pxl_gemm_bf16_pick_bn(int M, int N, int epi);
 int pxl_gemm_bf16_small_m(const void* A, const void* W, void* C, const void* residual, const void* bias,
                           int M, int N, int K, int lda, int ldw, int ldc, int splitk, int mode, int* status,
                           pxl_stream_t stream);
+// Clipped GLU in the epilogue: g = min(gate, limit), u = clamp(up, -limit, limit), C = g sigmoid(1.702 g) (u + 1).
+// W rows in groups of 128 (64 gate rows, the 64 up rows of the same outputs); C has N / 2 columns.
+int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, float limit,
+                      int bn, int* status, pxl_stream_t stream);
+// One product per attention head in one launch: for every head h < heads
+//   C[m, h * c_head + n] = sum_k A[m, h * a_head + k] * W[h * N + n, k]   (n < N, k < K)
+// optionally times sigmoid(gate[m, h * N + n]). bf16; K, N, strides and head offsets multiples of 8, pointers 16-byte
+// aligned.
+int pxl_gemm_bf16_heads(const void* A, const void* W, void* C, const void* gate, int M, int heads, int N, int K, int lda,
+                        int a_head, int ldw, int ldc, int c_head, int ldg, int* status, pxl_stream_t stream);
 // 1 when pxl_gemm_bf16(bn = 0) would use the small-M path for this shape and epilogue.
 int pxl_gemm_bf16_uses_small_m(int M, int N, int K, int epi);
 
@@ -297,6 +312,43 @@ int pxl_msa_select(const float* scores, int64_t ld, const int* positions, const 
                    const int* cu_q, int T, int B, int max_blocks, int page, int sparse_block, int topk,
                    int init_blocks, int local_blocks, int* v_tables, int64_t ld_vt, int* v_ctx,
                    pxl_stream_t stream);
+
+// ---- gemm_simt.cu: fp32 operands, and bf16 shapes the TMA rules exclude -----------------------------
+// C[m, h*c_head + n] = sum_k A[m, h*a_head + k] * W[h*N + n, k] (+ bias[h*N + n]) (+ residual at C's place)
+// (* sigmoid(gate[m, h*N + n])); fp32 accumulation in K order. in_f32: operands, bias and gate are fp32.
+int pxl_gemm_simt(const void* A, const void* W, void* C, const void* bias, const void* residual, const void* gate, int M,
+                  int N, int K, int64_t lda, int64_t ldw, int64_t ldc, int64_t ldg, int heads, int64_t a_head,
+                  int64_t c_head, int in_f32, int out_f32, pxl_stream_t stream);
+
+// ---- residual.cu: fp32 residual stream -----------------------------------------------------------------
+// out[t] = table[ids[t]] * scale (+ hash[row]), row = (prev[t] * mul_prev + ids[t] * mul_cur) mod buckets, or
+// `buckets` when prev[t] < 0. hash may be null.
+int pxl_embed_rows(const void* table, const int* ids, float scale, const void* hash, const int* prev, int64_t mul_prev,
+                   int64_t mul_cur, int64_t buckets, float* out, int T, int W, int64_t num_rows, int is_f32, int* status,
+                   pxl_stream_t stream);
+int pxl_f32_to_bf16(const float* x, void* out, int64_t n, pxl_stream_t stream);
+// x += mult * norm(y) * w in place; low (bf16) receives the sum when y is bf16. kind: PXL_NORM_*.
+int pxl_residual_norm(float* x, const void* y, const float* w, void* low, int T, int W, float eps, float mult, int kind,
+                      int y_f32, pxl_stream_t stream);
+// out[t] = norm(x[rows ? rows[t] : t]) * w
+int pxl_row_norm(const float* x, const float* w, const int* rows, int64_t num_rows, void* out, int T, int W, float eps,
+                 int kind, int out_f32, int* status, pxl_stream_t stream);
+// fp32 form of pxl_act_mul
+int pxl_act_mul_f32(const float* x, float* out, int T, int I, int mode, float limit, pxl_stream_t stream);
+
+// ---- latent_attn.cu / latent_attn_tc.cu: latent attention of any widths, window, sinks -------------------
+// proj [T, ld]: `heads` query heads of q_width columns (rotated part of R dims at q_rot_off) and, at kv_off, the raw
+// latent (L) | key part (R). Writes cache[slots[t]] = RMSnorm(latent) * norm_w | rotated key and the rotated query
+// parts to q_cat[t, h, L:]. Interleaved pairs; the first `rot` of the R dims are rotated. cos_sin [max_pos, rot].
+int pxl_latent_prep(const void* proj, int64_t ld, int kv_off, int heads, int q_width, int q_rot_off, const float* norm_w,
+                    const float* cos_sin, const int* positions, int max_pos, const int64_t* slots, void* cache,
+                    int64_t num_slots, void* q_cat, int T, int L, int R, int rot, float eps, int is_f32, int* status,
+                    pxl_stream_t stream);
+// out[t, h, :L] = attention of q[t, h, :L+R] over the cached rows of t's sequence (cu_q null: token t is the only
+// query of sequence t). The queries are the last tokens of ctx_lens[b]. window <= 0: no window; sinks may be null.
+int pxl_latent_attn(const void* q, const void* cache, const int* block_tables, const int* cu_q, const int* ctx_lens,
+                    void* out, const float* sinks, int B, int max_q, int H, int L, int R, int page, int max_blocks,
+                    int64_t num_blocks, float scale, int window, int is_f32, int* status, pxl_stream_t stream);
 
 // ---- stage_exec.cu: all layers of a dense GQA stage for one step behind one call --------------
 // The descriptor structs are defined in stage_exec.cu (mirrored by parallax_b200/engine/native_stage.py).

@@ -1,0 +1,311 @@
+// Rows of an fp32 residual stream: embedding (scaled, with an optional hashed second table), the update
+// x += mult * norm(y) * w fused with the low-precision copy the next product reads, norms of fp32 rows, and
+// activations in any precision. All statistics are fp32; the layer norm's variance is the mean of the squared
+// deviations from the mean (two passes over the row, which stays in registers when it is aligned).
+#include "common.cuh"
+#include "pxl_api.h"
+
+namespace {
+using namespace pxl;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&v)[8]) {
+  if constexpr (sizeof(T) == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+  } else {
+    const bf16x8 a = ld_bf16x8(p);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(a.u[j]);
+      v[2 * j] = f.x, v[2 * j + 1] = f.y;
+    }
+  }
+}
+template <typename T>
+__device__ __forceinline__ void store8(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  } else {
+    bf16x8 o;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o.u[j] = pack_bf16x2(v[2 * j], v[2 * j + 1]);
+    st_bf16x8(p, o);
+  }
+}
+
+// ---- embedding -------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128) embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ ids,
+                                                         float scale, const T* __restrict__ hash,
+                                                         const int* __restrict__ prev, int64_t mul_prev, int64_t mul_cur,
+                                                         int64_t buckets, float* __restrict__ out, int W,
+                                                         int64_t rows, int* status) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int64_t id = ids[t];
+  if (id < 0 || id >= rows) {
+    if (threadIdx.x == 0 && status) atomicCAS(status, 0, PXL_DEV_BAD_ROW_ID);
+    for (int i = threadIdx.x; i < W; i += blockDim.x) out[static_cast<int64_t>(t) * W + i] = 0.f;
+    return;
+  }
+  const T* src = table + id * W;
+  const T* h = nullptr;
+  if (hash) {
+    const int64_t p = prev[t];
+    int64_t row = buckets;
+    if (p >= 0) {
+      row = (p * mul_prev + id * mul_cur) % buckets;
+      if (row < 0) row += buckets;
+    }
+    h = hash + row * W;
+  }
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    float v = to_f(src[i]) * scale;
+    if (h) v += to_f(h[i]);
+    out[static_cast<int64_t>(t) * W + i] = v;
+  }
+}
+
+__global__ void __launch_bounds__(256) to_low_kernel(const float* __restrict__ x, bf16* __restrict__ out, int64_t n) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) * 4;
+  if (i + 3 < n) {
+    const float4 v = *reinterpret_cast<const float4*>(x + i);
+    uint2 o;
+    o.x = pack_bf16x2(v.x, v.y);
+    o.y = pack_bf16x2(v.z, v.w);
+    *reinterpret_cast<uint2*>(out + i) = o;
+  } else {
+    for (int64_t j = i; j < n; ++j) out[j] = __float2bfloat16(x[j]);
+  }
+}
+
+// ---- norms -----------------------------------------------------------------------------------------------
+// kUpdate: src = y (type TI), x updated in place, low = TO copy of x (null when TO is fp32).
+// else:    src = x (type TI, row index optional), low = norm(x) * w.
+struct NormArgs {
+  float* x;
+  const void* src;
+  const float* w;
+  void* low;
+  const int* rows;  // row gather (plain norm only)
+  int64_t num_rows;
+  int W;
+  float eps, mult;
+  int* status;
+};
+
+template <typename TI, typename TO, bool kUpdate, bool kLayer, int NV>
+__global__ void __launch_bounds__(256) norm_vec_kernel(const NormArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  int64_t r = t;
+  if (!kUpdate && a.rows) {
+    r = a.rows[t];
+    if (r < 0 || r >= a.num_rows) {
+      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_ROW_ID);
+      r = 0;
+    }
+  }
+  const TI* src = static_cast<const TI*>(a.src) + r * a.W;
+  float v[NV][8];
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.W) {
+      load8(src + c, v[i]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) sum += v[i][j];
+  }
+  float mean = 0.f;
+  if (kLayer) mean = block_reduce_sum(sum, red) / a.W;
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.W) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        v[i][j] -= mean;
+        sq = fmaf(v[i][j], v[i][j], sq);
+      }
+    }
+  }
+  sq = block_reduce_sum(sq, red);
+  const float inv = a.mult / sqrtf(sq / a.W + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c >= a.W) continue;
+    float w[8], o[8];
+    load8(a.w + c, w);
+    if constexpr (kUpdate) {
+      float* x = a.x + t * a.W + c;
+      load8(x, o);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] = fmaf(v[i][j] * inv, w[j], o[j]);
+      store8(x, o);
+      if constexpr (sizeof(TO) == 2) store8(static_cast<TO*>(a.low) + t * a.W + c, o);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] = v[i][j] * inv * w[j];
+      store8(static_cast<TO*>(a.low) + t * a.W + c, o);
+    }
+  }
+}
+
+// any width: three passes over the row in global memory (L1 keeps it)
+template <typename TI, typename TO, bool kUpdate, bool kLayer>
+__global__ void __launch_bounds__(256) norm_any_kernel(const NormArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  int64_t r = t;
+  if (!kUpdate && a.rows) {
+    r = a.rows[t];
+    if (r < 0 || r >= a.num_rows) {
+      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_ROW_ID);
+      r = 0;
+    }
+  }
+  const TI* src = static_cast<const TI*>(a.src) + r * a.W;
+  float mean = 0.f;
+  if (kLayer) {
+    float sum = 0.f;
+    for (int c = threadIdx.x; c < a.W; c += blockDim.x) sum += to_f(src[c]);
+    mean = block_reduce_sum(sum, red) / a.W;
+  }
+  float sq = 0.f;
+  for (int c = threadIdx.x; c < a.W; c += blockDim.x) {
+    const float d = to_f(src[c]) - mean;
+    sq = fmaf(d, d, sq);
+  }
+  sq = block_reduce_sum(sq, red);
+  const float inv = a.mult / sqrtf(sq / a.W + a.eps);
+  for (int c = threadIdx.x; c < a.W; c += blockDim.x) {
+    const float n = (to_f(src[c]) - mean) * inv;
+    TO* low = static_cast<TO*>(a.low) + t * a.W + c;
+    if constexpr (kUpdate) {
+      float* x = a.x + t * a.W + c;
+      const float o = fmaf(n, a.w[c], *x);
+      *x = o;
+      if constexpr (sizeof(TO) == 2) put(low, o);
+    } else {
+      put(low, n * a.w[c]);
+    }
+  }
+}
+
+template <typename TI, typename TO, bool kUpdate, bool kLayer>
+int launch_norm(const NormArgs& a, int T, bool vec, cudaStream_t stream) {
+  if (vec && a.W % 8 == 0 && a.W <= 256 * 8 * 8) {
+    const int nvec = a.W / 8;
+    const int threads = nvec >= 256 ? 256 : ceil_div(nvec, 32) * 32;
+    const int per = ceil_div(nvec, threads);
+    const dim3 g(T), b(threads);
+    if (per <= 1) pxl_host::launch(norm_vec_kernel<TI, TO, kUpdate, kLayer, 1>, g, b, 0, stream, a);
+    else if (per <= 2) pxl_host::launch(norm_vec_kernel<TI, TO, kUpdate, kLayer, 2>, g, b, 0, stream, a);
+    else if (per <= 4) pxl_host::launch(norm_vec_kernel<TI, TO, kUpdate, kLayer, 4>, g, b, 0, stream, a);
+    else pxl_host::launch(norm_vec_kernel<TI, TO, kUpdate, kLayer, 8>, g, b, 0, stream, a);
+  } else {
+    pxl_host::launch(norm_any_kernel<TI, TO, kUpdate, kLayer>, dim3(T), dim3(256), 0, stream, a);
+  }
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+template <typename TI, typename TO, bool kUpdate>
+int launch_norm(const NormArgs& a, int T, int kind, bool vec, cudaStream_t stream) {
+  return kind == PXL_NORM_LAYER ? launch_norm<TI, TO, kUpdate, true>(a, T, vec, stream)
+                                : launch_norm<TI, TO, kUpdate, false>(a, T, vec, stream);
+}
+inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+// ---- clipped GLU and friends in fp32 -------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) act_mul_f32_kernel(const float* __restrict__ x, float* __restrict__ out, int I,
+                                                          int64_t n, int mode, float limit) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  if (i >= n) return;
+  const int64_t t = i / I, c = i % I;
+  float g = x[t * 2 * I + c], u = x[t * 2 * I + I + c];
+  float y;
+  if (mode == 1) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    y = g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+  } else if (mode == 0) {
+    y = g / (1.f + expf(-g)) * u;
+  } else {
+    y = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  }
+  out[i] = y;
+}
+}  // namespace
+
+PXL_EXPORT int pxl_embed_rows(const void* table, const int* ids, float scale, const void* hash, const int* prev,
+                              int64_t mul_prev, int64_t mul_cur, int64_t buckets, float* out, int T, int W,
+                              int64_t num_rows, int is_f32, int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (W <= 0 || (hash && (prev == nullptr || buckets <= 0))) return PXL_ERR_INVALID_ARG;
+  if (is_f32)
+    pxl_host::launch(embed_rows_kernel<float>, dim3(T), dim3(128), 0, stream, static_cast<const float*>(table), ids, scale,
+                     static_cast<const float*>(hash), prev, mul_prev, mul_cur, buckets, out, W, num_rows, status);
+  else
+    pxl_host::launch(embed_rows_kernel<pxl::bf16>, dim3(T), dim3(128), 0, stream, static_cast<const pxl::bf16*>(table), ids,
+                     scale, static_cast<const pxl::bf16*>(hash), prev, mul_prev, mul_cur, buckets, out, W, num_rows, status);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
+PXL_EXPORT int pxl_f32_to_bf16(const float* x, void* out, int64_t n, cudaStream_t stream) {
+  if (n <= 0) return PXL_OK;
+  if (!aligned16(x) || !aligned16(out)) return PXL_ERR_INVALID_ARG;
+  pxl_host::launch(to_low_kernel, dim3(static_cast<unsigned>((n + 1023) / 1024)), dim3(256), 0, stream, x,
+                   static_cast<pxl::bf16*>(out), n);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
+PXL_EXPORT int pxl_residual_norm(float* x, const void* y, const float* w, void* low, int T, int W, float eps, float mult,
+                                 int kind, int y_f32, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (W <= 0 || (!y_f32 && low == nullptr)) return PXL_ERR_INVALID_ARG;
+  NormArgs a{x, y, w, low, nullptr, T, W, eps, mult, nullptr};
+  const bool vec = aligned16(x) && aligned16(y) && aligned16(w) && aligned16(low);
+  return y_f32 ? launch_norm<float, float, true>(a, T, kind, vec, stream)
+               : launch_norm<pxl::bf16, pxl::bf16, true>(a, T, kind, vec, stream);
+}
+
+PXL_EXPORT int pxl_row_norm(const float* x, const float* w, const int* rows, int64_t num_rows, void* out, int T, int W,
+                            float eps, int kind, int out_f32, int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (W <= 0) return PXL_ERR_INVALID_ARG;
+  NormArgs a{nullptr, x, w, out, rows, num_rows, W, eps, 1.f, status};
+  const bool vec = aligned16(x) && aligned16(w) && aligned16(out);
+  return out_f32 ? launch_norm<float, float, false>(a, T, kind, vec, stream)
+                 : launch_norm<float, pxl::bf16, false>(a, T, kind, vec, stream);
+}
+
+PXL_EXPORT int pxl_act_mul_f32(const float* x, float* out, int T, int I, int mode, float limit, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (I <= 0) return PXL_ERR_INVALID_ARG;
+  const int64_t n = static_cast<int64_t>(T) * I;
+  pxl_host::launch(act_mul_f32_kernel, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0, stream, x, out, I, n,
+                   mode, limit);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}

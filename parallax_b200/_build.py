@@ -42,8 +42,21 @@ def _nvcc() -> str:
     return cand
 
 
-def _sources() -> list[Path]:
+# Sources a model family needs when nothing has been built yet (the whole library otherwise): a fresh checkout
+# that only runs this family compiles these into a library of their own.
+FAMILY_SOURCES = {
+    "latent": ["elementwise", "gemm_simt", "gemm_tcgen05", "latent_attn", "residual", "sampler"],
+}
+
+
+def _sources(family: str | None = None) -> list[Path]:
+    if family is not None:
+        return [CSRC / f"{name}.cu" for name in FAMILY_SOURCES[family]]
     return sorted(CSRC.glob("*.cu"))
+
+
+def _headers() -> list[Path]:
+    return sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
 
 
 def _digest(paths: list[Path]) -> str:
@@ -55,30 +68,50 @@ def _digest(paths: list[Path]) -> str:
     return h.hexdigest()
 
 
-def lib_path() -> Path:
-    return OUT_DIR / LIB_NAME
+_active_family: str | None = None      # set when only a family's library is in use (see ensure_kernels)
 
 
-def is_fresh() -> bool:
-    stamp = OUT_DIR / "build.stamp"
-    if not lib_path().exists() or not stamp.exists():
+def lib_path(family: str | None = None) -> Path:
+    family = family or _active_family
+    return OUT_DIR / (LIB_NAME if family is None else f"libpxl_{family}.so")
+
+
+def _stamp(family: str | None) -> Path:
+    return OUT_DIR / ("build.stamp" if family is None else f"build.{family}.stamp")
+
+
+def is_fresh(family: str | None = None) -> bool:
+    out = OUT_DIR / LIB_NAME if family is None else lib_path(family)
+    if not out.exists() or not _stamp(family).exists():
         return False
-    deps = _sources() + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    return stamp.read_text().strip() == _digest(deps)
+    return _stamp(family).read_text().strip() == _digest(_sources(family) + _headers())
 
 
-def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` for sm_100a and link them into one shared library."""
-    if not force and is_fresh():
-        return lib_path()
+def ensure_kernels(family: str) -> Path:
+    """Kernels for one model family: the whole library if it is built and up to date, else the family's own,
+    compiled now if need be. Call before the first kernel of the process runs."""
+    global _active_family
+    if is_fresh() or family not in FAMILY_SOURCES:
+        return build_kernels()
+    build_kernels(family=family)
+    _active_family = family
+    return lib_path()
+
+
+def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool = False,
+                  family: str | None = None) -> Path:
+    """Compile every ``csrc/*.cu`` (or those of one family) for sm_100a and link them into one shared library."""
+    target = OUT_DIR / LIB_NAME if family is None else lib_path(family)
+    if not force and is_fresh(family):
+        return target
     OUT_DIR.mkdir(parents=True, exist_ok=True)
     obj_dir = OUT_DIR / "obj"
     obj_dir.mkdir(exist_ok=True)
     nvcc = _nvcc()
-    srcs = _sources()
+    srcs = _sources(family)
     if not srcs:
         raise RuntimeError(f"no CUDA sources under {CSRC}")
-    headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    headers = _headers()
     hdr_digest = _digest(headers)
 
     def compile_one(src: Path) -> Path:
@@ -100,13 +133,13 @@ def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool =
 
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(compile_one, srcs))
-    link = [nvcc, "-shared", "-o", str(lib_path()), *map(str, objs)]
+    link = [nvcc, "-shared", "-o", str(target), *map(str, objs)]
     res = subprocess.run(link, capture_output=True, text=True)
     if res.returncode != 0:
         sys.stderr.write(res.stdout + res.stderr)
-        raise RuntimeError("link of libpxl_kernels.so failed")
-    (OUT_DIR / "build.stamp").write_text(_digest(srcs + headers))
-    return lib_path()
+        raise RuntimeError(f"link of {target.name} failed")
+    _stamp(family).write_text(_digest(srcs + headers))
+    return target
 
 
 if __name__ == "__main__":

@@ -4,7 +4,8 @@ One cache object per decoder layer, chosen by layer kind (same taxonomy as the r
 hybrid cache, ``src/parallax/server/cache_manager.py:188-259``):
 
 * ``attention``      K, V            ``[blocks, Hkv, page, D]``
-* ``mla_attention``  latent | rope   ``[blocks, 1, page, kv_lora + rope]`` (one tensor)
+* ``mla_attention``  latent | rope   ``[blocks, 1, page, kv_lora + rope]`` (one tensor; the widths may differ
+                     from layer to layer)
 * ``dsa_attention``  MLA cache + lightning-indexer keys ``[blocks, 1, page, index_dim]``
 * ``linear``         conv state ``[slots, conv_dim, k-1]`` + recurrent state
                      ``[slots, Hv, Dv, Dk]`` (per request slot, not paged)
@@ -77,7 +78,7 @@ def bytes_per_block(cfg: ModelConfig, start: int, end: int, page: int, elem: int
             if kind == MSA_ATTENTION:
                 total += page * int(cfg.raw.get("index_head_dim") or 0) * elem
         elif kind in (MLA_ATTENTION, DSA_ATTENTION):
-            total += page * (cfg.kv_lora_rank + cfg.qk_rope_head_dim) * elem
+            total += page * sum(cfg.latent_dims(li)) * elem
             if kind == DSA_ATTENTION:
                 total += page * cfg.index_head_dim * elem
     return total
@@ -121,7 +122,7 @@ class KVPool:
                     lc.index_k = torch.zeros((num_blocks, 1, page_size, int(cfg.raw.get("index_head_dim") or 0)),
                                              device=self.device, dtype=dtype)
             elif kind in (MLA_ATTENTION, DSA_ATTENTION):
-                lc.k = torch.zeros((num_blocks, 1, page_size, cfg.kv_lora_rank + cfg.qk_rope_head_dim),
+                lc.k = torch.zeros((num_blocks, 1, page_size, sum(cfg.latent_dims(li))),
                                    device=self.device, dtype=dtype)
                 if kind == DSA_ATTENTION:
                     lc.index_k = torch.zeros((num_blocks, 1, page_size, cfg.index_head_dim),

@@ -21,6 +21,7 @@ class ForwardBatch:
     num_prefill_seqs: int = 0
     num_decode: int = 0
     input_ids: Optional[torch.Tensor] = None      # int32 [T] (first stage only)
+    prev_ids: Optional[torch.Tensor] = None       # int32 [T] token before each token, -1 = none (first stage, if needed)
     positions: Optional[torch.Tensor] = None      # int32 [T]
     slot_mapping: Optional[torch.Tensor] = None   # int64 [T]
     # prefill part
@@ -52,10 +53,10 @@ class BatchBuilder:
         self.max_tokens = max_tokens
         self.max_seqs = max_seqs
         self.max_blocks = max_blocks_per_seq
-        # int32 words: ids T, positions T, slots 2T (as int64), cu_q S+1, p_ctx S, d_ctx S,
-        # logit_rows S, block tables 2*S*MB (prefill and decode parts never overlap, but keep
+        # int32 words: ids T, previous ids T, positions T, slots 2T (as int64), logit rows up to T,
+        # cu_q S+1, p_ctx S, d_ctx S, block tables 2*S*MB (prefill and decode parts never overlap, but keep
         # room for both so that offsets are static)
-        words = 4 * max_tokens + 6 * max_seqs + 16 + max_seqs * max_blocks_per_seq + 64
+        words = 6 * max_tokens + 6 * max_seqs + 16 + max_seqs * max_blocks_per_seq + 64
         self.capacity = words
         pin = device.type == "cuda"
         self.host = torch.empty(words, dtype=torch.int32, pin_memory=pin)
@@ -76,6 +77,7 @@ class BatchBuilder:
         logit_rows: np.ndarray,
         seq_rows: Optional[np.ndarray] = None,
         extra: Optional[dict] = None,
+        prev_ids: Optional[np.ndarray] = None,
     ) -> ForwardBatch:
         if self._copied is not None:
             # the pinned buffer is about to be rewritten: the asynchronous copy of its previous
@@ -101,6 +103,8 @@ class BatchBuilder:
         spans = {}
         if input_ids is not None:
             spans["ids"] = put(input_ids.astype(np.int32, copy=False))
+            if prev_ids is not None:
+                spans["prev"] = put(prev_ids.astype(np.int32, copy=False))
         spans["pos"] = put(positions.astype(np.int32, copy=False))
         spans["slots"] = put(slots.astype(np.int64, copy=False).view(np.int32))
         if Bp:
@@ -136,6 +140,8 @@ class BatchBuilder:
         fb.h2d_bytes = total * 4
         if input_ids is not None:
             fb.input_ids = view("ids")
+            if prev_ids is not None:
+                fb.prev_ids = view("prev")
         fb.positions = view("pos")
         fb.slot_mapping = view("slots").view(torch.int64)
         if Bp:

@@ -66,11 +66,12 @@ class Planner:
                  max_num_tokens_per_batch: int, micro_batch_ratio: int = 1,
                  chunked_prefill_size: Optional[int] = 1024, enable_prefix_cache: bool = True,
                  max_total_length: int = 32768, request_timeout_s: Optional[float] = 600,
-                 eos_token_id=None, shared_state=None, linear_prefix_slots: int = 0):
+                 eos_token_id=None, shared_state=None, linear_prefix_slots: int = 0,
+                 max_requests: Optional[int] = None):
         self.cfg = cfg
         self.page_size = page_size
         max_blocks_per_seq = (max_total_length + page_size - 1) // page_size + 1
-        max_requests = max(max_batch_size * 2, 16)
+        max_requests = max_requests or max(max_batch_size * 2, 16)
         # hybrid models: a request's recurrent state lives in a slot of its own, and the prefix cache keeps
         # snapshots of that state at block boundaries (`linear_prefix_slots` of them) to resume from
         hybrid_slots = max_requests if (cfg.has_linear_layers and enable_prefix_cache and linear_prefix_slots > 0) else 0
@@ -111,6 +112,8 @@ class Planner:
         T = sum(s.num_tokens for s in ordered)
         ids = np.empty(T, dtype=np.int32)
         pos = np.empty(T, dtype=np.int32)
+        # models whose embedding also looks at the token before (-1: the sequence starts here)
+        prev_ids = np.empty(T, dtype=np.int32) if self.cfg.needs_prev_token else None
         rows_of_tok = np.empty(T, dtype=np.int32)
         logit_rows, owners = [], []
         o = 0
@@ -120,12 +123,18 @@ class Planner:
             n, st = s.num_tokens, s.start
             ids[o:o + n] = s.req.input_ids[st:st + n]
             pos[o:o + n] = np.arange(st, st + n, dtype=np.int32)
+            if prev_ids is not None:
+                prev_ids[o] = s.req.input_ids[st - 1] if st else -1
+                prev_ids[o + 1:o + n] = ids[o:o + n - 1]
             row = cache.get_row(s.req.request_id)
             rows_of_tok[o:o + n] = row
             p_q.append(n)
             p_ctx.append(st + n)
             p_rows.append(row)
-            if s.produces_token:
+            if s.logit_at is not None:
+                logit_rows.extend(o + k for k in s.logit_at)
+                owners.extend([s] * len(s.logit_at))
+            elif s.produces_token:
                 logit_rows.append(o + n - 1)
                 owners.append(s)
             o += n
@@ -134,18 +143,25 @@ class Planner:
         nd = len(decode)
         if nd:
             reqs_d = [s.req for s in decode]
-            d_ctx = np.fromiter((r.prompt_len + len(r.output_ids) for r in reqs_d), dtype=np.int32, count=nd)
+            d_ctx = np.fromiter((s.start + 1 for s in decode), dtype=np.int32, count=nd)
             d_rows = np.fromiter((cache.get_row(r.request_id) for r in reqs_d), dtype=np.int32, count=nd)
-            ids[o:o + nd] = np.fromiter((r.output_ids[-1] for r in reqs_d), dtype=np.int32, count=nd)
+            ids[o:o + nd] = np.fromiter((r.output_ids[-1] if r.output_ids else r.input_ids[-1] for r in reqs_d),
+                                        dtype=np.int32, count=nd)
+            if prev_ids is not None:
+                # known on the host even when a row's own token is still on its way: steps are at most one
+                # token ahead of what has been read back
+                prev_ids[o:o + nd] = np.fromiter((r.token_before_last() for r in reqs_d), dtype=np.int32, count=nd)
             if pending_index:
                 hit = [(o + i, pending_index[r.request_id]) for i, r in enumerate(reqs_d)
-                       if r.output_ids[-1] == PENDING_TOKEN and r.request_id in pending_index]
+                       if r.output_ids and r.output_ids[-1] == PENDING_TOKEN and r.request_id in pending_index]
                 if hit:
                     patch_rows, patch_src = (np.asarray(x, dtype=np.int32) for x in zip(*hit))
             pos[o:o + nd] = d_ctx - 1
             rows_of_tok[o:o + nd] = d_rows
-            logit_rows.extend(range(o, o + nd))
-            owners.extend(decode)
+            for i, s in enumerate(decode):
+                if s.logit_at is None or s.logit_at:
+                    logit_rows.append(o + i)
+                    owners.append(s)
             o += nd
         else:
             d_rows = np.empty(0, dtype=np.int32)
@@ -159,7 +175,7 @@ class Planner:
             seq_rows = np.fromiter((state_slot(s.req.request_id) for s in ordered), dtype=np.int32, count=len(ordered))
         else:
             seq_rows = np.concatenate([np.asarray(p_rows, dtype=np.int32), d_rows])
-        return dict(ordered=ordered, ids=ids, pos=pos, slots=slots, p_q=p_q, p_ctx=p_ctx,
+        return dict(ordered=ordered, ids=ids, prev_ids=prev_ids, pos=pos, slots=slots, p_q=p_q, p_ctx=p_ctx,
                     p_tables=p_tables, d_ctx=d_ctx, d_tables=d_tables,
                     logit_rows=np.asarray(logit_rows, dtype=np.int32), owners=owners, seq_rows=seq_rows,
                     patch_rows=patch_rows, patch_src=patch_src)
@@ -195,8 +211,10 @@ class Engine:
         kv_cache_dtype: Optional[str] = None,
         tokenizer=None,
         return_routed_experts: bool = False,
+        max_requests: Optional[int] = None,
     ):
-        """``tokenizer`` (anything with ``token_text(id)`` and ``eos_token_ids``) is only needed for requests
+        """``max_requests``: rows (block tables, state slots) for requests that are live at the same time; by
+        default twice the batch size. ``tokenizer`` (anything with ``token_text(id)`` and ``eos_token_ids``) is only needed for requests
         with a ``json_schema``: constrained decoding checks candidate tokens by their text."""
         self.tokenizer = tokenizer
         self.cfg = cfg
@@ -208,7 +226,7 @@ class Engine:
         # on-the-fly rotary embedding); a table cut at the advertised length was read out of bounds
         max_positions = max_total_length + 8
         self.stages: list[StageWorker] = []
-        max_requests = max(max_batch_size * 2, 16)
+        max_requests = max_requests or max(max_batch_size * 2, 16)
         # hybrid models resume a shared prefix from a snapshot of the recurrent state taken at a block
         # boundary (a recurrent state cannot be rebuilt from cached KV pages); the snapshots live in extra
         # state slots behind the requests' own
@@ -232,7 +250,7 @@ class Engine:
         self.planner = Planner(cfg, nb, page_size, max_batch_size, max_num_tokens_per_batch,
                                micro_batch_ratio, chunked_prefill_size, enable_prefix_cache,
                                max_total_length, request_timeout_s, eos_token_id, shared_state,
-                               linear_prefix_slots=self.linear_prefix_slots)
+                               linear_prefix_slots=self.linear_prefix_slots, max_requests=max_requests)
         self.scheduler = self.planner.scheduler
         self.cache = self.planner.cache
         if self.cache.needs_slots:
@@ -248,6 +266,7 @@ class Engine:
             async_scheduling = self.device.type == "cuda" and not _os.environ.get("PXL_SYNC_ENGINE")
         self.async_scheduling = bool(async_scheduling)
         self._in_flight: Optional[_InFlightStep] = None
+        self._fed: dict[str, Request] = {}      # requests driven by feed()
         self._host_slots = []
         if self.device.type == "cuda":
             for _ in range(3):
@@ -521,15 +540,11 @@ class Engine:
             extra = dict(extra or {}, lora_ids=rows)
         fb = self.builder.build(arrays["ids"], arrays["pos"], arrays["slots"], arrays["p_q"],
                                 arrays["p_ctx"], arrays["p_tables"], arrays["d_ctx"], arrays["d_tables"],
-                                arrays["logit_rows"], arrays["seq_rows"], extra=extra)
+                                arrays["logit_rows"], arrays["seq_rows"], extra=extra, prev_ids=arrays["prev_ids"])
         if "patch_rows" in fb.extras:
             ops.patch_ids(fb.input_ids, fb.extras["patch_rows"], prev.ids, fb.extras["patch_src"])
         owners = arrays["owners"]
-        h = None
-        for i, st in enumerate(self.stages):
-            h = st.run(fb, h)
-            if self.wire_hook is not None and i + 1 < len(self.stages):
-                h = self.wire_hook(h)
+        h = self._forward(fb)
         if self.keep_logits:
             self.last_logits = h
         ids = probs = None
@@ -560,6 +575,74 @@ class Engine:
             out += self._commit(cur)
         self.last_step_stats["wall_s"] = time.perf_counter() - t0
         return out
+
+    def _forward(self, fb) -> torch.Tensor:
+        """One pass of a packed batch through every stage: logits of ``fb.logit_rows``."""
+        h = None
+        for i, st in enumerate(self.stages):
+            h = st.run(fb, h)
+            if self.wire_hook is not None and i + 1 < len(self.stages):
+                h = self.wire_hook(h)
+        return h
+
+    @torch.inference_mode()
+    def feed(self, entries: list) -> Optional[torch.Tensor]:
+        """Teacher-forced step: ``entries`` is a list of ``(request_id, token_ids, places)``; the tokens continue
+        their requests (a new id admits a request) and run as ONE batch through the planner, cache, batch
+        builder and stages that :meth:`step` uses - slices of several tokens as prompt rows, single tokens of a
+        started request as decode rows. Nothing is sampled. Returns fp32 logits at the wanted places (indices
+        into the entry's tokens) in the order of the entries, or None when nothing is wanted. Requests fed this
+        way are not scheduled by :meth:`step`; end them with :meth:`release_fed`."""
+        cache = self.cache
+        seqs: list[ScheduledSeq] = []
+        for rid, tokens, places in entries:
+            tokens, places = [int(t) for t in tokens], [int(p) for p in places]
+            if not tokens or any(p < 0 or p >= len(tokens) for p in places):
+                raise ValueError(f"request {rid}: no tokens, or a wanted place outside them")
+            if any(t < 0 or t >= self.cfg.vocab_size for t in tokens):
+                raise ValueError(f"request {rid}: a token id outside the vocabulary")
+            req = self._fed.get(rid)
+            start = 0 if req is None else req.prompt_len
+            if start + len(tokens) > self.planner.max_total_length:
+                raise ValueError(f"request {rid} outgrows the engine's max_total_length")
+            if req is None:
+                ok, _ = cache.allocate_request(rid, len(tokens))
+                if not ok:
+                    raise RuntimeError(f"no room for request {rid}")
+                req = self._fed[rid] = Request(request_id=rid, input_ids=tokens)
+            else:
+                if len(tokens) > 1 and not cache.extend_request(rid, start + len(tokens)):
+                    raise RuntimeError(f"no KV room for {len(tokens)} more tokens of request {rid}")
+                req.input_ids.extend(tokens)
+                req.prompt_len += len(tokens)
+            seqs.append(ScheduledSeq(req, len(tokens), start, len(tokens) > 1 or start == 0, False, places))
+        arrays = self.planner.plan_arrays(seqs) if seqs else None
+        if arrays is None or len(arrays["ordered"]) != len(seqs):
+            if seqs:
+                raise RuntimeError("no KV room for a decoded token")
+            return None
+        fb = self.builder.build(arrays["ids"], arrays["pos"], arrays["slots"], arrays["p_q"], arrays["p_ctx"],
+                                arrays["p_tables"], arrays["d_ctx"], arrays["d_tables"], arrays["logit_rows"],
+                                arrays["seq_rows"], prev_ids=arrays["prev_ids"])
+        logits = self._forward(fb)
+        if self.device.type == "cuda":
+            from parallax_b200.ops import cuda as _cuda
+
+            _cuda.check_status(self.device)
+        if not arrays["owners"]:
+            return None
+        # rows come in plan order (prompt slices first); hand them out in the order of the entries
+        at: dict[int, list[int]] = {}
+        for row, s in enumerate(arrays["owners"]):
+            at.setdefault(id(s), []).append(row)
+        order = [row for s in seqs for row in at.get(id(s), [])]
+        return logits.float()[torch.tensor(order, dtype=torch.long, device=logits.device)]
+
+    def release_fed(self, rid: str) -> None:
+        """Give back what a request run by :meth:`feed` holds in the cache."""
+        if self._fed.pop(rid, None) is None:
+            raise ValueError(f"request {rid} not found")
+        self.cache.free_request(rid)
 
     # ------------------------------------------------------------------ the two halves of a step's bookkeeping
     def _read_back(self, cur: "_InFlightStep") -> None:

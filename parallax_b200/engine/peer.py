@@ -143,7 +143,8 @@ class PeerExecutor:
             return arrays, out
         fb = self.builder.build(arrays["ids"] if self.is_first else None, arrays["pos"], arrays["slots"],
                                 arrays["p_q"], arrays["p_ctx"], arrays["p_tables"], arrays["d_ctx"],
-                                arrays["d_tables"], arrays["logit_rows"], arrays["seq_rows"], extra=extra)
+                                arrays["d_tables"], arrays["logit_rows"], arrays["seq_rows"], extra=extra,
+                                prev_ids=arrays["prev_ids"])
         with torch.inference_mode():
             if self.is_last:
                 h = self.worker.model.embed_tokens(fb) if self.is_first else hidden
@@ -434,7 +435,8 @@ class PeerExecutor:
             return out
         # plan order is prefill first, then decode: order the hidden states the same way
         seqs.sort(key=lambda sp: 0 if sp[0].is_prefill else 1)
-        hidden_of = {id(s): pk.hidden_states.to(device=self.device, dtype=self.worker.dtype) for s, pk in seqs}
+        hidden_of = {id(s): pk.hidden_states.to(device=self.device, dtype=self.worker.model.hidden_dtype)
+                     for s, pk in seqs}
         arrays, res = self._run([s for s, _ in seqs], hidden_of)
         for s, pk in seqs:
             if s.req.is_finished:   # KV exhausted while appending a decode slot

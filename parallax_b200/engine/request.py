@@ -226,6 +226,14 @@ class Request:
             self.status = RequestStatus.DECODING
         return len(self.output_ids) - 1
 
+    def token_before_last(self) -> int:
+        """The token before the newest one (-1: there is none)."""
+        n = len(self.output_ids)
+        if n >= 2:
+            return self.output_ids[-2]
+        k = len(self.input_ids) - (2 - n)
+        return self.input_ids[k] if k >= 0 else -1
+
     def fill_token(self, index: int, token_id: int, prob: Optional[float] = None, now: Optional[float] = None) -> None:
         """The value of a reserved token arrived."""
         self.output_ids[index] = int(token_id)

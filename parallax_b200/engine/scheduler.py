@@ -43,6 +43,7 @@ class ScheduledSeq:
     start: int             # sequence position of the first token run in this step
     is_prefill: bool
     produces_token: bool   # last prompt chunk or decode step => a token is sampled
+    logit_at: Optional[list] = None   # places among this step's tokens whose logits are wanted (teacher forcing)
 
 
 class BatchScheduler:

@@ -4,7 +4,8 @@ A stage that owns decoder layers ``[start, end)`` needs: the embedding table if 
 first stage; the final norm and lm_head if it is the last stage (plus the embedding table
 when embeddings are tied); and every ``layers.N.*`` tensor with ``start <= N < end``. VLM
 checkpoints nest the text tower under ``language_model.``; those keys are mapped to the
-text-only layout first. Same selection rule as
+text-only layout first. Checkpoints of layer-list models use flat names (``embed``, ``l<i>.*``,
+``final.norm``, ``head``), selected by the same rule. Same selection rule as
 ``src/parallax/utils/weight_filter_utils.py:11-118``.
 """
 
@@ -16,7 +17,10 @@ from pathlib import Path
 from typing import Iterable, Optional
 
 _LM_PREFIXES = ("model.language_model.", "language_model.")
-_LAYER_RE = re.compile(r"(?:^|\.)layers\.(\d+)\.")
+_LAYER_RE = re.compile(r"(?:^|\.)layers\.(\d+)\.|^l(\d+)\.")
+# flat naming of layer-list checkpoints: embed, bigram, l<i>.*, final.norm, head
+_FLAT_FIRST = ("embed", "bigram")
+_FLAT_LAST = ("final.norm", "head")
 
 
 def normalize_weight_key(key: str) -> str:
@@ -33,11 +37,15 @@ def normalize_weight_key(key: str) -> str:
 
 def layer_index_of(key: str) -> Optional[int]:
     m = _LAYER_RE.search(key)
-    return int(m.group(1)) if m else None
+    return int(m.group(1) or m.group(2)) if m else None
 
 
 def should_include_weight_key(key: str, start_layer: int, end_layer: int, is_first_shard: bool,
                               is_last_shard: bool, tie_word_embeddings: bool = False) -> bool:
+    if key in _FLAT_FIRST:
+        return is_first_shard
+    if key in _FLAT_LAST:
+        return is_last_shard
     if key.startswith("model.") and "embed_tokens" in key:
         if is_first_shard:
             return True

@@ -83,9 +83,26 @@ class ModelConfig:
     quant_method: str = ""
     weight_block_size: Optional[list] = None
     dtype: str = "bfloat16"
+    # models whose config lists every layer with its own mixer / feed-forward sizes (models/layer_spec.py)
+    layer_specs: list = field(default_factory=list)
+    embedding_scale: float = 1.0
+    bigram: Optional[object] = None      # BigramSpec: hashed (previous token, token) embedding
+    residual_mult: float = 1.0           # factor of every sublayer's contribution to the residual
     raw: dict = field(default_factory=dict, repr=False)
 
     # ------------------------------------------------------------------ derived
+    @property
+    def needs_prev_token(self) -> bool:
+        """Whether the embedding of a token also depends on the token before it in its sequence."""
+        return self.bigram is not None
+
+    def latent_dims(self, layer_idx: int) -> tuple[int, int]:
+        """(latent width, rotated key width) of a latent-attention layer's cache row."""
+        if self.layer_specs:
+            m = self.layer_specs[layer_idx].mixer
+            return m.kv_rank, m.rot_dim
+        return self.kv_lora_rank, self.qk_rope_head_dim
+
     @property
     def is_moe(self) -> bool:
         return self.num_experts > 0
@@ -137,6 +154,8 @@ class ModelConfig:
         return any(self.layer_kind(i) == LINEAR for i in range(self.num_hidden_layers))
 
     def layer_window(self, layer_idx: int) -> int:
+        if self.layer_specs:
+            return self.layer_specs[layer_idx].mixer.window
         if not self.sliding_window:
             return 0
         if self.layer_types and layer_idx < len(self.layer_types):
@@ -144,6 +163,9 @@ class ModelConfig:
         return self.sliding_window
 
     def kv_bytes_per_token_per_layer(self, elem_bytes: int = 2) -> int:
+        if self.layer_specs:      # the mean over the layers
+            return -(-sum(sum(self.latent_dims(i)) for i in range(self.num_hidden_layers)) * elem_bytes
+                     // self.num_hidden_layers)
         if self.is_mla:
             return (self.kv_lora_rank + self.qk_rope_head_dim) * elem_bytes
         return 2 * self.num_key_value_heads * self.head_dim * elem_bytes
@@ -169,7 +191,33 @@ def normalize_hf_config(cfg: dict) -> dict:
     return cfg
 
 
+def config_from_layer_list(cfg: dict) -> ModelConfig:
+    """Config whose ``layers`` entry describes every layer by itself (see ``models/layer_spec.py``). The scalar
+    sizes of :class:`ModelConfig` hold the largest value of any layer: capacity estimates use them, the model
+    itself reads ``layer_specs``."""
+    from parallax_b200.models.layer_spec import parse_bigram, parse_layer
+
+    specs = [parse_layer(e) for e in cfg["layers"]]
+    if not specs:
+        raise ValueError("a layer-list config needs at least one layer")
+    emb = cfg.get("embedding") or {}
+    top = lambda f: max(f(s.mixer) for s in specs)  # noqa: E731
+    heads = top(lambda m: m.heads)
+    return ModelConfig(
+        architecture=cfg["architecture"], model_type=str(cfg["architecture"]).lower(), hidden_size=int(cfg["width"]),
+        num_hidden_layers=len(specs), num_attention_heads=heads, num_key_value_heads=heads,
+        head_dim=top(lambda m: m.q_width), intermediate_size=max([s.mlp.ff for s in specs if s.mlp] or [0]),
+        vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]), rope_theta=specs[0].mixer.rot.base,
+        max_position_embeddings=int(cfg.get("max_position_embeddings") or 32768),
+        kv_lora_rank=top(lambda m: m.kv_rank), qk_nope_head_dim=top(lambda m: m.dim),
+        qk_rope_head_dim=top(lambda m: m.rot_dim), v_head_dim=top(lambda m: m.vdim),
+        layer_specs=specs, embedding_scale=float(emb.get("scale", 1.0)), bigram=parse_bigram(emb),
+        residual_mult=float(cfg.get("residual_mult", 1.0)), raw=cfg)
+
+
 def config_from_hf(cfg: dict) -> ModelConfig:
+    if isinstance(cfg.get("layers"), list) and cfg.get("architecture"):
+        return config_from_layer_list(cfg)
     cfg = normalize_hf_config(cfg)
     arch = (cfg.get("architectures") or ["Qwen3ForCausalLM"])[0]
     mt = cfg.get("model_type", "")
@@ -334,6 +382,20 @@ def named_config(name: str) -> ModelConfig:
                                    index_head_dim=hd, index_block_size=sparse["sparse_block_size"],
                                    index_topk_blocks=sparse["sparse_topk_blocks"], index_local_blocks=1,
                                    max_position_embeddings=4096))
+    if n in {"tiny-piburax", "small-piburax", "piburax-1b", "piburax-8b"}:
+        # (layers, width, heads, dim, rot, vdim, rank, window, ff, vocab)
+        nl, w, h, d, r, v, k, win, ff, vocab = {
+            "tiny-piburax": (3, 64, 4, 16, 8, 24, 40, 20, 96, 260),
+            "small-piburax": (3, 512, 8, 64, 32, 64, 192, 100, 1024, 1024),
+            "piburax-1b": (16, 2048, 16, 128, 64, 128, 512, 1024, 5632, 32768),
+            "piburax-8b": (32, 4096, 32, 128, 64, 128, 512, 1024, 12288, 131072)}[n]
+        return config_from_hf(dict(
+            architecture="Piburax", vocab=vocab, width=w, norm=dict(eps=1e-6), residual_mult=0.4,
+            embedding=dict(scale=8.0, bigram=dict(buckets=4093, mul_prev=37, mul_cur=11)),
+            layers=[dict(type="latent_attention",
+                         mixer=dict(heads=h, dim=d, rot_dim=r, vdim=v, kv_rank=k, scale=(d + r) ** -0.5,
+                                    mask=dict(size=win), rot=dict(base=1e4, dims=r)),
+                         mlp=dict(kind="dense", ff=ff, limit=6.0)) for _ in range(nl)]))
     if n == "tiny":
         return config_from_hf(dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", hidden_size=256,
                                    num_hidden_layers=4, num_attention_heads=4, num_key_value_heads=2,

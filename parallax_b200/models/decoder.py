@@ -108,6 +108,11 @@ class DecoderStage(ExpertParallelMixin):
         self.routed_buf = None  # [kv slots, MoE layers, top-k] int16 when routed experts are recorded
         self._route_slots = None
 
+    @property
+    def hidden_dtype(self) -> torch.dtype:
+        """Dtype of the hidden states that travel between pipeline stages."""
+        return self.dtype
+
     # ------------------------------------------------------------------ weights
     def num_local_layers(self) -> int:
         return self.end_layer - self.start_layer
@@ -220,6 +225,7 @@ class DecoderStage(ExpertParallelMixin):
     # ------------------------------------------------------------------ online refit
     _LAYER_KEY = re.compile(r"(?:^|\.)layers\.(\d+)\.")
     _GLOBAL_KEYS = ("embed_tokens.weight", ".norm.weight", "lm_head.weight")
+    _GLOBAL_TENSORS = ("embed", "norm_w", "lm_head")
 
     @classmethod
     def _layer_of_key(cls, key: str) -> Optional[int]:
@@ -268,7 +274,8 @@ class DecoderStage(ExpertParallelMixin):
             glob = copy.copy(self)
             glob.start_layer = glob.end_layer = self.start_layer
             glob.layers, glob.kv_caches, glob._native, glob.lora = [], [], False, None
-            glob.embed = glob.norm_w = glob.lm_head = None
+            for name in self._GLOBAL_TENSORS:
+                setattr(glob, name, None)
             self._prepare_shadow(glob)
             try:
                 glob.load_weights(tensors)
@@ -279,7 +286,7 @@ class DecoderStage(ExpertParallelMixin):
             replaced |= self._adopt_layer(gi - self.start_layer, shadow)
         if glob is not None:
             tied = self.embed is not None and self.lm_head is not None and self.embed.data_ptr() == self.lm_head.data_ptr()
-            for name in ("embed", "norm_w", "lm_head"):
+            for name in self._GLOBAL_TENSORS:
                 new = getattr(glob, name)
                 if new is None or (tied and name == "lm_head"):
                     continue

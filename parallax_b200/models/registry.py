@@ -31,6 +31,8 @@ _REGISTRY: dict[str, str] = {
     "Qwen3NextForCausalLM": "hybrid",
     "Qwen3_5ForConditionalGeneration": "hybrid",
     "Qwen3_5MoeForConditionalGeneration": "hybrid",
+    # layer-list configs: windowed latent attention
+    "Piburax": "latent",
     # block-sparse (MSA)
     "MiniMaxM3SparseForCausalLM": "msa",
 }
@@ -45,6 +47,11 @@ def family_of(arch: str) -> str:
         return _REGISTRY[arch]
     except KeyError as e:
         raise ValueError(f"unsupported architecture {arch!r}; supported: {supported_architectures()}") from e
+
+
+def runs_in_float32(arch: str) -> bool:
+    """Whether the family's GPU stages also run in 32-bit throughout (``dtype=torch.float32``)."""
+    return family_of(arch) == "latent"
 
 
 def build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype, max_positions=None,
@@ -64,6 +71,12 @@ def build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtyp
 def _build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype, max_positions, tp_rank, tp_size,
                  tp_group, comm):
     fam = family_of(cfg.architecture)
+    if fam == "latent":
+        from parallax_b200.models.latent import LatentStage
+
+        if tp_size > 1:
+            raise ValueError(f"tensor parallelism is not available for {cfg.architecture}; use pipeline stages")
+        return LatentStage(cfg, start_layer, end_layer, device, dtype, max_positions=max_positions)
     if tp_size > 1 and fam != "decoder":
         from parallax_b200.models import tp_families
 

@@ -10,13 +10,15 @@ from __future__ import annotations
 import torch
 
 from . import reference
-from ._lib import EPI_F32, EPI_NONE, EPI_RESIDUAL, EPI_SILU_MUL, KernelError
+from .reference import NORM_LAYER, NORM_RMS
+from ._lib import EPI_CLIP_GLU, EPI_F32, EPI_NONE, EPI_RESIDUAL, EPI_SILU_MUL, KernelError
 
 _NAMES = [
     "linear", "rmsnorm", "qk_norm_rope_cache", "reshape_and_cache", "act_mul", "gather_rows",
     "add_inplace", "patch_ids", "attn_decode", "attn_prefill", "argmax", "apply_penalties", "sample", "moe_route", "moe_ffn",
     "mla_kv_prep", "mla_q_absorb", "mla_attn", "mla_unabsorb", "store_rows", "dsa_index_prep", "dsa_index_scores", "topk_select",
     "quant_fp8_rows", "linear_fp8", "moe_ffn_fp8", "causal_conv1d_silu", "gated_delta_rule", "sigmoid_gate_mul", "gate_mul_grouped", "row_dot", "msa_block_scores", "msa_select",
+    "embed_rows", "to_low", "residual_norm", "row_norm", "latent_prep", "head_linear", "latent_attn",
 ]
 
 
@@ -49,5 +51,5 @@ for _n in _NAMES:
 build_cos_sin = reference.build_cos_sin
 interleave_gate_up = reference.interleave_gate_up
 
-__all__ = _NAMES + ["build_cos_sin", "interleave_gate_up", "reference", "KernelError",
+__all__ = _NAMES + ["build_cos_sin", "interleave_gate_up", "reference", "KernelError", "NORM_LAYER", "NORM_RMS", "EPI_CLIP_GLU",
                     "EPI_NONE", "EPI_RESIDUAL", "EPI_SILU_MUL", "EPI_F32"]

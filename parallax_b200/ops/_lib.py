@@ -33,6 +33,7 @@ _ERRORS = {
 }
 
 EPI_NONE, EPI_RESIDUAL, EPI_SILU_MUL, EPI_F32 = 0, 1, 2, 3
+EPI_CLIP_GLU = 10
 
 
 class KernelError(RuntimeError):
@@ -109,6 +110,19 @@ _SIGS = {
     "pxl_msa_block_scores": [_P, _P, _P, _P, _P, _P, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                              c_float, _P],
     "pxl_msa_select": [_P, c_int64, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int64, _P, _P],
+    "pxl_gemm_bf16_glu": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P],
+    "pxl_gemm_bf16_heads": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P],
+    "pxl_gemm_simt": [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int64, c_int, c_int64,
+                      c_int64, c_int, c_int, _P],
+    "pxl_embed_rows": [_P, _P, c_float, _P, _P, c_int64, c_int64, c_int64, _P, c_int, c_int, c_int64, c_int, _P, _P],
+    "pxl_f32_to_bf16": [_P, _P, c_int64, _P],
+    "pxl_residual_norm": [_P, _P, _P, _P, c_int, c_int, c_float, c_float, c_int, c_int, _P],
+    "pxl_row_norm": [_P, _P, _P, c_int64, _P, c_int, c_int, c_float, c_int, c_int, _P, _P],
+    "pxl_act_mul_f32": [_P, _P, c_int, c_int, c_int, c_float, _P],
+    "pxl_latent_prep": [_P, c_int64, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P, _P, c_int64, _P, c_int, c_int, c_int,
+                        c_int, c_float, c_int, _P, _P],
+    "pxl_latent_attn": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64, c_float,
+                        c_int, c_int, _P, _P],
     "pxl_rmsnorm_strided": [_P, c_int64, _P, _P, c_int64, c_int, c_int, c_float, c_float, _P],
     "pxl_argmax": [_P, c_int, c_int64, c_int, c_int, _P, _P, _P, _P],
     "pxl_apply_penalties": [_P, c_int, c_int64, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P],

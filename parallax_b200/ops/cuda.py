@@ -13,7 +13,7 @@ from typing import Optional
 import torch
 
 from . import _lib
-from ._lib import EPI_F32, EPI_NONE, EPI_RESIDUAL, EPI_SILU_MUL, check
+from ._lib import EPI_CLIP_GLU, EPI_F32, EPI_NONE, EPI_RESIDUAL, EPI_SILU_MUL, check
 
 _status: dict[int, torch.Tensor] = {}
 _workspaces: dict[tuple[int, str], torch.Tensor] = {}
@@ -109,6 +109,28 @@ def workspace(device: torch.device, tag: str, nbytes: int) -> torch.Tensor:
 
 
 # ----------------------------------------------------------------------------- GEMM
+def _tma_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
+    """Whether bf16 operands ``x [M, K]``, ``w [N, K]`` fit the tensor-core GEMM (16-byte rows and bases)."""
+    return not ((x.shape[1] | w.shape[0] | x.stride(0) | w.stride(0)) & 7 or (x.data_ptr() | w.data_ptr()) & 15)
+
+
+def _linear_simt(x, w, bias=None, residual=None, epi: int = EPI_NONE, out=None) -> torch.Tensor:
+    assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16)
+    assert x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1] and x.stride(1) == 1 and w.stride(1) == 1
+    if residual is None and epi not in (EPI_NONE, EPI_F32):
+        raise _lib.KernelError("this epilogue needs bf16 operands with 16-byte aligned rows")
+    (M, K), N = x.shape, w.shape[0]
+    f32 = x.dtype == torch.float32
+    if out is None:
+        out = torch.empty((M, N), dtype=torch.float32 if f32 or epi == EPI_F32 else x.dtype, device=x.device)
+    assert residual is None or (residual.dtype == out.dtype and residual.stride() == out.stride())
+    check(_lib.lib().pxl_gemm_simt(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(bias), _ptr(residual), None, M, N, K,
+                                   x.stride(0), w.stride(0), out.stride(0), 0, 1, 0, 0, int(f32),
+                                   int(out.dtype == torch.float32), _stream(x.device)), "pxl_gemm_simt")
+    _count()
+    return out
+
+
 def linear(
     x: torch.Tensor,
     w: torch.Tensor,
@@ -117,8 +139,13 @@ def linear(
     epi: int = EPI_NONE,
     out: Optional[torch.Tensor] = None,
     bn: int = 0,
+    limit: float = 0.0,
 ) -> torch.Tensor:
-    """``x[M,K] @ w[N,K]^T`` on tcgen05 tensor cores with a fused epilogue."""
+    """``x[M,K] @ w[N,K]^T`` on tcgen05 tensor cores with a fused epilogue. fp32 operands, and bf16 operands
+    whose sizes or strides break the TMA rules, run on the FMA pipes (plain epilogues only). ``limit``: clip of
+    :data:`EPI_CLIP_GLU`."""
+    if x.dtype == torch.float32 or not _tma_ok(x, w):
+        return _linear_simt(x, w, bias, residual, epi, out)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     assert x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1]
     assert x.stride(1) == 1 and w.stride(1) == 1
@@ -126,7 +153,7 @@ def linear(
     N = w.shape[0]
     if residual is not None:
         epi = EPI_RESIDUAL
-    n_out = N // 2 if epi == EPI_SILU_MUL else N
+    n_out = N // 2 if epi in (EPI_SILU_MUL, EPI_CLIP_GLU) else N
     if out is None:
         out = torch.empty(
             (M, n_out), dtype=torch.float32 if epi == EPI_F32 else torch.bfloat16, device=x.device
@@ -135,6 +162,13 @@ def linear(
         return out
     if residual is not None:
         assert residual.shape == out.shape and residual.stride(0) == out.stride(0)
+    if epi == EPI_CLIP_GLU:
+        assert bias is None and limit > 0
+        check(_lib.lib().pxl_gemm_bf16_glu(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, x.stride(0), w.stride(0),
+                                           out.stride(0), limit, bn, status_tensor(x.device).data_ptr(),
+                                           _stream(x.device)), "pxl_gemm_bf16_glu")
+        _count()
+        return out
     code = _lib.lib().pxl_gemm_bf16(
         x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(residual), _ptr(bias), M, N, K,
         x.stride(0), w.stride(0), out.stride(0), epi, bn, status_tensor(x.device).data_ptr(),
@@ -328,6 +362,12 @@ def reshape_and_cache(
 def act_mul(x: torch.Tensor, mode: int = 0, limit: float = 7.0) -> torch.Tensor:
     T, I2 = x.shape
     out = torch.empty((T, I2 // 2), dtype=x.dtype, device=x.device)
+    if x.dtype == torch.float32:
+        assert x.is_contiguous()
+        check(_lib.lib().pxl_act_mul_f32(x.data_ptr(), out.data_ptr(), T, I2 // 2, mode, limit, _stream(x.device)),
+              "pxl_act_mul_f32")
+        _count()
+        return out
     check(_lib.lib().pxl_act_mul(x.data_ptr(), out.data_ptr(), T, I2 // 2, mode, limit,
                                  _stream(x.device)), "pxl_act_mul")
     _count()
@@ -925,3 +965,109 @@ def msa_select(scores, positions, block_tables, cu_q, page: int, sparse_block: i
                                     v_ctx.data_ptr(), _stream(scores.device)), "pxl_msa_select")
     _count()
     return v_tables, v_ctx
+
+
+# ---------------------------------------------------------------------------- fp32 residual, latent attention
+def embed_rows(table, ids, scale: float = 1.0, hash_table=None, prev_ids=None, mul_prev: int = 0, mul_cur: int = 0,
+               buckets: int = 0):
+    T, W = ids.numel(), table.shape[1]
+    assert table.is_contiguous() and ids.dtype == torch.int32
+    if hash_table is not None:
+        assert hash_table.is_contiguous() and hash_table.shape == (buckets + 1, W) and hash_table.dtype == table.dtype
+        assert prev_ids.dtype == torch.int32 and prev_ids.numel() == T
+    out = torch.empty((T, W), dtype=torch.float32, device=table.device)
+    check(_lib.lib().pxl_embed_rows(table.data_ptr(), ids.data_ptr(), scale, _ptr(hash_table), _ptr(prev_ids), mul_prev,
+                                    mul_cur, buckets, out.data_ptr(), T, W, table.shape[0],
+                                    int(table.dtype == torch.float32), status_tensor(table.device).data_ptr(),
+                                    _stream(table.device)), "pxl_embed_rows")
+    _count()
+    return out
+
+
+def to_low(x, dtype):
+    if dtype == torch.float32:
+        return x
+    assert x.dtype == torch.float32 and x.is_contiguous() and dtype == torch.bfloat16
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    check(_lib.lib().pxl_f32_to_bf16(x.data_ptr(), out.data_ptr(), x.numel(), _stream(x.device)), "pxl_f32_to_bf16")
+    _count()
+    return out
+
+
+def residual_norm(x, y, w, eps: float, mult: float = 1.0, kind: int = 0):
+    T, W = x.shape
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous()
+    assert y.shape == x.shape and w.numel() == W
+    f32 = y.dtype == torch.float32
+    low = x if f32 else torch.empty_like(y)
+    check(_lib.lib().pxl_residual_norm(x.data_ptr(), y.data_ptr(), w.data_ptr(), None if f32 else low.data_ptr(), T, W,
+                                       eps, mult, kind, int(f32), _stream(x.device)), "pxl_residual_norm")
+    _count()
+    return low
+
+
+def row_norm(x, w, eps: float, kind: int = 0, rows=None, dtype=None):
+    W = x.shape[1]
+    T = x.shape[0] if rows is None else rows.numel()
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.is_contiguous() and w.numel() == W
+    assert rows is None or rows.dtype == torch.int32
+    out = torch.empty((T, W), dtype=dtype or torch.float32, device=x.device)
+    check(_lib.lib().pxl_row_norm(x.data_ptr(), w.data_ptr(), _ptr(rows), x.shape[0], out.data_ptr(), T, W, eps, kind,
+                                  int(out.dtype == torch.float32), status_tensor(x.device).data_ptr(),
+                                  _stream(x.device)), "pxl_row_norm")
+    _count()
+    return out
+
+
+def latent_prep(proj, kv_off: int, q_heads: int, q_width: int, q_rot_off: int, norm_w, cos_sin, positions, slot_mapping,
+                cache, q_cat, eps: float, latent: int, rot_dim: int, rot: int):
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and proj.dtype == cache.dtype == q_cat.dtype and cos_sin.shape[1] == rot
+    assert cache.is_contiguous() and cache.shape[-1] == latent + rot_dim
+    assert q_cat.is_contiguous() and q_cat.shape == (T, q_heads, latent + rot_dim)
+    check(_lib.lib().pxl_latent_prep(proj.data_ptr(), proj.stride(0), kv_off, q_heads, q_width, q_rot_off,
+                                     norm_w.data_ptr(), cos_sin.data_ptr(), positions.data_ptr(), cos_sin.shape[0],
+                                     slot_mapping.data_ptr(), cache.data_ptr(), cache.numel() // cache.shape[-1],
+                                     q_cat.data_ptr(), T, latent, rot_dim, rot, eps, int(proj.dtype == torch.float32),
+                                     status_tensor(proj.device).data_ptr(), _stream(proj.device)), "pxl_latent_prep")
+    _count()
+
+
+def head_linear(x, x_head_stride: int, w, heads: int, out, gate=None):
+    T, K = x.shape[0], w.shape[1]
+    N = w.shape[0] // heads
+    assert x.stride(1) == 1 and w.is_contiguous() and out.shape == (T, heads, N) and out.stride(2) == 1
+    assert x.dtype == w.dtype == out.dtype and (gate is None or (gate.stride(1) == 1 and gate.dtype == x.dtype))
+    ldg = gate.stride(0) if gate is not None else 0
+    ld, hs = out.stride(0), out.stride(1)
+    sizes = K | N | x.stride(0) | x_head_stride | ld | hs | ldg
+    ptrs = x.data_ptr() | w.data_ptr() | out.data_ptr() | (gate.data_ptr() if gate is not None else 0)
+    if x.dtype == torch.bfloat16 and not sizes & 7 and not ptrs & 15:
+        check(_lib.lib().pxl_gemm_bf16_heads(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(gate), T, heads, N, K,
+                                             x.stride(0), x_head_stride, K, ld, hs, ldg,
+                                             status_tensor(x.device).data_ptr(), _stream(x.device)),
+              "pxl_gemm_bf16_heads")
+    else:
+        f32 = int(x.dtype == torch.float32)
+        check(_lib.lib().pxl_gemm_simt(x.data_ptr(), w.data_ptr(), out.data_ptr(), None, None, _ptr(gate), T, N, K,
+                                       x.stride(0), K, ld, ldg, heads, x_head_stride, hs, f32, f32, _stream(x.device)),
+              "pxl_gemm_simt")
+    _count()
+    return out
+
+
+def latent_attn(q_cat, cache, block_tables, cu_q, ctx_lens, scale: float, latent: int, window: int = 0, sinks=None,
+                max_q: int = 1, max_ctx: int = 0, out=None):
+    T, H, D = q_cat.shape
+    page, B = cache.shape[-2], ctx_lens.numel()
+    assert q_cat.is_contiguous() and cache.is_contiguous() and cache.shape[-1] == D and q_cat.dtype == cache.dtype
+    if out is None:
+        out = torch.empty((T, H, latent), dtype=q_cat.dtype, device=q_cat.device)
+    assert out.is_contiguous() and out.shape == (T, H, latent)
+    check(_lib.lib().pxl_latent_attn(q_cat.data_ptr(), cache.data_ptr(), block_tables.data_ptr(), _ptr(cu_q),
+                                     ctx_lens.data_ptr(), out.data_ptr(), _ptr(sinks), B, max_q, H, latent, D - latent,
+                                     page, block_tables.shape[1], cache.shape[0], float(scale), window,
+                                     int(q_cat.dtype == torch.float32), status_tensor(q_cat.device).data_ptr(),
+                                     _stream(q_cat.device)), "pxl_latent_attn")
+    _count()
+    return out

@@ -16,6 +16,7 @@ import math
 import torch
 
 EPI_NONE, EPI_RESIDUAL, EPI_SILU_MUL, EPI_F32 = 0, 1, 2, 3
+EPI_CLIP_GLU = 10
 
 
 def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
@@ -32,7 +33,7 @@ def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor
     return torch.cat([g, u], dim=1).reshape(2 * I, K).contiguous()
 
 
-def linear(x, w, bias=None, residual=None, epi: int = EPI_NONE, out=None, bn: int = 128):
+def linear(x, w, bias=None, residual=None, epi: int = EPI_NONE, out=None, bn: int = 128, limit: float = 0.0):
     y = x.float() @ w.float().t()
     if bias is not None:
         y = y + bias.float()
@@ -44,6 +45,9 @@ def linear(x, w, bias=None, residual=None, epi: int = EPI_NONE, out=None, bn: in
         h = 64
         yb = y.reshape(y.shape[0], N // 128, 2, h)
         y = (torch.nn.functional.silu(yb[:, :, 0]) * yb[:, :, 1]).reshape(y.shape[0], N // 2)
+    elif epi == EPI_CLIP_GLU:
+        yb = y.reshape(y.shape[0], w.shape[0] // 128, 2, 64)
+        y = act_mul(torch.cat([yb[:, :, 0], yb[:, :, 1]], -1), 1, limit).reshape(y.shape[0], w.shape[0] // 2)
     res = y if epi == EPI_F32 else y.to(x.dtype)
     if out is not None:
         out.copy_(res)
@@ -640,3 +644,113 @@ def msa_select(scores, positions, block_tables, cu_q, page: int, sparse_block: i
                                              torch.zeros_like(pages)).int()
         v_ctx[t] = (k - 1) * sparse_block + pos - cur * sparse_block + 1
     return v_tables, v_ctx
+
+
+# ---------------------------------------------------------------------------- fp32 residual, latent attention
+NORM_LAYER, NORM_RMS = 0, 1
+
+
+def _normalised(x, eps, kind: int):
+    xf = x.float()
+    if kind == NORM_LAYER:
+        xf = xf - xf.mean(-1, keepdim=True)
+    return xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def embed_rows(table, ids, scale: float = 1.0, hash_table=None, prev_ids=None, mul_prev: int = 0, mul_cur: int = 0,
+               buckets: int = 0):
+    """fp32 rows ``table[id] * scale``; with ``hash_table [buckets + 1, W]`` plus its row
+    ``(prev * mul_prev + id * mul_cur) mod buckets`` (row ``buckets`` where ``prev`` is negative)."""
+    x = table[ids.long()].float() * scale
+    if hash_table is not None:
+        prev = prev_ids.long()
+        row = torch.where(prev < 0, torch.full_like(prev, buckets), (prev * mul_prev + ids.long() * mul_cur) % buckets)
+        x = x + hash_table[row].float()
+    return x
+
+
+def to_low(x, dtype):
+    """fp32 residual rows as GEMM operand (the tensor itself when that is fp32 too)."""
+    return x if dtype == torch.float32 else x.to(dtype)
+
+
+def residual_norm(x, y, w, eps: float, mult: float = 1.0, kind: int = NORM_LAYER):
+    """In place on the fp32 residual: ``x += mult * norm(y) * w``. Returns ``x`` in ``y``'s dtype."""
+    x.add_(_normalised(y, eps, kind) * w.float() * mult)
+    return to_low(x, y.dtype)
+
+
+def row_norm(x, w, eps: float, kind: int = NORM_LAYER, rows=None, dtype=None):
+    """``norm(x[rows]) * w`` of fp32 rows in ``dtype``."""
+    x = x if rows is None else x[rows.long()]
+    return (_normalised(x, eps, kind) * w.float()).to(dtype or x.dtype)
+
+
+def _rotate_pairs(x, cos_sin, positions, dims: int):
+    """Interleaved rotation of the first ``dims`` entries of the last dimension; x ``[T, ..., R]`` fp32."""
+    cs = cos_sin[positions.long()].float()
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (dims // 2,)
+    c, s = cs[:, :dims // 2].reshape(shape), cs[:, dims // 2:dims].reshape(shape)
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    out = x.clone()
+    out[..., 0:dims:2] = u * c - v * s
+    out[..., 1:dims:2] = v * c + u * s
+    return out
+
+
+def latent_prep(proj, kv_off: int, q_heads: int, q_width: int, q_rot_off: int, norm_w, cos_sin, positions, slot_mapping,
+                cache, q_cat, eps: float, latent: int, rot_dim: int, rot: int):
+    """One step's latent-attention inputs out of the packed projection ``proj`` (columns: ``q_heads`` heads of
+    ``q_width``, and at ``kv_off`` the raw latent | rotated key part): RMS-normed latent and rotated key go to
+    the cache rows ``slot_mapping``, the rotated query parts to ``q_cat[:, :, latent:]``."""
+    T = proj.shape[0]
+    kv = proj[:, kv_off:kv_off + latent + rot_dim].float()
+    c = _normalised(kv[:, :latent], eps, NORM_RMS) * norm_w.float()
+    k = _rotate_pairs(kv[:, latent:], cos_sin, positions, rot)
+    flat = cache.view(-1, latent + rot_dim)
+    ok = slot_mapping >= 0
+    flat[slot_mapping[ok]] = torch.cat([c, k], -1)[ok].to(cache.dtype)
+    q = proj[:, :q_heads * q_width].reshape(T, q_heads, q_width)[..., q_rot_off:q_rot_off + rot_dim].float()
+    q_cat[:, :, latent:] = _rotate_pairs(q, cos_sin, positions, rot).to(q_cat.dtype)
+
+
+def head_linear(x, x_head_stride: int, w, heads: int, out, gate=None):
+    """Per-head product: ``out[t, h, :] = W_h x[t, h * x_head_stride : ... + K]`` with ``w [heads * N, K]``;
+    ``out [T, heads, N]`` may be strided. With ``gate [T, heads * N]`` times ``sigmoid(gate)``."""
+    T, K = x.shape[0], w.shape[1]
+    N = w.shape[0] // heads
+    xs = torch.stack([x[:, h * x_head_stride:h * x_head_stride + K] for h in range(heads)], 1).float()
+    y = torch.einsum("thk,hnk->thn", xs, w.view(heads, N, K).float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float().reshape(T, heads, N))
+    out.copy_(y.to(out.dtype))
+    return out
+
+
+def latent_attn(q_cat, cache, block_tables, cu_q, ctx_lens, scale: float, latent: int, window: int = 0, sinks=None,
+                max_q: int = 1, max_ctx: int = 0, out=None):
+    """Causal attention of ``q_cat [T, H, latent + R]`` over cached rows ``latent | R``; the values are the latent
+    parts. ``cu_q`` None: one query per sequence. ``window`` keys per query (0: all); ``sinks [H]`` fp32 add
+    ``exp(sink)`` to the denominator. ``out [T, H, latent]``."""
+    T, H, _ = q_cat.shape
+    page = cache.shape[-2]
+    flat = cache.view(-1, cache.shape[-1])
+    if out is None:
+        out = torch.empty((T, H, latent), dtype=q_cat.dtype, device=q_cat.device)
+    cu = list(range(T + 1)) if cu_q is None else cu_q.tolist()
+    for b, ctx in enumerate(ctx_lens.tolist()):
+        t0, t1 = cu[b], cu[b + 1]
+        if t1 <= t0:
+            continue
+        keys = torch.arange(ctx, device=q_cat.device)
+        rows = flat[block_tables[b].long()[keys // page] * page + keys % page].float()
+        pos = ctx - (t1 - t0) + torch.arange(t1 - t0, device=q_cat.device)
+        s = torch.einsum("thk,sk->hts", q_cat[t0:t1].float(), rows) * scale
+        dist = pos[:, None] - keys[None, :]
+        keep = (dist >= 0) & (dist < window) if window > 0 else dist >= 0
+        s = s.masked_fill(~keep, float("-inf"))
+        if sinks is not None:
+            s = torch.cat([s, sinks.float().view(H, 1, 1).expand(H, t1 - t0, 1)], -1)
+        p = torch.softmax(s, -1)[..., :ctx]
+        out[t0:t1] = torch.einsum("hts,sk->thk", p, rows[:, :latent]).to(out.dtype)
+    return out

@@ -233,8 +233,8 @@ class DistEngine:
         lane_batch = -(-max_batch_size // ep)
         lane_tokens = max(-(-max_num_tokens_per_batch // ep), lane_batch + 256) if ep > 1 else max_num_tokens_per_batch
         micro_seqs = max(1, max_batch_size // max(1, ratio))
-        # the largest plan: ids, positions (4 B) and slots (8 B) per token, one block table row per sequence
-        slot_bytes = 16 * (ep * lane_tokens + max_batch_size) + 4 * micro_seqs * (max_blocks + 8) + (64 << 10)
+        # the largest plan: ids, previous ids, positions (4 B) and slots (8 B) per token, one block table row per sequence
+        slot_bytes = 20 * (ep * lane_tokens + max_batch_size) + 4 * micro_seqs * (max_blocks + 8) + (64 << 10)
         slot_bytes = max(1 << 18, (slot_bytes + 4095) // 4096 * 4096)
         n_slots = max(8, self.max_in_flight + 6)
         box = [None]
@@ -415,7 +415,7 @@ class DistEngine:
         slot = self._recv_ring[self._recv_n % len(self._recv_ring)]
         self._recv_n += 1
         if slot.buf is None or slot.buf.shape[0] < rows:
-            slot.buf = torch.empty((max(rows, 256), H), dtype=self.worker.dtype, device=self.device)
+            slot.buf = torch.empty((max(rows, 256), H), dtype=self.worker.model.hidden_dtype, device=self.device)
             slot.free = None
             if self.device.type == "cuda" and self.topo.tp == 1:
                 # The memory comes from the compute stream's pool: it may be a block that a tensor of an
@@ -582,7 +582,8 @@ class DistEngine:
             fb = b.build(lp["ids"] if topo.is_first_stage else None, lp["pos"], lp["slots"], lp["p_q"],
                          lp["p_ctx"], lp["p_tables"], lp["d_ctx"], lp["d_tables"], lp["logit_rows"],
                          lp.get("seq_rows"),
-                         extra={"lora_ids": lp["lora_ids"]} if lp.get("lora_ids") is not None else None)
+                         extra={"lora_ids": lp["lora_ids"]} if lp.get("lora_ids") is not None else None,
+                         prev_ids=lp.get("prev_ids"))
             if lp.get("lora_ids") is not None:
                 fb.extras["lora_ids_host"] = lp["lora_ids"]
             self.h2d_bytes += fb.h2d_bytes
@@ -900,7 +901,7 @@ class DistEngine:
         owners = arrays["owners"]
         sps = [s.req.sampling_params for s in owners]
         greedy = all(sp.is_greedy for sp in sps)
-        lp = {k: arrays[k] for k in ("ids", "pos", "slots", "p_q", "p_ctx", "p_tables", "d_ctx", "d_tables",
+        lp = {k: arrays[k] for k in ("ids", "prev_ids", "pos", "slots", "p_q", "p_ctx", "p_tables", "d_ctx", "d_tables",
                                      "logit_rows", "seq_rows")}
         lp.update(n_logits=len(owners), greedy=greedy)
         if any(s.req.return_probs for s in owners):
