@@ -1,0 +1,435 @@
+// Latent attention on the 5th-generation tensor cores, prompts and decoding alike (bf16; see latent_attn.cu for
+// the op). One kernel serves every size with L + R <= 576.
+//
+// A query row is a (token, head) pair: q [T, H, L + R] is a matrix of T * H rows that all read the same cached
+// rows, so a CTA takes 128 consecutive rows of one sequence - 128 / H tokens (one token and a block of 128 heads
+// when H > 128) - and walks the keys that its first and last token may see in tiles of NK.
+//
+//   warp 4    : TMA producer. The query tile once (chunks of 64 columns, 128-byte swizzle), then tiles of cache
+//               rows (page boxes) through a ring. A cache row is key AND value: each tile is loaded once.
+//   warp 5    : MMA issuer. S = Q K^T over L + R (both operands K-major) into one of two TMEM score buffers, so
+//               the scores of tile i + 1 are computed while the softmax warps work on tile i; then O += P V, P
+//               from tensor memory, V taken MN-major from the same shared-memory tile (its first L columns).
+//   warps 0-3 : softmax, one row per thread (its TMEM lane): mask (causal, window), running reference maximum
+//               that only moves when a row grew by more than 2^8 (then the TMEM rows of O are rescaled), P
+//               back to tensor memory as bf16 (two buffers), row sums in fp32; at the end the sink and the
+//               division.
+//
+// O takes 64 TMEM columns per 64 latent columns and scores need room beside it, so a CTA accumulates at most 256
+// latent columns; wider latents run as several CTAs per query tile that repeat the scores (L = 512: two).
+// Every wait is bounded; on expiry the kernel records a status code, all roles unwind, TMEM is freed.
+#include "common.cuh"
+#include "pxl_api.h"
+
+namespace {
+using namespace pxl;
+
+constexpr int kRows = 128;
+constexpr int kQChunk = kRows * 128;   // bytes of 64 columns of the query tile
+constexpr int kMaxV = 4;               // 64-column latent chunks a CTA accumulates
+constexpr int kMaxStages = 4;
+constexpr int kProducerWarp = 4, kMmaWarp = 5;
+constexpr int kThreads = 192;
+constexpr int kBarBytes = 256;
+constexpr int kMaxSmem = 227 * 1024;
+constexpr float kLog2eF = 1.4426950408889634f;
+
+struct TcArgs {
+  const int* block_tables;
+  const int* cu_q;      // null: token i is the only query of sequence i
+  const int* ctx_lens;
+  bf16* out;            // [T, H, L]
+  const float* sinks;
+  int H, L, D, page, max_blocks, window, stages, vsplit, head_blocks;
+  int64_t num_blocks;
+  float scale_log2;
+  int* status;
+};
+
+__device__ __forceinline__ uint64_t desc_mn_sw128(uint32_t addr) {  // B stored [key rows, 64 columns]: MN-major
+  return umma_desc_k_sw128(addr);  // same fields: groups of 8 rows 1024 B apart, one 64-wide chunk addressed
+}
+__device__ __forceinline__ float fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// D[tmem] (+)= A[tmem] * B[smem desc]; A holds two bf16 per 32-bit column, one row per lane
+__device__ __forceinline__ void tc_mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc,
+                                              uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n"
+      :
+      : "r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_32x32b_x16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+      :
+      : "r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]),
+        "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+      : "memory");
+}
+
+template <int NK>
+__global__ void __launch_bounds__(kThreads, 1)
+latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv,
+                      const TcArgs a) {
+  constexpr int kKvChunk = NK * 128;  // bytes of 64 columns of a key tile
+  constexpr uint32_t kIdescS = umma_idesc(kRows, NK, 1, 1);
+  constexpr uint32_t kIdescPV = umma_idesc(kRows, 64, 1, 1) | (1u << 16);  // B (V) is MN-major
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const int nck = ceil_div(a.D, 64);
+  const uint32_t sm_q = smem_u32(smem);
+  const uint32_t sm_kv = sm_q + nck * kQChunk;
+  const uint32_t stage_bytes = nck * kKvChunk;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + nck * kQChunk + a.stages * stage_bytes);
+  // q_full | kv_full [kMaxStages] | kv_empty [kMaxStages] | s_full [2] | p_ready [2] | o_full [2]
+  const uint32_t q_full = smem_u32(bars), kv_full = q_full + 8, kv_empty = kv_full + 8 * kMaxStages,
+                 s_full = kv_empty + 8 * kMaxStages, p_ready = s_full + 16, o_full = p_ready + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * kMaxStages + 6);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  pdl_wait();
+  pdl_launch_dependents();
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = blockIdx.z, hb = blockIdx.y;
+  const int vs = blockIdx.x % a.vsplit, tile = blockIdx.x / a.vsplit;
+  const int t0 = a.cu_q ? a.cu_q[b] : b;
+  const int len = a.cu_q ? a.cu_q[b + 1] - t0 : 1;
+  const int ctx = a.ctx_lens[b];
+  const int h0 = hb * kRows;
+  const int heads = a.H - h0 < kRows ? a.H - h0 : kRows;  // heads per token of this tile
+  const int tpt = a.H <= kRows ? kRows / a.H : 1;         // tokens per tile
+  const int tok0 = tile * tpt;
+  if (tok0 >= len) return;  // uniform for the CTA, before any barrier or allocation
+  const int ntok = len - tok0 < tpt ? len - tok0 : tpt;
+  const int rows = ntok * heads;
+  const int64_t row0 = static_cast<int64_t>(t0 + tok0) * a.H + h0;  // row of q / out
+  const int pos0 = ctx - len + tok0;
+  const int hi = pos0 + ntok;  // keys [lo, hi) are visible to some row
+  const int lo = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;
+  const int t_begin = lo / NK;
+  const int n_tiles = ceil_div(hi, NK) - t_begin;
+  // latent chunks of this CTA
+  const int ncv = ceil_div(a.L, 64), per = ceil_div(ncv, a.vsplit);
+  const int v0 = vs * per;
+  const int nv = ncv - v0 < per ? ncv - v0 : per;
+
+  if (threadIdx.x == 0) {
+    *abort_flag = 0;
+    mbar_init(q_full, 1);
+    for (int s = 0; s < a.stages; ++s) {
+      mbar_init(kv_full + 8 * s, 1);
+      mbar_init(kv_empty + 8 * s, 1);
+    }
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(s_full + 8 * s, 1);
+      mbar_init(p_ready + 8 * s, 4);  // one arrival per softmax warp
+      mbar_init(o_full + 8 * s, 1);
+    }
+    mbar_fence_init();
+    fence_proxy_async_smem();
+    tma_prefetch_desc(&tm_q);
+    tma_prefetch_desc(&tm_kv);
+  }
+  const uint32_t tmem_cols = 64 * per + 3 * NK <= 256 ? 256 : 512;  // O | two score | two probability buffers
+  if (warp == kMmaWarp) {
+    tmem_alloc(smem_u32(tmem_slot), tmem_cols);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tm_o = *tmem_slot;             // O: 64 columns per latent chunk
+  const uint32_t tm_s = tm_o + 64 * per;        // two score buffers of NK columns
+  const uint32_t tm_p = tm_s + 2 * NK;          // two probability buffers of NK / 2 columns
+
+  if (warp == kProducerWarp) {
+    // ------------------------------------------------------------------ TMA producer
+    // Lane p looks up the block of piece p of the tile and issues its boxes: the block-table reads of a tile are
+    // in flight together and come before the wait for the stage.
+    if (lane == 0) {
+      mbar_arrive_expect_tx(q_full, nck * kQChunk);
+      for (int c = 0; c < nck; ++c)
+        tma_load_2d(sm_q + c * kQChunk, &tm_q, q_full, c * 64, static_cast<int>(row0));
+    }
+    const int* bt = a.block_tables + static_cast<int64_t>(b) * a.max_blocks;
+    const int box = a.page < NK ? a.page : NK;
+    const int pieces = NK / box;
+    for (int it = 0; it < n_tiles; ++it) {
+      const int stage = it % a.stages;
+      int64_t row = 0;
+      if (lane < pieces) {
+        int key = (t_begin + it) * NK + lane * box;
+        if (key >= ctx) key = (ctx - 1) / box * box;  // beyond the context: re-read its last piece (masked)
+        const int bi = key / a.page;
+        int64_t blk = bi < a.max_blocks ? bt[bi] : -1;
+        if (blk < 0 || blk >= a.num_blocks) {
+          if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_BLOCK_PREFILL);
+          blk = 0;
+        }
+        row = blk * a.page + key % a.page;
+      }
+      int okf = 1;
+      if (it >= a.stages && lane == 0)
+        okf = mbar_wait_bounded(kv_empty + 8 * stage, ((it / a.stages) - 1) & 1, abort_flag, a.status,
+                                PXL_DEV_TIMEOUT_EMPTY) ? 1 : 0;
+      okf = __shfl_sync(0xffffffffu, okf, 0);
+      if (!okf) break;
+      const uint32_t bar = kv_full + 8 * stage;
+      if (lane == 0) mbar_arrive_expect_tx(bar, stage_bytes);
+      __syncwarp();
+      if (lane < pieces) {
+        const uint32_t dst = sm_kv + stage * stage_bytes + lane * box * 128;
+        for (int c = 0; c < nck; ++c) tma_load_2d(dst + c * kKvChunk, &tm_kv, bar, c * 64, static_cast<int>(row));
+      }
+    }
+  } else if (warp == kMmaWarp) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0) {
+      const int ksteps = ceil_div(a.D, 16);
+      auto issue_s = [&](int it) {  // S[it % 2] = Q K(it)^T
+        const uint32_t k_addr = sm_kv + (it % a.stages) * stage_bytes;
+        const uint32_t d_tmem = tm_s + (it & 1) * NK;
+        for (int ks = 0; ks < ksteps; ++ks) {
+          const uint32_t in = (ks & 3) * 32;
+          tc_mma_f16(d_tmem, umma_desc_k_sw128(sm_q + (ks >> 2) * kQChunk + in),
+                     umma_desc_k_sw128(k_addr + (ks >> 2) * kKvChunk + in), kIdescS, ks > 0 ? 1u : 0u);
+        }
+        tc_commit(s_full + 8 * (it & 1));
+      };
+      bool ok = mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
+      ok = ok && mbar_wait_bounded(kv_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
+      if (ok) {
+        tc_fence_after_sync();
+        issue_s(0);
+      }
+      for (int it = 0; ok && it < n_tiles; ++it) {
+        const int stage = it % a.stages;
+        if (it + 1 < n_tiles) {
+          // scores of the next tile while the softmax warps work on this one
+          ok = mbar_wait_bounded(kv_full + 8 * ((it + 1) % a.stages), ((it + 1) / a.stages) & 1, abort_flag, a.status,
+                                 PXL_DEV_TIMEOUT_FULL);
+          if (!ok) break;
+          tc_fence_after_sync();
+          issue_s(it + 1);
+        }
+        ok = mbar_wait_bounded(p_ready + 8 * (it & 1), (it >> 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_TMEM_EMPTY);
+        if (!ok) break;
+        tc_fence_after_sync();
+        const uint32_t v_addr = sm_kv + stage * stage_bytes + v0 * kKvChunk;
+        for (int c = 0; c < nv; ++c) {
+#pragma unroll
+          for (int ks = 0; ks < NK / 16; ++ks)
+            tc_mma_f16_ts(tm_o + c * 64, tm_p + (it & 1) * (NK / 2) + ks * 8, desc_mn_sw128(v_addr + c * kKvChunk + ks * 2048),
+                          kIdescPV, (it > 0 || ks > 0) ? 1u : 0u);
+        }
+        tc_commit(o_full + 8 * (it & 1));
+        tc_commit(kv_empty + 8 * stage);  // the rows of this stage are no longer read
+      }
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax warps
+    const int r = warp * 32 + lane;  // query row = TMEM lane
+    const int pos = pos0 + r / heads, head = h0 + r % heads;
+    const bool row_valid = r < rows;
+    const int key_lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+    const int key_hi = row_valid ? pos + 1 : 0;
+    const uint32_t lane_sel = static_cast<uint32_t>(warp * 32) << 16;
+    float m_run = -INFINITY, l_run = 0.f;
+    int failed = 0;
+    for (int it = 0; it < n_tiles; ++it) {
+      const int par = it & 1;
+      failed = mbar_wait_bounded(s_full + 8 * par, (it >> 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_TMEM_FULL) ? 0 : 1;
+      failed = __any_sync(0xffffffffu, failed);  // warp-uniform: the TMEM accesses below are warp-wide
+      if (failed) break;
+      tc_fence_after_sync();
+      uint32_t sc[NK];
+#pragma unroll
+      for (int c = 0; c < NK; c += 32)
+        tmem_ld_32x32b_x32(tm_s + par * NK + c + lane_sel, *reinterpret_cast<uint32_t(*)[32]>(&sc[c]));
+      tmem_ld_wait();
+      const int key0 = (t_begin + it) * NK;
+      const int ma = key_lo - key0, me = key_hi - key0;  // this row sees columns [ma, me)
+      if (!__all_sync(0xffffffffu, ma <= 0 && me >= NK)) {
+#pragma unroll
+        for (int j = 0; j < NK; ++j)
+          if (j < ma || j >= me) sc[j] = 0xff800000u;  // -inf
+      }
+      float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+      for (int j = 0; j < NK; j += 4) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) m4[k] = fmaxf(m4[k], __uint_as_float(sc[j + k]));
+      }
+      const float m_new = fmaxf(m_run, fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * a.scale_log2);  // scale > 0
+      if (it == 0) {
+        m_run = m_new;
+      } else if (__any_sync(0xffffffffu, m_new > m_run + 8.f)) {
+        // O accumulates relative to m_run: move the reference and rescale, once O of the tile before is complete
+        failed = mbar_wait_bounded(o_full + 8 * (par ^ 1), ((it - 1) >> 1) & 1, abort_flag, a.status,
+                                   PXL_DEV_TIMEOUT_TMEM_FULL) ? 0 : 1;
+        failed = __any_sync(0xffffffffu, failed);
+        if (failed) break;
+        const float corr = fast_exp2(m_run - (m_new == -INFINITY ? 0.f : m_new));
+        m_run = m_new;
+        l_run *= corr;
+        tc_fence_after_sync();
+        for (int c = 0; c < nv * 64; c += 32) {
+          uint32_t v[32];
+          tmem_ld_32x32b_x32(tm_o + lane_sel + c, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) * corr);
+          tmem_st_32x32b_x32(tm_o + lane_sel + c, v);
+        }
+        tmem_st_wait();
+      }
+      const float m_use = (m_run == -INFINITY) ? 0.f : m_run;
+      // the P buffer was last read by the product of tile it - 2
+      if (it >= 2) {
+        failed = mbar_wait_bounded(o_full + 8 * par, ((it - 2) >> 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_TMEM_FULL) ? 0 : 1;
+        failed = __any_sync(0xffffffffu, failed);
+        if (failed) break;
+        tc_fence_after_sync();
+      }
+      float sum2[2] = {0.f, 0.f};
+      uint32_t pk[NK / 2];
+#pragma unroll
+      for (int j = 0; j < NK; j += 2) {
+        const float p0 = fast_exp2(fmaf(__uint_as_float(sc[j]), a.scale_log2, -m_use));
+        const float p1 = fast_exp2(fmaf(__uint_as_float(sc[j + 1]), a.scale_log2, -m_use));
+        sum2[0] += p0;
+        sum2[1] += p1;
+        pk[j >> 1] = pack_bf16x2(p0, p1);
+      }
+      l_run += sum2[0] + sum2[1];
+#pragma unroll
+      for (int c = 0; c < NK / 2; c += 16)
+        tmem_st_32x32b_x16(tm_p + par * (NK / 2) + c + lane_sel, *reinterpret_cast<uint32_t(*)[16]>(&pk[c]));
+      tmem_st_wait();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_ready + 8 * par);
+    }
+    if (!failed)
+      failed = mbar_wait_bounded(o_full + 8 * ((n_tiles - 1) & 1), ((n_tiles - 1) >> 1) & 1, abort_flag, a.status,
+                                 PXL_DEV_TIMEOUT_TMEM_FULL) ? 0 : 1;
+    failed = __any_sync(0xffffffffu, failed);
+    if (!failed) {
+      float denom = l_run, f = 1.f;
+      if (a.sinks && row_valid) {
+        const float sink = a.sinks[head] * kLog2eF;
+        const float M = fmaxf(m_run, sink);
+        f = exp2f(m_run - M);
+        denom = denom * f + exp2f(sink - M);
+      }
+      const float inv = denom > 0.f ? f / denom : 0.f;
+      bf16* dst = a.out + (row0 + r) * a.L + v0 * 64;
+      const int ncol = a.L - v0 * 64 < nv * 64 ? a.L - v0 * 64 : nv * 64;
+      tc_fence_after_sync();
+      for (int c = 0; c < nv * 64; c += 32) {
+        uint32_t v[32];
+        tmem_ld_32x32b_x32(tm_o + lane_sel + c, v);
+        tmem_ld_wait();
+#pragma unroll
+        for (int c8 = 0; c8 < 32; c8 += 8) {
+          bf16x8 ov;
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            ov.u[j] = pack_bf16x2(__uint_as_float(v[c8 + 2 * j]) * inv, __uint_as_float(v[c8 + 2 * j + 1]) * inv);
+          if (row_valid && c + c8 < ncol) st_bf16x8(dst + c + c8, ov);
+        }
+      }
+      tc_fence_before_sync();
+    }
+  }
+
+  // ---------------------------------------------------------------------- teardown
+  __syncwarp();
+  if (*abort_flag) __nanosleep(200000);  // loads that are still in flight must land before smem is released
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  if (warp == kMmaWarp) tmem_dealloc(tm_o, tmem_cols);
+}
+
+int smem_bytes(int nck, int nk, int stages) { return 1024 + nck * kQChunk + stages * nck * nk * 128 + kBarBytes; }
+
+// keys per tile and ring stages for a row width; false when two stages do not fit
+bool plan_tiles(int D, int page, int* nk, int* stages) {
+  const int nck = ceil_div(D, 64);
+  for (const int cand : {64, 32}) {
+    if (page % cand != 0 && cand % page != 0) continue;
+    int s = kMaxStages;
+    while (s >= 2 && smem_bytes(nck, cand, s) > kMaxSmem) --s;
+    if (s >= 2) {
+      *nk = cand;
+      *stages = s;
+      return true;
+    }
+  }
+  return false;
+}
+
+template <int NK>
+int launch_tc(const CUtensorMap& tq, const CUtensorMap& tkv, const TcArgs& a, dim3 grid, cudaStream_t stream) {
+  static bool configured[64] = {false};
+  const int dev = pxl_host::current_device_slot();
+  if (!configured[dev]) {
+    if (cudaFuncSetAttribute(latent_attn_tc_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem) != cudaSuccess)
+      return PXL_ERR_CUDA;
+    configured[dev] = true;
+  }
+  pxl_host::launch(latent_attn_tc_kernel<NK>, grid, dim3(kThreads), smem_bytes(ceil_div(a.D, 64), NK, a.stages), stream, tq,
+                   tkv, a);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+}  // namespace
+
+PXL_EXPORT int pxl_latent_attn_tc_supported(int L, int R, int page, float scale) {
+  int nk, stages;
+  return L > 0 && R >= 0 && L % 8 == 0 && R % 8 == 0 && page > 0 && page % 8 == 0 && scale > 0.f &&
+         plan_tiles(L + R, page, &nk, &stages);
+}
+
+PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* block_tables, const int* cu_q,
+                                  const int* ctx_lens, void* out, const float* sinks, int B, int max_q, int total_q, int H,
+                                  int L, int R, int page, int max_blocks, int64_t num_blocks, float scale, int window,
+                                  int* status, cudaStream_t stream) {
+  if (B <= 0 || max_q <= 0 || total_q <= 0) return PXL_OK;
+  if (H <= 0 || B > 65535 || !pxl_latent_attn_tc_supported(L, R, page, scale)) return PXL_ERR_INVALID_ARG;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15)
+    return PXL_ERR_INVALID_ARG;
+  if (num_blocks * page >= (1ll << 31) || static_cast<int64_t>(total_q) * H >= (1ll << 31)) return PXL_ERR_TOO_LARGE;
+  TcArgs a{};
+  int nk = 0;
+  plan_tiles(L + R, page, &nk, &a.stages);
+  a.block_tables = block_tables;
+  a.cu_q = cu_q;
+  a.ctx_lens = ctx_lens;
+  a.out = static_cast<pxl::bf16*>(out);
+  a.sinks = sinks;
+  a.H = H, a.L = L, a.D = L + R, a.page = page, a.max_blocks = max_blocks, a.window = window, a.num_blocks = num_blocks;
+  a.vsplit = pxl::ceil_div(pxl::ceil_div(L, 64), kMaxV);
+  a.head_blocks = pxl::ceil_div(H, kRows);
+  a.scale_log2 = scale * kLog2eF;
+  a.status = status;
+  CUtensorMap tq, tkv;
+  if (!pxl_host::make_tmap_2d(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, q, static_cast<uint64_t>(total_q) * H, a.D, a.D, kRows,
+                              64) ||
+      !pxl_host::make_tmap_2d(&tkv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cache, static_cast<uint64_t>(num_blocks) * page, a.D,
+                              a.D, page < nk ? page : nk, 64))
+    return PXL_ERR_TENSORMAP;
+  const int tpt = H <= kRows ? kRows / H : 1;
+  const dim3 grid(pxl::ceil_div(max_q, tpt) * a.vsplit, a.head_blocks, B);
+  return nk == 64 ? launch_tc<64>(tq, tkv, a, grid, stream) : launch_tc<32>(tq, tkv, a, grid, stream);
+}

@@ -349,6 +349,11 @@ int pxl_latent_prep(const void* proj, int64_t ld, int kv_off, int heads, int q_w
 int pxl_latent_attn(const void* q, const void* cache, const int* block_tables, const int* cu_q, const int* ctx_lens,
                     void* out, const float* sinks, int B, int max_q, int H, int L, int R, int page, int max_blocks,
                     int64_t num_blocks, float scale, int window, int is_f32, int* status, pxl_stream_t stream);
+// bf16 tensor-core form of pxl_latent_attn (L and R multiples of 8, L + R <= 576, scale > 0; total_q = rows of q).
+int pxl_latent_attn_tc_supported(int L, int R, int page, float scale);
+int pxl_latent_attn_tc(const void* q, const void* cache, const int* block_tables, const int* cu_q, const int* ctx_lens,
+                       void* out, const float* sinks, int B, int max_q, int total_q, int H, int L, int R, int page,
+                       int max_blocks, int64_t num_blocks, float scale, int window, int* status, pxl_stream_t stream);
 
 // ---- stage_exec.cu: all layers of a dense GQA stage for one step behind one call --------------
 // The descriptor structs are defined in stage_exec.cu (mirrored by parallax_b200/engine/native_stage.py).

@@ -45,7 +45,7 @@ def _nvcc() -> str:
 # Sources a model family needs when nothing has been built yet (the whole library otherwise): a fresh checkout
 # that only runs this family compiles these into a library of their own.
 FAMILY_SOURCES = {
-    "latent": ["elementwise", "gemm_simt", "gemm_tcgen05", "latent_attn", "residual", "sampler"],
+    "latent": ["elementwise", "gemm_simt", "gemm_tcgen05", "latent_attn", "latent_attn_tc", "residual", "sampler"],
 }
 
 

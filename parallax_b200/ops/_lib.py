@@ -123,6 +123,9 @@ _SIGS = {
                         c_int, c_float, c_int, _P, _P],
     "pxl_latent_attn": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64, c_float,
                         c_int, c_int, _P, _P],
+    "pxl_latent_attn_tc_supported": [c_int, c_int, c_int, c_float],
+    "pxl_latent_attn_tc": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64,
+                           c_float, c_int, _P, _P],
     "pxl_rmsnorm_strided": [_P, c_int64, _P, _P, c_int64, c_int, c_int, c_float, c_float, _P],
     "pxl_argmax": [_P, c_int, c_int64, c_int, c_int, _P, _P, _P, _P],
     "pxl_apply_penalties": [_P, c_int, c_int64, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P],

@@ -1064,6 +1064,15 @@ def latent_attn(q_cat, cache, block_tables, cu_q, ctx_lens, scale: float, latent
     if out is None:
         out = torch.empty((T, H, latent), dtype=q_cat.dtype, device=q_cat.device)
     assert out.is_contiguous() and out.shape == (T, H, latent)
+    if q_cat.dtype == torch.bfloat16 and not (q_cat.data_ptr() | out.data_ptr() | cache.data_ptr()) & 15 \
+            and _lib.lib().pxl_latent_attn_tc_supported(latent, D - latent, page, scale):
+        check(_lib.lib().pxl_latent_attn_tc(q_cat.data_ptr(), cache.data_ptr(), block_tables.data_ptr(), _ptr(cu_q),
+                                            ctx_lens.data_ptr(), out.data_ptr(), _ptr(sinks), B, max_q, T, H, latent,
+                                            D - latent, page, block_tables.shape[1], cache.shape[0], float(scale), window,
+                                            status_tensor(q_cat.device).data_ptr(), _stream(q_cat.device)),
+              "pxl_latent_attn_tc")
+        _count()
+        return out
     check(_lib.lib().pxl_latent_attn(q_cat.data_ptr(), cache.data_ptr(), block_tables.data_ptr(), _ptr(cu_q),
                                      ctx_lens.data_ptr(), out.data_ptr(), _ptr(sinks), B, max_q, H, latent, D - latent,
                                      page, block_tables.shape[1], cache.shape[0], float(scale), window,
