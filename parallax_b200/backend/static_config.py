@@ -52,6 +52,10 @@ def get_param_bytes_per_element(config: dict, model_name: str = "") -> float:
 
 
 def model_info_from_config(config: dict, model_name: str) -> ModelInfo:
+    if isinstance(config.get("layers"), list):      # layer-list config: no model-wide sizes in the file itself
+        from parallax_b200.models.config import config_from_hf
+
+        return ModelInfo.from_model_config(config_from_hf(config), model_name)
     experts = config.get("num_local_experts") or config.get("num_experts") or config.get("n_routed_experts")
     kvh = config.get("num_key_value_heads") or config.get("num_attention_groups") or 0
     pb = get_param_bytes_per_element(config, model_name)
