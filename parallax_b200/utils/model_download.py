@@ -68,7 +68,7 @@ def selective_model_download(model: str, start_layer: Optional[int] = None, end_
         return p
     root = _snapshot(model, METADATA_PATTERNS, local_files_only)
     cfg = json.loads((root / "config.json").read_text())
-    n = int((cfg.get("text_config") or cfg).get("num_hidden_layers", 0))
+    n = int((cfg.get("text_config") or cfg).get("num_hidden_layers", 0)) or len(cfg.get("layers") or [])
     index_file = root / "model.safetensors.index.json"
     if start_layer is None or end_layer is None or not index_file.exists():
         return _snapshot(model, METADATA_PATTERNS + ["*.safetensors"], local_files_only)
