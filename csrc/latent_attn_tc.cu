@@ -25,9 +25,9 @@ namespace {
 using namespace pxl;
 
 constexpr int kRows = 128;
-constexpr int kQChunk = kRows * 128;   // bytes of 64 columns of the query tile
+constexpr int kQChunk = kRows * 128;   // bytes of 64 columns of a full query tile
 constexpr int kMaxV = 4;               // 64-column latent chunks a CTA accumulates
-constexpr int kMaxStages = 4;
+constexpr int kMaxStages = 6;
 constexpr int kProducerWarp = 4, kMmaWarp = 5;
 constexpr int kThreads = 192;
 constexpr int kBarBytes = 256;
@@ -41,6 +41,7 @@ struct TcArgs {
   bf16* out;            // [T, H, L]
   const float* sinks;
   int H, L, D, page, max_blocks, window, stages, vsplit, head_blocks;
+  int q_rows;           // rows of the query tile kept in shared memory (decoding: the heads of one token)
   int64_t num_blocks;
   float scale_log2;
   int* status;
@@ -48,6 +49,19 @@ struct TcArgs {
 
 __device__ __forceinline__ uint64_t desc_mn_sw128(uint32_t addr) {  // B stored [key rows, 64 columns]: MN-major
   return umma_desc_k_sw128(addr);  // same fields: groups of 8 rows 1024 B apart, one 64-wide chunk addressed
+}
+__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {  // never suspends, unlike mbar_try_wait
+  uint32_t ok;
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t"
+      "}\n"
+      : "=r"(ok)
+      : "r"(bar), "r"(parity)
+      : "memory");
+  return ok != 0;
 }
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
@@ -87,10 +101,13 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const int nck = ceil_div(a.D, 64);
+  // The MMA always reads 128 rows. With fewer in shared memory the rest are whatever follows (other chunks, the
+  // key ring): those rows' scores are masked and their outputs never stored.
+  const uint32_t q_chunk = a.q_rows * 128;
   const uint32_t sm_q = smem_u32(smem);
-  const uint32_t sm_kv = sm_q + nck * kQChunk;
+  const uint32_t sm_kv = sm_q + nck * q_chunk;
   const uint32_t stage_bytes = nck * kKvChunk;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + nck * kQChunk + a.stages * stage_bytes);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + nck * q_chunk + a.stages * stage_bytes);
   // q_full | kv_full [kMaxStages] | kv_empty [kMaxStages] | s_full [2] | p_ready [2] | o_full [2]
   const uint32_t q_full = smem_u32(bars), kv_full = q_full + 8, kv_empty = kv_full + 8 * kMaxStages,
                  s_full = kv_empty + 8 * kMaxStages, p_ready = s_full + 16, o_full = p_ready + 16;
@@ -157,9 +174,9 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     // Lane p looks up the block of piece p of the tile and issues its boxes: the block-table reads of a tile are
     // in flight together and come before the wait for the stage.
     if (lane == 0) {
-      mbar_arrive_expect_tx(q_full, nck * kQChunk);
+      mbar_arrive_expect_tx(q_full, nck * q_chunk);
       for (int c = 0; c < nck; ++c)
-        tma_load_2d(sm_q + c * kQChunk, &tm_q, q_full, c * 64, static_cast<int>(row0));
+        tma_load_2d(sm_q + c * q_chunk, &tm_q, q_full, c * 64, static_cast<int>(row0));
     }
     const int* bt = a.block_tables + static_cast<int64_t>(b) * a.max_blocks;
     const int box = a.page < NK ? a.page : NK;
@@ -201,31 +218,13 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         const uint32_t d_tmem = tm_s + (it & 1) * NK;
         for (int ks = 0; ks < ksteps; ++ks) {
           const uint32_t in = (ks & 3) * 32;
-          tc_mma_f16(d_tmem, umma_desc_k_sw128(sm_q + (ks >> 2) * kQChunk + in),
+          tc_mma_f16(d_tmem, umma_desc_k_sw128(sm_q + (ks >> 2) * q_chunk + in),
                      umma_desc_k_sw128(k_addr + (ks >> 2) * kKvChunk + in), kIdescS, ks > 0 ? 1u : 0u);
         }
         tc_commit(s_full + 8 * (it & 1));
       };
-      bool ok = mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
-      ok = ok && mbar_wait_bounded(kv_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
-      if (ok) {
-        tc_fence_after_sync();
-        issue_s(0);
-      }
-      for (int it = 0; ok && it < n_tiles; ++it) {
-        const int stage = it % a.stages;
-        if (it + 1 < n_tiles) {
-          // scores of the next tile while the softmax warps work on this one
-          ok = mbar_wait_bounded(kv_full + 8 * ((it + 1) % a.stages), ((it + 1) / a.stages) & 1, abort_flag, a.status,
-                                 PXL_DEV_TIMEOUT_FULL);
-          if (!ok) break;
-          tc_fence_after_sync();
-          issue_s(it + 1);
-        }
-        ok = mbar_wait_bounded(p_ready + 8 * (it & 1), (it >> 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_TMEM_EMPTY);
-        if (!ok) break;
-        tc_fence_after_sync();
-        const uint32_t v_addr = sm_kv + stage * stage_bytes + v0 * kKvChunk;
+      auto issue_pv = [&](int it) {  // O += P(it) V(it)
+        const uint32_t v_addr = sm_kv + (it % a.stages) * stage_bytes + v0 * kKvChunk;
         for (int c = 0; c < nv; ++c) {
 #pragma unroll
           for (int ks = 0; ks < NK / 16; ++ks)
@@ -233,7 +232,41 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
                           kIdescPV, (it > 0 || ks > 0) ? 1u : 0u);
         }
         tc_commit(o_full + 8 * (it & 1));
-        tc_commit(kv_empty + 8 * stage);  // the rows of this stage are no longer read
+        tc_commit(kv_empty + 8 * (it % a.stages));  // the rows of this stage are no longer read
+      };
+      // Whichever is ready goes next: the scores of a tile whose rows have landed (at most one tile ahead of the
+      // products: two score buffers), or the product of a tile whose probabilities are written. A load in flight
+      // never holds back a product, which is what frees the ring for the load after it.
+      bool ok = mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
+      int next_s = 0, next_pv = 0;
+      uint64_t since = 0;
+      uint32_t spins = 0;
+      while (ok && next_pv < n_tiles) {
+        bool moved = false;
+        if (next_s < n_tiles && next_s <= next_pv + 1 &&
+            mbar_test(kv_full + 8 * (next_s % a.stages), (next_s / a.stages) & 1)) {
+          tc_fence_after_sync();
+          issue_s(next_s++);
+          moved = true;
+        }
+        if (next_pv < next_s && mbar_test(p_ready + 8 * (next_pv & 1), (next_pv >> 1) & 1)) {
+          tc_fence_after_sync();
+          issue_pv(next_pv++);
+          moved = true;
+        }
+        if (moved) {
+          spins = 0;
+          since = 0;
+        } else if ((++spins & 0x3ffu) == 0) {
+          const uint64_t now = global_timer_ns();
+          if (since == 0) since = now;
+          if (*abort_flag) ok = false;
+          if (now - since > kWaitLimitNs) {
+            *abort_flag = 1;
+            if (a.status) atomicCAS(a.status, 0, PXL_DEV_TIMEOUT_TMEM_EMPTY);
+            ok = false;
+          }
+        }
       }
     }
   } else {
@@ -362,15 +395,19 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   if (warp == kMmaWarp) tmem_dealloc(tm_o, tmem_cols);
 }
 
-int smem_bytes(int nck, int nk, int stages) { return 1024 + nck * kQChunk + stages * nck * nk * 128 + kBarBytes; }
+int smem_bytes(int nck, int q_rows, int nk, int stages) {
+  const int tiles = nck * q_rows * 128 + stages * nck * nk * 128;
+  const int reach = (nck - 1) * q_rows * 128 + kQChunk;  // what the MMA reads of the query tile
+  return 1024 + (tiles > reach ? tiles : reach) + kBarBytes;
+}
 
 // keys per tile and ring stages for a row width; false when two stages do not fit
-bool plan_tiles(int D, int page, int* nk, int* stages) {
+bool plan_tiles(int D, int q_rows, int page, int* nk, int* stages) {
   const int nck = ceil_div(D, 64);
   for (const int cand : {64, 32}) {
     if (page % cand != 0 && cand % page != 0) continue;
     int s = kMaxStages;
-    while (s >= 2 && smem_bytes(nck, cand, s) > kMaxSmem) --s;
+    while (s >= 2 && smem_bytes(nck, q_rows, cand, s) > kMaxSmem) --s;
     if (s >= 2) {
       *nk = cand;
       *stages = s;
@@ -389,7 +426,7 @@ int launch_tc(const CUtensorMap& tq, const CUtensorMap& tkv, const TcArgs& a, di
       return PXL_ERR_CUDA;
     configured[dev] = true;
   }
-  pxl_host::launch(latent_attn_tc_kernel<NK>, grid, dim3(kThreads), smem_bytes(ceil_div(a.D, 64), NK, a.stages), stream, tq,
+  pxl_host::launch(latent_attn_tc_kernel<NK>, grid, dim3(kThreads), smem_bytes(ceil_div(a.D, 64), a.q_rows, NK, a.stages), stream, tq,
                    tkv, a);
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }
@@ -398,7 +435,7 @@ int launch_tc(const CUtensorMap& tq, const CUtensorMap& tkv, const TcArgs& a, di
 PXL_EXPORT int pxl_latent_attn_tc_supported(int L, int R, int page, float scale) {
   int nk, stages;
   return L > 0 && R >= 0 && L % 8 == 0 && R % 8 == 0 && page > 0 && page % 8 == 0 && scale > 0.f &&
-         plan_tiles(L + R, page, &nk, &stages);
+         plan_tiles(L + R, kRows, page, &nk, &stages);
 }
 
 PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* block_tables, const int* cu_q,
@@ -412,7 +449,10 @@ PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* b
   if (num_blocks * page >= (1ll << 31) || static_cast<int64_t>(total_q) * H >= (1ll << 31)) return PXL_ERR_TOO_LARGE;
   TcArgs a{};
   int nk = 0;
-  plan_tiles(L + R, page, &nk, &a.stages);
+  // short queries (decoding) leave most of the tile's rows empty: keep only the others, and more keys in flight
+  const int rows = max_q * (H < kRows ? H : kRows);
+  a.q_rows = rows >= kRows ? kRows : pxl::ceil_div(rows, 8) * 8;
+  plan_tiles(L + R, a.q_rows, page, &nk, &a.stages);
   a.block_tables = block_tables;
   a.cu_q = cu_q;
   a.ctx_lens = ctx_lens;
@@ -424,8 +464,8 @@ PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* b
   a.scale_log2 = scale * kLog2eF;
   a.status = status;
   CUtensorMap tq, tkv;
-  if (!pxl_host::make_tmap_2d(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, q, static_cast<uint64_t>(total_q) * H, a.D, a.D, kRows,
-                              64) ||
+  if (!pxl_host::make_tmap_2d(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, q, static_cast<uint64_t>(total_q) * H, a.D, a.D,
+                              a.q_rows, 64) ||
       !pxl_host::make_tmap_2d(&tkv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cache, static_cast<uint64_t>(num_blocks) * page, a.D,
                               a.D, page < nk ? page : nk, 64))
     return PXL_ERR_TENSORMAP;

@@ -28,7 +28,7 @@ MIXED = oracle.random_config([L(), L(heads=4, dim=8, rot_dim=16, vdim=8, kv_rank
 # sizes that no vector or tile width divides
 ODD = oracle.random_config([L(heads=3, dim=7, rot_dim=6, vdim=5, kv_rank=19, window=5, ff=33),
                             L(heads=2, dim=5, rot_dim=2, vdim=11, kv_rank=10, window=33, ff=14)],
-                           vocab=37, width=30, bigram=(11, 1, 1), mult=1.0, emb_scale=1.0, eps=1e-3)
+                           vocab=37, width=30, bigram=(11, 1, 1), mult=0.5, emb_scale=1.0, eps=1e-3)
 # equal sizes everywhere, no bigram table, a window of one (a token sees itself only) and one that never ends
 EQUAL = oracle.random_config([L(heads=4, dim=32, rot_dim=32, vdim=32, kv_rank=32, window=1, ff=64),
                               L(heads=4, dim=32, rot_dim=32, vdim=32, kv_rank=32, window=1000, ff=64)],

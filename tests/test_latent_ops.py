@@ -70,8 +70,8 @@ def test_residual_norm(target, width):
         xg = x.to(dev).clone()
         low = ops.residual_norm(xg, y.to(dev), w.to(dev), 1e-4, 0.7, kind)
         want = x.double() + 0.7 * norm(y.double(), w, 1e-4)
-        assert rel(xg, want) < 1e-5 and low.dtype == dt
-        assert rel(low, want) < tol(dt, 1e-5, 4e-3)
+        assert rel(xg, want) < 3e-5 and low.dtype == dt
+        assert rel(low, want) < tol(dt, 3e-5, 4e-3)
 
 
 @pytest.mark.parametrize("target", TARGETS)
