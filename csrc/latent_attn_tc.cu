@@ -3,20 +3,24 @@
 //
 // A query row is a (token, head) pair: q [T, H, L + R] is a matrix of T * H rows that all read the same cached
 // rows, so a CTA takes 128 consecutive rows of one sequence - 128 / H tokens (one token and a block of 128 heads
-// when H > 128) - and walks the keys that its first and last token may see in tiles of NK.
+// when H > 128) - and walks the keys that its first and last token may see in tiles of 64.
 //
 //   warp 4    : TMA producer. The query tile once (chunks of 64 columns, 128-byte swizzle), then tiles of cache
-//               rows (page boxes) through a ring. A cache row is key AND value: each tile is loaded once.
-//   warp 5    : MMA issuer. S = Q K^T over L + R (both operands K-major) into one of two TMEM score buffers, so
-//               the scores of tile i + 1 are computed while the softmax warps work on tile i; then O += P V, P
-//               from tensor memory, V taken MN-major from the same shared-memory tile (its first L columns).
+//               rows (page boxes), chunk by chunk. A cache row is key AND value and is loaded once: the chunks this
+//               CTA accumulates as values go to whole-tile V buffers, all others - needed for the scores only - to a
+//               ring of chunk slots that are free again as soon as the scores have read them.
+//   warp 5    : MMA issuer. S = Q K^T over L + R (both operands K-major) into one of two TMEM score buffers, chunk
+//               by chunk as the loads land, so the scores of tile i + 1 are computed while the softmax warps work
+//               on tile i; then O += P V, P from tensor memory, V taken MN-major from the V buffer, all of its
+//               columns by one instruction per 16 keys (narrow instructions cost almost as much as wide ones).
 //   warps 0-3 : softmax, one row per thread (its TMEM lane): mask (causal, window), running reference maximum
 //               that only moves when a row grew by more than 2^8 (then the TMEM rows of O are rescaled), P
 //               back to tensor memory as bf16 (two buffers), row sums in fp32; at the end the sink and the
 //               division.
 //
 // O takes 64 TMEM columns per 64 latent columns and scores need room beside it, so a CTA accumulates at most 256
-// latent columns; wider latents run as several CTAs per query tile that repeat the scores (L = 512: two).
+// latent columns; wider latents run as several CTAs per query tile that repeat the scores (L = 512: two). The host
+// sizes the ring and the number of V buffers to what the query tile leaves of shared memory.
 // Every wait is bounded; on expiry the kernel records a status code, all roles unwind, TMEM is freed.
 #include "common.cuh"
 #include "pxl_api.h"
@@ -27,10 +31,12 @@ using namespace pxl;
 constexpr int kRows = 128;
 constexpr int kQChunk = kRows * 128;   // bytes of 64 columns of a full query tile
 constexpr int kMaxV = 4;               // 64-column latent chunks a CTA accumulates
-constexpr int kMaxStages = 6;
+constexpr int NK = 64;                 // keys per tile
+constexpr int kKvChunk = NK * 128;     // bytes of 64 columns of a key tile
+constexpr int kMaxSlots = 16, kMaxVBufs = 3;
 constexpr int kProducerWarp = 4, kMmaWarp = 5;
 constexpr int kThreads = 192;
-constexpr int kBarBytes = 256;
+constexpr int kBarBytes = 512;
 constexpr int kMaxSmem = 227 * 1024;
 constexpr float kLog2eF = 1.4426950408889634f;
 
@@ -40,15 +46,17 @@ struct TcArgs {
   const int* ctx_lens;
   bf16* out;            // [T, H, L]
   const float* sinks;
-  int H, L, D, page, max_blocks, window, stages, vsplit, head_blocks;
+  int H, L, D, page, max_blocks, window, vsplit, head_blocks;
+  int k_slots, v_bufs;  // ring slots for score-only chunks, buffers for value chunks
   int q_rows;           // rows of the query tile kept in shared memory (decoding: the heads of one token)
   int64_t num_blocks;
   float scale_log2;
   int* status;
 };
 
-__device__ __forceinline__ uint64_t desc_mn_sw128(uint32_t addr) {  // B stored [key rows, 64 columns]: MN-major
-  return umma_desc_k_sw128(addr);  // same fields: groups of 8 rows 1024 B apart, one 64-wide chunk addressed
+// B stored as 64-column chunks of [key rows, 64]: MN-major, 8-row groups 1024 B apart, chunks kKvChunk apart
+__device__ __forceinline__ uint64_t desc_mn_sw128(uint32_t addr) {
+  return (umma_desc_k_sw128(addr) & ~(0x3fffull << 16)) | (static_cast<uint64_t>(kKvChunk >> 4) << 16);
 }
 __device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {  // never suspends, unlike mbar_try_wait
   uint32_t ok;
@@ -91,13 +99,10 @@ __device__ __forceinline__ void tmem_st_32x32b_x16(uint32_t taddr, const uint32_
       : "memory");
 }
 
-template <int NK>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv,
                       const TcArgs a) {
-  constexpr int kKvChunk = NK * 128;  // bytes of 64 columns of a key tile
   constexpr uint32_t kIdescS = umma_idesc(kRows, NK, 1, 1);
-  constexpr uint32_t kIdescPV = umma_idesc(kRows, 64, 1, 1) | (1u << 16);  // B (V) is MN-major
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const int nck = ceil_div(a.D, 64);
@@ -105,20 +110,27 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   // key ring): those rows' scores are masked and their outputs never stored.
   const uint32_t q_chunk = a.q_rows * 128;
   const uint32_t sm_q = smem_u32(smem);
-  const uint32_t sm_kv = sm_q + nck * q_chunk;
-  const uint32_t stage_bytes = nck * kKvChunk;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + nck * q_chunk + a.stages * stage_bytes);
-  // q_full | kv_full [kMaxStages] | kv_empty [kMaxStages] | s_full [2] | p_ready [2] | o_full [2]
-  const uint32_t q_full = smem_u32(bars), kv_full = q_full + 8, kv_empty = kv_full + 8 * kMaxStages,
-                 s_full = kv_empty + 8 * kMaxStages, p_ready = s_full + 16, o_full = p_ready + 16;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * kMaxStages + 6);
+  // latent chunks of this CTA
+  const int vs = blockIdx.x % a.vsplit, tile = blockIdx.x / a.vsplit;
+  const int ncv = ceil_div(a.L, 64), per = ceil_div(ncv, a.vsplit);
+  const int v0 = vs * per;
+  const int nv = ncv - v0 < per ? ncv - v0 : per;
+  const int nkc = nck - nv;                                   // chunks that only the scores read
+  auto k_chunk = [&](int j) { return j < v0 ? j : j + nv; };  // their column chunks
+  const uint32_t sm_v = sm_q + nck * q_chunk;
+  const uint32_t sm_k = sm_v + a.v_bufs * per * kKvChunk;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + nck * q_chunk + (a.v_bufs * per + a.k_slots) * kKvChunk);
+  // q_full | v_full, v_empty [kMaxVBufs] | k_full, k_empty [kMaxSlots] | s_full, p_ready, o_full [2]
+  const uint32_t q_full = smem_u32(bars), v_full = q_full + 8, v_empty = v_full + 8 * kMaxVBufs,
+                 k_full = v_empty + 8 * kMaxVBufs, k_empty = k_full + 8 * kMaxSlots, s_full = k_empty + 8 * kMaxSlots,
+                 p_ready = s_full + 16, o_full = p_ready + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * kMaxVBufs + 2 * kMaxSlots + 6);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   pdl_wait();
   pdl_launch_dependents();
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = blockIdx.z, hb = blockIdx.y;
-  const int vs = blockIdx.x % a.vsplit, tile = blockIdx.x / a.vsplit;
   const int t0 = a.cu_q ? a.cu_q[b] : b;
   const int len = a.cu_q ? a.cu_q[b + 1] - t0 : 1;
   const int ctx = a.ctx_lens[b];
@@ -135,17 +147,17 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   const int lo = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;
   const int t_begin = lo / NK;
   const int n_tiles = ceil_div(hi, NK) - t_begin;
-  // latent chunks of this CTA
-  const int ncv = ceil_div(a.L, 64), per = ceil_div(ncv, a.vsplit);
-  const int v0 = vs * per;
-  const int nv = ncv - v0 < per ? ncv - v0 : per;
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
     mbar_init(q_full, 1);
-    for (int s = 0; s < a.stages; ++s) {
-      mbar_init(kv_full + 8 * s, 1);
-      mbar_init(kv_empty + 8 * s, 1);
+    for (int s = 0; s < a.v_bufs; ++s) {
+      mbar_init(v_full + 8 * s, 1);
+      mbar_init(v_empty + 8 * s, 1);
+    }
+    for (int s = 0; s < a.k_slots; ++s) {
+      mbar_init(k_full + 8 * s, 1);
+      mbar_init(k_empty + 8 * s, 1);
     }
     for (int s = 0; s < 2; ++s) {
       mbar_init(s_full + 8 * s, 1);
@@ -171,8 +183,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 
   if (warp == kProducerWarp) {
     // ------------------------------------------------------------------ TMA producer
-    // Lane p looks up the block of piece p of the tile and issues its boxes: the block-table reads of a tile are
-    // in flight together and come before the wait for the stage.
+    // Lane p looks up the block of piece p of the tile and issues that piece's boxes.
     if (lane == 0) {
       mbar_arrive_expect_tx(q_full, nck * q_chunk);
       for (int c = 0; c < nck; ++c)
@@ -181,9 +192,20 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const int* bt = a.block_tables + static_cast<int64_t>(b) * a.max_blocks;
     const int box = a.page < NK ? a.page : NK;
     const int pieces = NK / box;
-    for (int it = 0; it < n_tiles; ++it) {
-      const int stage = it % a.stages;
-      int64_t row = 0;
+    bool ok = true;
+    // wait for the buffer behind `bar_empty` to be free again (its `use`-th use), announce `bytes`
+    auto acquire = [&](uint32_t bar_empty, uint32_t bar_full, int use, uint32_t bytes) {
+      int okf = 1;
+      if (lane == 0) {
+        if (use > 0)
+          okf = mbar_wait_bounded(bar_empty, (use - 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_EMPTY) ? 1 : 0;
+        if (okf) mbar_arrive_expect_tx(bar_full, bytes);
+      }
+      return __shfl_sync(0xffffffffu, okf, 0) != 0;
+    };
+    int slot = 0, slot_use = 0;
+    for (int it = 0; ok && it < n_tiles; ++it) {
+      int row = 0;
       if (lane < pieces) {
         int key = (t_begin + it) * NK + lane * box;
         if (key >= ctx) key = (ctx - 1) / box * box;  // beyond the context: re-read its last piece (masked)
@@ -193,66 +215,84 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
           if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_BLOCK_PREFILL);
           blk = 0;
         }
-        row = blk * a.page + key % a.page;
+        row = static_cast<int>(blk * a.page + key % a.page);
       }
-      int okf = 1;
-      if (it >= a.stages && lane == 0)
-        okf = mbar_wait_bounded(kv_empty + 8 * stage, ((it / a.stages) - 1) & 1, abort_flag, a.status,
-                                PXL_DEV_TIMEOUT_EMPTY) ? 1 : 0;
-      okf = __shfl_sync(0xffffffffu, okf, 0);
-      if (!okf) break;
-      const uint32_t bar = kv_full + 8 * stage;
-      if (lane == 0) mbar_arrive_expect_tx(bar, stage_bytes);
-      __syncwarp();
-      if (lane < pieces) {
-        const uint32_t dst = sm_kv + stage * stage_bytes + lane * box * 128;
-        for (int c = 0; c < nck; ++c) tma_load_2d(dst + c * kKvChunk, &tm_kv, bar, c * 64, static_cast<int>(row));
+      const uint32_t piece_off = lane * box * 128;
+      for (int j = 0; ok && j < nkc; ++j) {
+        ok = acquire(k_empty + 8 * slot, k_full + 8 * slot, slot_use, kKvChunk);
+        if (ok && lane < pieces)
+          tma_load_2d(sm_k + slot * kKvChunk + piece_off, &tm_kv, k_full + 8 * slot, k_chunk(j) * 64, row);
+        if (++slot == a.k_slots) {
+          slot = 0;
+          ++slot_use;
+        }
+      }
+      if (!ok) break;
+      const int vb = it % a.v_bufs;
+      ok = acquire(v_empty + 8 * vb, v_full + 8 * vb, it / a.v_bufs, nv * kKvChunk);
+      if (ok && lane < pieces) {
+        const uint32_t dst = sm_v + vb * per * kKvChunk + piece_off;
+        for (int c = 0; c < nv; ++c) tma_load_2d(dst + c * kKvChunk, &tm_kv, v_full + 8 * vb, (v0 + c) * 64, row);
       }
     }
   } else if (warp == kMmaWarp) {
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
-      const int ksteps = ceil_div(a.D, 16);
-      auto issue_s = [&](int it) {  // S[it % 2] = Q K(it)^T
-        const uint32_t k_addr = sm_kv + (it % a.stages) * stage_bytes;
-        const uint32_t d_tmem = tm_s + (it & 1) * NK;
-        for (int ks = 0; ks < ksteps; ++ks) {
-          const uint32_t in = (ks & 3) * 32;
-          tc_mma_f16(d_tmem, umma_desc_k_sw128(sm_q + (ks >> 2) * q_chunk + in),
-                     umma_desc_k_sw128(k_addr + (ks >> 2) * kKvChunk + in), kIdescS, ks > 0 ? 1u : 0u);
-        }
-        tc_commit(s_full + 8 * (it & 1));
+      const uint32_t idesc_pv = umma_idesc(kRows, 64 * nv, 1, 1) | (1u << 16);  // B (V) is MN-major
+      const uint64_t dq0 = umma_desc_k_sw128(sm_q);
+      // descriptors advance by 16-byte units: 2 per k-step inside a chunk (columns past D are zeros on both sides)
+      auto s_chunk = [&](int it, int col_chunk, uint32_t rows_addr, bool first) {  // S[it % 2] (+)= Q[:, chunk] K[:, chunk]^T
+        const uint64_t dq = dq0 + static_cast<uint64_t>(col_chunk) * (q_chunk >> 4), dk = umma_desc_k_sw128(rows_addr);
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks)
+          tc_mma_f16(tm_s + (it & 1) * NK, dq + 2 * ks, dk + 2 * ks, kIdescS, first && ks == 0 ? 0u : 1u);
       };
       auto issue_pv = [&](int it) {  // O += P(it) V(it)
-        const uint32_t v_addr = sm_kv + (it % a.stages) * stage_bytes + v0 * kKvChunk;
-        for (int c = 0; c < nv; ++c) {
+        const int vb = it % a.v_bufs;
+        const uint64_t dv = desc_mn_sw128(sm_v + vb * per * kKvChunk);
 #pragma unroll
-          for (int ks = 0; ks < NK / 16; ++ks)
-            tc_mma_f16_ts(tm_o + c * 64, tm_p + (it & 1) * (NK / 2) + ks * 8, desc_mn_sw128(v_addr + c * kKvChunk + ks * 2048),
-                          kIdescPV, (it > 0 || ks > 0) ? 1u : 0u);
-        }
+        for (int ks = 0; ks < NK / 16; ++ks)
+          tc_mma_f16_ts(tm_o, tm_p + (it & 1) * (NK / 2) + ks * 8, dv + 128 * ks, idesc_pv, (it > 0 || ks > 0) ? 1u : 0u);
         tc_commit(o_full + 8 * (it & 1));
-        tc_commit(kv_empty + 8 * (it % a.stages));  // the rows of this stage are no longer read
+        tc_commit(v_empty + 8 * vb);
       };
-      // Whichever is ready goes next: the scores of a tile whose rows have landed (at most one tile ahead of the
-      // products: two score buffers), or the product of a tile whose probabilities are written. A load in flight
-      // never holds back a product, which is what frees the ring for the load after it.
+      // Whichever is ready goes next: the product of a tile whose probabilities are written, or the next chunk of the
+      // scores (at most one tile ahead of the products: two score buffers). A load in flight never holds back a
+      // product, which is what frees the buffers for the loads after it.
       bool ok = mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
-      int next_s = 0, next_pv = 0;
+      int next_s = 0, next_pv = 0;   // tiles whose scores / products come next
+      int j = 0, slot = 0, slot_phase = 0;  // score-only chunk of tile next_s and its ring slot
       uint64_t since = 0;
       uint32_t spins = 0;
       while (ok && next_pv < n_tiles) {
         bool moved = false;
-        if (next_s < n_tiles && next_s <= next_pv + 1 &&
-            mbar_test(kv_full + 8 * (next_s % a.stages), (next_s / a.stages) & 1)) {
-          tc_fence_after_sync();
-          issue_s(next_s++);
-          moved = true;
-        }
         if (next_pv < next_s && mbar_test(p_ready + 8 * (next_pv & 1), (next_pv >> 1) & 1)) {
           tc_fence_after_sync();
           issue_pv(next_pv++);
           moved = true;
+        }
+        if (next_s < n_tiles && next_s <= next_pv + 1) {
+          if (j < nkc) {
+            if (mbar_test(k_full + 8 * slot, slot_phase)) {
+              tc_fence_after_sync();
+              s_chunk(next_s, k_chunk(j), sm_k + slot * kKvChunk, j == 0);
+              tc_commit(k_empty + 8 * slot);  // free again once these have read it
+              ++j;
+              if (++slot == a.k_slots) {
+                slot = 0;
+                slot_phase ^= 1;
+              }
+              moved = true;
+            }
+          } else if (mbar_test(v_full + 8 * (next_s % a.v_bufs), (next_s / a.v_bufs) & 1)) {
+            tc_fence_after_sync();
+            const uint32_t v = sm_v + (next_s % a.v_bufs) * per * kKvChunk;
+            for (int c = 0; c < nv; ++c) s_chunk(next_s, v0 + c, v + c * kKvChunk, nkc == 0 && c == 0);
+            tc_commit(s_full + 8 * (next_s & 1));
+            ++next_s;
+            j = 0;
+            moved = true;
+          }
         }
         if (moved) {
           spins = 0;
@@ -395,47 +435,39 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   if (warp == kMmaWarp) tmem_dealloc(tm_o, tmem_cols);
 }
 
-int smem_bytes(int nck, int q_rows, int nk, int stages) {
-  const int tiles = nck * q_rows * 128 + stages * nck * nk * 128;
-  const int reach = (nck - 1) * q_rows * 128 + kQChunk;  // what the MMA reads of the query tile
-  return 1024 + (tiles > reach ? tiles : reach) + kBarBytes;
-}
+struct TilePlan {
+  int k_slots, v_bufs, smem;
+};
 
-// keys per tile and ring stages for a row width; false when two stages do not fit
-bool plan_tiles(int D, int q_rows, int page, int* nk, int* stages) {
-  const int nck = ceil_div(D, 64);
-  for (const int cand : {64, 32}) {
-    if (page % cand != 0 && cand % page != 0) continue;
-    int s = kMaxStages;
-    while (s >= 2 && smem_bytes(nck, q_rows, cand, s) > kMaxSmem) --s;
-    if (s >= 2) {
-      *nk = cand;
-      *stages = s;
-      return true;
+// Ring slots and V buffers beside a query tile of q_rows rows; false when the sizes do not fit.
+bool plan_tiles(int L, int D, int q_rows, int page, TilePlan* p) {
+  if (page % 8 != 0 || (page % NK != 0 && NK % page != 0)) return false;
+  const int nck = ceil_div(D, 64), ncv = ceil_div(L, 64);
+  const int vsplit = ceil_div(ncv, kMaxV), per = ceil_div(ncv, vsplit);
+  const int nkc = nck - (ncv - (vsplit - 1) * per);  // score-only chunks of the CTA that has most of them
+  const int q_bytes = nck * q_rows * 128;
+  const int slots = (kMaxSmem - 1024 - kBarBytes - q_bytes) / kKvChunk;
+  p->k_slots = 0;
+  for (int vb = kMaxVBufs; vb >= 1; --vb) {
+    const int ks = slots - vb * per;
+    if (ks >= (vb > 1 ? nkc + 1 : (nkc > 0 ? 1 : 0))) {
+      p->v_bufs = vb;
+      p->k_slots = ks < kMaxSlots ? ks : kMaxSlots;
+      if (p->k_slots < 1) p->k_slots = 1;
+      const int tiles = q_bytes + (vb * per + p->k_slots) * kKvChunk;
+      const int reach = (nck - 1) * q_rows * 128 + kQChunk;  // what the MMA reads of the query tile
+      p->smem = 1024 + (tiles > reach ? tiles : reach) + kBarBytes;
+      return p->smem <= kMaxSmem;
     }
   }
   return false;
 }
-
-template <int NK>
-int launch_tc(const CUtensorMap& tq, const CUtensorMap& tkv, const TcArgs& a, dim3 grid, cudaStream_t stream) {
-  static bool configured[64] = {false};
-  const int dev = pxl_host::current_device_slot();
-  if (!configured[dev]) {
-    if (cudaFuncSetAttribute(latent_attn_tc_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem) != cudaSuccess)
-      return PXL_ERR_CUDA;
-    configured[dev] = true;
-  }
-  pxl_host::launch(latent_attn_tc_kernel<NK>, grid, dim3(kThreads), smem_bytes(ceil_div(a.D, 64), a.q_rows, NK, a.stages), stream, tq,
-                   tkv, a);
-  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
-}
 }  // namespace
 
 PXL_EXPORT int pxl_latent_attn_tc_supported(int L, int R, int page, float scale) {
-  int nk, stages;
+  TilePlan plan;
   return L > 0 && R >= 0 && L % 8 == 0 && R % 8 == 0 && page > 0 && page % 8 == 0 && scale > 0.f &&
-         plan_tiles(L + R, kRows, page, &nk, &stages);
+         plan_tiles(L, L + R, kRows, page, &plan);
 }
 
 PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* block_tables, const int* cu_q,
@@ -448,11 +480,13 @@ PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* b
     return PXL_ERR_INVALID_ARG;
   if (num_blocks * page >= (1ll << 31) || static_cast<int64_t>(total_q) * H >= (1ll << 31)) return PXL_ERR_TOO_LARGE;
   TcArgs a{};
-  int nk = 0;
+  TilePlan plan;
   // short queries (decoding) leave most of the tile's rows empty: keep only the others, and more keys in flight
   const int rows = max_q * (H < kRows ? H : kRows);
   a.q_rows = rows >= kRows ? kRows : pxl::ceil_div(rows, 8) * 8;
-  plan_tiles(L + R, a.q_rows, page, &nk, &a.stages);
+  if (!plan_tiles(L, L + R, a.q_rows, page, &plan)) return PXL_ERR_INVALID_ARG;
+  a.k_slots = plan.k_slots;
+  a.v_bufs = plan.v_bufs;
   a.block_tables = block_tables;
   a.cu_q = cu_q;
   a.ctx_lens = ctx_lens;
@@ -467,9 +501,17 @@ PXL_EXPORT int pxl_latent_attn_tc(const void* q, const void* cache, const int* b
   if (!pxl_host::make_tmap_2d(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, q, static_cast<uint64_t>(total_q) * H, a.D, a.D,
                               a.q_rows, 64) ||
       !pxl_host::make_tmap_2d(&tkv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cache, static_cast<uint64_t>(num_blocks) * page, a.D,
-                              a.D, page < nk ? page : nk, 64))
+                              a.D, page < NK ? page : NK, 64))
     return PXL_ERR_TENSORMAP;
   const int tpt = H <= kRows ? kRows / H : 1;
   const dim3 grid(pxl::ceil_div(max_q, tpt) * a.vsplit, a.head_blocks, B);
-  return nk == 64 ? launch_tc<64>(tq, tkv, a, grid, stream) : launch_tc<32>(tq, tkv, a, grid, stream);
+  static bool configured[64] = {false};
+  const int dev = pxl_host::current_device_slot();
+  if (!configured[dev]) {
+    if (cudaFuncSetAttribute(latent_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem) != cudaSuccess)
+      return PXL_ERR_CUDA;
+    configured[dev] = true;
+  }
+  pxl_host::launch(latent_attn_tc_kernel, grid, dim3(kThreads), plan.smem, stream, tq, tkv, a);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }
