@@ -76,17 +76,57 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// D[tmem] (+)= A[tmem] * B[smem desc]; A holds two bf16 per 32-bit column, one row per lane
-__device__ __forceinline__ void tc_mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc,
-                                              uint32_t accumulate) {
+// The MMA warp runs its loop with all lanes, so that addresses and descriptors stay in uniform registers (a loop in one
+// lane moves them there before every instruction and issues at half the rate); `leader` is non-zero in the lane
+// that issues.
+__device__ __forceinline__ uint32_t elect_leader() {
+  uint32_t r;
   asm volatile(
       "{\n\t"
       ".reg .pred p;\n\t"
+      "elect.sync _|p, 0xffffffff;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t"
+      "}\n"
+      : "=r"(r));
+  return r;
+}
+// D[tmem] (+)= A[smem desc] * B[smem desc]
+__device__ __forceinline__ void mma_ss(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate,
+                                       uint32_t leader) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p, q;\n\t"
       "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "setp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
       "}\n"
       :
-      : "r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
+      : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(leader)
+      : "memory");
+}
+// D[tmem] (+)= A[tmem] * B[smem desc]; A holds two bf16 per 32-bit column, one row per lane
+__device__ __forceinline__ void mma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate,
+                                       uint32_t leader) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p, q;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "setp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n"
+      :
+      : "r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(leader)
+      : "memory");
+}
+__device__ __forceinline__ void commit(uint32_t bar, uint32_t leader) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred q;\n\t"
+      "setp.ne.b32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t"
+      "}\n"
+      :
+      : "r"(bar), "r"(leader)
       : "memory");
 }
 __device__ __forceinline__ void tmem_st_32x32b_x16(uint32_t taddr, const uint32_t (&r)[16]) {
@@ -129,7 +169,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   pdl_wait();
   pdl_launch_dependents();
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
   const int b = blockIdx.z, hb = blockIdx.y;
   const int t0 = a.cu_q ? a.cu_q[b] : b;
   const int len = a.cu_q ? a.cu_q[b + 1] - t0 : 1;
@@ -146,7 +186,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   const int hi = pos0 + ntok;  // keys [lo, hi) are visible to some row
   const int lo = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;
   const int t_begin = lo / NK;
-  const int n_tiles = ceil_div(hi, NK) - t_begin;
+  const int n_tiles = __shfl_sync(0xffffffffu, ceil_div(hi, NK) - t_begin, 0);
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
@@ -237,46 +277,48 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     }
   } else if (warp == kMmaWarp) {
     // ------------------------------------------------------------------ MMA issuer
-    if (lane == 0) {
+    {
+      const uint32_t leader = elect_leader();
       const uint32_t idesc_pv = umma_idesc(kRows, 64 * nv, 1, 1) | (1u << 16);  // B (V) is MN-major
       const uint64_t dq0 = umma_desc_k_sw128(sm_q);
       // descriptors advance by 16-byte units: 2 per k-step inside a chunk (columns past D are zeros on both sides)
+      auto ready = [](uint32_t bar, uint32_t parity) { return __all_sync(0xffffffffu, mbar_test(bar, parity)) != 0; };
       auto s_chunk = [&](int it, int col_chunk, uint32_t rows_addr, bool first) {  // S[it % 2] (+)= Q[:, chunk] K[:, chunk]^T
         const uint64_t dq = dq0 + static_cast<uint64_t>(col_chunk) * (q_chunk >> 4), dk = umma_desc_k_sw128(rows_addr);
 #pragma unroll
         for (int ks = 0; ks < 4; ++ks)
-          tc_mma_f16(tm_s + (it & 1) * NK, dq + 2 * ks, dk + 2 * ks, kIdescS, first && ks == 0 ? 0u : 1u);
+          mma_ss(tm_s + (it & 1) * NK, dq + 2 * ks, dk + 2 * ks, kIdescS, first && ks == 0 ? 0u : 1u, leader);
       };
       auto issue_pv = [&](int it) {  // O += P(it) V(it)
         const int vb = it % a.v_bufs;
         const uint64_t dv = desc_mn_sw128(sm_v + vb * per * kKvChunk);
 #pragma unroll
         for (int ks = 0; ks < NK / 16; ++ks)
-          tc_mma_f16_ts(tm_o, tm_p + (it & 1) * (NK / 2) + ks * 8, dv + 128 * ks, idesc_pv, (it > 0 || ks > 0) ? 1u : 0u);
-        tc_commit(o_full + 8 * (it & 1));
-        tc_commit(v_empty + 8 * vb);
+          mma_ts(tm_o, tm_p + (it & 1) * (NK / 2) + ks * 8, dv + 128 * ks, idesc_pv, (it > 0 || ks > 0) ? 1u : 0u, leader);
+        commit(o_full + 8 * (it & 1), leader);
+        commit(v_empty + 8 * vb, leader);
       };
       // Whichever is ready goes next: the product of a tile whose probabilities are written, or the next chunk of the
       // scores (at most one tile ahead of the products: two score buffers). A load in flight never holds back a
       // product, which is what frees the buffers for the loads after it.
-      bool ok = mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL);
+      bool ok = __all_sync(0xffffffffu, mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL));
       int next_s = 0, next_pv = 0;   // tiles whose scores / products come next
       int j = 0, slot = 0, slot_phase = 0;  // score-only chunk of tile next_s and its ring slot
       uint64_t since = 0;
       uint32_t spins = 0;
       while (ok && next_pv < n_tiles) {
         bool moved = false;
-        if (next_pv < next_s && mbar_test(p_ready + 8 * (next_pv & 1), (next_pv >> 1) & 1)) {
+        if (next_pv < next_s && ready(p_ready + 8 * (next_pv & 1), (next_pv >> 1) & 1)) {
           tc_fence_after_sync();
           issue_pv(next_pv++);
           moved = true;
         }
         if (next_s < n_tiles && next_s <= next_pv + 1) {
           if (j < nkc) {
-            if (mbar_test(k_full + 8 * slot, slot_phase)) {
+            if (ready(k_full + 8 * slot, slot_phase)) {
               tc_fence_after_sync();
               s_chunk(next_s, k_chunk(j), sm_k + slot * kKvChunk, j == 0);
-              tc_commit(k_empty + 8 * slot);  // free again once these have read it
+              commit(k_empty + 8 * slot, leader);  // free again once these have read it
               ++j;
               if (++slot == a.k_slots) {
                 slot = 0;
@@ -284,11 +326,11 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
               }
               moved = true;
             }
-          } else if (mbar_test(v_full + 8 * (next_s % a.v_bufs), (next_s / a.v_bufs) & 1)) {
+          } else if (ready(v_full + 8 * (next_s % a.v_bufs), (next_s / a.v_bufs) & 1)) {
             tc_fence_after_sync();
             const uint32_t v = sm_v + (next_s % a.v_bufs) * per * kKvChunk;
             for (int c = 0; c < nv; ++c) s_chunk(next_s, v0 + c, v + c * kKvChunk, nkc == 0 && c == 0);
-            tc_commit(s_full + 8 * (next_s & 1));
+            commit(s_full + 8 * (next_s & 1), leader);
             ++next_s;
             j = 0;
             moved = true;
@@ -300,12 +342,12 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         } else if ((++spins & 0x3ffu) == 0) {
           const uint64_t now = global_timer_ns();
           if (since == 0) since = now;
-          if (*abort_flag) ok = false;
-          if (now - since > kWaitLimitNs) {
+          const bool late = now - since > kWaitLimitNs;
+          if (late && leader) {
             *abort_flag = 1;
             if (a.status) atomicCAS(a.status, 0, PXL_DEV_TIMEOUT_TMEM_EMPTY);
-            ok = false;
           }
+          ok = __all_sync(0xffffffffu, !late && !*abort_flag);
         }
       }
     }
