@@ -76,7 +76,7 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// The MMA warp runs its loop with all lanes, so that addresses and descriptors stay in uniform registers (a loop in one
+// The MMA and producer warps run their loops with all lanes, so that addresses and descriptors stay in uniform registers (a loop in one
 // lane moves them there before every instruction and issues at half the rate); `leader` is non-zero in the lane
 // that issues.
 __device__ __forceinline__ uint32_t elect_leader() {
@@ -116,6 +116,18 @@ __device__ __forceinline__ void mma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_
       "}\n"
       :
       : "r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(leader)
+      : "memory");
+}
+__device__ __forceinline__ void tma_box(uint32_t smem_dst, const CUtensorMap* tmap, uint32_t bar, int x, int y,
+                                        uint32_t leader) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred q;\n\t"
+      "setp.ne.b32 q, %5, 0;\n\t"
+      "@q cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n\t"
+      "}\n"
+      :
+      : "r"(smem_dst), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(bar), "r"(x), "r"(y), "r"(leader)
       : "memory");
 }
 __device__ __forceinline__ void commit(uint32_t bar, uint32_t leader) {
@@ -223,30 +235,27 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 
   if (warp == kProducerWarp) {
     // ------------------------------------------------------------------ TMA producer
-    // Lane p looks up the block of piece p of the tile and issues that piece's boxes.
-    if (lane == 0) {
-      mbar_arrive_expect_tx(q_full, nck * q_chunk);
-      for (int c = 0; c < nck; ++c)
-        tma_load_2d(sm_q + c * q_chunk, &tm_q, q_full, c * 64, static_cast<int>(row0));
-    }
+    // Lane p looks up the block of piece p of the tile; one lane issues all boxes.
+    const uint32_t leader = elect_leader();
+    if (leader) mbar_arrive_expect_tx(q_full, nck * q_chunk);
+    __syncwarp();
+    for (int c = 0; c < nck; ++c) tma_box(sm_q + c * q_chunk, &tm_q, q_full, c * 64, static_cast<int>(row0), leader);
     const int* bt = a.block_tables + static_cast<int64_t>(b) * a.max_blocks;
     const int box = a.page < NK ? a.page : NK;
     const int pieces = NK / box;
     bool ok = true;
     // wait for the buffer behind `bar_empty` to be free again (its `use`-th use), announce `bytes`
     auto acquire = [&](uint32_t bar_empty, uint32_t bar_full, int use, uint32_t bytes) {
-      int okf = 1;
-      if (lane == 0) {
-        if (use > 0)
-          okf = mbar_wait_bounded(bar_empty, (use - 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_EMPTY) ? 1 : 0;
-        if (okf) mbar_arrive_expect_tx(bar_full, bytes);
-      }
-      return __shfl_sync(0xffffffffu, okf, 0) != 0;
+      bool free = true;
+      if (use > 0)
+        free = __all_sync(0xffffffffu, mbar_wait_bounded(bar_empty, (use - 1) & 1, abort_flag, a.status, PXL_DEV_TIMEOUT_EMPTY));
+      if (free && leader) mbar_arrive_expect_tx(bar_full, bytes);
+      __syncwarp();
+      return free;
     };
-    int slot = 0, slot_use = 0;
-    for (int it = 0; ok && it < n_tiles; ++it) {
+    auto tile_row = [&](int it) {  // cache row of this lane's piece of tile `it`
       int row = 0;
-      if (lane < pieces) {
+      if (lane < pieces && it < n_tiles) {
         int key = (t_begin + it) * NK + lane * box;
         if (key >= ctx) key = (ctx - 1) / box * box;  // beyond the context: re-read its last piece (masked)
         const int bi = key / a.page;
@@ -257,23 +266,36 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         }
         row = static_cast<int>(blk * a.page + key % a.page);
       }
-      const uint32_t piece_off = lane * box * 128;
+      return row;
+    };
+    int slot = 0, slot_use = 0, vb = 0, vb_use = 0;
+    int row = tile_row(0);
+    for (int it = 0; ok && it < n_tiles; ++it) {
+      const int next_row = tile_row(it + 1);  // its table reads are in flight while this tile is issued
       for (int j = 0; ok && j < nkc; ++j) {
         ok = acquire(k_empty + 8 * slot, k_full + 8 * slot, slot_use, kKvChunk);
-        if (ok && lane < pieces)
-          tma_load_2d(sm_k + slot * kKvChunk + piece_off, &tm_kv, k_full + 8 * slot, k_chunk(j) * 64, row);
+        if (ok)
+          for (int p = 0; p < pieces; ++p)
+            tma_box(sm_k + slot * kKvChunk + p * box * 128, &tm_kv, k_full + 8 * slot, k_chunk(j) * 64,
+                    __shfl_sync(0xffffffffu, row, p), leader);
         if (++slot == a.k_slots) {
           slot = 0;
           ++slot_use;
         }
       }
       if (!ok) break;
-      const int vb = it % a.v_bufs;
-      ok = acquire(v_empty + 8 * vb, v_full + 8 * vb, it / a.v_bufs, nv * kKvChunk);
-      if (ok && lane < pieces) {
-        const uint32_t dst = sm_v + vb * per * kKvChunk + piece_off;
-        for (int c = 0; c < nv; ++c) tma_load_2d(dst + c * kKvChunk, &tm_kv, v_full + 8 * vb, (v0 + c) * 64, row);
+      ok = acquire(v_empty + 8 * vb, v_full + 8 * vb, vb_use, nv * kKvChunk);
+      if (ok)
+        for (int p = 0; p < pieces; ++p) {
+          const int r = __shfl_sync(0xffffffffu, row, p);
+          for (int c = 0; c < nv; ++c)
+            tma_box(sm_v + (vb * per + c) * kKvChunk + p * box * 128, &tm_kv, v_full + 8 * vb, (v0 + c) * 64, r, leader);
+        }
+      if (++vb == a.v_bufs) {
+        vb = 0;
+        ++vb_use;
       }
+      row = next_row;
     }
   } else if (warp == kMmaWarp) {
     // ------------------------------------------------------------------ MMA issuer
