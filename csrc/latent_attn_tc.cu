@@ -311,52 +311,55 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         for (int ks = 0; ks < 4; ++ks)
           mma_ss(tm_s + (it & 1) * NK, dq + 2 * ks, dk + 2 * ks, kIdescS, first && ks == 0 ? 0u : 1u, leader);
       };
-      auto issue_pv = [&](int it) {  // O += P(it) V(it)
-        const int vb = it % a.v_bufs;
-        const uint64_t dv = desc_mn_sw128(sm_v + vb * per * kKvChunk);
-#pragma unroll
-        for (int ks = 0; ks < NK / 16; ++ks)
-          mma_ts(tm_o, tm_p + (it & 1) * (NK / 2) + ks * 8, dv + 128 * ks, idesc_pv, (it > 0 || ks > 0) ? 1u : 0u, leader);
-        commit(o_full + 8 * (it & 1), leader);
-        commit(v_empty + 8 * vb, leader);
-      };
       // Whichever is ready goes next: the product of a tile whose probabilities are written, or the next chunk of the
       // scores (at most one tile ahead of the products: two score buffers). A load in flight never holds back a
       // product, which is what frees the buffers for the loads after it.
       bool ok = __all_sync(0xffffffffu, mbar_wait_bounded(q_full, 0, abort_flag, a.status, PXL_DEV_TIMEOUT_FULL));
       int next_s = 0, next_pv = 0;   // tiles whose scores / products come next
       int j = 0, slot = 0, slot_phase = 0;  // score-only chunk of tile next_s and its ring slot
+      int s_vb = 0, s_vb_phase = 0, pv_vb = 0;
       uint64_t since = 0;
       uint32_t spins = 0;
       while (ok && next_pv < n_tiles) {
         bool moved = false;
-        if (next_pv < next_s && ready(p_ready + 8 * (next_pv & 1), (next_pv >> 1) & 1)) {
-          tc_fence_after_sync();
-          issue_pv(next_pv++);
-          moved = true;
-        }
         if (next_s < n_tiles && next_s <= next_pv + 1) {
-          if (j < nkc) {
-            if (ready(k_full + 8 * slot, slot_phase)) {
-              tc_fence_after_sync();
-              s_chunk(next_s, k_chunk(j), sm_k + slot * kKvChunk, j == 0);
-              commit(k_empty + 8 * slot, leader);  // free again once these have read it
-              ++j;
-              if (++slot == a.k_slots) {
-                slot = 0;
-                slot_phase ^= 1;
-              }
-              moved = true;
-            }
-          } else if (ready(v_full + 8 * (next_s % a.v_bufs), (next_s / a.v_bufs) & 1)) {
+          while (j < nkc && ready(k_full + 8 * slot, slot_phase)) {
             tc_fence_after_sync();
-            const uint32_t v = sm_v + (next_s % a.v_bufs) * per * kKvChunk;
+            s_chunk(next_s, k_chunk(j), sm_k + slot * kKvChunk, j == 0);
+            commit(k_empty + 8 * slot, leader);  // free again once these have read it
+            ++j;
+            if (++slot == a.k_slots) {
+              slot = 0;
+              slot_phase ^= 1;
+            }
+            moved = true;
+          }
+          if (j == nkc && ready(v_full + 8 * s_vb, s_vb_phase)) {
+            tc_fence_after_sync();
+            const uint32_t v = sm_v + s_vb * per * kKvChunk;
             for (int c = 0; c < nv; ++c) s_chunk(next_s, v0 + c, v + c * kKvChunk, nkc == 0 && c == 0);
             commit(s_full + 8 * (next_s & 1), leader);
             ++next_s;
             j = 0;
+            if (++s_vb == a.v_bufs) {
+              s_vb = 0;
+              s_vb_phase ^= 1;
+            }
             moved = true;
           }
+        }
+        if (next_pv < next_s && ready(p_ready + 8 * (next_pv & 1), (next_pv >> 1) & 1)) {  // O += P V
+          tc_fence_after_sync();
+          const uint64_t dv = desc_mn_sw128(sm_v + pv_vb * per * kKvChunk);
+          const uint32_t p = tm_p + (next_pv & 1) * (NK / 2);
+#pragma unroll
+          for (int ks = 0; ks < NK / 16; ++ks)
+            mma_ts(tm_o, p + ks * 8, dv + 128 * ks, idesc_pv, (next_pv > 0 || ks > 0) ? 1u : 0u, leader);
+          commit(o_full + 8 * (next_pv & 1), leader);
+          commit(v_empty + 8 * pv_vb, leader);
+          ++next_pv;
+          if (++pv_vb == a.v_bufs) pv_vb = 0;
+          moved = true;
         }
         if (moved) {
           spins = 0;
