@@ -5,6 +5,7 @@
     python benchmarks/profile_case.py gemm_mid     # mid-M cluster split-K GEMM, 320 x 4096 x 12288
     python benchmarks/profile_case.py attn_decode  # paged GQA decode, 256 seqs x 2048 ctx
     python benchmarks/profile_case.py attn_prefill # ragged prefill, 4 x 2048
+    python benchmarks/profile_case.py latent_attn  # windowed latent attention, 4096-token prompt, 32 heads
     python benchmarks/profile_case.py step         # 2 engine steps of a 4-layer Qwen3-8B-shaped
                                                    # model at 64 concurrent (launch list)
     python benchmarks/profile_case.py decode_step  # same, decode rows only (small-M GEMMs); decode_step_8: 8 rows
@@ -154,9 +155,31 @@ def case_step(steps: int = 2, conc: int = 64, with_prefill: bool = True):
     cu.check_status(torch.device("cuda:0"))
 
 
+def case_latent_attn(iters: int = 2, T: int = 4096, H: int = 32, L: int = 512, R: int = 64, window: int = 1024, page: int = 16):
+    q = torch.randn(T, H, L + R, device="cuda", dtype=torch.bfloat16) * 0.3
+    cache = torch.randn(T // page, 1, page, L + R, device="cuda", dtype=torch.bfloat16)
+    table = torch.randperm(T // page, device="cuda").to(torch.int32).view(1, -1)
+    cu_q = torch.tensor([0, T], dtype=torch.int32, device="cuda")
+    ctx = torch.tensor([T], dtype=torch.int32, device="cuda")
+    sinks = torch.zeros(H, device="cuda")
+    out = torch.empty(T, H, L, device="cuda", dtype=torch.bfloat16)
+
+    def run():
+        cu.latent_attn(q, cache, table, cu_q, ctx, (L + R) ** -0.5, L, window, sinks, T, T, out=out)
+
+    run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStart()
+    for _ in range(iters):
+        run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStop()
+    cu.check_status(q.device)
+
+
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "gemm"
-    {"gemm": case_gemm, "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
+    {"gemm": case_gemm, "latent_attn": case_latent_attn, "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
      "gemm_small": case_gemm_small, "gemm_mid": case_gemm_mid, "step": case_step, "decode_step": lambda: case_step(conc=64, with_prefill=False),
      "decode_step_8": lambda: case_step(conc=8, with_prefill=False)}[which]()
     print(f"profile case {which}: ok")
