@@ -148,9 +148,11 @@ def run_multi_gpu(args, cfg, name: str, path: Optional[str]) -> None:
     dp_lanes = ep_size if (getattr(args, "enable_dp_attention", False) and ep_size > 1 and cfg.is_moe) else 1
     tp_size = args.tp_size if dp_lanes > 1 else max(args.tp_size, ep_size)
     device_type = "cuda" if torch.cuda.is_available() else "cpu"
+    from parallax_b200.models.registry import runs_in_float32
+
+    dtypes = ("bfloat16", "float16") + (("float32",) if runs_in_float32(cfg.architecture) else ())
     spec = dict(model_path=path, model_name=name.split("/")[-1], pp=args.pp_size, tp=tp_size, ep=dp_lanes,
-                device_type=device_type,
-                dtype=args.dtype if args.dtype in ("bfloat16", "float16") else "bfloat16",
+                device_type=device_type, dtype=args.dtype if args.dtype in dtypes else "bfloat16",
                 page_size=args.kv_block_size, kv_fraction=args.kv_cache_memory_fraction,
                 kv_cache_dtype=getattr(args, "kv_cache_dtype", None),
                 max_batch_size=args.max_batch_size, max_num_tokens_per_batch=args.max_num_tokens_per_batch,

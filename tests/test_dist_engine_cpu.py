@@ -69,6 +69,11 @@ def test_dist_engine_matches_single_process(pp, tp, tmp_path):
     assert got["probe"]["device_ms"] > 0 and got["probe"]["h2d_bytes"] > 0
 
 
+def test_layer_list_model_over_pipeline_ranks(tmp_path):
+    """fp32 hidden states between stages and the previous-token ids of the embedding travel with the plans."""
+    assert _run_group(2, 1, tmp_path, model="tiny-piburax")["outputs"] == _single(model="tiny-piburax")
+
+
 def test_rank0_executor_thread_and_aligned_rows(tmp_path):
     """Rank 0 launching its stage from a thread of its own, three micro-batches in flight and prompt
     slices trimmed to a row multiple: same tokens as the single-process engine."""

@@ -46,6 +46,15 @@ def _run_pipeline(cfg, spans, prompts, max_new, **kw):
     return [r.output_ids for r in reqs], peers
 
 
+def test_three_peers_of_a_layer_list_model():
+    cfg = named_config("tiny-piburax")
+    prompts = _prompts(3, 41, cfg.vocab_size, seed=4)
+    want = Engine(cfg, device="cpu", num_blocks=128, max_batch_size=8).generate(
+        prompts, SamplingParams(max_new_tokens=9, temperature=0.0, ignore_eos=True))
+    got, peers = _run_pipeline(cfg, [(0, 1), (1, 2), (2, 3)], prompts, 9)
+    assert got == want and all(not p.cache.reqs for p in peers)
+
+
 def test_three_peers_match_single_engine():
     cfg = named_config("tiny")
     prompts = _prompts(3, 41, cfg.vocab_size, seed=4)
