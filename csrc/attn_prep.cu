@@ -1,0 +1,362 @@
+// Around softmax attention with grouped heads, rows of any size in bf16 or fp32:
+//
+//  * pxl_conv_qkv_prep: one launch per layer and step turns the packed projection q | k | v into queries and
+//    cache rows: short causal convolution per channel (y_t = sum_j w[j] u[t - taps + 1 + j], zeros before the
+//    sequence), RMS norm over the whole q row and the whole k row, half-split rotation, and the scatter of k and
+//    v into their pages. Heads are padded with zeros to `cols` columns. v is neither normed nor rotated.
+//  * pxl_conv_state_update: the last taps - 1 projected rows of every prompt slice become the state of its slot
+//    (a launch of its own: the first tokens of the slice read the state that its last tokens replace; a decoded
+//    token reads and replaces it in pxl_conv_qkv_prep itself).
+//  * pxl_gated_rows: concatenated heads, optionally RMS-normed together, times sigmoid(gate), into the columns of
+//    the output product's operand.
+//
+// All arithmetic is fp32.
+#include "common.cuh"
+#include "pxl_api.h"
+
+namespace {
+using namespace pxl;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+// VEC consecutive elements (VEC == 8: 16-byte aligned)
+template <int VEC, typename T>
+__device__ __forceinline__ void load_v(const T* p, float (&v)[VEC]) {
+  if constexpr (VEC == 1) {
+    v[0] = to_f(*p);
+  } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4) {
+      const float4 a = *reinterpret_cast<const float4*>(p + i);
+      v[i] = a.x, v[i + 1] = a.y, v[i + 2] = a.z, v[i + 3] = a.w;
+    }
+  } else {
+    const bf16x8 a = ld_bf16x8(p);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(a.u[j]);
+      v[2 * j] = f.x, v[2 * j + 1] = f.y;
+    }
+  }
+}
+template <int VEC, typename T>
+__device__ __forceinline__ void store_v(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 1) {
+    put(p, v[0]);
+  } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4)
+      *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+  } else {
+    bf16x8 o;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o.u[j] = pack_bf16x2(v[2 * j], v[2 * j + 1]);
+    st_bf16x8(p, o);
+  }
+}
+
+struct PrepArgs {
+  const void* proj;  // [T, ld]
+  int64_t ld;
+  int q_off, k_off, v_off;      // first column of each part (k and v absent: G == 0)
+  int H, G, dk, dv, cols, rot, taps;
+  const void* conv_w;           // [taps, C] over channels q | k | v, or null
+  void* conv_state;             // [slots, taps - 1, C]: previous projected values, oldest first
+  int num_state_slots;
+  const float* q_norm;
+  const float* k_norm;
+  const float* cos_sin;         // [max_pos, rot]: cos | sin halves
+  const int* positions;
+  int max_pos;
+  const int* seq_cu;            // [seqs + 1] token ranges: prompt slices first, then one token per decoded sequence
+  const int* seq_slots;
+  int prefill_seqs, prefill_tokens, T;
+  const int64_t* slots;         // cache row of every token
+  int64_t num_slots;
+  int page;
+  void* k_cache;                // [blocks, G, page, cols]
+  void* v_cache;
+  void* q_out;                  // [T, H, cols]
+  float eps;
+  int* status;
+};
+
+// y = norm_w * inv * row (or the convolved row itself), rotated; VEC elements of one head from d0
+template <int VEC>
+__device__ __forceinline__ void rotated(const float* row, const float* w, float inv, const float* cs, int dk, int rot,
+                                        int d0, float (&o)[VEC]) {
+  const int half = rot / 2;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) {
+    const int d = d0 + j;
+    if (d >= dk) {
+      o[j] = 0.f;
+      continue;
+    }
+    float y = row[d] * inv * w[d];
+    if (d < half) y = y * cs[d] - row[d + half] * inv * w[d + half] * cs[half + d];
+    else if (d < rot) y = y * cs[d - half] + row[d - half] * inv * w[d - half] * cs[d];
+    o[j] = y;
+  }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) conv_qkv_prep_kernel(const PrepArgs a, int tokens_per_cta) {
+  extern __shared__ float row[];  // convolved q | k of one token
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int Cq = a.H * a.dk, Ck = a.G * a.dk, Cv = a.G * a.dv, C = Cq + Ck + Cv;
+  const int back = a.conv_w ? a.taps - 1 : 0;
+  const T* w = static_cast<const T*>(a.conv_w);
+  const int first = blockIdx.x * tokens_per_cta;
+  int seq = 0;
+  if (first < a.prefill_tokens) {  // last slice that starts at or before the token
+    int lo = 0, hi = a.prefill_seqs - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) / 2;
+      if (a.seq_cu[mid] <= first) lo = mid;
+      else hi = mid - 1;
+    }
+    seq = lo;
+  }
+  for (int t = first; t < a.T && t < first + tokens_per_cta; ++t) {
+    const bool decoded = t >= a.prefill_tokens;
+    if (decoded) seq = a.prefill_seqs + t - a.prefill_tokens;
+    else
+      while (a.seq_cu[seq + 1] <= t) ++seq;
+    const int li = t - a.seq_cu[seq];
+    int pos = a.positions[t];
+    const T* cur = static_cast<const T*>(a.proj) + static_cast<int64_t>(t) * a.ld;
+    T* state = nullptr;
+    if (back) {
+      const int slot = a.seq_slots[seq];
+      if (slot >= 0 && slot < a.num_state_slots) state = static_cast<T*>(a.conv_state) + static_cast<int64_t>(slot) * back * C;
+      else if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_INDEX);
+    }
+    int64_t cslot = a.G ? a.slots[t] : -1;
+    if (cslot >= a.num_slots) {
+      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_SLOT);
+      cslot = -1;
+    }
+    const int64_t blk = cslot / a.page, in_page = cslot % a.page;
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
+      const int col = c < Cq ? a.q_off + c : c < Cq + Ck ? a.k_off + c - Cq : a.v_off + c - Cq - Ck;
+      float u[VEC], y[VEC];
+      load_v<VEC>(cur + col, u);
+      if (w) {
+        float wv[VEC];
+        load_v<VEC>(w + static_cast<int64_t>(back) * C + c, wv);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) y[j] = wv[j] * u[j];
+        for (int b = back; b >= 1; --b) {
+          if (pos - b < 0) continue;
+          float h[VEC];
+          if (b <= li) {
+            load_v<VEC>(cur - static_cast<int64_t>(b) * a.ld + col, h);
+          } else {
+            if (!state) continue;
+            load_v<VEC>(state + static_cast<int64_t>(back + li - b) * C + c, h);
+          }
+          load_v<VEC>(w + static_cast<int64_t>(back - b) * C + c, wv);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) y[j] = fmaf(wv[j], h[j], y[j]);
+        }
+        if (decoded && state) {  // this thread is the only reader and writer of these channels
+          for (int m = 0; m + 1 < back; ++m) {
+            float h[VEC];
+            load_v<VEC>(state + static_cast<int64_t>(m + 1) * C + c, h);
+            store_v<VEC>(state + static_cast<int64_t>(m) * C + c, h);
+          }
+          store_v<VEC>(state + static_cast<int64_t>(back - 1) * C + c, u);
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) y[j] = u[j];
+      }
+      if (c < Cq + Ck) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          row[c + j] = y[j];
+          if (c < Cq) sq = fmaf(y[j], y[j], sq);
+          else sk = fmaf(y[j], y[j], sk);
+        }
+      } else if (cslot >= 0) {
+        const int vc = c - Cq - Ck, g = vc / a.dv;
+        store_v<VEC>(static_cast<T*>(a.v_cache) + ((blk * a.G + g) * a.page + in_page) * a.cols + vc % a.dv, y);
+      }
+    }
+    sq = block_reduce_sum(sq, red);
+    if (a.G) sk = block_reduce_sum(sk, red);
+    if (pos < 0 || pos >= a.max_pos) {
+      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
+      pos = 0;
+    }
+    const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
+    const float inv_q = 1.f / sqrtf(sq / Cq + a.eps), inv_k = a.G ? 1.f / sqrtf(sk / Ck + a.eps) : 0.f;
+    const int per = a.cols / VEC;
+    for (int i = threadIdx.x; i < (a.H + a.G) * per; i += blockDim.x) {
+      const int h = i / per, d0 = i % per * VEC;
+      float o[VEC];
+      if (h < a.H) {
+        rotated<VEC>(row + h * a.dk, a.q_norm + h * a.dk, inv_q, cs, a.dk, a.rot, d0, o);
+        store_v<VEC>(static_cast<T*>(a.q_out) + (static_cast<int64_t>(t) * a.H + h) * a.cols + d0, o);
+      } else if (cslot >= 0) {
+        const int g = h - a.H;
+        rotated<VEC>(row + Cq + g * a.dk, a.k_norm + g * a.dk, inv_k, cs, a.dk, a.rot, d0, o);
+        store_v<VEC>(static_cast<T*>(a.k_cache) + ((blk * a.G + g) * a.page + in_page) * a.cols + d0, o);
+        if (d0 + VEC > a.dv) {  // zero columns behind the value
+          T* v = static_cast<T*>(a.v_cache) + ((blk * a.G + g) * a.page + in_page) * a.cols;
+          for (int d = d0 > a.dv ? d0 : a.dv; d < d0 + VEC; ++d) put(v + d, 0.f);
+        }
+      }
+    }
+    __syncthreads();  // the next token overwrites the row
+  }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) conv_state_update_kernel(const PrepArgs a) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int Cq = a.H * a.dk, Ck = a.G * a.dk, C = Cq + Ck + a.G * a.dv, back = a.taps - 1;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC, seq = blockIdx.y;
+  if (c >= C) return;
+  const int t0 = a.seq_cu[seq], n = a.seq_cu[seq + 1] - t0, slot = a.seq_slots[seq];
+  if (n <= 0) return;
+  if (slot < 0 || slot >= a.num_state_slots) {
+    if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_INDEX);
+    return;
+  }
+  const int col = c < Cq ? a.q_off + c : c < Cq + Ck ? a.k_off + c - Cq : a.v_off + c - Cq - Ck;
+  T* state = static_cast<T*>(a.conv_state) + static_cast<int64_t>(slot) * back * C + c;
+  for (int m = 0; m < back; ++m) {
+    const int li = n - back + m;  // entry m holds the value at this place of the slice, or an older one
+    float h[VEC];
+    if (li >= 0) load_v<VEC>(static_cast<const T*>(a.proj) + static_cast<int64_t>(t0 + li) * a.ld + col, h);
+    else load_v<VEC>(state + static_cast<int64_t>(m + n) * C, h);
+    store_v<VEC>(state + static_cast<int64_t>(m) * C, h);
+  }
+}
+
+struct GateArgs {
+  const void* x;        // [T, heads, x_cols]
+  int heads, x_cols, dv;
+  const void* gate;     // [T, ldg], heads * dv columns
+  int64_t ldg;
+  const float* norm_w;  // [heads * dv] or null
+  float eps;
+  void* out;            // [T, ldo], out_cols columns: heads * dv, then zeros
+  int64_t ldo;
+  int out_cols;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) gated_rows_kernel(const GateArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const int N = a.heads * a.dv;
+  const T* x = static_cast<const T*>(a.x) + t * a.heads * a.x_cols;
+  const T* g = static_cast<const T*>(a.gate) + t * a.ldg;
+  T* out = static_cast<T*>(a.out) + t * a.ldo;
+  float inv = 1.f;
+  if (a.norm_w) {
+    float sq = 0.f;
+    for (int c = threadIdx.x * VEC; c < N; c += blockDim.x * VEC) {
+      float v[VEC];
+      load_v<VEC>(x + c / a.dv * a.x_cols + c % a.dv, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) sq = fmaf(v[j], v[j], sq);
+    }
+    inv = 1.f / sqrtf(block_reduce_sum(sq, red) / N + a.eps);
+  }
+  for (int c = threadIdx.x * VEC; c < N; c += blockDim.x * VEC) {
+    float v[VEC], gv[VEC];
+    load_v<VEC>(x + c / a.dv * a.x_cols + c % a.dv, v);
+    load_v<VEC>(g + c, gv);
+    if (a.norm_w) {
+      float w[VEC];
+      load_v<VEC>(a.norm_w + c, w);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] /= 1.f + expf(-gv[j]);
+    store_v<VEC>(out + c, v);
+  }
+  for (int c = N + threadIdx.x; c < a.out_cols; c += blockDim.x) put(out + c, 0.f);
+}
+
+inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+template <typename T, int VEC>
+int launch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
+  if (update) {
+    const int C = a.H * a.dk + a.G * (a.dk + a.dv);
+    pxl_host::launch(conv_state_update_kernel<T, VEC>, dim3(ceil_div(C, 256 * VEC), a.prefill_seqs), dim3(256), 0, stream, a);
+  } else {
+    const size_t smem = sizeof(float) * (a.H + a.G) * a.dk;
+    if (smem > 220 * 1024) return PXL_ERR_TOO_LARGE;
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(conv_qkv_prep_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                 static_cast<int>(smem)) != cudaSuccess)
+      return PXL_ERR_CUDA;
+    const int per = a.prefill_tokens >= 4 * 8 * pxl_host::num_sms() ? 4 : 1;  // neighbours share taps through L1
+    pxl_host::launch(conv_qkv_prep_kernel<T, VEC>, dim3(ceil_div(a.T, per)), dim3(256), smem, stream, a, per);
+  }
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
+template <typename T>
+int dispatch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
+  const bool vec = !((a.q_off | a.k_off | a.v_off | a.dk | a.dv | a.cols | (a.rot / 2) | static_cast<int>(a.ld)) & 7) &&
+                   aligned16(a.proj) && aligned16(a.conv_w) && aligned16(a.conv_state) && aligned16(a.k_cache) &&
+                   aligned16(a.v_cache) && aligned16(a.q_out);
+  return vec ? launch_prep<T, 8>(a, update, stream) : launch_prep<T, 1>(a, update, stream);
+}
+
+inline bool bad_prep(const PrepArgs& a) {
+  return a.H <= 0 || a.G < 0 || a.dk <= 0 || (a.G && a.dv <= 0) || a.cols < a.dk || (a.G && a.cols < a.dv) || a.rot < 0 ||
+         a.rot > a.dk || (a.rot & 1) || a.taps < 1 || a.page <= 0 || (a.taps > 1 && a.conv_w && a.conv_state == nullptr);
+}
+}  // namespace
+
+PXL_EXPORT int pxl_conv_qkv_prep(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int H, int G, int dk, int dv,
+                                 int cols, int rot, int taps, const void* conv_w, void* conv_state, int num_state_slots,
+                                 const float* q_norm, const float* k_norm, const float* cos_sin, const int* positions,
+                                 int max_pos, const int* seq_cu, const int* seq_slots, int prefill_seqs, int prefill_tokens,
+                                 int T, const int64_t* slots, int64_t num_slots, int page, void* k_cache, void* v_cache,
+                                 void* q_out, float eps, int is_f32, int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  PrepArgs a{proj, ld, q_off, k_off, v_off, H, G, dk, dv, cols, rot, taps, conv_w, conv_state, num_state_slots, q_norm, k_norm,
+             cos_sin, positions, max_pos, seq_cu, seq_slots, prefill_seqs, prefill_tokens, T, slots, num_slots, page, k_cache,
+             v_cache, q_out, eps, status};
+  if (bad_prep(a)) return PXL_ERR_INVALID_ARG;
+  int code = is_f32 ? dispatch_prep<float>(a, false, stream) : dispatch_prep<pxl::bf16>(a, false, stream);
+  if (code == PXL_OK && conv_w && taps > 1 && prefill_seqs > 0)
+    code = is_f32 ? dispatch_prep<float>(a, true, stream) : dispatch_prep<pxl::bf16>(a, true, stream);
+  return code;
+}
+
+PXL_EXPORT int pxl_gated_rows(const void* x, int heads, int x_cols, int dv, const void* gate, int64_t ldg,
+                              const float* norm_w, float eps, void* out, int64_t ldo, int out_cols, int T, int is_f32,
+                              cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (heads <= 0 || dv <= 0 || x_cols < dv || out_cols < heads * dv) return PXL_ERR_INVALID_ARG;
+  const GateArgs a{x, heads, x_cols, dv, gate, ldg, norm_w, eps, out, ldo, out_cols};
+  const bool vec = !((x_cols | dv | static_cast<int>(ldg) | static_cast<int>(ldo)) & 7) && aligned16(x) && aligned16(gate) &&
+                   aligned16(out) && aligned16(norm_w);
+  if (is_f32) {
+    if (vec) pxl_host::launch(gated_rows_kernel<float, 8>, dim3(T), dim3(256), 0, stream, a);
+    else pxl_host::launch(gated_rows_kernel<float, 1>, dim3(T), dim3(256), 0, stream, a);
+  } else {
+    if (vec) pxl_host::launch(gated_rows_kernel<pxl::bf16, 8>, dim3(T), dim3(256), 0, stream, a);
+    else pxl_host::launch(gated_rows_kernel<pxl::bf16, 1>, dim3(T), dim3(256), 0, stream, a);
+  }
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}

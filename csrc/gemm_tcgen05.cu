@@ -59,6 +59,9 @@ struct GemmEpilogueArgs {
   bf16* const* row_ptrs; // EPI_SCATTER: destination of every output row (null = drop), N elements each
   uint32_t* done_counter;  // EPI_SCATTER: local counter for the "last CTA publishes the flags" step
   float act_limit;           // EPI_CLIP_GLU
+  int act;                   // EPI_GLU: 0 silu, 2 gelu (tanh form)
+  const float* row_gate;     // EPI_GLU: optional, row m times sigmoid(row_gate[m * ld_row_gate])
+  int64_t ld_row_gate;
   const bf16* gate;          // EPI_GATE: [M, ldg], indexed by the row of W like the bias
   int ldg;
   // EPI_SPLITK_T (operands swapped: accumulator row = output column, accumulator column = token)
@@ -417,9 +420,13 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
       }
       const int row = tc.a_row + q * 32 + lane;
       const uint32_t t_row = tmem_base + acc * BN + (static_cast<uint32_t>(q * 32) << 16);
-      if constexpr (EPI == PXL_EPI_SILU_MUL || EPI == PXL_EPI_CLIP_GLU) {
+      if constexpr (EPI == PXL_EPI_SILU_MUL || EPI == PXL_EPI_CLIP_GLU || EPI == PXL_EPI_GLU) {
         // W rows come in groups of 128: 64 gate rows then the 64 up rows of the same outputs
         const int n_out = N / 2;
+        float row_scale = 1.f;
+        if constexpr (EPI == PXL_EPI_GLU) {
+          if (ep.row_gate && row < M_end) row_scale = 1.f / (1.f + __expf(-ep.row_gate[row * ep.ld_row_gate]));
+        }
 #pragma unroll 1
         for (int c = 0; c < BN / 2; c += 32) {
           const int grp = c / 64, cin = c % 64;
@@ -448,6 +455,13 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                     g1 = g1 / (1.f + __expf(-1.702f * g1));
                     u0 = fminf(fmaxf(u0, -lim), lim) + 1.f;
                     u1 = fminf(fmaxf(u1, -lim), lim) + 1.f;
+                  } else if constexpr (EPI == PXL_EPI_GLU) {
+                    // gelu, tanh form: z (1 + tanh(s)) / 2 = z / (1 + exp(-2 s))
+                    const bool gelu = ep.act == 2;
+                    const float s0 = gelu ? 1.5957691216057308f * (g0 + 0.044715f * g0 * g0 * g0) : g0;
+                    const float s1 = gelu ? 1.5957691216057308f * (g1 + 0.044715f * g1 * g1 * g1) : g1;
+                    g0 = g0 / (1.f + __expf(-s0)) * row_scale;
+                    g1 = g1 / (1.f + __expf(-s1)) * row_scale;
                   } else {
                     g0 = g0 / (1.f + __expf(-g0));
                     g1 = g1 / (1.f + __expf(-g1));
@@ -1423,9 +1437,11 @@ PXL_EXPORT int pxl_gemm_bf16(const void* A, const void* W, void* C, const void* 
   }
 }
 
-// Clipped GLU epilogue (see pxl_api.h): tiles of 128 or 256 columns of W.
-PXL_EXPORT int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,
-                                 float limit, int bn, int* status, cudaStream_t stream) {
+// Gated-activation epilogues (see pxl_api.h): tiles of 128 or 256 columns of W.
+namespace {
+template <int EPI>
+int gemm_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, GemmEpilogueArgs ep, int bn,
+             int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return PXL_ERR_INVALID_ARG;
   if ((K % 8) || (lda % 8) || (ldw % 8) || (ldc % 8) || (N % 128)) return PXL_ERR_INVALID_ARG;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C)) & 15)
@@ -1436,14 +1452,30 @@ PXL_EXPORT int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, i
   if (!pxl_host::make_tmap_2d(&ta, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, M, K, lda, BM, BK) ||
       !pxl_host::make_tmap_2d(&tb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, N, K, ldw, bn, BK))
     return PXL_ERR_TENSORMAP;
-  GemmEpilogueArgs ep{};
   ep.C = static_cast<pxl::bf16*>(C);
   ep.ldc = ldc;
-  ep.act_limit = limit;
   GemmGroupArgs grp{};
-  if (bn == 256)
-    return launch_gemm<256, PXL_EPI_CLIP_GLU>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
-  return launch_gemm<128, PXL_EPI_CLIP_GLU>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+  if (bn == 256) return launch_gemm<256, EPI>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+  return launch_gemm<128, EPI>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+}
+}  // namespace
+
+PXL_EXPORT int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,
+                                 float limit, int bn, int* status, cudaStream_t stream) {
+  GemmEpilogueArgs ep{};
+  ep.act_limit = limit;
+  return gemm_glu<PXL_EPI_CLIP_GLU>(A, W, C, M, N, K, lda, ldw, ldc, ep, bn, status, stream);
+}
+
+PXL_EXPORT int pxl_gemm_bf16_act_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc,
+                                     int act, const float* row_gate, int64_t ld_row_gate, int bn, int* status,
+                                     cudaStream_t stream) {
+  if (act != 0 && act != 2) return PXL_ERR_INVALID_ARG;
+  GemmEpilogueArgs ep{};
+  ep.act = act;
+  ep.row_gate = row_gate;
+  ep.ld_row_gate = ld_row_gate;
+  return gemm_glu<PXL_EPI_GLU>(A, W, C, M, N, K, lda, ldw, ldc, ep, bn, status, stream);
 }
 
 // Per-head products (see pxl_api.h). K columns past a head's K meet zeros: the tensor map of W ends at K.

@@ -6,10 +6,13 @@
 //   mode 0  softmax over all experts, top-k, optional renormalisation (Qwen3-MoE, GPT-OSS
 //           style; the reference gets it from mlx-lm's switch layers, src/parallax/models/
 //           qwen3_moe.py)
+//           With a correction bias the choice is by score + bias, the weights stay the scores.
 //   mode 1  sigmoid scores, selection on score + per-expert correction bias with optional
 //           group-limited routing, weights = unbiased scores renormalised and scaled
 //           (DeepSeek-V3 "noaux_tc"; MiniMax-M3 uses the ungrouped form,
 //           src/parallax/models/minimax_m3.py:155-173)
+// In either mode the choice can be limited to the topk_group best of n_group groups of neighbouring experts; a
+// group counts as its best selection score (group_top 1) or the sum of its two best (group_top 2).
 #include "common.cuh"
 #include "pxl_api.h"
 
@@ -27,8 +30,8 @@ __device__ __forceinline__ float load_score(const void* p, size_t i) {
 // One warp per token.
 template <bool BF16>
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const void* __restrict__ logits, const float* __restrict__ e_bias, int T, int E,
-                 int k, int mode, int renorm, int n_group, int topk_group, float routed_scale,
+moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __restrict__ e_bias, int T, int E,
+                 int k, int mode, int renorm, int n_group, int topk_group, int group_top, float routed_scale,
                  int* __restrict__ out_ids, float* __restrict__ out_w) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
@@ -40,7 +43,7 @@ moe_route_kernel(const void* __restrict__ logits, const float* __restrict__ e_bi
 #pragma unroll
   for (int j = 0; j < kMaxEPL; ++j) {
     const int e = j * 32 + lane;
-    s[j] = (j < epl && e < E) ? load_score<BF16>(logits, static_cast<size_t>(t) * E + e) : -INFINITY;
+    s[j] = (j < epl && e < E) ? load_score<BF16>(logits, static_cast<size_t>(t) * ld + e) : -INFINITY;
     mx = fmaxf(mx, s[j]);
   }
   if (mode == 0) {
@@ -57,7 +60,7 @@ moe_route_kernel(const void* __restrict__ logits, const float* __restrict__ e_bi
     for (int j = 0; j < kMaxEPL; ++j) {
       const int e = j * 32 + lane;
       s[j] *= inv;
-      sel[j] = (j < epl && e < E) ? s[j] : -INFINITY;
+      sel[j] = (j < epl && e < E) ? s[j] + (e_bias ? e_bias[e] : 0.f) : -INFINITY;
     }
   } else {
 #pragma unroll
@@ -67,51 +70,51 @@ moe_route_kernel(const void* __restrict__ logits, const float* __restrict__ e_bi
       s[j] = ok ? 1.f / (1.f + __expf(-s[j])) : 0.f;
       sel[j] = ok ? s[j] + (e_bias ? e_bias[e] : 0.f) : -INFINITY;
     }
-    if (n_group > 1 && topk_group < n_group) {
-      // group score = sum of the two best selection scores inside the group
-      const int gsize = E / n_group;
-      float gscore_mine = -INFINITY;  // lane g (< n_group) holds the score of group g
-      for (int g = 0; g < n_group; ++g) {
-        float b1 = -INFINITY, b2 = -INFINITY;
-#pragma unroll
-        for (int j = 0; j < kMaxEPL; ++j) {
-          const int e = j * 32 + lane;
-          if (j < epl && e < E && e / gsize == g) {
-            if (sel[j] > b1) { b2 = b1; b1 = sel[j]; }
-            else if (sel[j] > b2) b2 = sel[j];
-          }
-        }
-        // merge (b1, b2) pairs across lanes
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          const float o1 = __shfl_xor_sync(0xffffffffu, b1, o);
-          const float o2 = __shfl_xor_sync(0xffffffffu, b2, o);
-          const float n1 = fmaxf(b1, o1);
-          const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
-          b1 = n1; b2 = n2;
-        }
-        if (lane == g) gscore_mine = b1 + (b2 == -INFINITY ? 0.f : b2);
-      }
-      // pick topk_group groups; keep a bitmask of allowed groups (n_group <= 32)
-      unsigned allowed = 0;
-      float gs = lane < n_group ? gscore_mine : -INFINITY;
-      for (int it = 0; it < topk_group; ++it) {
-        float best = gs;
-        int arg = lane;
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-          const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-          if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-        }
-        allowed |= 1u << arg;
-        if (lane == arg) gs = -INFINITY;
-      }
+  }
+  if (n_group > 1 && topk_group < n_group) {
+    // group score: its best selection score, or the sum of its two best
+    const int gsize = E / n_group;
+    float gscore_mine = -INFINITY;  // lane g (< n_group) holds the score of group g
+    for (int g = 0; g < n_group; ++g) {
+      float b1 = -INFINITY, b2 = -INFINITY;
 #pragma unroll
       for (int j = 0; j < kMaxEPL; ++j) {
         const int e = j * 32 + lane;
-        if (j < epl && e < E && !((allowed >> (e / gsize)) & 1u)) sel[j] = -INFINITY;
+        if (j < epl && e < E && e / gsize == g) {
+          if (sel[j] > b1) { b2 = b1; b1 = sel[j]; }
+          else if (sel[j] > b2) b2 = sel[j];
+        }
       }
+      // merge (b1, b2) pairs across lanes
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float o1 = __shfl_xor_sync(0xffffffffu, b1, o);
+        const float o2 = __shfl_xor_sync(0xffffffffu, b2, o);
+        const float n1 = fmaxf(b1, o1);
+        const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
+        b1 = n1; b2 = n2;
+      }
+      if (lane == g) gscore_mine = b1 + (group_top == 1 || b2 == -INFINITY ? 0.f : b2);
+    }
+    // pick topk_group groups; keep a bitmask of allowed groups (n_group <= 32)
+    unsigned allowed = 0;
+    float gs = lane < n_group ? gscore_mine : -INFINITY;
+    for (int it = 0; it < topk_group; ++it) {
+      float best = gs;
+      int arg = lane;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+        if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+      }
+      allowed |= 1u << arg;
+      if (lane == arg) gs = -INFINITY;
+    }
+#pragma unroll
+    for (int j = 0; j < kMaxEPL; ++j) {
+      const int e = j * 32 + lane;
+      if (j < epl && e < E && !((allowed >> (e / gsize)) & 1u)) sel[j] = -INFINITY;
     }
   }
   // iterative top-k over the warp
@@ -272,19 +275,19 @@ inline int check_launch() { return cudaGetLastError() == cudaSuccess ? PXL_OK : 
 
 }  // namespace
 
-PXL_EXPORT int pxl_moe_route(const void* logits, int logits_bf16, const float* e_bias, int T, int E,
-                             int k, int mode, int renorm, int n_group, int topk_group,
+PXL_EXPORT int pxl_moe_route(const void* logits, int64_t ld, int logits_bf16, const float* e_bias, int T, int E,
+                             int k, int mode, int renorm, int n_group, int topk_group, int group_top,
                              float routed_scale, int* out_ids, float* out_w, pxl_stream_t stream) {
   if (T <= 0) return PXL_OK;
   if (E <= 0 || E > 32 * kMaxEPL || k <= 0 || k > 32 || k > E) return PXL_ERR_INVALID_ARG;
   if (n_group > 32 || (n_group > 1 && E % n_group)) return PXL_ERR_INVALID_ARG;
   const unsigned grid = (T + 3) / 4;
   if (logits_bf16)
-    moe_route_kernel<true><<<grid, 128, 0, stream>>>(logits, e_bias, T, E, k, mode, renorm, n_group,
-                                                     topk_group, routed_scale, out_ids, out_w);
+    moe_route_kernel<true><<<grid, 128, 0, stream>>>(logits, ld, e_bias, T, E, k, mode, renorm, n_group,
+                                                     topk_group, group_top, routed_scale, out_ids, out_w);
   else
-    moe_route_kernel<false><<<grid, 128, 0, stream>>>(logits, e_bias, T, E, k, mode, renorm,
-                                                      n_group, topk_group, routed_scale, out_ids,
+    moe_route_kernel<false><<<grid, 128, 0, stream>>>(logits, ld, e_bias, T, E, k, mode, renorm,
+                                                      n_group, topk_group, group_top, routed_scale, out_ids,
                                                       out_w);
   return check_launch();
 }

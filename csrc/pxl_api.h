@@ -28,6 +28,7 @@ typedef struct CUstream_st* pxl_stream_t;
 #define PXL_EPI_SPLITK_C 7  // internal: small-M path, the K ranges of a tile form a cluster and reduce over DSMEM
 #define PXL_EPI_SPLITK_CN 8 // internal: mid-M path (operands not swapped), K ranges of a tile reduce inside a cluster
 #define PXL_EPI_GATE 9      // internal: C = (A W^T) * sigmoid(gate)      bf16 out (pxl_gemm_bf16_heads)
+#define PXL_EPI_GLU 11      // act(gate) * up (* sigmoid(row gate)), arranged alike (pxl_gemm_bf16_act_glu)
 #define PXL_EPI_CLIP_GLU 10 // clipped GLU of gate / up groups arranged as for PXL_EPI_SILU_MUL (pxl_gemm_bf16_glu)
 
 #define PXL_NORM_LAYER 0    // (x - mean) / sqrt(variance + eps)
@@ -56,6 +57,10 @@ int pxl_gemm_bf16_small_m(const void* A, const void* W, void* C, const void* res
 // W rows in groups of 128 (64 gate rows, the 64 up rows of the same outputs); C has N / 2 columns.
 int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, float limit,
                       int bn, int* status, pxl_stream_t stream);
+// Gated activation in the epilogue: C = act(g) u, act 0 = silu, 2 = gelu (tanh form); with row_gate (fp32) row m times
+// sigmoid(row_gate[m * ld_row_gate]). W and C as above.
+int pxl_gemm_bf16_act_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
+                          const float* row_gate, int64_t ld_row_gate, int bn, int* status, pxl_stream_t stream);
 // One product per attention head in one launch: for every head h < heads
 //   C[m, h * c_head + n] = sum_k A[m, h * a_head + k] * W[h * N + n, k]   (n < N, k < K)
 // optionally times sigmoid(gate[m, h * N + n]). bf16; K, N, strides and head offsets multiples of 8, pointers 16-byte
@@ -173,11 +178,11 @@ int pxl_sample(const void* logits, int logits_bf16, int64_t ld, int B, int V,
 
 // ---- moe.cu ------------------------------------------------------------------
 // Router: scores [T, E] fp32/bf16 logits -> top-k expert ids and weights.
-// mode 0: softmax then top-k (optionally renormalised); mode 1: sigmoid + per-expert
-// correction bias for selection, grouped top-k (n_group/topk_group, 1/1 = none),
-// weights = sigmoid scores renormalised and scaled by routed_scale.
-int pxl_moe_route(const void* logits, int logits_bf16, const float* e_bias, int T, int E, int k,
-                  int mode, int renorm, int n_group, int topk_group, float routed_scale,
+// Scores: softmax (mode 0) or sigmoid (mode 1). Selection by score + e_bias (optional), limited to the topk_group
+// best of n_group groups (1/1 = none; a group counts as the sum of its group_top best, group_top 1 or 2). Weights =
+// scores, optionally renormalised, times routed_scale. ld: elements between rows of logits.
+int pxl_moe_route(const void* logits, int64_t ld, int logits_bf16, const float* e_bias, int T, int E, int k,
+                  int mode, int renorm, int n_group, int topk_group, int group_top, float routed_scale,
                   int* out_ids, float* out_w, pxl_stream_t stream);
 
 int pxl_moe_align(const int* ids, int T, int k, int E, int e_lo, int e_hi, int* counts,
@@ -319,6 +324,10 @@ int pxl_msa_select(const float* scores, int64_t ld, const int* positions, const 
 int pxl_gemm_simt(const void* A, const void* W, void* C, const void* bias, const void* residual, const void* gate, int M,
                   int N, int K, int64_t lda, int64_t ldw, int64_t ldc, int64_t ldg, int heads, int64_t a_head,
                   int64_t c_head, int in_f32, int out_f32, pxl_stream_t stream);
+// Grouped form over the device tile lists of pxl_moe_align: C[r, :N] = A[a_rows ? a_rows[r] : r] . W_expert^T
+int pxl_gemm_simt_grouped(const void* A, const void* W, void* C, const int* a_rows, int N, int K, int64_t lda, int64_t ldw,
+                          int64_t ldc, const int* mt_expert, const int* mt_row0, const int* mt_row_end, const int* num_mt,
+                          int max_m_tiles, int is_f32, pxl_stream_t stream);
 
 // ---- residual.cu: fp32 residual stream -----------------------------------------------------------------
 // out[t] = table[ids[t]] * scale (+ hash[row]), row = (prev[t] * mul_prev + ids[t] * mul_cur) mod buckets, or
@@ -335,6 +344,48 @@ int pxl_row_norm(const float* x, const float* w, const int* rows, int64_t num_ro
                  int kind, int out_f32, int* status, pxl_stream_t stream);
 // fp32 form of pxl_act_mul
 int pxl_act_mul_f32(const float* x, float* out, int T, int I, int mode, float limit, pxl_stream_t stream);
+
+// x += y (+ sum_j weights[t, j] * (pos_of[t, j] >= 0 ? rows[pos_of[t, j]] : h[t])) in place; with a norm weight w:
+// low = x / sqrt(mean(x^2) + eps) * w. y, rows, h and low are bf16, or fp32 when y_f32.
+int pxl_residual_add(float* x, const void* y, int64_t ldy, const void* rows, int64_t ldr, int64_t num_rows,
+                     const int* pos_of, const float* weights, int k, const void* h, const float* w, void* low, int T, int W,
+                     float eps, int y_f32, int* status, pxl_stream_t stream);
+// out[t, c] = act(gate) * up (* sigmoid(row_gate[t * ldg])) of x [T, 2 I] with gate / up columns in alternating groups
+// of 64; mode 0 = silu, 2 = gelu (tanh form)
+int pxl_glu_act(const void* x, const float* row_gate, int64_t ldg, void* out, int64_t ldo, int T, int I, int mode, int is_f32,
+                pxl_stream_t stream);
+
+// ---- attn_prep.cu: in front of and behind softmax attention with grouped heads ---------------------------
+// proj [T, ld]: q (H x dk columns from q_off), k (G x dk), v (G x dv; G == 0: no keys and values). Convolution taps
+// conv_w [taps, q | k | v channels] (null: none) over each sequence's tokens with the state slots conv_state
+// [slots, taps - 1, channels]; RMS norm over the whole q and k rows; rotation of the first `rot` dimensions of a head
+// (pairs i, i + rot / 2). q_out [T, H, cols] and the pages get heads padded with zeros to `cols`. Sequences: seq_cu
+// [n + 1], the first prefill_seqs are slices (prefill_tokens tokens), each later one is one decoded token.
+int pxl_conv_qkv_prep(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int H, int G, int dk, int dv, int cols,
+                      int rot, int taps, const void* conv_w, void* conv_state, int num_state_slots, const float* q_norm,
+                      const float* k_norm, const float* cos_sin, const int* positions, int max_pos, const int* seq_cu,
+                      const int* seq_slots, int prefill_seqs, int prefill_tokens, int T, const int64_t* slots,
+                      int64_t num_slots, int page, void* k_cache, void* v_cache, void* q_out, float eps, int is_f32,
+                      int* status, pxl_stream_t stream);
+// out[t, h * dv + d] = x[t, h, d] (, RMS-normed over all heads * norm_w) * sigmoid(gate[t, h * dv + d]); columns up to
+// out_cols are zeroed. x [T, heads, x_cols].
+int pxl_gated_rows(const void* x, int heads, int x_cols, int dv, const void* gate, int64_t ldg, const float* norm_w, float eps,
+                   void* out, int64_t ldo, int out_cols, int T, int is_f32, pxl_stream_t stream);
+
+// ---- attention_any.cu: paged attention of any head size, bf16 or fp32, on the FMA pipes ------------------
+// Arguments as pxl_attn_prefill; cu_q null: token i is the only query of sequence i.
+int pxl_attn_any(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const int* block_tables,
+                 const int* cu_q, const int* ctx_lens, void* out, int64_t out_stride, const float* sinks, int B, int max_q,
+                 int Hq, int Hkv, int D, int page, int max_blocks, int64_t num_blocks, float scale, int window, int is_f32,
+                 int* status, pxl_stream_t stream);
+
+// ---- lightning_attn.cu: linear attention with a fixed decay per head ------------------------------------
+// q, k [T, H x dk] and v [T, H x dv] are columns of proj, all passed through silu here. state [slots, H, dk, dv] fp32,
+// decay_pow [H, pow_len = 65]: decay^0 .. decay^64. Sequences as for pxl_conv_qkv_prep.
+int pxl_lightning_attn(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int H, int dk, int dv,
+                       const float* decay_pow, int pow_len, float* state, int num_slots, const int* seq_cu,
+                       const int* seq_slots, const int* positions, void* out, int64_t ldo, int prefill_seqs, int decode_seqs,
+                       int is_f32, int* status, pxl_stream_t stream);
 
 // ---- latent_attn.cu / latent_attn_tc.cu: latent attention of any widths, window, sinks -------------------
 // proj [T, ld]: `heads` query heads of q_width columns (rotated part of R dims at q_rot_off) and, at kv_off, the raw

@@ -1,6 +1,7 @@
 // Rows of an fp32 residual stream: embedding (scaled, with an optional hashed second table), the update
-// x += mult * norm(y) * w fused with the low-precision copy the next product reads, norms of fp32 rows, and
-// activations in any precision. All statistics are fp32; the layer norm's variance is the mean of the squared
+// x += mult * norm(y) * w fused with the low-precision copy the next product reads, the update x += y + weighted
+// expert rows fused with the norm that the next layer starts with, norms of fp32 rows, and gated activations in any
+// precision. All statistics are fp32; the layer norm's variance is the mean of the squared
 // deviations from the mean (two passes over the row, which stays in registers when it is aligned).
 #include "common.cuh"
 #include "pxl_api.h"
@@ -236,6 +237,145 @@ int launch_norm(const NormArgs& a, int T, int kind, bool vec, cudaStream_t strea
 }
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
+// ---- x += y + sum of chosen experts' rows; low = RMSnorm(x) * w ------------------------------------------
+struct AddArgs {
+  float* x;
+  const void* y;         // [T, ldy]
+  int64_t ldy;
+  const void* rows;      // [P, ldr] expert outputs, or null
+  int64_t ldr, num_rows;
+  const int* pos_of;     // [T, k]: row of the pair in `rows`; negative: the identity expert, whose output is h[t]
+  const float* weights;  // [T, k]
+  int k;
+  const void* h;         // [T, W]
+  const float* w;        // norm weight, or null (no norm)
+  void* low;
+  int W;
+  float eps;
+  int* status;
+};
+
+template <typename T>
+__device__ __forceinline__ const T* expert_row(const AddArgs& a, int64_t t, int j) {
+  const int64_t r = a.pos_of[t * a.k + j];
+  if (r < 0) return static_cast<const T*>(a.h) + t * a.W;
+  if (r >= a.num_rows) {
+    if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_ROW_ID);
+    return static_cast<const T*>(a.h) + t * a.W;
+  }
+  return static_cast<const T*>(a.rows) + r * a.ldr;
+}
+
+// NV vectors of 8 elements per thread
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) residual_add_vec_kernel(const AddArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  float v[NV][8], f[8];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.W) {
+      load8(static_cast<const T*>(a.y) + t * a.ldy + c, v[i]);
+      load8(a.x + t * a.W + c, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] += f[j];
+    }
+  }
+  if (a.rows) {
+    for (int e = 0; e < a.k; ++e) {
+      const T* r = expert_row<T>(a, t, e);
+      const float g = a.weights[t * a.k + e];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * blockDim.x + threadIdx.x) * 8;
+        if (c < a.W) {
+          load8(r + c, f);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[i][j] = fmaf(g, f[j], v[i][j]);
+        }
+      }
+    }
+  }
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.W) {
+      store8(a.x + t * a.W + c, v[i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sq = fmaf(v[i][j], v[i][j], sq);
+    }
+  }
+  if (!a.w) return;
+  const float inv = 1.f / sqrtf(block_reduce_sum(sq, red) / a.W + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < a.W) {
+      load8(a.w + c, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= v[i][j] * inv;
+      store8(static_cast<T*>(a.low) + t * a.W + c, f);
+    }
+  }
+}
+
+// any width
+template <typename T>
+__global__ void __launch_bounds__(256) residual_add_any_kernel(const AddArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  float* x = a.x + t * a.W;
+  float sq = 0.f;
+  for (int c = threadIdx.x; c < a.W; c += blockDim.x) {
+    float v = x[c] + to_f(static_cast<const T*>(a.y)[t * a.ldy + c]);
+    if (a.rows)
+      for (int e = 0; e < a.k; ++e) v = fmaf(a.weights[t * a.k + e], to_f(expert_row<T>(a, t, e)[c]), v);
+    x[c] = v;
+    sq = fmaf(v, v, sq);
+  }
+  if (!a.w) return;
+  const float inv = 1.f / sqrtf(block_reduce_sum(sq, red) / a.W + a.eps);
+  for (int c = threadIdx.x; c < a.W; c += blockDim.x) put(static_cast<T*>(a.low) + t * a.W + c, x[c] * inv * a.w[c]);
+}
+
+template <typename T>
+int launch_add(const AddArgs& a, int rows, bool vec, cudaStream_t stream) {
+  if (vec && a.W % 8 == 0 && a.W <= 256 * 8 * 8) {
+    const int nvec = a.W / 8, threads = nvec >= 256 ? 256 : ceil_div(nvec, 32) * 32, per = ceil_div(nvec, threads);
+    const dim3 g(rows), b(threads);
+    if (per <= 1) pxl_host::launch(residual_add_vec_kernel<T, 1>, g, b, 0, stream, a);
+    else if (per <= 2) pxl_host::launch(residual_add_vec_kernel<T, 2>, g, b, 0, stream, a);
+    else if (per <= 4) pxl_host::launch(residual_add_vec_kernel<T, 4>, g, b, 0, stream, a);
+    else pxl_host::launch(residual_add_vec_kernel<T, 8>, g, b, 0, stream, a);
+  } else {
+    pxl_host::launch(residual_add_any_kernel<T>, dim3(rows), dim3(256), 0, stream, a);
+  }
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
+// ---- gated activation of gate / up columns interleaved in groups of 64 --------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) glu_act_kernel(const T* __restrict__ x, const float* __restrict__ row_gate, int64_t ldg,
+                                                      T* __restrict__ out, int64_t ldo, int I, int64_t n, int mode) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  if (i >= n) return;
+  const int64_t t = i / I, c = i % I, col = c / 64 * 128 + c % 64;
+  const float g = to_f(x[t * 2 * I + col]), u = to_f(x[t * 2 * I + col + 64]);
+  // gelu, tanh form: z (1 + tanh(s)) / 2 = z / (1 + exp(-2 s))
+  const float s = mode == 2 ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;
+  float y = g / (1.f + expf(-s)) * u;
+  if (row_gate) y /= 1.f + expf(-row_gate[t * ldg]);
+  put(out + t * ldo + c, y);
+}
+
 // ---- clipped GLU and friends in fp32 -------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) act_mul_f32_kernel(const float* __restrict__ x, float* __restrict__ out, int I,
                                                           int64_t n, int mode, float limit) {
@@ -307,5 +447,31 @@ PXL_EXPORT int pxl_act_mul_f32(const float* x, float* out, int T, int I, int mod
   const int64_t n = static_cast<int64_t>(T) * I;
   pxl_host::launch(act_mul_f32_kernel, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0, stream, x, out, I, n,
                    mode, limit);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
+PXL_EXPORT int pxl_residual_add(float* x, const void* y, int64_t ldy, const void* rows, int64_t ldr, int64_t num_rows,
+                                const int* pos_of, const float* weights, int k, const void* h, const float* w, void* low,
+                                int T, int W, float eps, int y_f32, int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (W <= 0 || (w && !low) || (rows && (!pos_of || !weights || !h || k <= 0))) return PXL_ERR_INVALID_ARG;
+  const AddArgs a{x, y, ldy, rows, ldr, num_rows, pos_of, weights, k, h, w, low, W, eps, status};
+  const bool vec = aligned16(x) && aligned16(y) && aligned16(rows) && aligned16(h) && aligned16(w) && aligned16(low) &&
+                   ldy % 8 == 0 && ldr % 8 == 0;
+  return y_f32 ? launch_add<float>(a, T, vec, stream) : launch_add<pxl::bf16>(a, T, vec, stream);
+}
+
+PXL_EXPORT int pxl_glu_act(const void* x, const float* row_gate, int64_t ldg, void* out, int64_t ldo, int T, int I, int mode,
+                           int is_f32, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (I <= 0 || I % 64 || (mode != 0 && mode != 2)) return PXL_ERR_INVALID_ARG;
+  const int64_t n = static_cast<int64_t>(T) * I;
+  const dim3 grid(static_cast<unsigned>((n + 255) / 256));
+  if (is_f32)
+    pxl_host::launch(glu_act_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(x), row_gate, ldg,
+                     static_cast<float*>(out), ldo, I, n, mode);
+  else
+    pxl_host::launch(glu_act_kernel<pxl::bf16>, grid, dim3(256), 0, stream, static_cast<const pxl::bf16*>(x), row_gate, ldg,
+                     static_cast<pxl::bf16*>(out), ldo, I, n, mode);
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }

@@ -46,6 +46,8 @@ def _nvcc() -> str:
 # that only runs this family compiles these into a library of their own.
 FAMILY_SOURCES = {
     "latent": ["elementwise", "gemm_simt", "gemm_tcgen05", "latent_attn", "latent_attn_tc", "residual", "sampler"],
+    "parallel_block": ["attention", "attention_any", "attention_prefill_tc", "attn_prep", "elementwise", "gemm_simt",
+                       "gemm_tcgen05", "lightning_attn", "moe", "residual", "sampler"],
 }
 
 

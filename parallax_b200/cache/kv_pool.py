@@ -3,12 +3,16 @@
 One cache object per decoder layer, chosen by layer kind (same taxonomy as the reference's
 hybrid cache, ``src/parallax/server/cache_manager.py:188-259``):
 
-* ``attention``      K, V            ``[blocks, Hkv, page, D]``
+* ``attention``      K, V            ``[blocks, Hkv, page, D]`` (heads and columns may differ from layer to layer; none
+                     for a layer that reads another layer's)
 * ``mla_attention``  latent | rope   ``[blocks, 1, page, kv_lora + rope]`` (one tensor; the widths may differ
                      from layer to layer)
 * ``dsa_attention``  MLA cache + lightning-indexer keys ``[blocks, 1, page, index_dim]``
 * ``linear``         conv state ``[slots, conv_dim, k-1]`` + recurrent state
                      ``[slots, Hv, Dv, Dk]`` (per request slot, not paged)
+
+Any layer may keep per-request slots beside its pages (``ModelConfig.slot_dims``), e.g. the window of a short
+convolution in front of softmax attention.
 
 Layouts are chosen for the sm_100a kernels (whole pages of one head are contiguous), not
 for compatibility with the reference's Metal layouts.
@@ -21,8 +25,7 @@ from typing import Optional
 
 import torch
 
-from parallax_b200.models.config import (ATTENTION, DSA_ATTENTION, LINEAR, MLA_ATTENTION,
-                                         MSA_ATTENTION, ModelConfig)
+from parallax_b200.models.config import ATTENTION, DSA_ATTENTION, MLA_ATTENTION, MSA_ATTENTION, ModelConfig
 
 
 @dataclass
@@ -57,12 +60,13 @@ def kv_cache_torch_dtype(name: Optional[str], model_dtype):
     raise ValueError(f"unknown KV cache dtype {name!r} (auto, bf16, fp8_e4m3)")
 
 
-def linear_dims(cfg: ModelConfig, tp: int = 1) -> tuple[int, int, int, int, int]:
-    """(conv_dim, conv_kernel-1, num_v_heads, v_head_dim, k_head_dim) of a gated-delta layer."""
-    hk, hv = cfg.linear_num_key_heads // tp, cfg.linear_num_value_heads // tp
-    dk, dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
-    conv_dim = 2 * hk * dk + hv * dv
-    return conv_dim, max(cfg.linear_conv_kernel_dim - 1, 0), hv, dv, dk
+def slot_dims(cfg: ModelConfig, layer: int, tp: int = 1) -> tuple:
+    """``ModelConfig.slot_dims`` of one tensor-parallel rank, ``(None, None)`` for a layer without slots."""
+    conv, rec = cfg.slot_dims(layer) or (None, None)
+    if tp > 1:
+        conv = conv and (conv[0] // tp, conv[1])
+        rec = rec and (rec[0] // tp, *rec[1:])
+    return conv, rec
 
 
 def bytes_per_block(cfg: ModelConfig, start: int, end: int, page: int, elem: int = 2, tp: int = 1,
@@ -73,8 +77,8 @@ def bytes_per_block(cfg: ModelConfig, start: int, end: int, page: int, elem: int
     for li in range(start, end):
         kind = cfg.layer_kind(li)
         if kind in (ATTENTION, MSA_ATTENTION):
-            hkv = max(1, cfg.num_key_value_heads // tp)
-            total += 2 * hkv * page * cfg.head_dim * kv_elem
+            heads, cols = cfg.kv_dims(li) or (0, 0)
+            total += 2 * (heads and max(1, heads // tp)) * page * cols * kv_elem
             if kind == MSA_ATTENTION:
                 total += page * int(cfg.raw.get("index_head_dim") or 0) * elem
         elif kind in (MLA_ATTENTION, DSA_ATTENTION):
@@ -87,9 +91,8 @@ def bytes_per_block(cfg: ModelConfig, start: int, end: int, page: int, elem: int
 def bytes_per_linear_slot(cfg: ModelConfig, start: int, end: int, elem: int = 2, tp: int = 1) -> int:
     total = 0
     for li in range(start, end):
-        if cfg.layer_kind(li) == LINEAR:
-            conv_dim, km1, hv, dv, dk = linear_dims(cfg, tp)
-            total += conv_dim * km1 * elem + hv * dv * dk * 4
+        conv, rec = slot_dims(cfg, li, tp)
+        total += (conv[0] * conv[1] * elem if conv else 0) + (rec[0] * rec[1] * rec[2] * 4 if rec else 0)
     return total
 
 
@@ -112,10 +115,11 @@ class KVPool:
             kind = cfg.layer_kind(li)
             lc = LayerCache(kind)
             if kind in (ATTENTION, MSA_ATTENTION):
-                hkv = max(1, cfg.num_key_value_heads // tp)
-                shape = (num_blocks, hkv, page_size, cfg.head_dim)
-                lc.k = torch.zeros(shape, device=self.device, dtype=kv_dt)
-                lc.v = torch.zeros(shape, device=self.device, dtype=kv_dt)
+                dims = cfg.kv_dims(li)
+                if dims is not None:
+                    shape = (num_blocks, max(1, dims[0] // tp), page_size, dims[1])
+                    lc.k = torch.zeros(shape, device=self.device, dtype=kv_dt)
+                    lc.v = torch.zeros(shape, device=self.device, dtype=kv_dt)
                 if kv_dt == torch.float8_e4m3fn:
                     lc.k_scale, lc.v_scale = float(kv_scale[0]), float(kv_scale[1])
                 if kind == MSA_ATTENTION:
@@ -127,24 +131,23 @@ class KVPool:
                 if kind == DSA_ATTENTION:
                     lc.index_k = torch.zeros((num_blocks, 1, page_size, cfg.index_head_dim),
                                              device=self.device, dtype=dtype)
-            elif kind == LINEAR:
-                conv_dim, km1, hv, dv, dk = linear_dims(cfg, tp)
-                lc.conv_state = torch.zeros((num_linear_slots, conv_dim, km1), device=self.device, dtype=dtype)
-                lc.rec_state = torch.zeros((num_linear_slots, hv, dv, dk), device=self.device,
-                                           dtype=torch.float32)
+            conv, rec = slot_dims(cfg, li, tp)
+            if conv is not None:
+                lc.conv_state = torch.zeros((num_linear_slots, *conv), device=self.device, dtype=dtype)
+            if rec is not None:
+                lc.rec_state = torch.zeros((num_linear_slots, *rec), device=self.device, dtype=torch.float32)
             self.layers.append(lc)
 
     def zero_slot(self, slot: int) -> None:
-        for lc in self.layers:
-            if lc.kind == LINEAR:
-                lc.conv_state[slot].zero_()
-                lc.rec_state[slot].zero_()
+        for t in self._slot_tensors():
+            t[slot].zero_()
 
     def copy_slot(self, dst: int, src: int) -> None:
-        for lc in self.layers:
-            if lc.kind == LINEAR:
-                lc.conv_state[dst].copy_(lc.conv_state[src])
-                lc.rec_state[dst].copy_(lc.rec_state[src])
+        for t in self._slot_tensors():
+            t[dst].copy_(t[src])
+
+    def _slot_tensors(self):
+        return [t for lc in self.layers for t in (lc.conv_state, lc.rec_state) if t is not None]
 
     def nbytes(self) -> int:
         n = 0

@@ -25,10 +25,10 @@ def plan_kv_blocks(cfg: ModelConfig, start: int, end: int, page_size: int, devic
 
     kv_elem = torch.empty(0, dtype=kv_cache_torch_dtype(kv_cache_dtype, dtype)).element_size()
     per_block = bytes_per_block(cfg, start, end, page_size, torch.empty(0, dtype=dtype).element_size(), tp, kv_elem)
-    if per_block == 0:
-        return 0
     if device.type != "cuda":
         n = cpu_default_blocks
+    elif per_block == 0:        # no layer of the stage has pages: block ids cost nothing here
+        n = 1 << 16
     else:
         free, _total = torch.cuda.mem_get_info(device)
         n = int(free * fraction) // per_block

@@ -103,6 +103,24 @@ class ModelConfig:
             return m.kv_rank, m.rot_dim
         return self.kv_lora_rank, self.qk_rope_head_dim
 
+    def kv_dims(self, layer_idx: int) -> Optional[tuple[int, int]]:
+        """(heads, columns per head) of a softmax-attention layer's cached keys and values; None for a layer that
+        reads another layer's."""
+        if self.layer_specs:
+            return self.layer_specs[layer_idx].mixer.kv_dims
+        return self.num_key_value_heads, self.head_dim
+
+    def slot_dims(self, layer_idx: int) -> Optional[tuple]:
+        """What a layer keeps per request instead of per token: ``(shape of a short convolution's last inputs or None,
+        shape of a recurrent state or None)``; None for a layer that keeps nothing."""
+        if self.layer_specs:
+            return self.layer_specs[layer_idx].mixer.slot_dims
+        if self.layer_kind(layer_idx) != LINEAR:
+            return None
+        hk, hv = self.linear_num_key_heads, self.linear_num_value_heads
+        dk, dv = self.linear_key_head_dim, self.linear_value_head_dim
+        return (2 * hk * dk + hv * dv, max(self.linear_conv_kernel_dim - 1, 0)), (hv, dv, dk)
+
     @property
     def is_moe(self) -> bool:
         return self.num_experts > 0
@@ -128,6 +146,8 @@ class ModelConfig:
     def layer_is_moe(self, layer_idx: int) -> bool:
         if not self.is_moe:
             return False
+        if self.layer_specs:
+            return hasattr(self.layer_specs[layer_idx].mlp, "experts")
         if layer_idx in self.mlp_only_layers:
             return False
         if layer_idx < self.first_k_dense_replace:
@@ -135,6 +155,8 @@ class ModelConfig:
         return (layer_idx + 1) % max(1, self.moe_layer_freq) == 0 if self.moe_layer_freq > 1 else True
 
     def layer_kind(self, layer_idx: int) -> str:
+        if self.layer_specs:
+            return self.layer_specs[layer_idx].mixer.kind
         if self.layer_types and layer_idx < len(self.layer_types):
             if self.layer_types[layer_idx] == "linear_attention":
                 return LINEAR
@@ -151,7 +173,8 @@ class ModelConfig:
 
     @property
     def has_linear_layers(self) -> bool:
-        return any(self.layer_kind(i) == LINEAR for i in range(self.num_hidden_layers))
+        """Whether some layer keeps a state per request (recurrent state, window of a short convolution)."""
+        return any(self.slot_dims(i) is not None for i in range(self.num_hidden_layers))
 
     def layer_window(self, layer_idx: int) -> int:
         if self.layer_specs:
@@ -164,8 +187,14 @@ class ModelConfig:
 
     def kv_bytes_per_token_per_layer(self, elem_bytes: int = 2) -> int:
         if self.layer_specs:      # the mean over the layers
-            return -(-sum(sum(self.latent_dims(i)) for i in range(self.num_hidden_layers)) * elem_bytes
-                     // self.num_hidden_layers)
+            rows = 0
+            for i in range(self.num_hidden_layers):
+                if self.layer_kind(i) == MLA_ATTENTION:
+                    rows += sum(self.latent_dims(i))
+                elif self.kv_dims(i) is not None:
+                    heads, cols = self.kv_dims(i)
+                    rows += 2 * heads * cols
+            return -(-rows * elem_bytes // self.num_hidden_layers)
         if self.is_mla:
             return (self.kv_lora_rank + self.qk_rope_head_dim) * elem_bytes
         return 2 * self.num_key_value_heads * self.head_dim * elem_bytes
@@ -195,22 +224,30 @@ def config_from_layer_list(cfg: dict) -> ModelConfig:
     """Config whose ``layers`` entry describes every layer by itself (see ``models/layer_spec.py``). The scalar
     sizes of :class:`ModelConfig` hold the largest value of any layer: capacity estimates use them, the model
     itself reads ``layer_specs``."""
-    from parallax_b200.models.layer_spec import parse_bigram, parse_layer
+    from parallax_b200.models.layer_spec import parse_bigram, parse_layers
 
-    specs = [parse_layer(e) for e in cfg["layers"]]
+    specs = parse_layers(cfg["architecture"], cfg["layers"])
     if not specs:
         raise ValueError("a layer-list config needs at least one layer")
     emb = cfg.get("embedding") or {}
-    top = lambda f: max(f(s.mixer) for s in specs)  # noqa: E731
-    heads = top(lambda m: m.heads)
+    mlps = [s.mlp for s in specs if s.mlp]
+
+    def top(objs, name):
+        return max((getattr(o, name, None) or 0 for o in objs), default=0)
+
+    mixers = [s.mixer for s in specs]
+    latent, routed = [m for m in mixers if m.kind == MLA_ATTENTION], [m for m in mlps if hasattr(m, "experts")]
     return ModelConfig(
         architecture=cfg["architecture"], model_type=str(cfg["architecture"]).lower(), hidden_size=int(cfg["width"]),
-        num_hidden_layers=len(specs), num_attention_heads=heads, num_key_value_heads=heads,
-        head_dim=top(lambda m: m.q_width), intermediate_size=max([s.mlp.ff for s in specs if s.mlp] or [0]),
-        vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]), rope_theta=specs[0].mixer.rot.base,
+        num_hidden_layers=len(specs), num_attention_heads=top(mixers, "heads"), num_key_value_heads=top(mixers, "kv_heads"),
+        head_dim=top(mixers, "q_width"), intermediate_size=top(mlps, "ff"),
+        vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]),
+        rope_theta=next((m.rot.base for m in mixers if hasattr(m, "rot")), 1e4),
         max_position_embeddings=int(cfg.get("max_position_embeddings") or 32768),
-        kv_lora_rank=top(lambda m: m.kv_rank), qk_nope_head_dim=top(lambda m: m.dim),
-        qk_rope_head_dim=top(lambda m: m.rot_dim), v_head_dim=top(lambda m: m.vdim),
+        kv_lora_rank=top(latent, "kv_rank"), qk_nope_head_dim=top(latent, "dim"),
+        qk_rope_head_dim=top(latent, "rot_dim"), v_head_dim=top(mixers, "vdim"),
+        num_experts=top(routed, "experts"), num_experts_per_tok=top(routed, "top"), moe_intermediate_size=top(routed, "ff"),
+        shared_expert_intermediate_size=top([m.shared for m in routed], "ff"),
         layer_specs=specs, embedding_scale=float(emb.get("scale", 1.0)), bigram=parse_bigram(emb),
         residual_mult=float(cfg.get("residual_mult", 1.0)), raw=cfg)
 

@@ -327,7 +327,8 @@ class DecoderStage(ExpertParallelMixin):
         slots = self._route_slots
         if slots is not None and slots.shape[0] == ids.shape[0]:
             # rows without a KV slot (negative) are parked in the last row of the buffer, which no request reads
-            self.routed_buf[torch.where(slots < 0, self.routed_buf.shape[0] - 1, slots), j] = ids.to(torch.int16)
+            rows = torch.where(slots < 0, self.routed_buf.shape[0] - 1, slots)
+            self.routed_buf[rows, j, :ids.shape[1]] = ids.to(torch.int16)     # (layers may choose fewer; -1 behind)
 
     def routed_experts_of(self, slots: torch.Tensor) -> torch.Tensor:
         """``[len(slots), MoE layers, top-k]`` for the given KV slots (int64, on this device)."""

@@ -22,64 +22,24 @@ cores; fp32 where the design keeps fp32) or entirely in fp32 (``dtype=torch.floa
 
 from __future__ import annotations
 
-import re
-from typing import Optional
-
 import torch
 
 from parallax_b200 import ops
 from parallax_b200.engine.batch import ForwardBatch
-from parallax_b200.models.config import ModelConfig
-from parallax_b200.models.decoder import DecoderStage
-from parallax_b200.models.layer_spec import LayerSpec, RotarySpec
+from parallax_b200.models.layer_list import LayerListStage, ListedLayer, pad_rows
 
 
-def _pad_rows(w: torch.Tensor, multiple: int) -> torch.Tensor:
-    extra = -w.shape[0] % multiple
-    if not extra:
-        return w.contiguous()
-    return torch.cat([w, w.new_zeros((extra,) + tuple(w.shape[1:]))], 0).contiguous()
+class LatentLayer(ListedLayer):
+    __slots__ = ("w_in", "kv_norm", "w_uk_s", "w_uv", "sinks", "w_o", "norm1", "norm2", "w_gu", "w_down", "moe")
 
 
-class LatentLayer:
-    __slots__ = ("spec", "layer_idx", "cos_sin", "w_in", "kv_norm", "w_uk_s", "w_uv", "sinks", "w_o", "norm1", "norm2",
-                 "w_gu", "w_down", "moe")
+class LatentStage(LayerListStage):
+    layer_class = LatentLayer
 
-    def __init__(self):
-        for s in self.__slots__:
-            setattr(self, s, None)
-
-
-class LatentStage(DecoderStage):
-    _LAYER_KEY = re.compile(r"(?:^|\.)l(\d+)\.")
-    _GLOBAL_KEYS = ("embed", "bigram", "final.norm", "head")
-    _GLOBAL_TENSORS = ("embed", "bigram", "norm_w", "lm_head")
-
-    def __init__(self, cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype=None,
-                 max_positions: Optional[int] = None):
-        super().__init__(cfg, start_layer, end_layer, device, dtype, max_positions)
-        if self.dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"{cfg.architecture} runs in bfloat16 or float32, not {self.dtype}")
-        del self.lora                   # no per-request adapters for this family (checked with hasattr)
-        self.bigram: Optional[torch.Tensor] = None
-        self.layers = [LatentLayer() for _ in range(start_layer, end_layer)]
-        self.cos_sin = None             # tables are per layer: base and width are
-        self._tables: dict[RotarySpec, torch.Tensor] = {}
-        for gi, lw in enumerate(self.layers, start_layer):
-            self._describe(lw, gi)
+    def __init__(self, *args, **kwargs):
+        super().__init__(*args, **kwargs)
         # gate / up rows interleaved for the fused epilogue, or stacked for the separate activation kernel
-        self.fused_glu = self.dtype == torch.bfloat16 and cfg.hidden_size % 8 == 0
-
-    @property
-    def hidden_dtype(self) -> torch.dtype:
-        return torch.float32
-
-    def _describe(self, lw: LatentLayer, gi: int) -> None:
-        lw.layer_idx, lw.spec = gi, self.cfg.layer_specs[gi]
-        rot = lw.spec.mixer.rot
-        if rot not in self._tables:
-            self._tables[rot] = ops.build_cos_sin(self.max_positions, rot.dims, rot.base, device=self.device)
-        lw.cos_sin = self._tables[rot]
+        self.fused_glu = self.dtype == torch.bfloat16 and self.cfg.hidden_size % 8 == 0
 
     # ------------------------------------------------------------------ weights
     def weight_shapes(self, gi: int) -> dict[str, tuple]:
@@ -95,67 +55,13 @@ class LatentStage(DecoderStage):
                        p + "mlp.down": (W, spec.mlp.ff)})
         return sh
 
-    def init_random(self, seed: int = 0, std: float = 0.02) -> None:
-        cfg, dev = self.cfg, self.device
-        g = torch.Generator(device=dev)
-
-        def rnd(shape, k):
-            g.manual_seed(seed * 1000003 + k)
-            return (torch.randn(*shape, generator=g, device=dev, dtype=torch.float32) * std).to(torch.bfloat16)
-
-        W = cfg.hidden_size
-        tensors = {}
-        if self.is_first:
-            tensors["embed"] = rnd((cfg.vocab_size, W), 900001)
-            if cfg.bigram is not None:
-                tensors["bigram"] = rnd((cfg.bigram.buckets + 1, W), 900003)
-        if self.is_last:
-            tensors["final.norm"], tensors["head"] = torch.ones(W, device=dev), rnd((cfg.vocab_size, W), 900002)
-        self._load_globals(tensors)
-        for gi, lw in enumerate(self.layers, self.start_layer):      # layer by layer: one raw copy at a time
-            layer = {name: (torch.ones(shape, device=dev) if "norm" in name else rnd(shape, gi * 32 + i))
-                     for i, (name, shape) in enumerate(self.weight_shapes(gi).items())}
-            self._load_layer(lw, gi, layer)
-
-    def load_weights(self, tensors: dict[str, torch.Tensor]) -> None:
-        self._load_globals(tensors)
-        for gi, lw in enumerate(self.layers, self.start_layer):
-            self._load_layer(lw, gi, tensors)
-
-    @staticmethod
-    def _take(tensors, name: str, shape: tuple) -> torch.Tensor:
-        t = tensors.get(name)
-        if t is None:
-            raise KeyError(f"missing weight {name}")
-        if tuple(t.shape) != tuple(shape):
-            raise ValueError(f"weight {name} has shape {tuple(t.shape)}, the config says {tuple(shape)}")
-        return t
-
-    def _load_globals(self, tensors) -> None:
-        cfg, W = self.cfg, self.cfg.hidden_size
-
-        def get(name, shape, dtype=self.dtype):
-            return self._take(tensors, name, shape).to(device=self.device, dtype=dtype).contiguous()
-
-        if self.is_first:
-            self.embed = get("embed", (cfg.vocab_size, W))
-            if cfg.bigram is not None:
-                self.bigram = get("bigram", (cfg.bigram.buckets + 1, W))
-        if self.is_last:
-            self.norm_w = get("final.norm", (W,), torch.float32)
-            self.lm_head = _pad_rows(get("head", (cfg.vocab_size, W)), 8)
-
     def _load_layer(self, lw: LatentLayer, gi: int, tensors) -> None:
         self._describe(lw, gi)
-        spec: LayerSpec = lw.spec
-        m, p = spec.mixer, f"l{gi}."
-        shapes = self.weight_shapes(gi)
-
-        def get(name, dtype=self.dtype):
-            return self._take(tensors, p + name, shapes[p + name]).to(device=self.device, dtype=dtype).contiguous()
+        spec, get = lw.spec, self._getter(gi, tensors)
+        m = spec.mixer
 
         # the three products that read x, one matrix: queries | latent and rotated key | output gate
-        lw.w_in = torch.cat([_pad_rows(get("mix." + n), 8) for n in ("q", "dkv", "g")], 0).contiguous()
+        lw.w_in = torch.cat([pad_rows(get("mix." + n), 8) for n in ("q", "dkv", "g")], 0).contiguous()
         lw.kv_norm = get("mix.dkv.norm", torch.float32)
         # score = (W_uk^T q) . c: the key up-projection acts on the query
         lw.w_uk_s = get("mix.uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(-1, m.dim).contiguous()
@@ -166,32 +72,16 @@ class LatentStage(DecoderStage):
         if spec.mlp is not None:
             lw.norm2 = get("norm2", torch.float32)
             if self.fused_glu:
-                gate, up = _pad_rows(get("mlp.gate"), 64), _pad_rows(get("mlp.up"), 64)
+                gate, up = pad_rows(get("mlp.gate"), 64), pad_rows(get("mlp.up"), 64)
                 lw.w_gu = ops.interleave_gate_up(gate, up)
             else:
-                gate, up = _pad_rows(get("mlp.gate"), 8), _pad_rows(get("mlp.up"), 8)
+                gate, up = pad_rows(get("mlp.gate"), 8), pad_rows(get("mlp.up"), 8)
                 lw.w_gu = torch.cat([gate, up], 0)
             # padded rows give activations of zero; the down projection gets zero columns for them
             down = get("mlp.down")
             lw.w_down = torch.nn.functional.pad(down, (0, gate.shape[0] - spec.mlp.ff)).contiguous()
 
-    def update_weights(self, tensors) -> int:
-        """Online refit: layers named in ``tensors`` are rebuilt by the loader and moved into the live weights."""
-        return self.reload_layers(tensors)
-
-    def weight_bytes(self) -> int:
-        ts = [self.embed, self.bigram, self.norm_w, self.lm_head]
-        ts += [getattr(lw, s) for lw in self.layers for s in LatentLayer.__slots__ if s != "cos_sin"]
-        return sum(t.numel() * t.element_size() for t in ts if isinstance(t, torch.Tensor))
-
     # ------------------------------------------------------------------ forward
-    def embed_tokens(self, fb: ForwardBatch) -> torch.Tensor:
-        b = self.cfg.bigram
-        if b is None:
-            return ops.embed_rows(self.embed, fb.input_ids, self.cfg.embedding_scale)
-        return ops.embed_rows(self.embed, fb.input_ids, self.cfg.embedding_scale, self.bigram, fb.prev_ids,
-                              b.mul_prev, b.mul_cur, b.buckets)
-
     def _mixer(self, lw: LatentLayer, li: int, xl: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
         m, T = lw.spec.mixer, xl.shape[0]
         L, R = m.kv_rank, m.rot_dim
@@ -233,8 +123,3 @@ class LatentStage(DecoderStage):
             if lw.spec.mlp is not None:
                 xl = ops.residual_norm(h, self._feed_forward(lw, xl), lw.norm2, eps, mult)
         return h
-
-    def logits(self, h: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
-        rows = fb.logit_rows if fb.num_logits else None
-        hn = ops.row_norm(h[:0] if rows is None else h, self.norm_w, self.cfg.rms_norm_eps, rows=rows, dtype=self.dtype)
-        return ops.linear(hn, self.lm_head, epi=ops.EPI_F32)[:, :self.cfg.vocab_size]

@@ -33,6 +33,8 @@ _REGISTRY: dict[str, str] = {
     "Qwen3_5MoeForConditionalGeneration": "hybrid",
     # layer-list configs: windowed latent attention
     "Piburax": "latent",
+    # layer-list configs: attention / lightning layers beside (not before) their feed-forward
+    "Zudepel": "parallel_block",
     # block-sparse (MSA)
     "MiniMaxM3SparseForCausalLM": "msa",
 }
@@ -51,7 +53,7 @@ def family_of(arch: str) -> str:
 
 def runs_in_float32(arch: str) -> bool:
     """Whether the family's GPU stages also run in 32-bit throughout (``dtype=torch.float32``)."""
-    return family_of(arch) == "latent"
+    return family_of(arch) in ("latent", "parallel_block")
 
 
 def build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype, max_positions=None,
@@ -71,12 +73,14 @@ def build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtyp
 def _build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype, max_positions, tp_rank, tp_size,
                  tp_group, comm):
     fam = family_of(cfg.architecture)
-    if fam == "latent":
+    if fam in ("latent", "parallel_block"):
         from parallax_b200.models.latent import LatentStage
+        from parallax_b200.models.parallel_block import ParallelBlockStage
 
         if tp_size > 1:
             raise ValueError(f"tensor parallelism is not available for {cfg.architecture}; use pipeline stages")
-        return LatentStage(cfg, start_layer, end_layer, device, dtype, max_positions=max_positions)
+        cls = LatentStage if fam == "latent" else ParallelBlockStage
+        return cls(cfg, start_layer, end_layer, device, dtype, max_positions=max_positions)
     if tp_size > 1 and fam != "decoder":
         from parallax_b200.models import tp_families
 

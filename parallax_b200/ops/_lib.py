@@ -84,7 +84,7 @@ _SIGS = {
                          c_int, c_int, c_int, c_int, c_int64, c_float, c_int, _P, _P],
     "pxl_attn_prefill_tc": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int, c_int,
                             c_int, c_int, c_int, c_int, c_int64, c_float, c_int, _P, _P],
-    "pxl_moe_route": [_P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, _P],
+    "pxl_moe_route": [_P, c_int64, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, _P],
     "pxl_moe_align": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, _P],
     "pxl_moe_gather": [_P, _P, _P, _P, c_int, c_int, _P],
     "pxl_moe_combine": [_P, _P, _P, _P, _P, c_int, c_int, c_int, _P],
@@ -126,6 +126,17 @@ _SIGS = {
     "pxl_latent_attn_tc_supported": [c_int, c_int, c_int, c_float],
     "pxl_latent_attn_tc": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64,
                            c_float, c_int, _P, _P],
+    "pxl_gemm_bf16_act_glu": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int64, c_int, _P, _P],
+    "pxl_gemm_simt_grouped": [_P, _P, _P, _P, c_int, c_int, c_int64, c_int64, c_int64, _P, _P, _P, _P, c_int, c_int, _P],
+    "pxl_residual_add": [_P, _P, c_int64, _P, c_int64, c_int64, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_float, c_int, _P, _P],
+    "pxl_glu_act": [_P, _P, c_int64, _P, c_int64, c_int, c_int, c_int, c_int, _P],
+    "pxl_conv_qkv_prep": [_P, c_int64] + [c_int] * 10 + [_P, _P, c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P,
+                          c_int64, c_int, _P, _P, _P, c_float, c_int, _P, _P],
+    "pxl_gated_rows": [_P, c_int, c_int, c_int, _P, c_int64, _P, c_float, _P, c_int64, c_int, c_int, c_int, _P],
+    "pxl_attn_any": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64,
+                     c_float, c_int, c_int, _P, _P],
+    "pxl_lightning_attn": [_P, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, _P, c_int64,
+                           c_int, c_int, c_int, _P, _P],
     "pxl_rmsnorm_strided": [_P, c_int64, _P, _P, c_int64, c_int, c_int, c_float, c_float, _P],
     "pxl_argmax": [_P, c_int, c_int64, c_int, c_int, _P, _P, _P, _P],
     "pxl_apply_penalties": [_P, c_int, c_int64, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P],

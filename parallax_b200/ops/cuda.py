@@ -410,6 +410,24 @@ def add_inplace(y: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------ attention
+def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, window, sinks, out):
+    """FMA-pipe form: fp32, any head size, any number of query heads per key head."""
+    T, Hq, D = q.shape
+    Hkv, page = k_cache.shape[1], k_cache.shape[2]
+    assert k_cache.dtype == v_cache.dtype == q.dtype and out.stride(2) == 1 and out.stride(1) == D
+    check(_lib.lib().pxl_attn_any(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
+                                  _ptr(cu_q), ctx_lens.data_ptr(), out.data_ptr(), out.stride(0), _ptr(sinks),
+                                  ctx_lens.numel(), max_q, Hq, Hkv, D, page, block_tables.shape[1], k_cache.shape[0],
+                                  float(scale), window, int(q.dtype == torch.float32), status_tensor(q.device).data_ptr(),
+                                  _stream(q.device)), "pxl_attn_any")
+    _count()
+    return out
+
+
+def _attn_on_tensor_cores(q, k_cache, scale: float, max_group: int) -> bool:
+    return q.dtype == torch.bfloat16 and q.shape[2] in (64, 128) and q.shape[1] // k_cache.shape[1] <= max_group and scale > 0
+
+
 def attn_decode(
     q: torch.Tensor,
     k_cache: torch.Tensor,
@@ -431,6 +449,8 @@ def attn_decode(
     Hkv, page = k_cache.shape[1], k_cache.shape[2]
     if out is None:
         out = torch.empty((B, Hq, D), dtype=q.dtype, device=q.device)
+    if not _is_fp8_cache(k_cache) and not _attn_on_tensor_cores(q, k_cache, scale, 16):
+        return _attn_any(q, k_cache, v_cache, block_tables, None, ctx_lens, 1, scale, window, sinks, out)
     if max_ctx <= 0:
         max_ctx = block_tables.shape[1] * page
     if num_splits <= 0:
@@ -485,6 +505,8 @@ def attn_prefill(
     B = ctx_lens.numel()
     if T == 0 or B == 0:
         return out
+    if not _is_fp8_cache(k_cache) and not _attn_on_tensor_cores(q, k_cache, scale, 64):
+        return _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window, sinks, out)
     if _is_fp8_cache(k_cache):
         check(
             _lib.lib().pxl_attn_prefill_fp8(
@@ -577,14 +599,14 @@ def sample(
 
 # ------------------------------------------------------------------------------ MoE
 def moe_route(logits: torch.Tensor, e_bias: Optional[torch.Tensor], k: int, mode: int = 0, renorm: bool = True,
-              n_group: int = 1, topk_group: int = 1, routed_scale: float = 1.0):
+              n_group: int = 1, topk_group: int = 1, routed_scale: float = 1.0, group_top: int = 2):
     """Router logits ``[T, E]`` -> (expert ids int32 ``[T, k]``, weights fp32 ``[T, k]``)."""
     T, E = logits.shape
-    assert logits.is_contiguous()
+    assert logits.stride(1) == 1
     ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
-    check(_lib.lib().pxl_moe_route(logits.data_ptr(), int(logits.dtype == torch.bfloat16), _ptr(e_bias), T, E, k,
-                                   mode, int(renorm), n_group, topk_group, routed_scale, ids.data_ptr(),
+    check(_lib.lib().pxl_moe_route(logits.data_ptr(), logits.stride(0), int(logits.dtype == torch.bfloat16), _ptr(e_bias), T,
+                                   E, k, mode, int(renorm), n_group, topk_group, group_top, routed_scale, ids.data_ptr(),
                                    w.data_ptr(), _stream(logits.device)), "pxl_moe_route")
     _count()
     return ids, w
@@ -681,6 +703,62 @@ def moe_ffn(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w1: torch
         act = act_mul(gu, mode=act_mode, limit=limit)
     y = grouped_linear(act, w2, plan, num_experts, bias=b2)
     return moe_combine(y, plan, weights, base, x.shape[0])
+
+
+def routed_ffn(x, ids, weights, w1, w2, num_experts: int):
+    """Gated (SiLU) experts; rows stay in expert order for :func:`residual_add` to pick up. ``w1 [E * 2 I, W]`` gate / up
+    rows interleaved per expert, ``w2 [E * N, I]`` (N >= W: padded outputs). Ids >= ``num_experts`` are identity experts."""
+    plan = moe_align(ids, num_experts)
+    if x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
+        n = w2.shape[0] // num_experts
+        act = grouped_linear(moe_gather(x, plan), w1, plan, num_experts, epi=EPI_SILU_MUL)
+        y = grouped_linear(act, w2, plan, num_experts, bn=0 if n % 128 == 0 else 64)
+    else:
+        act = _glu_act(_grouped_simt(x, w1, plan, num_experts, plan.src_tok), 0)
+        y = _grouped_simt(act, w2, plan, num_experts, None)
+    return y, plan.pos_of, weights
+
+
+def _grouped_simt(x, w, plan, num_experts: int, a_rows):
+    N, K = w.shape[0] // num_experts, w.shape[1]
+    assert x.dtype == w.dtype and x.stride(1) == 1 and x.shape[1] == K
+    out = torch.empty((plan.max_rows, N), dtype=x.dtype, device=x.device)
+    check(_lib.lib().pxl_gemm_simt_grouped(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(a_rows), N, K, x.stride(0),
+                                           w.stride(0), N, plan.mt_expert.data_ptr(), plan.mt_row0.data_ptr(),
+                                           plan.mt_row_end.data_ptr(), plan.num_mt.data_ptr(), plan.max_mt,
+                                           int(x.dtype == torch.float32), _stream(x.device)), "pxl_gemm_simt_grouped")
+    _count()
+    return out
+
+
+def _glu_act(x, act: int, row_gate=None, out=None):
+    T, I = x.shape[0], x.shape[1] // 2
+    assert x.is_contiguous()
+    if out is None:
+        out = torch.empty((T, I), dtype=x.dtype, device=x.device)
+    assert out.stride(1) == 1 and out.dtype == x.dtype
+    check(_lib.lib().pxl_glu_act(x.data_ptr(), _ptr(row_gate), row_gate.stride(0) if row_gate is not None else 0,
+                                 out.data_ptr(), out.stride(0), T, I, act, int(x.dtype == torch.float32), _stream(x.device)),
+          "pxl_glu_act")
+    _count()
+    return out
+
+
+def glu_linear(x, w_gu, act: int = 0, row_gate=None, out=None):
+    T, N = x.shape[0], w_gu.shape[0]
+    assert row_gate is None or row_gate.dtype == torch.float32
+    if out is None:
+        out = torch.empty((T, N // 2), dtype=x.dtype, device=x.device)
+    if T == 0:
+        return out
+    if x.dtype == torch.float32 or not _tma_ok(x, w_gu) or out.stride(0) & 7 or out.data_ptr() & 15:
+        return _glu_act(linear(x, w_gu), act, row_gate, out)
+    check(_lib.lib().pxl_gemm_bf16_act_glu(x.data_ptr(), w_gu.data_ptr(), out.data_ptr(), T, N, x.shape[1], x.stride(0),
+                                           w_gu.stride(0), out.stride(0), act, _ptr(row_gate),
+                                           row_gate.stride(0) if row_gate is not None else 0, 0,
+                                           status_tensor(x.device).data_ptr(), _stream(x.device)), "pxl_gemm_bf16_act_glu")
+    _count()
+    return out
 
 
 def as_c_int_p(t: torch.Tensor) -> ctypes.c_void_p:
@@ -1079,4 +1157,73 @@ def latent_attn(q_cat, cache, block_tables, cu_q, ctx_lens, scale: float, latent
                                      int(q_cat.dtype == torch.float32), status_tensor(q_cat.device).data_ptr(),
                                      _stream(q_cat.device)), "pxl_latent_attn")
     _count()
+    return out
+
+
+# ---------------------------------------------------------------------------- convolved attention, lightning attention
+def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None):
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.stride(1) == 1 and y.shape == x.shape
+    low = torch.empty((T, W), dtype=y.dtype, device=x.device) if w is not None else None
+    rows, pos_of, weights = routed or (None, None, None)
+    if routed:
+        assert rows.dtype == h.dtype == y.dtype and h.is_contiguous() and weights.is_contiguous() and rows.shape[1] >= W
+    check(_lib.lib().pxl_residual_add(x.data_ptr(), y.data_ptr(), y.stride(0), _ptr(rows), rows.stride(0) if routed else 0,
+                                      rows.shape[0] if routed else 0, _ptr(pos_of), _ptr(weights),
+                                      weights.shape[1] if routed else 0, _ptr(h if routed else None), _ptr(w), _ptr(low), T, W,
+                                      eps, int(y.dtype == torch.float32), status_tensor(x.device).data_ptr(),
+                                      _stream(x.device)), "pxl_residual_add")
+    _count()
+    return low
+
+
+def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, conv_w, conv_state, q_norm, k_norm, cos_sin,
+                  positions, seq_cu, seq_slots, prefill_seqs: int, prefill_tokens: int, slot_mapping, k_cache, v_cache, q_out,
+                  eps: float):
+    T = proj.shape[0]
+    cols, rot = q_out.shape[2], cos_sin.shape[1]
+    own = k_cache is not None
+    taps = conv_w.shape[0] if conv_w is not None else 1
+    state = conv_state if taps > 1 else None
+    assert proj.stride(1) == 1 and q_out.is_contiguous() and q_out.dtype == proj.dtype
+    assert conv_w is None or (conv_w.is_contiguous() and conv_w.dtype == proj.dtype)
+    assert state is None or (state.is_contiguous() and state.dtype == proj.dtype
+                             and state.shape[1:] == (taps - 1, conv_w.shape[1]))
+    if own:
+        assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == proj.dtype
+        assert k_cache.shape[1] == kv_heads and k_cache.shape[3] == v_cache.shape[3] == cols
+    check(_lib.lib().pxl_conv_qkv_prep(
+        proj.data_ptr(), proj.stride(0), *offs, heads, kv_heads if own else 0, dim, vdim, cols, rot, taps, _ptr(conv_w),
+        _ptr(state), state.shape[0] if state is not None else 0, q_norm.data_ptr(), _ptr(k_norm), cos_sin.data_ptr(),
+        positions.data_ptr(), cos_sin.shape[0], seq_cu.data_ptr(), seq_slots.data_ptr(), prefill_seqs, prefill_tokens, T,
+        slot_mapping.data_ptr(), k_cache.shape[0] * k_cache.shape[2] if own else 0, k_cache.shape[2] if own else 1,
+        _ptr(k_cache), _ptr(v_cache), q_out.data_ptr(), eps, int(proj.dtype == torch.float32),
+        status_tensor(proj.device).data_ptr(), _stream(proj.device)), "pxl_conv_qkv_prep")
+    _count(2 if taps > 1 and prefill_seqs else 1)
+
+
+def gated_rows(x, vdim: int, gate, out, norm_w=None, eps: float = 0.0):
+    T, heads, cols = x.shape
+    assert x.is_contiguous() and gate.stride(1) == 1 and out.stride(1) == 1 and x.dtype == gate.dtype == out.dtype
+    check(_lib.lib().pxl_gated_rows(x.data_ptr(), heads, cols, vdim, gate.data_ptr(), gate.stride(0), _ptr(norm_w), eps,
+                                    out.data_ptr(), out.stride(0), out.shape[1], T, int(x.dtype == torch.float32),
+                                    _stream(x.device)), "pxl_gated_rows")
+    _count()
+    return out
+
+
+def lightning_attn(proj, offs, heads: int, dim: int, vdim: int, decay_pow, state, positions, seq_cu, seq_slots,
+                   prefill_seqs: int, out=None):
+    T = proj.shape[0]
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=proj.dtype, device=proj.device)
+    assert proj.stride(1) == 1 and out.is_contiguous() and out.dtype == proj.dtype and decay_pow.dtype == torch.float32
+    assert state.is_contiguous() and state.dtype == torch.float32 and state.shape[1:] == (heads, dim, vdim)
+    n = seq_slots.numel()
+    check(_lib.lib().pxl_lightning_attn(proj.data_ptr(), proj.stride(0), *offs, heads, dim, vdim, decay_pow.data_ptr(),
+                                        decay_pow.shape[1], state.data_ptr(), state.shape[0], seq_cu.data_ptr(),
+                                        seq_slots.data_ptr(), positions.data_ptr(), out.data_ptr(), heads * vdim, prefill_seqs,
+                                        n - prefill_seqs, int(proj.dtype == torch.float32),
+                                        status_tensor(proj.device).data_ptr(), _stream(proj.device)), "pxl_lightning_attn")
+    _count((prefill_seqs > 0) + (n > prefill_seqs))
     return out

@@ -309,22 +309,19 @@ def sample(logits, temperature, top_k, top_p, min_p, uniform, want_prob: bool = 
     return (ids, probs_out) if want_prob else ids
 
 
-def moe_route(logits, e_bias, k, mode=0, renorm=True, n_group=1, topk_group=1, routed_scale=1.0):
-    """Top-k expert selection (see csrc/moe.cu for the two modes)."""
+def moe_route(logits, e_bias, k, mode=0, renorm=True, n_group=1, topk_group=1, routed_scale=1.0, group_top=2):
+    """Top-k expert selection (see csrc/moe.cu): softmax (mode 0) or sigmoid (mode 1) scores, chosen by score + ``e_bias``
+    within the ``topk_group`` best of ``n_group`` groups (by the sum of their ``group_top`` best)."""
     lf = logits.float()
     T, E = lf.shape
-    if mode == 0:
-        s = torch.softmax(lf, dim=-1)
-        sel = s
-    else:
-        s = torch.sigmoid(lf)
-        sel = s + (e_bias.float() if e_bias is not None else 0.0)
-        if n_group > 1 and topk_group < n_group:
-            g = sel.view(T, n_group, E // n_group)
-            gscore = g.topk(2, dim=-1).values.sum(-1)
-            keep = torch.zeros_like(gscore, dtype=torch.bool)
-            keep.scatter_(1, gscore.topk(topk_group, dim=-1).indices, True)
-            sel = g.masked_fill(~keep[:, :, None], float("-inf")).reshape(T, E)
+    s = torch.softmax(lf, dim=-1) if mode == 0 else torch.sigmoid(lf)
+    sel = s + (e_bias.float() if e_bias is not None else 0.0)
+    if n_group > 1 and topk_group < n_group:
+        g = sel.view(T, n_group, E // n_group)
+        gscore = g.topk(min(group_top, E // n_group), dim=-1).values.sum(-1)
+        keep = torch.zeros_like(gscore, dtype=torch.bool)
+        keep.scatter_(1, gscore.topk(topk_group, dim=-1).indices, True)
+        sel = g.masked_fill(~keep[:, :, None], float("-inf")).reshape(T, E)
     ids = sel.topk(k, dim=-1).indices
     w = s.gather(1, ids)
     if renorm:
@@ -753,4 +750,132 @@ def latent_attn(q_cat, cache, block_tables, cu_q, ctx_lens, scale: float, latent
             s = torch.cat([s, sinks.float().view(H, 1, 1).expand(H, t1 - t0, 1)], -1)
         p = torch.softmax(s, -1)[..., :ctx]
         out[t0:t1] = torch.einsum("hts,sk->thk", p, rows[:, :latent]).to(out.dtype)
+    return out
+
+
+# ---------------------------------------------------------------------------- convolved attention, lightning attention
+def glu_linear(x, w_gu, act: int = 0, row_gate=None, out=None):
+    """``act(gate) * up`` of ``x @ w_gu^T`` (gate / up rows interleaved by :func:`interleave_gate_up`); ``act`` 0 = SiLU,
+    2 = GELU (tanh form). ``row_gate [T]`` fp32: rows times ``sigmoid(row_gate)``."""
+    y = (x.float() @ w_gu.float().t()).view(x.shape[0], -1, 2, 64)
+    g = torch.nn.functional.gelu(y[:, :, 0], approximate="tanh") if act == 2 else torch.nn.functional.silu(y[:, :, 0])
+    res = (g * y[:, :, 1]).reshape(x.shape[0], -1)
+    if row_gate is not None:
+        res = res * torch.sigmoid(row_gate.float())[:, None]
+    if out is None:
+        return res.to(x.dtype)
+    out.copy_(res)
+    return out
+
+
+def routed_ffn(x, ids, weights, w1, w2, num_experts: int):
+    """Outputs of the chosen gated (SiLU) experts for :func:`residual_add`: ``(rows, pos_of, weights)``, where
+    ``rows[pos_of[t, j]]`` is expert ``ids[t, j]``'s output. ``w1 [E * 2 I, W]`` gate / up rows interleaved per expert,
+    ``w2 [E * N, I]``. Ids >= ``num_experts`` are identity experts: position -1."""
+    T, k = ids.shape
+    n1, n2 = w1.shape[0] // num_experts, w2.shape[0] // num_experts
+    rows = torch.zeros((T * k, n2), dtype=x.dtype, device=x.device)
+    pos = torch.arange(T * k, device=x.device).view(T, k)
+    for e in range(num_experts):
+        tok, slot = (ids == e).nonzero(as_tuple=True)
+        if tok.numel():
+            act = glu_linear(x[tok], w1[e * n1:(e + 1) * n1])
+            rows[tok * k + slot] = linear(act, w2[e * n2:(e + 1) * n2])
+    return rows, torch.where(ids < num_experts, pos, torch.full_like(pos, -1)).to(torch.int32), weights
+
+
+def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None):
+    """In place on the fp32 residual: ``x += y`` plus the weighted expert rows of :func:`routed_ffn` (an identity
+    expert's row is ``h[t]``). With a norm weight returns ``rmsnorm(x) * w`` in ``y``'s dtype."""
+    W = x.shape[1]
+    x.add_(y.float())
+    if routed is not None:
+        rows, pos, wt = routed
+        val = torch.where(pos[:, :, None] < 0, h[:, None, :].float(), rows[pos.clamp_min(0).long()][:, :, :W].float())
+        x.add_((val * wt.float()[:, :, None]).sum(1))
+    return None if w is None else (_normalised(x, eps, NORM_RMS) * w.float()).to(y.dtype)
+
+
+def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, conv_w, conv_state, q_norm, k_norm, cos_sin,
+                  positions, seq_cu, seq_slots, prefill_seqs: int, prefill_tokens: int, slot_mapping, k_cache, v_cache, q_out,
+                  eps: float):
+    """Queries and cache rows of one step out of the packed projection: q, k, v start at columns ``offs`` of ``proj``.
+    Causal convolution per channel (``conv_w [taps, channels]`` over q | k | v, or None) with the state slots
+    ``conv_state [slots, taps - 1, channels]``, RMS norm over the whole q and k rows, half-split rotation
+    (``cos_sin [positions, dims]``). ``q_out [T, heads, cols]`` and the pages ``[blocks, kv_heads, page, cols]`` get heads
+    padded with zeros; without caches only q is made."""
+    T, cols, rot = proj.shape[0], q_out.shape[2], cos_sin.shape[1]
+    own = k_cache is not None
+    widths = [heads * dim] + ([kv_heads * dim, kv_heads * vdim] if own else [])
+    u = torch.cat([proj[:, o:o + n] for o, n in zip(offs, widths)], 1).float()
+    y = u
+    if conv_w is not None:
+        taps, wf = conv_w.shape[0], conv_w.float()
+        y = torch.empty_like(u)
+        cu = seq_cu.tolist()
+        for b in range(len(cu) - 1):
+            t0, t1, slot = cu[b], cu[b + 1], int(seq_slots[b])
+            if t1 <= t0:
+                continue
+            hist = u.new_zeros((0, u.shape[1]))
+            if taps > 1:
+                hist = conv_state[slot].float().clone()
+                start = int(positions[t0])
+                if start < taps - 1:       # zeros before the sequence
+                    hist[:taps - 1 - start] = 0
+            full = torch.cat([hist, u[t0:t1]], 0)
+            y[t0:t1] = sum(wf[j] * full[j:j + t1 - t0] for j in range(taps))
+            if taps > 1:
+                conv_state[slot] = full[-(taps - 1):].to(conv_state.dtype)
+    cs = cos_sin[positions.long()].float()[:, None]
+    c, s = cs[..., :rot // 2], cs[..., rot // 2:]
+
+    def rotate(x, norm_w, n):
+        x = (_normalised(x, eps, NORM_RMS) * norm_w.float()).view(T, n, dim)
+        a, b = x[..., :rot // 2], x[..., rot // 2:rot]
+        return torch.cat([a * c - b * s, b * c + a * s, x[..., rot:]], -1)
+
+    pad = torch.nn.functional.pad
+    q_out.copy_(pad(rotate(y[:, :widths[0]], q_norm, heads), (0, cols - dim)))
+    if own:
+        k = rotate(y[:, widths[0]:widths[0] + widths[1]], k_norm, kv_heads)
+        v = y[:, widths[0] + widths[1]:].view(T, kv_heads, vdim)
+        reshape_and_cache(pad(k, (0, cols - dim)), pad(v, (0, cols - vdim)), slot_mapping, k_cache, v_cache)
+
+
+def gated_rows(x, vdim: int, gate, out, norm_w=None, eps: float = 0.0):
+    """``out[:, :heads * vdim] = heads side by side (, rmsnorm over them all * norm_w) * sigmoid(gate)``, zeros behind;
+    ``x [T, heads, cols]``, of which the first ``vdim`` columns count."""
+    y = x[:, :, :vdim].reshape(x.shape[0], -1).float()
+    n = y.shape[1]
+    if norm_w is not None:
+        y = _normalised(y, eps, NORM_RMS) * norm_w.float()
+    out[:, :n] = (y * torch.sigmoid(gate.float())).to(out.dtype)
+    out[:, n:] = 0
+    return out
+
+
+def lightning_attn(proj, offs, heads: int, dim: int, vdim: int, decay_pow, state, positions, seq_cu, seq_slots,
+                   prefill_seqs: int, out=None):
+    """``S <- decay S + k v^T``, ``o = S^T q`` per head, with q, k, v = silu of the columns at ``offs``; states
+    ``[slots, heads, dim, vdim]`` fp32, ``decay_pow[h, n]`` = decay^n. Returns ``[T, heads, vdim]``."""
+    T = proj.shape[0]
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=proj.dtype, device=proj.device)
+
+    def part(o, d):
+        return torch.nn.functional.silu(proj[:, o:o + heads * d].float()).to(proj.dtype).float().view(T, heads, d)
+
+    q, k, v = part(offs[0], dim), part(offs[1], dim), part(offs[2], vdim)
+    decay = decay_pow[:, 1].float()[:, None, None]
+    cu = seq_cu.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1, slot = cu[b], cu[b + 1], int(seq_slots[b])
+        if t1 <= t0:
+            continue
+        S = torch.zeros_like(state[slot]) if int(positions[t0]) == 0 else state[slot].clone()
+        for t in range(t0, t1):
+            S = decay * S + k[t][:, :, None] * v[t][:, None, :]
+            out[t] = torch.einsum("hkv,hk->hv", S, q[t]).to(out.dtype)
+        state[slot] = S
     return out
