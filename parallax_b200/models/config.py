@@ -122,6 +122,11 @@ class ModelConfig:
         return (2 * hk * dk + hv * dv, max(self.linear_conv_kernel_dim - 1, 0)), (hv, dv, dk)
 
     @property
+    def linked_layers(self) -> list[tuple[int, int]]:
+        """Pairs (layer that owns keys and values, later layer that reads them): both belong in one pipeline stage."""
+        return [(s.mixer.kv_from, i) for i, s in enumerate(self.layer_specs) if s.mixer.kv_from is not None]
+
+    @property
     def is_moe(self) -> bool:
         return self.num_experts > 0
 
@@ -433,6 +438,30 @@ def named_config(name: str) -> ModelConfig:
                          mixer=dict(heads=h, dim=d, rot_dim=r, vdim=v, kv_rank=k, scale=(d + r) ** -0.5,
                                     mask=dict(size=win), rot=dict(base=1e4, dims=r)),
                          mlp=dict(kind="dense", ff=ff, limit=6.0)) for _ in range(nl)]))
+    if n in {"tiny-zudepel", "small-zudepel", "zudepel-1b", "zudepel-8b"}:
+        # layer list: q = attention with its own keys, s = attention that reads the last q's, l = lightning
+        # (layers, width, heads, kv heads, dim, vdim, lightning heads, dim, vdim, ff, experts, identity, top, groups, expert ff, vocab)
+        pattern, w, h, g, d, v, lh, ld, lv, ff, ex, ident, top, groups, eff, vocab = {
+            "tiny-zudepel": ("qslq", 64, 4, 2, 16, 24, 4, 16, 8, 96, 6, 2, 2, (4, 2), 32, 260),
+            "small-zudepel": ("lqlsq", 512, 8, 2, 64, 64, 4, 128, 64, 1024, 14, 2, 4, (4, 2), 256, 1024),
+            "zudepel-1b": ("lllq" * 4, 2048, 16, 4, 128, 128, 16, 128, 128, 5632, 30, 2, 4, (4, 2), 768, 32768),
+            "zudepel-8b": ("lllqllls" * 4, 4096, 32, 8, 128, 128, 32, 128, 128, 12288, 60, 4, 4, (8, 4), 1536, 131072)}[n]
+        layers, last = [], None
+        for i, kind in enumerate(pattern):
+            if kind == "l":
+                layers.append(dict(type="lightning", mlp=dict(kind="dense", ff=ff),
+                                   mixer=dict(heads=lh, dim=ld, vdim=lv, decay=[1 - 2.0 ** -(1 + j % 10) for j in range(lh)])))
+                continue
+            mixer = dict(heads=h, kv_heads=g, dim=d, vdim=v, conv=4, scale=d ** -0.5, rot=dict(base=1e4, dims=d))
+            if kind == "s":
+                mixer["kv_from"] = last
+            else:
+                last = i
+            layers.append(dict(type="attention", mixer=mixer,
+                               mlp=dict(kind="moe", expert=dict(ff=eff), shared=dict(ff=eff),
+                                        router=dict(experts=ex, identity=ident, top=top,
+                                                    groups=dict(count=groups[0], keep=groups[1])))))
+        return config_from_hf(dict(architecture="Zudepel", vocab=vocab, width=w, norm=dict(eps=1e-6), layers=layers))
     if n == "tiny":
         return config_from_hf(dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", hidden_size=256,
                                    num_hidden_layers=4, num_attention_heads=4, num_key_value_heads=2,

@@ -61,10 +61,11 @@ def cu_launch_count() -> int:
     return cu.launch_count
 
 
-def split_layers(num_layers: int, pp: int) -> list[tuple[int, int]]:
+def split_layers(num_layers: int, pp: int, linked=()) -> list[tuple[int, int]]:
     """Contiguous split, as even as the layer count allows (what water-filling yields for identical
     GPUs). The remainder layers go to the stages in the middle: the first stage also hosts the
-    scheduler and the embedding, the last one the lm_head and the sampler."""
+    scheduler and the embedding, the last one the lm_head and the sampler. ``linked``: pairs of layers that
+    must share a stage (one reads the other's cache); a cut between them moves to the nearest place it may be."""
     base, rem = divmod(num_layers, pp)
     extra = [0] * pp
     order = list(range(1, pp - 1)) + [0, pp - 1] if pp > 2 else list(range(pp))
@@ -75,7 +76,20 @@ def split_layers(num_layers: int, pp: int) -> list[tuple[int, int]]:
         n = base + extra[i]
         out.append((s, s + n))
         s += n
-    return out
+    free = [c for c in range(1, num_layers) if not any(a < c <= b for a, b in linked)]
+    cuts = [e for _, e in out[:-1]]
+    if all(c in free for c in cuts):
+        return out
+    if len(free) < pp - 1:
+        raise ValueError(f"{num_layers} layers with shared caches cannot be cut into {pp} stages")
+    moved, lo = [], 0
+    for i, c in enumerate(cuts):        # leave enough places for the cuts that follow
+        choices = free[lo:len(free) - (len(cuts) - 1 - i)]
+        best = min(choices, key=lambda f: abs(f - c))
+        moved.append(best)
+        lo = free.index(best) + 1
+    edges = [0, *moved, num_layers]
+    return list(zip(edges, edges[1:]))
 
 
 @dataclass
@@ -245,7 +259,7 @@ class DistEngine:
         if rank != 0:
             self.chan = CtrlChannel(box[0], create=False, n_readers=world - 1, reader_index=rank - 1, slots=n_slots,
                                     slot_bytes=slot_bytes)
-        start, end = split_layers(cfg.num_hidden_layers, pp)[topo.pp_rank]
+        start, end = split_layers(cfg.num_hidden_layers, pp, cfg.linked_layers)[topo.pp_rank]
         comm = None
         from parallax_b200.models.registry import family_of
 

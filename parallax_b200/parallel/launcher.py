@@ -74,7 +74,7 @@ def build_dist_engine(spec: dict):
     if spec.get("model_path"):
         from parallax_b200.loader.shard_loader import ShardLoader, apply_lora_adapter
 
-        start, end = split_layers(cfg.num_hidden_layers, pp)[rank // (tp * spec.get("ep", 1))]
+        start, end = split_layers(cfg.num_hidden_layers, pp, cfg.linked_layers)[rank // (tp * spec.get("ep", 1))]
         weights = ShardLoader(spec["model_path"], start, end).load_weights("cpu", None)
         for lp in spec.get("lora_paths") or []:
             apply_lora_adapter(weights, lp)

@@ -74,6 +74,16 @@ def test_layer_list_model_over_pipeline_ranks(tmp_path):
     assert _run_group(2, 1, tmp_path, model="tiny-piburax")["outputs"] == _single(model="tiny-piburax")
 
 
+def test_layers_that_share_a_cache_stay_in_one_stage(tmp_path):
+    assert split_layers(4, 2, [(0, 1)]) == [(0, 2), (2, 4)]                # the even cut is free
+    assert split_layers(4, 2, [(1, 2)]) in ([(0, 1), (1, 4)], [(0, 3), (3, 4)])
+    assert split_layers(6, 3, [(1, 2), (3, 5)]) == [(0, 1), (1, 3), (3, 6)]
+    with pytest.raises(ValueError, match="shared caches"):
+        split_layers(4, 3, [(0, 2)])
+    # state slots of convolutions and recurrent layers on both ranks
+    assert _run_group(2, 1, tmp_path, model="tiny-zudepel")["outputs"] == _single(model="tiny-zudepel")
+
+
 def test_rank0_executor_thread_and_aligned_rows(tmp_path):
     """Rank 0 launching its stage from a thread of its own, three micro-batches in flight and prompt
     slices trimmed to a row multiple: same tokens as the single-process engine."""

@@ -2,6 +2,7 @@
 request_to_proto / proto_to_request, as the reference's executor test does
 (tests/test_executor.py:67-285). The result must equal the single-engine run."""
 
+import pytest
 import torch
 
 from parallax_b200.engine.engine import Engine
@@ -46,12 +47,13 @@ def _run_pipeline(cfg, spans, prompts, max_new, **kw):
     return [r.output_ids for r in reqs], peers
 
 
-def test_three_peers_of_a_layer_list_model():
-    cfg = named_config("tiny-piburax")
+@pytest.mark.parametrize("name,layers", [("tiny-piburax", [(0, 1), (1, 2), (2, 3)]), ("tiny-zudepel", [(0, 2), (2, 3), (3, 4)])])
+def test_three_peers_of_a_layer_list_model(name, layers):
+    cfg = named_config(name)
     prompts = _prompts(3, 41, cfg.vocab_size, seed=4)
     want = Engine(cfg, device="cpu", num_blocks=128, max_batch_size=8).generate(
         prompts, SamplingParams(max_new_tokens=9, temperature=0.0, ignore_eos=True))
-    got, peers = _run_pipeline(cfg, [(0, 1), (1, 2), (2, 3)], prompts, 9)
+    got, peers = _run_pipeline(cfg, layers, prompts, 9)
     assert got == want and all(not p.cache.reqs for p in peers)
 
 
