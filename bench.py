@@ -496,13 +496,16 @@ def main() -> None:
     ap.add_argument("--micro-batches", type=int, default=0, help="pipeline modes: micro-batches in flight")
     ap.add_argument("--parallelism", default="auto",
                     help="auto (the workload's layout on N GPUs) | dp | pp | pp<P>tp<T> | ep<E> | pp<P>ep<E>")
-    ap.add_argument("--design", default="", choices=["", "piburax"],
+    ap.add_argument("--design", default="", choices=["", "piburax", "zudepel"],
                     help="instead of the workload: layer throughput of this design beside the closest other model of equal "
                          "sizes, and its kernels against their rooflines (one GPU)")
     ap.add_argument("--design-sizes", default="1b,8b")
     args = ap.parse_args()
     if args.design:
-        from benchmarks.bench_latent import run as run_design
+        if args.design == "piburax":
+            from benchmarks.bench_latent import run as run_design
+        else:
+            from benchmarks.bench_parallel_block import run as run_design
 
         sampler = ClockSampler(0)
         sampler.start()

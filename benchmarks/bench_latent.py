@@ -30,6 +30,7 @@ from parallax_b200.models.registry import build_stage  # noqa: E402
 from parallax_b200.ops import cuda as cu  # noqa: E402
 
 PAGE = 16
+SLOTS = 128        # requests with a state of their own
 LAYERS = {"1b": 12, "8b": 4}
 
 
@@ -60,9 +61,12 @@ class Stack:
         self.stage = build_stage(cfg, 0, cfg.num_hidden_layers, self.dev, torch.bfloat16, max_positions=16384)
         self.stage.init_random(1)
         self.blocks = -(-tokens // PAGE)
-        self.pool = KVPool(cfg, 0, cfg.num_hidden_layers, self.blocks, PAGE, self.dev, torch.bfloat16)
+        self.pool = KVPool(cfg, 0, cfg.num_hidden_layers, self.blocks, PAGE, self.dev, torch.bfloat16,
+                           num_linear_slots=SLOTS if cfg.has_linear_layers else 0)
         for lc in self.pool.layers:
-            lc.k.normal_(0, 0.5)
+            for t in (lc.k, lc.v, lc.conv_state, lc.rec_state):
+                if t is not None:
+                    t.normal_(0, 0.5)
         self.stage.attach_kv(self.pool.layers)
 
     def batch(self, prefill: list, decode: list):
@@ -83,7 +87,8 @@ class Stack:
         T, n_p = len(pos), len(prefill)
         b = BatchBuilder(self.dev, T, len(pages), tables.shape[1])
         fb = b.build(np.zeros(T, np.int32), pos, slots, prefill, prefill, tables[:n_p] if n_p else None,
-                     np.asarray(decode, dtype=np.int32), tables[n_p:] if decode else None, np.zeros(0, np.int32))
+                     np.asarray(decode, dtype=np.int32), tables[n_p:] if decode else None, np.zeros(0, np.int32),
+                    np.arange(len(pages), dtype=np.int32))
         fb.keep = b
         return fb
 

@@ -77,7 +77,7 @@ def engine(name, target, **kw):
 
 
 def errors(got, want):
-    got, want = got.double().cpu(), want.double()
+    got, want = got.double().cpu(), want.double().cpu()
     d = got - want
     d = d - d.mean(-1, keepdim=True)
     return d.pow(2).mean(-1).sqrt() / want.std(-1)
