@@ -6,6 +6,7 @@
     python benchmarks/profile_case.py attn_decode  # paged GQA decode, 256 seqs x 2048 ctx
     python benchmarks/profile_case.py attn_prefill # ragged prefill, 4 x 2048
     python benchmarks/profile_case.py latent_attn  # windowed latent attention, 4096-token prompt, 32 heads
+    python benchmarks/profile_case.py lightning    # chunked lightning attention, 4096-token prompt, 32 heads
     python benchmarks/profile_case.py step         # 2 engine steps of a 4-layer Qwen3-8B-shaped
                                                    # model at 64 concurrent (launch list)
     python benchmarks/profile_case.py decode_step  # same, decode rows only (small-M GEMMs); decode_step_8: 8 rows
@@ -177,9 +178,30 @@ def case_latent_attn(iters: int = 2, T: int = 4096, H: int = 32, L: int = 512, R
     cu.check_status(q.device)
 
 
+def case_lightning(iters: int = 2, T: int = 4096, H: int = 32, D: int = 128):
+    proj = torch.randn(T, 4 * H * D, device="cuda", dtype=torch.bfloat16)
+    pw = (torch.linspace(0.5, 0.999, H, dtype=torch.float64)[:, None] ** torch.arange(65)).float().cuda()
+    state = torch.zeros(1, H, D, D, device="cuda")
+    pos, cu_seq = torch.arange(T, dtype=torch.int32, device="cuda"), torch.tensor([0, T], dtype=torch.int32, device="cuda")
+    slot = torch.zeros(1, dtype=torch.int32, device="cuda")
+    out = torch.empty(T, H, D, device="cuda", dtype=torch.bfloat16)
+
+    def run():
+        cu.lightning_attn(proj, (0, H * D, 2 * H * D), H, D, D, pw, state, pos, cu_seq, slot, 1, out=out)
+
+    run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStart()
+    for _ in range(iters):
+        run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStop()
+    cu.check_status(proj.device)
+
+
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "gemm"
-    {"gemm": case_gemm, "latent_attn": case_latent_attn, "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
+    {"gemm": case_gemm, "latent_attn": case_latent_attn, "lightning": case_lightning, "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
      "gemm_small": case_gemm_small, "gemm_mid": case_gemm_mid, "step": case_step, "decode_step": lambda: case_step(conc=64, with_prefill=False),
      "decode_step_8": lambda: case_step(conc=8, with_prefill=False)}[which]()
     print(f"profile case {which}: ok")

@@ -84,35 +84,52 @@ struct PrepArgs {
   int* status;
 };
 
-// y = norm_w * inv * row (or the convolved row itself), rotated; VEC elements of one head from d0
+// inv * row, rotated; VEC elements of one head from d0, all in one part of the head (rot / 2 is a multiple of VEC)
 template <int VEC>
-__device__ __forceinline__ void rotated(const float* row, const float* w, float inv, const float* cs, int dk, int rot,
-                                        int d0, float (&o)[VEC]) {
+__device__ __forceinline__ void rotated(const float* row, float inv, const float* cs, int dk, int rot, int d0, float (&o)[VEC]) {
   const int half = rot / 2;
+  if (d0 >= dk) {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+    return;
+  }
+  load_v<VEC>(row + d0, o);
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) o[j] *= inv;
+  if (d0 >= rot) return;
+  const bool lower = d0 < half;
+  const int f = lower ? d0 : d0 - half;  // pair
+  float c[VEC], sn[VEC], other[VEC];
+  load_v<VEC>(cs + f, c);
+  load_v<VEC>(cs + half + f, sn);
+  load_v<VEC>(row + (lower ? d0 + half : f), other);
 #pragma unroll
   for (int j = 0; j < VEC; ++j) {
-    const int d = d0 + j;
-    if (d >= dk) {
-      o[j] = 0.f;
-      continue;
-    }
-    float y = row[d] * inv * w[d];
-    if (d < half) y = y * cs[d] - row[d + half] * inv * w[d + half] * cs[half + d];
-    else if (d < rot) y = y * cs[d - half] + row[d - half] * inv * w[d - half] * cs[d];
-    o[j] = y;
+    const float x = other[j] * inv;
+    o[j] = lower ? o[j] * c[j] - x * sn[j] : o[j] * c[j] + x * sn[j];
   }
 }
 
+// both sums over the block; red holds 64 floats
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  a = warp_reduce_sum(a);
+  b = warp_reduce_sum(b);
+  if (lane == 0) red[warp] = a, red[32 + warp] = b;
+  __syncthreads();
+  return make_float2(warp_reduce_sum(lane < nwarps ? red[lane] : 0.f), warp_reduce_sum(lane < nwarps ? red[32 + lane] : 0.f));
+}
+
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) conv_qkv_prep_kernel(const PrepArgs a, int tokens_per_cta) {
-  extern __shared__ float row[];  // convolved q | k of one token
-  __shared__ float red[32];
+__global__ void __launch_bounds__(512) conv_qkv_prep_kernel(const PrepArgs a, int begin, int tokens_per_cta) {
+  extern __shared__ __align__(16) float row[];  // convolved q | k of one token, times the norm weights
+  __shared__ float red[64];
   pdl_wait();
   pdl_launch_dependents();
   const int Cq = a.H * a.dk, Ck = a.G * a.dk, Cv = a.G * a.dv, C = Cq + Ck + Cv;
   const int back = a.conv_w ? a.taps - 1 : 0;
   const T* w = static_cast<const T*>(a.conv_w);
-  const int first = blockIdx.x * tokens_per_cta;
+  const int first = begin + blockIdx.x * tokens_per_cta;
   int seq = 0;
   if (first < a.prefill_tokens) {  // last slice that starts at or before the token
     int lo = 0, hi = a.prefill_seqs - 1;
@@ -142,7 +159,8 @@ __global__ void __launch_bounds__(256) conv_qkv_prep_kernel(const PrepArgs a, in
       if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_SLOT);
       cslot = -1;
     }
-    const int64_t blk = cslot / a.page, in_page = cslot % a.page;
+    const int in_page = cslot >= 0 ? static_cast<int>(static_cast<uint32_t>(cslot) % static_cast<uint32_t>(a.page)) : 0;
+    const int64_t blk = cslot >= 0 ? static_cast<uint32_t>(cslot) / static_cast<uint32_t>(a.page) : 0;
     float sq = 0.f, sk = 0.f;
     for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
       const int col = c < Cq ? a.q_off + c : c < Cq + Ck ? a.k_off + c - Cq : a.v_off + c - Cq - Ck;
@@ -179,40 +197,168 @@ __global__ void __launch_bounds__(256) conv_qkv_prep_kernel(const PrepArgs a, in
         for (int j = 0; j < VEC; ++j) y[j] = u[j];
       }
       if (c < Cq + Ck) {
+        float nw[VEC], sum = 0.f;
+        load_v<VEC>(c < Cq ? a.q_norm + c : a.k_norm + c - Cq, nw);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
-          row[c + j] = y[j];
-          if (c < Cq) sq = fmaf(y[j], y[j], sq);
-          else sk = fmaf(y[j], y[j], sk);
+          sum = fmaf(y[j], y[j], sum);
+          y[j] *= nw[j];
         }
+        (c < Cq ? sq : sk) += sum;
+        store_v<VEC>(row + c, y);
       } else if (cslot >= 0) {
         const int vc = c - Cq - Ck, g = vc / a.dv;
         store_v<VEC>(static_cast<T*>(a.v_cache) + ((blk * a.G + g) * a.page + in_page) * a.cols + vc % a.dv, y);
       }
     }
-    sq = block_reduce_sum(sq, red);
-    if (a.G) sk = block_reduce_sum(sk, red);
+    const float2 sums = block_sum2(sq, sk, red);  // (its barrier also publishes the row)
     if (pos < 0 || pos >= a.max_pos) {
       if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
       pos = 0;
     }
     const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
-    const float inv_q = 1.f / sqrtf(sq / Cq + a.eps), inv_k = a.G ? 1.f / sqrtf(sk / Ck + a.eps) : 0.f;
+    const float inv_q = 1.f / sqrtf(sums.x / Cq + a.eps), inv_k = a.G ? 1.f / sqrtf(sums.y / Ck + a.eps) : 0.f;
     const int per = a.cols / VEC;
     for (int i = threadIdx.x; i < (a.H + a.G) * per; i += blockDim.x) {
       const int h = i / per, d0 = i % per * VEC;
       float o[VEC];
       if (h < a.H) {
-        rotated<VEC>(row + h * a.dk, a.q_norm + h * a.dk, inv_q, cs, a.dk, a.rot, d0, o);
+        rotated<VEC>(row + h * a.dk, inv_q, cs, a.dk, a.rot, d0, o);
         store_v<VEC>(static_cast<T*>(a.q_out) + (static_cast<int64_t>(t) * a.H + h) * a.cols + d0, o);
       } else if (cslot >= 0) {
         const int g = h - a.H;
-        rotated<VEC>(row + Cq + g * a.dk, a.k_norm + g * a.dk, inv_k, cs, a.dk, a.rot, d0, o);
+        rotated<VEC>(row + Cq + g * a.dk, inv_k, cs, a.dk, a.rot, d0, o);
         store_v<VEC>(static_cast<T*>(a.k_cache) + ((blk * a.G + g) * a.page + in_page) * a.cols + d0, o);
         if (d0 + VEC > a.dv) {  // zero columns behind the value
           T* v = static_cast<T*>(a.v_cache) + ((blk * a.G + g) * a.page + in_page) * a.cols;
           for (int d = d0 > a.dv ? d0 : a.dv; d < d0 + VEC; ++d) put(v + d, 0.f);
         }
+      }
+    }
+    __syncthreads();  // the next token overwrites the row
+  }
+}
+
+// Prompt slices in bf16: a thread keeps its NV vectors of 8 channels for a run of tokens - weights, norm weights and
+// the last TAPS - 1 inputs stay in registers, one load per token and vector - and the next token's input is on its way
+// while this one is normed, rotated and stored.
+constexpr int run_threads(int nv) { return nv == 1 ? 768 : nv == 2 ? 512 : 448; }  // what the registers allow
+template <int TAPS, int NV>
+__global__ void __launch_bounds__(run_threads(NV)) conv_qkv_prep_run_kernel(const PrepArgs a, int run) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[64];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int Cq = a.H * a.dk, Ck = a.G * a.dk, C = Cq + Ck + a.G * a.dv;
+  constexpr int kBack = TAPS - 1;
+  const bf16* w = static_cast<const bf16*>(a.conv_w);
+  const int first = blockIdx.x * run, last = first + run < a.prefill_tokens ? first + run : a.prefill_tokens;
+  int seq = 0;
+  {
+    int lo = 0, hi = a.prefill_seqs - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) / 2;
+      if (a.seq_cu[mid] <= first) lo = mid;
+      else hi = mid - 1;
+    }
+    seq = lo;
+  }
+  const bf16x8 zero8 = {{0u, 0u, 0u, 0u}};
+  int col[NV], ch[NV], v_off[NV];  // column of proj, channel, place in a token's value rows (values only)
+  bf16x8 wt[NV][TAPS], hist[NV][kBack > 0 ? kBack : 1], next[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    ch[i] = c;
+    col[i] = c < Cq ? a.q_off + c : c < Cq + Ck ? a.k_off + c - Cq : a.v_off + c - Cq - Ck;
+    const int vc = c - Cq - Ck;
+    v_off[i] = vc >= 0 && c < C ? vc / a.dv * a.page * a.cols + vc % a.dv : 0;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wt[i][j] = c < C ? ld_bf16x8(w + static_cast<int64_t>(j) * C + c) : zero8;
+    next[i] = c < C ? ld_bf16x8(static_cast<const bf16*>(a.proj) + static_cast<int64_t>(first) * a.ld + col[i]) : zero8;
+  }
+  const int per = a.cols / 8, outs = (a.H + a.G) * per;
+  for (int t = first; t < last; ++t) {
+    while (a.seq_cu[seq + 1] <= t) ++seq;
+    const int li = t - a.seq_cu[seq];
+    int pos = a.positions[t];
+    const bf16* cur = static_cast<const bf16*>(a.proj) + static_cast<int64_t>(t) * a.ld;
+    if (kBack > 0 && (t == first || li == 0)) {  // the inputs before this run, or of this sequence's earlier steps
+      const int slot = a.seq_slots[seq];
+      const bool ok = slot >= 0 && slot < a.num_state_slots;
+      if (!ok && threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_INDEX);
+      const bf16* state = static_cast<const bf16*>(a.conv_state) + static_cast<int64_t>(ok ? slot : 0) * kBack * C;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int j = 0; j < kBack; ++j) {
+          const int b = kBack - j;
+          hist[i][j] = zero8;
+          if (ch[i] >= C || pos - b < 0) continue;
+          if (b <= li) hist[i][j] = ld_bf16x8(cur - static_cast<int64_t>(b) * a.ld + col[i]);
+          else if (ok) hist[i][j] = ld_bf16x8(state + static_cast<int64_t>(li + j) * C + ch[i]);
+        }
+    }
+    int64_t cslot = a.G ? a.slots[t] : -1;
+    if (cslot >= a.num_slots) {
+      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_SLOT);
+      cslot = -1;
+    }
+    const uint32_t us = cslot >= 0 ? static_cast<uint32_t>(cslot) : 0u, page = static_cast<uint32_t>(a.page);
+    // first element of (block, head 0, place in the page); heads are page * cols apart
+    const int64_t kv0 = (static_cast<int64_t>(us / page) * a.G * a.page + us % page) * a.cols;
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      if (ch[i] >= C) continue;
+      float y[8] = {};
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const bf16x8& x = j < kBack ? hist[i][j < kBack ? j : 0] : next[i];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 xf = unpack_bf16x2(x.u[e]), wf = unpack_bf16x2(wt[i][j].u[e]);
+          y[2 * e] = fmaf(wf.x, xf.x, y[2 * e]);
+          y[2 * e + 1] = fmaf(wf.y, xf.y, y[2 * e + 1]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j + 1 < kBack; ++j) hist[i][j] = hist[i][j + 1];
+      if constexpr (kBack > 0) hist[i][kBack - 1] = next[i];
+      if (t + 1 < last) next[i] = ld_bf16x8(cur + a.ld + col[i]);
+      if (ch[i] < Cq + Ck) {
+        float nw[8], sum = 0.f;
+        load_v<8>(ch[i] < Cq ? a.q_norm + ch[i] : a.k_norm + ch[i] - Cq, nw);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          sum = fmaf(y[e], y[e], sum);
+          y[e] *= nw[e];
+        }
+        (ch[i] < Cq ? sq : sk) += sum;
+        store_v<8>(row + ch[i], y);
+      } else if (cslot >= 0) {
+        store_v<8>(static_cast<bf16*>(a.v_cache) + kv0 + v_off[i], y);
+      }
+    }
+    const float2 sums = block_sum2(sq, sk, red);
+    if (pos < 0 || pos >= a.max_pos) {
+      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
+      pos = 0;
+    }
+    const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
+    const float inv_q = 1.f / sqrtf(sums.x / Cq + a.eps), inv_k = a.G ? 1.f / sqrtf(sums.y / Ck + a.eps) : 0.f;
+    for (int i = threadIdx.x; i < outs; i += blockDim.x) {
+      const int h = i / per, d0 = (i - h * per) * 8;
+      float o[8];
+      if (h < a.H) {
+        rotated<8>(row + h * a.dk, inv_q, cs, a.dk, a.rot, d0, o);
+        store_v<8>(static_cast<bf16*>(a.q_out) + (static_cast<int64_t>(t) * a.H + h) * a.cols + d0, o);
+      } else if (cslot >= 0) {
+        const int g = h - a.H;
+        const int64_t at = kv0 + static_cast<int64_t>(g) * a.page * a.cols + d0;
+        rotated<8>(row + Cq + g * a.dk, inv_k, cs, a.dk, a.rot, d0, o);
+        store_v<8>(static_cast<bf16*>(a.k_cache) + at, o);
+        if (d0 >= a.dv) st_bf16x8(static_cast<bf16*>(a.v_cache) + at, zero8);  // zero columns behind the value
       }
     }
     __syncthreads();  // the next token overwrites the row
@@ -295,6 +441,44 @@ __global__ void __launch_bounds__(256) gated_rows_kernel(const GateArgs a) {
 
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
+template <typename K>
+bool opt_in_smem(K kern, size_t smem) {
+  return smem <= 48 * 1024 ||
+         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) == cudaSuccess;
+}
+
+template <int TAPS, int NV>
+bool launch_run(const PrepArgs& a, int threads, size_t smem, cudaStream_t stream) {
+  if (!opt_in_smem(conv_qkv_prep_run_kernel<TAPS, NV>, smem)) return false;
+  int run = ceil_div(a.prefill_tokens, pxl_host::num_sms());
+  if (run < 4) run = 4;
+  if (run > 64) run = 64;
+  pxl_host::launch(conv_qkv_prep_run_kernel<TAPS, NV>, dim3(ceil_div(a.prefill_tokens, run)), dim3(threads), smem, stream, a, run);
+  return true;
+}
+
+// the prompt slices of an aligned bf16 step; false: sizes this kernel does not take
+bool launch_run(const PrepArgs& a, size_t smem, cudaStream_t stream) {
+  const int vecs = (a.H * a.dk + a.G * (a.dk + a.dv)) / 8;
+  int nv = 1;
+  while (nv <= 3 && vecs > nv * run_threads(nv)) ++nv;
+  if (!a.conv_w || nv > 3) return false;
+  const int threads = ceil_div(ceil_div(vecs, nv), 32) * 32;
+#define PXL_RUN(N)                                                          \
+  case N:                                                                   \
+    return nv == 1   ? launch_run<N, 1>(a, threads, smem, stream)           \
+           : nv == 2 ? launch_run<N, 2>(a, threads, smem, stream)           \
+                     : launch_run<N, 3>(a, threads, smem, stream)
+  switch (a.taps) {
+    PXL_RUN(1);
+    PXL_RUN(2);
+    PXL_RUN(3);
+    PXL_RUN(4);
+    default: return false;
+  }
+#undef PXL_RUN
+}
+
 template <typename T, int VEC>
 int launch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
   if (update) {
@@ -303,11 +487,16 @@ int launch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
   } else {
     const size_t smem = sizeof(float) * (a.H + a.G) * a.dk;
     if (smem > 220 * 1024) return PXL_ERR_TOO_LARGE;
-    if (smem > 48 * 1024 && cudaFuncSetAttribute(conv_qkv_prep_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                                 static_cast<int>(smem)) != cudaSuccess)
-      return PXL_ERR_CUDA;
-    const int per = a.prefill_tokens >= 4 * 8 * pxl_host::num_sms() ? 4 : 1;  // neighbours share taps through L1
-    pxl_host::launch(conv_qkv_prep_kernel<T, VEC>, dim3(ceil_div(a.T, per)), dim3(256), smem, stream, a, per);
+    if (!opt_in_smem(conv_qkv_prep_kernel<T, VEC>, smem)) return PXL_ERR_CUDA;
+    int begin = 0;
+    if constexpr (VEC == 8 && sizeof(T) == 2) {
+      if (a.prefill_tokens > 0 && launch_run(a, smem, stream)) begin = a.prefill_tokens;
+    }
+    if (begin < a.T) {
+      // long prompts: neighbours share taps through L1; few tokens: more threads for each
+      const int sms = pxl_host::num_sms(), per = a.T - begin >= 16 * sms ? 4 : 1, threads = a.T - begin <= 2 * sms ? 512 : 256;
+      pxl_host::launch(conv_qkv_prep_kernel<T, VEC>, dim3(ceil_div(a.T - begin, per)), dim3(threads), smem, stream, a, begin, per);
+    }
   }
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }
@@ -316,13 +505,14 @@ template <typename T>
 int dispatch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
   const bool vec = !((a.q_off | a.k_off | a.v_off | a.dk | a.dv | a.cols | (a.rot / 2) | static_cast<int>(a.ld)) & 7) &&
                    aligned16(a.proj) && aligned16(a.conv_w) && aligned16(a.conv_state) && aligned16(a.k_cache) &&
-                   aligned16(a.v_cache) && aligned16(a.q_out);
+                   aligned16(a.v_cache) && aligned16(a.q_out) && aligned16(a.q_norm) && aligned16(a.k_norm) &&
+                   aligned16(a.cos_sin);
   return vec ? launch_prep<T, 8>(a, update, stream) : launch_prep<T, 1>(a, update, stream);
 }
 
 inline bool bad_prep(const PrepArgs& a) {
   return a.H <= 0 || a.G < 0 || a.dk <= 0 || (a.G && a.dv <= 0) || a.cols < a.dk || (a.G && a.cols < a.dv) || a.rot < 0 ||
-         a.rot > a.dk || (a.rot & 1) || a.taps < 1 || a.page <= 0 || (a.taps > 1 && a.conv_w && a.conv_state == nullptr);
+         a.rot > a.dk || (a.rot & 1) || a.taps < 1 || a.page <= 0 || a.num_slots >= (1ll << 31) || (a.taps > 1 && a.conv_w && a.conv_state == nullptr);
 }
 }  // namespace
 

@@ -19,8 +19,6 @@
 namespace {
 using namespace pxl;
 
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ float silu(float v) { return v / (1.f + expf(-v)); }
@@ -186,10 +184,6 @@ int launch_recurrent(const LightningArgs& a, int seq0, int n, cudaStream_t strea
 constexpr int kVS = 32;  // columns of v (and of the state) per CTA
 constexpr int kWarps = 8;
 
-__device__ __forceinline__ void split(float v, bf16& hi, bf16& lo) {
-  hi = __float2bfloat16(v);
-  lo = __float2bfloat16(v - __bfloat162float(hi));
-}
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(a, b);
   const float2 f = unpack_bf16x2(hi);

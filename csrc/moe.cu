@@ -27,8 +27,8 @@ __device__ __forceinline__ float load_score(const void* p, size_t i) {
   else return static_cast<const float*>(p)[i];
 }
 
-// One warp per token.
-template <bool BF16>
+// One warp per token; EPL: experts a lane holds (expert e belongs to lane e % 32).
+template <bool BF16, int EPL>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __restrict__ e_bias, int T, int E,
                  int k, int mode, int renorm, int n_group, int topk_group, int group_top, float routed_scale,
@@ -37,11 +37,11 @@ moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __res
   const int t = blockIdx.x * 4 + warp;
   if (t >= T) return;
   const int epl = (E + 31) / 32;
-  float s[kMaxEPL];    // unbiased score (softmax prob or sigmoid)
-  float sel[kMaxEPL];  // selection score
+  float s[EPL];    // unbiased score (softmax prob or sigmoid)
+  float sel[EPL];  // selection score
   float mx = -INFINITY;
 #pragma unroll
-  for (int j = 0; j < kMaxEPL; ++j) {
+  for (int j = 0; j < EPL; ++j) {
     const int e = j * 32 + lane;
     s[j] = (j < epl && e < E) ? load_score<BF16>(logits, static_cast<size_t>(t) * ld + e) : -INFINITY;
     mx = fmaxf(mx, s[j]);
@@ -50,21 +50,21 @@ moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __res
     mx = warp_reduce_max(mx);
     float sum = 0.f;
 #pragma unroll
-    for (int j = 0; j < kMaxEPL; ++j) {
+    for (int j = 0; j < EPL; ++j) {
       s[j] = (s[j] == -INFINITY) ? 0.f : __expf(s[j] - mx);
       sum += s[j];
     }
     sum = warp_reduce_sum(sum);
     const float inv = 1.f / sum;
 #pragma unroll
-    for (int j = 0; j < kMaxEPL; ++j) {
+    for (int j = 0; j < EPL; ++j) {
       const int e = j * 32 + lane;
       s[j] *= inv;
       sel[j] = (j < epl && e < E) ? s[j] + (e_bias ? e_bias[e] : 0.f) : -INFINITY;
     }
   } else {
 #pragma unroll
-    for (int j = 0; j < kMaxEPL; ++j) {
+    for (int j = 0; j < EPL; ++j) {
       const int e = j * 32 + lane;
       const bool ok = j < epl && e < E;
       s[j] = ok ? 1.f / (1.f + __expf(-s[j])) : 0.f;
@@ -78,7 +78,7 @@ moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __res
     for (int g = 0; g < n_group; ++g) {
       float b1 = -INFINITY, b2 = -INFINITY;
 #pragma unroll
-      for (int j = 0; j < kMaxEPL; ++j) {
+      for (int j = 0; j < EPL; ++j) {
         const int e = j * 32 + lane;
         if (j < epl && e < E && e / gsize == g) {
           if (sel[j] > b1) { b2 = b1; b1 = sel[j]; }
@@ -112,7 +112,7 @@ moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __res
       if (lane == arg) gs = -INFINITY;
     }
 #pragma unroll
-    for (int j = 0; j < kMaxEPL; ++j) {
+    for (int j = 0; j < EPL; ++j) {
       const int e = j * 32 + lane;
       if (j < epl && e < E && !((allowed >> (e / gsize)) & 1u)) sel[j] = -INFINITY;
     }
@@ -126,7 +126,7 @@ moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __res
     int arg = 0x7fffffff;
     float best_s = 0.f;
 #pragma unroll
-    for (int j = 0; j < kMaxEPL; ++j) {
+    for (int j = 0; j < EPL; ++j) {
       const int e = j * 32 + lane;
       if (j < epl && e < E && (sel[j] > best || (sel[j] == best && e < arg))) {
         best = sel[j]; arg = e; best_s = s[j];
@@ -141,7 +141,7 @@ moe_route_kernel(const void* __restrict__ logits, int64_t ld, const float* __res
     }
     if (arg != 0x7fffffff && (arg & 31) == lane) {
 #pragma unroll
-      for (int j = 0; j < kMaxEPL; ++j)
+      for (int j = 0; j < EPL; ++j)
         if (j == (arg >> 5)) sel[j] = -INFINITY;  // static indices keep sel[] in registers
     }
     wsum += best_s;
@@ -282,13 +282,23 @@ PXL_EXPORT int pxl_moe_route(const void* logits, int64_t ld, int logits_bf16, co
   if (E <= 0 || E > 32 * kMaxEPL || k <= 0 || k > 32 || k > E) return PXL_ERR_INVALID_ARG;
   if (n_group > 32 || (n_group > 1 && E % n_group)) return PXL_ERR_INVALID_ARG;
   const unsigned grid = (T + 3) / 4;
-  if (logits_bf16)
-    moe_route_kernel<true><<<grid, 128, 0, stream>>>(logits, ld, e_bias, T, E, k, mode, renorm, n_group,
-                                                     topk_group, group_top, routed_scale, out_ids, out_w);
-  else
-    moe_route_kernel<false><<<grid, 128, 0, stream>>>(logits, ld, e_bias, T, E, k, mode, renorm,
-                                                      n_group, topk_group, group_top, routed_scale, out_ids,
-                                                      out_w);
+  const int epl = (E + 31) / 32;
+#define PXL_ROUTE(B16, EPL)                                                                                        \
+  moe_route_kernel<B16, EPL><<<grid, 128, 0, stream>>>(logits, ld, e_bias, T, E, k, mode, renorm, n_group, topk_group, \
+                                                       group_top, routed_scale, out_ids, out_w)
+#define PXL_ROUTE_EPL(B16)          \
+  if (epl <= 1) PXL_ROUTE(B16, 1);  \
+  else if (epl <= 2) PXL_ROUTE(B16, 2); \
+  else if (epl <= 4) PXL_ROUTE(B16, 4); \
+  else if (epl <= 8) PXL_ROUTE(B16, 8); \
+  else PXL_ROUTE(B16, kMaxEPL)
+  if (logits_bf16) {
+    PXL_ROUTE_EPL(true);
+  } else {
+    PXL_ROUTE_EPL(false);
+  }
+#undef PXL_ROUTE_EPL
+#undef PXL_ROUTE
   return check_launch();
 }
 
