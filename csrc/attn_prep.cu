@@ -277,11 +277,16 @@ __global__ void __launch_bounds__(run_threads(NV)) conv_qkv_prep_run_kernel(cons
     for (int j = 0; j < TAPS; ++j) wt[i][j] = c < C ? ld_bf16x8(w + static_cast<int64_t>(j) * C + c) : zero8;
     next[i] = c < C ? ld_bf16x8(static_cast<const bf16*>(a.proj) + static_cast<int64_t>(first) * a.ld + col[i]) : zero8;
   }
+  float* cs = row + Cq + Ck;  // cosines | sines of the token: fetched while it is convolved
   const int per = a.cols / 8, outs = (a.H + a.G) * per;
   for (int t = first; t < last; ++t) {
     while (a.seq_cu[seq + 1] <= t) ++seq;
     const int li = t - a.seq_cu[seq];
-    int pos = a.positions[t];
+    const int pos = a.positions[t];
+    const int table_row = pos < 0 || pos >= a.max_pos ? 0 : pos;
+    float4 angle;
+    if (threadIdx.x * 4 < a.rot)
+      angle = *reinterpret_cast<const float4*>(a.cos_sin + static_cast<int64_t>(table_row) * a.rot + threadIdx.x * 4);
     const bf16* cur = static_cast<const bf16*>(a.proj) + static_cast<int64_t>(t) * a.ld;
     if (kBack > 0 && (t == first || li == 0)) {  // the inputs before this run, or of this sequence's earlier steps
       const int slot = a.seq_slots[seq];
@@ -340,12 +345,9 @@ __global__ void __launch_bounds__(run_threads(NV)) conv_qkv_prep_run_kernel(cons
         store_v<8>(static_cast<bf16*>(a.v_cache) + kv0 + v_off[i], y);
       }
     }
+    if (threadIdx.x * 4 < a.rot) *reinterpret_cast<float4*>(cs + threadIdx.x * 4) = angle;
+    if (pos != table_row && threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
     const float2 sums = block_sum2(sq, sk, red);
-    if (pos < 0 || pos >= a.max_pos) {
-      if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
-      pos = 0;
-    }
-    const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
     const float inv_q = 1.f / sqrtf(sums.x / Cq + a.eps), inv_k = a.G ? 1.f / sqrtf(sums.y / Ck + a.eps) : 0.f;
     for (int i = threadIdx.x; i < outs; i += blockDim.x) {
       const int h = i / per, d0 = (i - h * per) * 8;
@@ -464,6 +466,8 @@ bool launch_run(const PrepArgs& a, size_t smem, cudaStream_t stream) {
   while (nv <= 3 && vecs > nv * run_threads(nv)) ++nv;
   if (!a.conv_w || nv > 3) return false;
   const int threads = ceil_div(ceil_div(vecs, nv), 32) * 32;
+  if (a.rot > 4 * threads) return false;
+  smem += sizeof(float) * a.rot;
 #define PXL_RUN(N)                                                          \
   case N:                                                                   \
     return nv == 1   ? launch_run<N, 1>(a, threads, smem, stream)           \
