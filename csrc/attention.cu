@@ -147,6 +147,19 @@ __device__ __forceinline__ void pv_16x16(const uint32_t (&pf)[4], uint32_t v_sme
   }
 }
 
+// Tiles of the keys [0, keep) and [lo, hi), first to last: those of the kept keys that lie before the window's first tile,
+// then the window's (keep <= 0: none kept).
+struct KeyTiles {
+  int front, first, total;
+  __device__ KeyTiles(int lo, int hi, int keep) {
+    first = lo / TILE;
+    const int kept = keep > 0 ? ceil_div(keep, TILE) : 0;
+    front = kept < first ? kept : first;
+    total = hi > lo ? front + ceil_div(hi, TILE) - first : 0;
+  }
+  __device__ int operator[](int i) const { return i < front ? i : first + i - front; }
+};
+
 __device__ __forceinline__ float quad_max(float v) {
   v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
   v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
@@ -166,7 +179,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
                    const int* __restrict__ ctx_lens, bf16* __restrict__ out,
                    float* __restrict__ workspace, const float* __restrict__ sinks, int Hq, int Hkv,
                    int page_size, int max_blocks, int64_t num_blocks, float scale_log2, int window,
-                   int num_splits, float v_scale, int* status) {
+                   int keep, int num_splits, float v_scale, int* status) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int TILE_BYTES = TILE * D * 2;
   const uint32_t k_smem0 = smem_u32(smem);
@@ -178,11 +191,10 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
   const int ctx = ctx_lens[b];
   const int hi = ctx;
   const int lo = (window > 0 && ctx > window) ? ctx - window : 0;
-  const int tile_lo = lo / TILE;
-  const int tiles_total = hi > lo ? ceil_div(hi, TILE) - tile_lo : 0;
-  const int per_split = ceil_div(tiles_total, num_splits);
-  const int t_begin = tile_lo + split * per_split;
-  const int t_end = min(tile_lo + tiles_total, t_begin + per_split);
+  const KeyTiles tiles(lo, hi, keep);
+  const int per_split = ceil_div(tiles.total, num_splits);
+  const int t_begin = split * per_split;
+  const int t_end = min(tiles.total, t_begin + per_split);
 
   KVTileArgs ka{k_cache, v_cache, block_tables + static_cast<size_t>(b) * max_blocks, max_blocks,
                 num_blocks, Hkv, kvh, page_size};
@@ -210,19 +222,19 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
   float l_run[2] = {0.f, 0.f};
 
   int buf = 0;
-  if (t_begin < t_end) load_kv_tile<D, FP8>(ka, t_begin * TILE, hi, k_smem0, v_smem0, status);
+  if (t_begin < t_end) load_kv_tile<D, FP8>(ka, tiles[t_begin] * TILE, hi, k_smem0, v_smem0, status);
   cp_async_commit();
   for (int t = t_begin; t < t_end; ++t) {
     cp_async_wait<0>();
     __syncthreads();
     if (t + 1 < t_end)
-      load_kv_tile<D, FP8>(ka, (t + 1) * TILE, hi, k_smem0 + (buf ^ 1) * TILE_BYTES,
+      load_kv_tile<D, FP8>(ka, tiles[t + 1] * TILE, hi, k_smem0 + (buf ^ 1) * TILE_BYTES,
                       v_smem0 + (buf ^ 1) * TILE_BYTES, status);
     cp_async_commit();
 
     const int r0 = warp * 16;
-    const int tok_base = t * TILE + r0;
-    if (tok_base < hi && tok_base + 16 > lo) {  // warp-uniform
+    const int tok_base = tiles[t] * TILE + r0;
+    if (tok_base < hi && (tok_base + 16 > lo || tok_base < keep)) {  // warp-uniform
       float s[2][4];
 #pragma unroll
       for (int j = 0; j < 2; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
@@ -233,7 +245,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int tok = tok_base + j * 8 + 2 * (lane & 3) + (e & 1);
-          const bool valid = tok < hi && tok >= lo;
+          const bool valid = tok < hi && (tok >= lo || tok < keep);
           s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
         }
@@ -349,7 +361,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
                        const bf16* __restrict__ q, int64_t q_stride, const int* __restrict__ block_tables,
                        const int* __restrict__ ctx_lens, bf16* __restrict__ out, float* __restrict__ workspace,
                        const float* __restrict__ sinks, int Hq, int Hkv, int page_size, int max_blocks,
-                       int64_t num_blocks, float scale_log2, int window, int num_splits, int* status) {
+                       int64_t num_blocks, float scale_log2, int window, int keep, int num_splits, int* status) {
   constexpr int D = 128;
   constexpr int TILE_BYTES = TILE * D * 2;
   extern __shared__ uint8_t smem_raw[];
@@ -368,11 +380,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   const int ctx = ctx_lens[b];
   const int hi = ctx;
   const int lo = (window > 0 && ctx > window) ? ctx - window : 0;
-  const int tile_lo = lo / TILE;
-  const int tiles_total = hi > lo ? ceil_div(hi, TILE) - tile_lo : 0;
-  const int per_split = ceil_div(tiles_total, num_splits);
-  const int t_begin = tile_lo + split * per_split;
-  const int t_end = min(tile_lo + tiles_total, t_begin + per_split);
+  const KeyTiles tiles(lo, hi, keep);
+  const int per_split = ceil_div(tiles.total, num_splits);
+  const int t_begin = split * per_split;
+  const int t_end = min(tiles.total, t_begin + per_split);
   const int n_tiles = t_end > t_begin ? t_end - t_begin : 0;
   const int* bt = block_tables + static_cast<size_t>(b) * max_blocks;
   const int ppt = TILE / page_size;  // pages per tile
@@ -399,7 +410,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int stage = it % kDecStages;
       int blk = 0;
       if (lane < ppt) {
-        int bi = (t_begin + it) * ppt + lane;
+        int bi = tiles[t_begin + it] * ppt + lane;
         if (bi * page_size >= hi) bi = (hi - 1) / page_size;  // beyond the context: re-read the last page (masked)
         blk = bi < max_blocks ? bt[bi] : -1;
         if (blk < 0 || blk >= num_blocks) {
@@ -457,11 +468,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       failed = 1;
       break;  // reported to the whole CTA at the barrier behind the loop
     }
-    const int t = t_begin + it;
     const uint32_t k_smem = stage0 + stage * 2 * TILE_BYTES, v_smem = k_smem + TILE_BYTES;
     const int r0 = warp * 16;
-    const int tok_base = t * TILE + r0;
-    if (tok_base < hi && tok_base + 16 > lo) {  // warp-uniform
+    const int tok_base = tiles[t_begin + it] * TILE + r0;
+    if (tok_base < hi && (tok_base + 16 > lo || tok_base < keep)) {  // warp-uniform
       float s[2][4];
 #pragma unroll
       for (int j = 0; j < 2; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
@@ -472,7 +482,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int tok = tok_base + j * 8 + 2 * (lane & 3) + (e & 1);
-          const bool valid = tok < hi && tok >= lo;
+          const bool valid = tok < hi && (tok >= lo || tok < keep);
           s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
         }
@@ -605,7 +615,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
                     const int* __restrict__ cu_q, const int* __restrict__ ctx_lens,
                     bf16* __restrict__ out, int64_t out_stride, const float* __restrict__ sinks,
                     int Hq, int Hkv, int page_size, int max_blocks, int64_t num_blocks,
-                    float scale_log2, int window, float v_scale, int* status) {
+                    float scale_log2, int window, int keep, float v_scale, int* status) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int TILE_BYTES = TILE * D * 2;
   const uint32_t k_smem0 = smem_u32(smem);
@@ -663,8 +673,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
   const int c_tok_last = min(q_len - 1, qt * TQ + TQ - 1);
   const int c_hi = prefix + c_tok_last + 1;  // exclusive
   const int c_lo = (window > 0 && prefix + qt * TQ >= window) ? prefix + qt * TQ - window + 1 : 0;
-  const int t_begin = c_lo / TILE;
-  const int t_end = ceil_div(c_hi, TILE);
+  const KeyTiles tiles(c_lo, c_hi, keep);
 
   KVTileArgs ka{k_cache, v_cache, block_tables + static_cast<size_t>(b) * max_blocks, max_blocks,
                 num_blocks, Hkv, kvh, page_size};
@@ -676,18 +685,18 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
   float l_run[2] = {0.f, 0.f};
 
   int buf = 0;
-  load_kv_tile<D, FP8>(ka, t_begin * TILE, c_hi, k_smem0, v_smem0, status);
+  load_kv_tile<D, FP8>(ka, tiles[0] * TILE, c_hi, k_smem0, v_smem0, status);
   cp_async_commit();
-  for (int t = t_begin; t < t_end; ++t) {
+  for (int t = 0; t < tiles.total; ++t) {
     cp_async_wait<0>();
     __syncthreads();
-    if (t + 1 < t_end)
-      load_kv_tile<D, FP8>(ka, (t + 1) * TILE, c_hi, k_smem0 + (buf ^ 1) * TILE_BYTES,
+    if (t + 1 < tiles.total)
+      load_kv_tile<D, FP8>(ka, tiles[t + 1] * TILE, c_hi, k_smem0 + (buf ^ 1) * TILE_BYTES,
                       v_smem0 + (buf ^ 1) * TILE_BYTES, status);
     cp_async_commit();
 
-    const int tok0 = t * TILE;
-    if (warp_active && tok0 <= w_hi && tok0 + TILE > w_lo) {
+    const int tok0 = tiles[t] * TILE;
+    if (warp_active && tok0 <= w_hi && (tok0 + TILE > w_lo || tok0 < keep)) {
       const uint32_t ks_addr = k_smem0 + buf * TILE_BYTES;
       const uint32_t vs_addr = v_smem0 + buf * TILE_BYTES;
       float s[8][4];
@@ -703,7 +712,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
         for (int e = 0; e < 4; ++e) {
           const int h = e >> 1;
           const int tok = tok0 + j * 8 + 2 * (lane & 3) + (e & 1);
-          const bool valid = tok <= rpos[h] && tok >= rlo[h];
+          const bool valid = tok <= rpos[h] && (tok >= rlo[h] || tok < keep);
           s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
           mx[h] = fmaxf(mx[h], s[j][e]);
         }
@@ -795,7 +804,7 @@ namespace {
 int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
                      const int* block_tables, const int* ctx_lens, void* out, float* workspace,
                      const float* sinks, int B, int Hq, int Hkv, int D, int page_size, int max_blocks,
-                     int64_t num_blocks, float scale, int window, int num_splits, int max_ctx,
+                     int64_t num_blocks, float scale, int window, int keep_first, int num_splits, int max_ctx,
                      bool cache_fp8, float k_scale, float v_scale, int* status, pxl_stream_t stream) {
   if (B <= 0) return PXL_OK;
   if (Hkv <= 0 || Hq % Hkv || Hq / Hkv > 16 || page_size <= 0) return PXL_ERR_INVALID_ARG;
@@ -820,7 +829,7 @@ int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache, const
     }
     pxl_host::launch(attn_decode_tma_kernel, grid, kDecThreads, SMEM, stream,
         tk, tv, static_cast<const bf16*>(q), q_stride, block_tables, ctx_lens, static_cast<bf16*>(out), workspace,
-        sinks, Hq, Hkv, page_size, max_blocks, num_blocks, scale_log2, window, num_splits, status);
+        sinks, Hq, Hkv, page_size, max_blocks, num_blocks, scale_log2, window, keep_first, num_splits, status);
     if (num_splits > 1)
       pxl_host::launch(attn_decode_reduce_kernel<128>, dim3(Hq, B), 128, 0, stream, workspace, sinks,
                        static_cast<bf16*>(out), Hq, num_splits);
@@ -839,7 +848,7 @@ int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache, const
     attn_decode_kernel<DD, F8><<<grid, 128, SMEM, stream>>>(                                     \
         static_cast<const bf16*>(q), q_stride, k_cache, v_cache, block_tables, ctx_lens,         \
         static_cast<bf16*>(out), workspace, sinks, Hq, Hkv, page_size, max_blocks, num_blocks,   \
-        scale_log2 * k_scale, window, num_splits, v_scale, status);                              \
+        scale_log2 * k_scale, window, keep_first, num_splits, v_scale, status);                  \
     if (num_splits > 1)                                                                          \
       attn_decode_reduce_kernel<DD><<<dim3(Hq, B), DD, 0, stream>>>(                             \
           workspace, sinks, static_cast<bf16*>(out), Hq, num_splits);                            \
@@ -863,10 +872,10 @@ PXL_EXPORT int pxl_attn_decode(const void* q, int64_t q_stride, const void* k_ca
                                const int* block_tables, const int* ctx_lens, void* out,
                                float* workspace, const float* sinks, int B, int Hq, int Hkv, int D,
                                int page_size, int max_blocks, int64_t num_blocks, float scale,
-                               int window, int num_splits, int max_ctx, int* status,
+                               int window, int keep_first, int num_splits, int max_ctx, int* status,
                                pxl_stream_t stream) {
   return attn_decode_impl(q, q_stride, k_cache, v_cache, block_tables, ctx_lens, out, workspace, sinks,
-                          B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, num_splits,
+                          B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, keep_first, num_splits,
                           max_ctx, false, 1.f, 1.f, status, stream);
 }
 
@@ -882,7 +891,7 @@ PXL_EXPORT int pxl_attn_decode_fp8(const void* q, int64_t q_stride, const void* 
                                    int* status, pxl_stream_t stream) {
   if (!(k_scale > 0.f) || !(v_scale > 0.f)) return PXL_ERR_INVALID_ARG;
   return attn_decode_impl(q, q_stride, k_cache, v_cache, block_tables, ctx_lens, out, workspace, sinks,
-                          B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, num_splits,
+                          B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, 0, num_splits,
                           max_ctx, true, k_scale, v_scale, status, stream);
 }
 
@@ -891,7 +900,7 @@ int attn_prefill_impl(const void* q, int64_t q_stride, const void* k_cache, cons
                       const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                       int64_t out_stride, const float* sinks, int B, int max_q_len, int Hq, int Hkv,
                       int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                      int window, bool cache_fp8, float k_scale, float v_scale, int* status,
+                      int window, int keep_first, bool cache_fp8, float k_scale, float v_scale, int* status,
                       pxl_stream_t stream) {
   if (B <= 0 || max_q_len <= 0) return PXL_OK;
   if (Hkv <= 0 || Hq % Hkv || Hq / Hkv > 64 || page_size <= 0) return PXL_ERR_INVALID_ARG;
@@ -911,7 +920,7 @@ int attn_prefill_impl(const void* q, int64_t q_stride, const void* k_cache, cons
     attn_prefill_kernel<DD, F8><<<grid, 128, SMEM, stream>>>(                                    \
         static_cast<const bf16*>(q), q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens,   \
         static_cast<bf16*>(out), out_stride, sinks, Hq, Hkv, page_size, max_blocks, num_blocks,  \
-        scale_log2 * k_scale, window, v_scale, status);                                          \
+        scale_log2 * k_scale, window, keep_first, v_scale, status);                              \
   }
   if (cache_fp8) {
     if (D == 128) PXL_PRE(128, true)
@@ -932,10 +941,10 @@ PXL_EXPORT int pxl_attn_prefill(const void* q, int64_t q_stride, const void* k_c
                                 const int* ctx_lens, void* out, int64_t out_stride,
                                 const float* sinks, int B, int max_q_len, int Hq, int Hkv, int D,
                                 int page_size, int max_blocks, int64_t num_blocks, float scale,
-                                int window, int* status, pxl_stream_t stream) {
+                                int window, int keep_first, int* status, pxl_stream_t stream) {
   return attn_prefill_impl(q, q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens, out, out_stride,
                            sinks, B, max_q_len, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale,
-                           window, false, 1.f, 1.f, status, stream);
+                           window, keep_first, false, 1.f, 1.f, status, stream);
 }
 
 // Prefix-aware prefill over e4m3 caches (see pxl_attn_decode_fp8).
@@ -949,7 +958,7 @@ PXL_EXPORT int pxl_attn_prefill_fp8(const void* q, int64_t q_stride, const void*
   if (!(k_scale > 0.f) || !(v_scale > 0.f)) return PXL_ERR_INVALID_ARG;
   return attn_prefill_impl(q, q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens, out, out_stride,
                            sinks, B, max_q_len, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale,
-                           window, true, k_scale, v_scale, status, stream);
+                           window, 0, true, k_scale, v_scale, status, stream);
 }
 
 // ----------------------------------------------------------------------------------------
@@ -1002,6 +1011,6 @@ PXL_EXPORT int pxl_attn_decode_static_scratch(const void* q, int64_t q_stride, c
   // Every (sequence, head, split) partial that the reduction reads is written by the main
   // kernel of this same call, so the array needs no clearing between calls.
   return pxl_attn_decode(q, q_stride, k_cache, v_cache, block_tables, ctx_lens, out, scratch, sinks,
-                         B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, num_splits,
+                         B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, 0, num_splits,
                          0, status, stream);
 }

@@ -1,6 +1,6 @@
 // Paged attention with grouped heads on the FMA pipes, bf16 or fp32, any head size: what the tensor-core kernels
 // (attention.cu, attention_prefill_tc.cu) do not take - fp32 models, head sizes other than 64 and 128, many query
-// heads per key head. Causal, optional sliding window, optional sink per head (exp(sink) in the softmax
+// heads per key head. Causal, optional sliding window (which may keep a sequence's first keys), optional sink per head (exp(sink) in the softmax
 // denominator, no key, no value, not scaled). Cache layout as in attention.cu: K, V = [blocks, Hkv, page, D].
 //
 // One CTA per (query token, up to four query heads of one key head); keys stream through shared memory in small
@@ -31,7 +31,7 @@ struct AnyArgs {
   void* out;
   int64_t out_stride;
   const float* sinks;
-  int Hq, Hkv, D, page, max_blocks, window;
+  int Hq, Hkv, D, page, max_blocks, window, keep;
   int64_t num_blocks;
   float scale;
   int* status;
@@ -52,6 +52,8 @@ __global__ void __launch_bounds__(kThreads) attn_any_kernel(const AnyArgs a) {
   const int64_t t = t0 + ti;
   const int pos = a.ctx_lens[b] - len + ti;
   const int lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+  // the visible keys are [0, keep) and [lo, pos], walked as one run
+  const int keep = a.keep < lo ? a.keep : lo, total = keep + pos + 1 - lo;
   float* q = sm;                    // [kHG][D]
   float* acc = q + kHG * D;         // [kHG][D]
   float* ks = acc + kHG * D;        // [kTile][D]
@@ -69,11 +71,11 @@ __global__ void __launch_bounds__(kThreads) attn_any_kernel(const AnyArgs a) {
   }
   const int* bt = a.block_tables + static_cast<int64_t>(b) * a.max_blocks;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int k0 = lo; k0 <= pos; k0 += kTile) {
-    const int n = pos + 1 - k0 < kTile ? pos + 1 - k0 : kTile;
+  for (int k0 = 0; k0 < total; k0 += kTile) {
+    const int n = total - k0 < kTile ? total - k0 : kTile;
     __syncthreads();
     for (int i = threadIdx.x; i < n * D; i += kThreads) {
-      const int kp = k0 + i / D, pg = kp / a.page;
+      const int at = k0 + i / D, kp = at < keep ? at : at - keep + lo, pg = kp / a.page;
       int64_t blk = pg < a.max_blocks ? bt[pg] : -1;
       if (blk < 0 || blk >= a.num_blocks) {
         if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_BLOCK_PREFILL);
@@ -145,10 +147,10 @@ int launch_any(const AnyArgs& a, int B, int max_q, cudaStream_t stream) {
 PXL_EXPORT int pxl_attn_any(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const int* block_tables,
                             const int* cu_q, const int* ctx_lens, void* out, int64_t out_stride, const float* sinks, int B,
                             int max_q, int Hq, int Hkv, int D, int page, int max_blocks, int64_t num_blocks, float scale,
-                            int window, int is_f32, int* status, cudaStream_t stream) {
+                            int window, int keep_first, int is_f32, int* status, cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return PXL_OK;
   if (Hkv <= 0 || Hq % Hkv || D <= 0 || page <= 0 || B > 65535) return PXL_ERR_INVALID_ARG;
   AnyArgs a{q, q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens, out, out_stride, sinks, Hq, Hkv, D, page, max_blocks,
-            window, num_blocks, scale, status};
+            window, keep_first, num_blocks, scale, status};
   return is_f32 ? launch_any<float>(a, B, max_q, stream) : launch_any<pxl::bf16>(a, B, max_q, stream);
 }

@@ -71,7 +71,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
                        const __grid_constant__ CUtensorMap tm_v, const int* __restrict__ block_tables,
                        const int* __restrict__ cu_q, const int* __restrict__ ctx_lens, bf16* __restrict__ out,
                        int64_t out_stride, const float* __restrict__ sinks, int Hq, int Hkv, int page_size,
-                       int max_blocks, int64_t num_blocks, float scale_log2, int window, int* status) {
+                       int max_blocks, int64_t num_blocks, float scale_log2, int window, int keep, int* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sm0 = smem_u32(smem);
@@ -98,8 +98,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
   const int rows = L - q0 < kQ ? L - q0 : kQ;           // valid query rows
   const int hi = pos0 + rows;                           // keys [lo, hi) are visible to some row
   const int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
-  const int t_begin = lo / kT;
-  const int n_tiles = ceil_div(hi, kT) - t_begin;
+  // tiles of keys: those of the kept first keys before the window's first tile, then the window's
+  const int t_window = lo / kT, kept = keep > 0 ? ceil_div(keep, kT) : 0, front = kept < t_window ? kept : t_window;
+  const int n_tiles = front + ceil_div(hi, kT) - t_window;
+  auto tile_of = [&](int it) { return it < front ? it : t_window + it - front; };
   const int* bt = block_tables + static_cast<size_t>(b) * max_blocks;
 
   if (threadIdx.x == 0) {
@@ -143,7 +145,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       const int stage = it % kStages;
       int blk = 0;
       if (lane < ppt) {
-        int bi = (t_begin + it) * ppt + lane;
+        int bi = tile_of(it) * ppt + lane;
         if (bi * page_size >= ctx) bi = (ctx - 1) / page_size;  // beyond the context: re-read the last page (masked)
         blk = bi < max_blocks ? bt[bi] : -1;
         if (blk < 0 || blk >= num_blocks) {
@@ -252,9 +254,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         failed = mbar_wait_bounded(s_full + 8 * (it & 1), (it >> 1) & 1, abort_flag, status, PXL_DEV_TIMEOUT_TMEM_FULL) ? 0 : 1;
       failed = __any_sync(0xffffffffu, failed);  // warp-uniform: the TMEM loads below are warp-wide
       const uint32_t t_s = tmem_base + (it & 1) * kT + hc * 64 + lane_sel;
-      const int tile_key0 = (t_begin + it) * kT;
+      const int tile_key0 = tile_of(it) * kT;
       // interior tile: every key is visible to every row of the block, no masking needed
-      const bool interior = tile_key0 + kT - 1 <= pos0 && (window <= 0 || tile_key0 >= pos0 + kQ - window);
+      const bool interior = tile_key0 + kT - 1 <= pos0 &&
+                            (window <= 0 || tile_key0 >= pos0 + kQ - window || tile_key0 + kT <= keep);
       // this thread's 64 scores stay in registers between the maximum and the exponentials
       uint32_t sc[64];
       float mx = -INFINITY;
@@ -264,12 +267,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         tmem_ld_32x32b_x32(t_s + 32, *reinterpret_cast<uint32_t(*)[32]>(&sc[32]));
         tmem_ld_wait();
         if (!interior) {
-          // keys this thread's row may see among its 64 columns: [a, e)
+          // keys this thread's row may see among its 64 columns: [a, e), and those before f
           const int key0 = tile_key0 + hc * 64;
-          const int a = key_lo - key0, e = (row_valid ? q_pos + 1 : 0) - key0;
+          const int a = key_lo - key0, e = (row_valid ? q_pos + 1 : 0) - key0, f = keep - key0;
 #pragma unroll
           for (int j = 0; j < 64; ++j)
-            if (j < a || j >= e) sc[j] = 0xff800000u;  // -inf
+            if ((j < a && j >= f) || j >= e) sc[j] = 0xff800000u;  // -inf
         }
         float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -389,7 +392,7 @@ PXL_EXPORT int pxl_attn_prefill_tc(const void* q, int64_t q_stride, const void* 
                                    const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                                    int64_t out_stride, const float* sinks, int B, int max_q_len, int total_q, int Hq,
                                    int Hkv, int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                                   int window, int* status, cudaStream_t stream) {
+                                   int window, int keep_first, int* status, cudaStream_t stream) {
   if (B <= 0 || max_q_len <= 0 || total_q <= 0) return PXL_OK;
   if (D != kD || Hkv <= 0 || Hq % Hkv) return PXL_ERR_INVALID_ARG;
   if (page_size != 16 && page_size != 32 && page_size != 64) return PXL_ERR_INVALID_ARG;
@@ -415,6 +418,6 @@ PXL_EXPORT int pxl_attn_prefill_tc(const void* q, int64_t q_stride, const void* 
   dim3 grid(pxl::ceil_div(max_q_len, kQ), Hq, B);
   pxl_host::launch(attn_prefill_tc_kernel, grid, kThreads, kSmemBytes, stream,
       tq, tk, tv, block_tables, cu_q, ctx_lens, static_cast<pxl::bf16*>(out), out_stride, sinks, Hq, Hkv, page_size,
-      max_blocks, num_blocks, scale * kLog2eF, window, status);
+      max_blocks, num_blocks, scale * kLog2eF, window, keep_first, status);
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }

@@ -3,12 +3,13 @@
 //  * pxl_conv_qkv_prep: one launch per layer and step turns the packed projection q | k | v into queries and
 //    cache rows: short causal convolution per channel (y_t = sum_j w[j] u[t - taps + 1 + j], zeros before the
 //    sequence), RMS norm over the whole q row and the whole k row, half-split rotation, and the scatter of k and
-//    v into their pages. Heads are padded with zeros to `cols` columns. v is neither normed nor rotated.
+//    v into their pages. Heads are padded with zeros to `cols` columns. v is neither normed nor rotated. Without
+//    convolution and norms a kernel of its own does the rest, in which no thread waits for another.
 //  * pxl_conv_state_update: the last taps - 1 projected rows of every prompt slice become the state of its slot
 //    (a launch of its own: the first tokens of the slice read the state that its last tokens replace; a decoded
 //    token reads and replaces it in pxl_conv_qkv_prep itself).
-//  * pxl_gated_rows: concatenated heads, optionally RMS-normed together, times sigmoid(gate), into the columns of
-//    the output product's operand.
+//  * pxl_gated_rows: concatenated heads, optionally RMS-normed together or one by one, times sigmoid(gate) and a factor,
+//    into the columns of the output product's operand.
 //
 // All arithmetic is fp32.
 #include "common.cuh"
@@ -367,6 +368,59 @@ __global__ void __launch_bounds__(run_threads(NV)) conv_qkv_prep_run_kernel(cons
   }
 }
 
+// Neither convolution nor norms: every vector of an output head is made by one thread from the projection.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) rotate_qkv_kernel(const PrepArgs a, int64_t n) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  if (i >= n) return;
+  const int per = a.cols / VEC, heads = a.H + 2 * a.G;
+  const int d0 = static_cast<int>(i % per) * VEC, h = static_cast<int>(i / per % heads);
+  const int64_t t = i / per / heads;
+  int pos = a.positions[t];
+  if (pos < 0 || pos >= a.max_pos) {
+    if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
+    pos = 0;
+  }
+  const T* row = static_cast<const T*>(a.proj) + t * a.ld;
+  const bool value = h >= a.H + a.G;
+  const T* src = h < a.H ? row + a.q_off + h * a.dk : value ? row + a.v_off + (h - a.H - a.G) * a.dv : row + a.k_off + (h - a.H) * a.dk;
+  const int width = value ? a.dv : a.dk, half = a.rot / 2;
+  float o[VEC];
+  if (d0 >= width) {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+  } else {
+    load_v<VEC>(src + d0, o);
+    if (!value && d0 < a.rot) {
+      const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
+      const bool lower = d0 < half;
+      const int f = lower ? d0 : d0 - half;
+      float c[VEC], sn[VEC], x[VEC];
+      load_v<VEC>(cs + f, c);
+      load_v<VEC>(cs + half + f, sn);
+      load_v<VEC>(src + (lower ? d0 + half : f), x);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = lower ? o[j] * c[j] - x[j] * sn[j] : o[j] * c[j] + x[j] * sn[j];
+    }
+  }
+  if (h < a.H) {
+    store_v<VEC>(static_cast<T*>(a.q_out) + (t * a.H + h) * a.cols + d0, o);
+    return;
+  }
+  const int64_t slot = a.slots[t];
+  if (slot < 0) return;
+  if (slot >= a.num_slots) {
+    if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_SLOT);
+    return;
+  }
+  const uint32_t us = static_cast<uint32_t>(slot), page = static_cast<uint32_t>(a.page);
+  const int g = value ? h - a.H - a.G : h - a.H;
+  T* pages = static_cast<T*>(value ? a.v_cache : a.k_cache);
+  store_v<VEC>(pages + ((static_cast<int64_t>(us / page) * a.G + g) * a.page + us % page) * a.cols + d0, o);
+}
+
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256) conv_state_update_kernel(const PrepArgs a) {
   pdl_wait();
@@ -397,7 +451,8 @@ struct GateArgs {
   const void* gate;     // [T, ldg], heads * dv columns
   int64_t ldg;
   const float* norm_w;  // [heads * dv] or null
-  float eps;
+  float eps, scale;
+  int per_head;         // the norm's statistics are those of one head
   void* out;            // [T, ldo], out_cols columns: heads * dv, then zeros
   int64_t ldo;
   int out_cols;
@@ -414,7 +469,22 @@ __global__ void __launch_bounds__(256) gated_rows_kernel(const GateArgs a) {
   const T* g = static_cast<const T*>(a.gate) + t * a.ldg;
   T* out = static_cast<T*>(a.out) + t * a.ldo;
   float inv = 1.f;
-  if (a.norm_w) {
+  extern __shared__ float head_inv[];  // per_head: [heads]
+  if (a.norm_w && a.per_head) {
+    const int lane = threadIdx.x & 31;
+    for (int h = threadIdx.x >> 5; h < a.heads; h += blockDim.x >> 5) {  // one warp per head
+      float sq = 0.f;
+      for (int c = lane * VEC; c < a.dv; c += 32 * VEC) {
+        float v[VEC];
+        load_v<VEC>(x + static_cast<int64_t>(h) * a.x_cols + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) sq = fmaf(v[j], v[j], sq);
+      }
+      sq = warp_reduce_sum(sq);
+      if (lane == 0) head_inv[h] = 1.f / sqrtf(sq / a.dv + a.eps);
+    }
+    __syncthreads();
+  } else if (a.norm_w) {
     float sq = 0.f;
     for (int c = threadIdx.x * VEC; c < N; c += blockDim.x * VEC) {
       float v[VEC];
@@ -431,11 +501,12 @@ __global__ void __launch_bounds__(256) gated_rows_kernel(const GateArgs a) {
     if (a.norm_w) {
       float w[VEC];
       load_v<VEC>(a.norm_w + c, w);
+      const float f = a.per_head ? head_inv[c / a.dv] : inv;
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
+      for (int j = 0; j < VEC; ++j) v[j] *= f * w[j];
     }
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) v[j] /= 1.f + expf(-gv[j]);
+    for (int j = 0; j < VEC; ++j) v[j] *= a.scale / (1.f + expf(-gv[j]));
     store_v<VEC>(out + c, v);
   }
   for (int c = N + threadIdx.x; c < a.out_cols; c += blockDim.x) put(out + c, 0.f);
@@ -485,7 +556,10 @@ bool launch_run(const PrepArgs& a, size_t smem, cudaStream_t stream) {
 
 template <typename T, int VEC>
 int launch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
-  if (update) {
+  if (!a.conv_w && !a.q_norm) {
+    const int64_t n = static_cast<int64_t>(a.T) * (a.H + 2 * a.G) * (a.cols / VEC);
+    pxl_host::launch(rotate_qkv_kernel<T, VEC>, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0, stream, a, n);
+  } else if (update) {
     const int C = a.H * a.dk + a.G * (a.dk + a.dv);
     pxl_host::launch(conv_state_update_kernel<T, VEC>, dim3(ceil_div(C, 256 * VEC), a.prefill_seqs), dim3(256), 0, stream, a);
   } else {
@@ -516,7 +590,8 @@ int dispatch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
 
 inline bool bad_prep(const PrepArgs& a) {
   return a.H <= 0 || a.G < 0 || a.dk <= 0 || (a.G && a.dv <= 0) || a.cols < a.dk || (a.G && a.cols < a.dv) || a.rot < 0 ||
-         a.rot > a.dk || (a.rot & 1) || a.taps < 1 || a.page <= 0 || a.num_slots >= (1ll << 31) || (a.taps > 1 && a.conv_w && a.conv_state == nullptr);
+         a.rot > a.dk || (a.rot & 1) || a.taps < 1 || a.page <= 0 || a.num_slots >= (1ll << 31) || (a.q_norm == nullptr && a.conv_w) ||
+         (a.G && (a.q_norm == nullptr) != (a.k_norm == nullptr)) || (a.taps > 1 && a.conv_w && a.conv_state == nullptr);
 }
 }  // namespace
 
@@ -538,19 +613,21 @@ PXL_EXPORT int pxl_conv_qkv_prep(const void* proj, int64_t ld, int q_off, int k_
 }
 
 PXL_EXPORT int pxl_gated_rows(const void* x, int heads, int x_cols, int dv, const void* gate, int64_t ldg,
-                              const float* norm_w, float eps, void* out, int64_t ldo, int out_cols, int T, int is_f32,
-                              cudaStream_t stream) {
+                              const float* norm_w, float eps, int per_head, float scale, void* out, int64_t ldo, int out_cols,
+                              int T, int is_f32, cudaStream_t stream) {
   if (T <= 0) return PXL_OK;
+  const size_t smem = norm_w && per_head ? sizeof(float) * heads : 0;
+  if (smem > 40 * 1024) return PXL_ERR_TOO_LARGE;
   if (heads <= 0 || dv <= 0 || x_cols < dv || out_cols < heads * dv) return PXL_ERR_INVALID_ARG;
-  const GateArgs a{x, heads, x_cols, dv, gate, ldg, norm_w, eps, out, ldo, out_cols};
+  const GateArgs a{x, heads, x_cols, dv, gate, ldg, norm_w, eps, scale, per_head, out, ldo, out_cols};
   const bool vec = !((x_cols | dv | static_cast<int>(ldg) | static_cast<int>(ldo)) & 7) && aligned16(x) && aligned16(gate) &&
                    aligned16(out) && aligned16(norm_w);
   if (is_f32) {
-    if (vec) pxl_host::launch(gated_rows_kernel<float, 8>, dim3(T), dim3(256), 0, stream, a);
-    else pxl_host::launch(gated_rows_kernel<float, 1>, dim3(T), dim3(256), 0, stream, a);
+    if (vec) pxl_host::launch(gated_rows_kernel<float, 8>, dim3(T), dim3(256), smem, stream, a);
+    else pxl_host::launch(gated_rows_kernel<float, 1>, dim3(T), dim3(256), smem, stream, a);
   } else {
-    if (vec) pxl_host::launch(gated_rows_kernel<pxl::bf16, 8>, dim3(T), dim3(256), 0, stream, a);
-    else pxl_host::launch(gated_rows_kernel<pxl::bf16, 1>, dim3(T), dim3(256), 0, stream, a);
+    if (vec) pxl_host::launch(gated_rows_kernel<pxl::bf16, 8>, dim3(T), dim3(256), smem, stream, a);
+    else pxl_host::launch(gated_rows_kernel<pxl::bf16, 1>, dim3(T), dim3(256), smem, stream, a);
   }
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }

@@ -59,7 +59,10 @@ struct GemmEpilogueArgs {
   bf16* const* row_ptrs; // EPI_SCATTER: destination of every output row (null = drop), N elements each
   uint32_t* done_counter;  // EPI_SCATTER: local counter for the "last CTA publishes the flags" step
   float act_limit;           // EPI_CLIP_GLU
-  int act;                   // EPI_GLU: 0 silu, 2 gelu (tanh form)
+  int act;                   // EPI_GLU: 0 silu, 2 gelu (tanh form); EPI_ACT: 2 gelu, 3 square of relu
+  const bf16* table;         // EPI_ACT: optional, row m times table[ids[m] * ld_table + column]
+  const int* ids;
+  int64_t ld_table, num_ids;
   const float* row_gate;     // EPI_GLU: optional, row m times sigmoid(row_gate[m * ld_row_gate])
   int64_t ld_row_gate;
   const bf16* gate;          // EPI_GATE: [M, ldg], indexed by the row of W like the bias
@@ -535,6 +538,17 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
         }
       } else {
         const int col0 = n_blk * BN;
+        int64_t table_row = 0;
+        if constexpr (EPI == PXL_EPI_ACT) {
+          if (ep.table && row < M_end) {
+            int64_t id = ep.ids[row];
+            if (id < 0 || id >= ep.num_ids) {
+              if (status) atomicCAS(status, 0, PXL_DEV_BAD_ROW_ID);
+              id = 0;
+            }
+            table_row = id * ep.ld_table;
+          }
+        }
 #pragma unroll 1
         for (int c0 = 0; c0 < BN; c0 += 32) {
           uint32_t r[32];
@@ -577,6 +591,23 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                       const float2 bb = unpack_bf16x2(gg.u[j]);
                       f[2 * j] *= 1.f / (1.f + __expf(-bb.x));
                       f[2 * j + 1] *= 1.f / (1.f + __expf(-bb.y));
+                    }
+                  }
+                }
+                if constexpr (EPI == PXL_EPI_ACT) {
+#pragma unroll
+                  for (int j = 0; j < 8; ++j) {
+                    const float z = f[j], p = fmaxf(z, 0.f);
+                    // gelu, tanh form: z (1 + tanh(s)) / 2 = z / (1 + exp(-2 s))
+                    f[j] = ep.act == 3 ? p * p : z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+                  }
+                  if (ep.table) {
+                    const bf16x8 b = ld_bf16x8(ep.table + table_row + col);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                      const float2 bb = unpack_bf16x2(b.u[j]);
+                      f[2 * j] *= bb.x;
+                      f[2 * j + 1] *= bb.y;
                     }
                   }
                 }
@@ -1476,6 +1507,36 @@ PXL_EXPORT int pxl_gemm_bf16_act_glu(const void* A, const void* W, void* C, int 
   ep.row_gate = row_gate;
   ep.ld_row_gate = ld_row_gate;
   return gemm_glu<PXL_EPI_GLU>(A, W, C, M, N, K, lda, ldw, ldc, ep, bn, status, stream);
+}
+
+// Activation epilogue (see pxl_api.h).
+PXL_EXPORT int pxl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
+                                 const void* table, int64_t ld_table, const int* ids, int64_t num_ids, int* status,
+                                 cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || (act != 2 && act != 3) || (table && !ids)) return PXL_ERR_INVALID_ARG;
+  if ((K % 8) || (lda % 8) || (ldw % 8) || (ldc % 8) || (N % 8) || (ld_table % 8)) return PXL_ERR_INVALID_ARG;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C) |
+       reinterpret_cast<uintptr_t>(table)) & 15)
+    return PXL_ERR_INVALID_ARG;
+  const int bn = pxl_gemm_bf16_pick_bn(M, N, PXL_EPI_ACT);
+  CUtensorMap ta, tb;
+  if (!pxl_host::make_tmap_2d(&ta, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, M, K, lda, BM, BK) ||
+      !pxl_host::make_tmap_2d(&tb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, N, K, ldw, bn, BK))
+    return PXL_ERR_TENSORMAP;
+  GemmEpilogueArgs ep{};
+  ep.C = static_cast<pxl::bf16*>(C);
+  ep.ldc = ldc;
+  ep.act = act;
+  ep.table = static_cast<const pxl::bf16*>(table);
+  ep.ids = ids;
+  ep.ld_table = ld_table;
+  ep.num_ids = num_ids;
+  GemmGroupArgs grp{};
+  switch (bn) {
+    case 256: return launch_gemm<256, PXL_EPI_ACT>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+    case 128: return launch_gemm<128, PXL_EPI_ACT>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+    default: return launch_gemm<64, PXL_EPI_ACT>(ta, tb, ep, grp, GemmCommArgs{}, 0, M, N, K, status, stream);
+  }
 }
 
 // Per-head products (see pxl_api.h). K columns past a head's K meet zeros: the tensor map of W ends at K.

@@ -3,7 +3,8 @@
 // and an optional learned sink per head (exp(sink) in the softmax denominator, no key, no value, not scaled).
 //
 //  * pxl_latent_prep: one launch per layer and step turns the packed projection into cache rows (RMS norm of
-//    the latent, interleaved rotation of the key part) and the rotated query parts.
+//    the latent, interleaved rotation of the key part) and the rotated query parts. Where queries go through a normed
+//    latent of their own, pxl_latent_rows makes the cache rows and that latent, and pxl_latent_queries the rotated parts.
 //  * pxl_latent_attn: FMA-pipe kernel for fp32 models and for bf16 sizes that the tensor-core kernel
 //    (latent_attn_tc.cu) does not take. One CTA per (query token, group of heads); keys stream through shared
 //    memory in small tiles with an online softmax.
@@ -19,14 +20,20 @@ __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
 
 struct PrepArgs {
-  const void* proj;  // [T, ld]: query heads from column 0, latent | key part at kv_off
+  const void* proj;  // [T, ld]: latent | key part at kv_off
   int64_t ld;
-  int kv_off, heads, q_width, q_rot_off, L, R, rot;
+  int kv_off;
+  const void* q;     // [T, ldq]: query heads from column 0 (null: none)
+  int64_t ldq;
+  int heads, q_width, q_rot_off, L, R, rot;
+  int cq_off, cq_rank;  // query latent in proj (cq_rank 0: none), normed into c_q [T, cq_rank]
+  const float* cq_norm;
+  void* c_q;
   const float* norm_w;
   const float* cos_sin;  // [max_pos, rot]: cos | sin halves
   const int* positions;
   const int64_t* slots;
-  void* cache;    // [num_slots, L + R]
+  void* cache;    // [num_slots, L + R] (null: no cache rows)
   void* q_cat;    // [T, heads, L + R]: columns L.. written here
   int64_t num_slots;
   int max_pos;
@@ -48,21 +55,34 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepArgs a) {
     pos = 0;
   }
   const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
-  int64_t slot = a.slots[t];
+  int64_t slot = a.cache ? a.slots[t] : -1;
   if (slot >= a.num_slots) {
     if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_SLOT);
     slot = -1;
   }
   const int row_w = a.L + a.R;
+  if (a.cq_rank > 0) {  // query latent
+    const T* c = row + a.cq_off;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < a.cq_rank; i += blockDim.x) {
+      const float v = to_f(c[i]);
+      sq = fmaf(v, v, sq);
+    }
+    const float inv = 1.f / sqrtf(block_reduce_sum(sq, red) / a.cq_rank + a.eps);
+    T* dst = static_cast<T*>(a.c_q) + t * a.cq_rank;
+    for (int i = threadIdx.x; i < a.cq_rank; i += blockDim.x) put(dst + i, to_f(c[i]) * inv * a.cq_norm[i]);
+  }
   // cache row
   const T* c = row + a.kv_off;
-  float sq = 0.f;
-  for (int i = threadIdx.x; i < a.L; i += blockDim.x) {
-    const float v = to_f(c[i]);
-    sq = fmaf(v, v, sq);
+  float inv = 0.f;
+  if (a.cache) {
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < a.L; i += blockDim.x) {
+      const float v = to_f(c[i]);
+      sq = fmaf(v, v, sq);
+    }
+    inv = 1.f / sqrtf(block_reduce_sum(sq, red) / a.L + a.eps);
   }
-  sq = block_reduce_sum(sq, red);
-  const float inv = 1.f / sqrtf(sq / a.L + a.eps);
   if (slot >= 0) {
     T* dst = static_cast<T*>(a.cache) + slot * row_w;
     for (int i = threadIdx.x; i < a.L; i += blockDim.x) put(dst + i, to_f(c[i]) * inv * a.norm_w[i]);
@@ -74,11 +94,13 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepArgs a) {
     for (int i = a.rot + threadIdx.x; i < a.R; i += blockDim.x) dst[a.L + i] = c[a.L + i];
   }
   // rotated query parts
+  if (a.q == nullptr) return;
+  const T* q_row = static_cast<const T*>(a.q) + t * a.ldq;
   T* q_out = static_cast<T*>(a.q_cat) + t * a.heads * row_w + a.L;
   const int rest = a.R - a.rot, per = half + rest;
   for (int i = threadIdx.x; i < a.heads * per; i += blockDim.x) {
     const int h = i / per, j = i % per;
-    const T* q = row + static_cast<int64_t>(h) * a.q_width + a.q_rot_off;
+    const T* q = q_row + static_cast<int64_t>(h) * a.q_width + a.q_rot_off;
     T* o = q_out + static_cast<int64_t>(h) * row_w;
     if (j < half) {
       const float u = to_f(q[2 * j]), v = to_f(q[2 * j + 1]);
@@ -210,6 +232,12 @@ int launch_simt(const AttnArgs& a, int B, int max_q, cudaStream_t stream) {
   pxl_host::launch(latent_attn_simt_kernel<T>, grid, dim3(kThreads), smem, stream, a);
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }
+
+int launch_prep(const PrepArgs& a, int T, int is_f32, cudaStream_t stream) {
+  if (is_f32) pxl_host::launch(latent_prep_kernel<float>, dim3(T), dim3(256), 0, stream, a);
+  else pxl_host::launch(latent_prep_kernel<pxl::bf16>, dim3(T), dim3(256), 0, stream, a);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
 }  // namespace
 
 PXL_EXPORT int pxl_latent_prep(const void* proj, int64_t ld, int kv_off, int heads, int q_width, int q_rot_off,
@@ -218,11 +246,30 @@ PXL_EXPORT int pxl_latent_prep(const void* proj, int64_t ld, int kv_off, int hea
                                int rot, float eps, int is_f32, int* status, cudaStream_t stream) {
   if (T <= 0) return PXL_OK;
   if (heads <= 0 || L <= 0 || R < 0 || rot < 0 || rot > R || (rot % 2) || q_rot_off + R > q_width) return PXL_ERR_INVALID_ARG;
-  PrepArgs a{proj, ld, kv_off, heads, q_width, q_rot_off, L, R, rot, norm_w, cos_sin, positions, slots,
-             cache, q_cat, num_slots, max_pos, eps, status};
-  if (is_f32) pxl_host::launch(latent_prep_kernel<float>, dim3(T), dim3(256), 0, stream, a);
-  else pxl_host::launch(latent_prep_kernel<pxl::bf16>, dim3(T), dim3(256), 0, stream, a);
-  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+  const PrepArgs a{proj, ld, kv_off, proj, ld, heads, q_width, q_rot_off, L, R, rot, 0, 0, nullptr, nullptr, norm_w, cos_sin,
+                   positions, slots, cache, q_cat, num_slots, max_pos, eps, status};
+  return launch_prep(a, T, is_f32, stream);
+}
+
+PXL_EXPORT int pxl_latent_rows(const void* proj, int64_t ld, int q_off, int q_rank, const float* q_norm, void* c_q, int kv_off,
+                               const float* norm_w, const float* cos_sin, const int* positions, int max_pos,
+                               const int64_t* slots, void* cache, int64_t num_slots, int T, int L, int R, int rot, float eps,
+                               int is_f32, int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (q_rank <= 0 || L <= 0 || R < 0 || rot < 0 || rot > R || (rot % 2) || !cache) return PXL_ERR_INVALID_ARG;
+  const PrepArgs a{proj, ld, kv_off, nullptr, 0, 0, 0, 0, L, R, rot, q_off, q_rank, q_norm, c_q, norm_w, cos_sin, positions, slots,
+                   cache, nullptr, num_slots, max_pos, eps, status};
+  return launch_prep(a, T, is_f32, stream);
+}
+
+PXL_EXPORT int pxl_latent_queries(const void* q, int64_t ldq, int heads, int q_width, int q_rot_off, const float* cos_sin,
+                                  const int* positions, int max_pos, void* q_cat, int T, int L, int R, int rot, int is_f32,
+                                  int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (heads <= 0 || L <= 0 || R < 0 || rot < 0 || rot > R || (rot % 2) || q_rot_off + R > q_width) return PXL_ERR_INVALID_ARG;
+  const PrepArgs a{q, ldq, 0, q, ldq, heads, q_width, q_rot_off, L, R, rot, 0, 0, nullptr, nullptr, nullptr, cos_sin, positions,
+                   nullptr, nullptr, q_cat, 0, max_pos, 0.f, status};
+  return launch_prep(a, T, is_f32, stream);
 }
 
 PXL_EXPORT int pxl_latent_attn(const void* q, const void* cache, const int* block_tables, const int* cu_q,

@@ -232,6 +232,43 @@ moe_gather_kernel(const bf16* __restrict__ x, const int* __restrict__ src_tok,
     st_bf16x8(dst + v * 8, ld_bf16x8(src + v * 8));
 }
 
+// x_perm[pos_of[t, j], :] = weights[t, j] * x[t, :]: rows in expert order whose routing weight is part of the input. One CTA
+// per token reads its row once.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const T* __restrict__ x, int64_t ldx, const int* __restrict__ pos_of,
+                                                               const float* __restrict__ w, T* __restrict__ x_perm, int k, int H) {
+  const int64_t t = blockIdx.x;
+  for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+    float v[VEC];
+    if constexpr (VEC == 8) {
+      const bf16x8 b = ld_bf16x8(x + t * ldx + c);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = unpack_bf16x2(b.u[j]);
+        v[2 * j] = f.x, v[2 * j + 1] = f.y;
+      }
+    } else {
+      if constexpr (sizeof(T) == 4) v[0] = x[t * ldx + c];
+      else v[0] = __bfloat162float(x[t * ldx + c]);
+    }
+    for (int s = 0; s < k; ++s) {
+      const int p = pos_of[t * k + s];
+      if (p < 0) continue;
+      const float f = w[t * k + s];
+      T* dst = x_perm + static_cast<int64_t>(p) * H + c;
+      if constexpr (VEC == 8) {
+        bf16x8 o;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o.u[j] = pack_bf16x2(v[2 * j] * f, v[2 * j + 1] * f);
+        st_bf16x8(dst, o);
+      } else {
+        if constexpr (sizeof(T) == 4) *dst = v[0] * f;
+        else *dst = __float2bfloat16(v[0] * f);
+      }
+    }
+  }
+}
+
 // out[t, :] = (base ? base[t, :] : 0) + sum_j w[t, j] * y_perm[pos_of[t*k + j], :]
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const bf16* __restrict__ y_perm, const int* __restrict__ pos_of,
@@ -326,6 +363,23 @@ PXL_EXPORT int pxl_moe_gather(const void* x, const int* src_tok, const int* n_ro
   if (H % 8) return PXL_ERR_INVALID_ARG;
   moe_gather_kernel<<<max_rows, 128, 0, stream>>>(static_cast<const bf16*>(x), src_tok, n_rows,
                                                   static_cast<bf16*>(x_perm), H);
+  return check_launch();
+}
+
+PXL_EXPORT int pxl_moe_scatter_rows(const void* x, int64_t ldx, const int* pos_of, const float* w, void* x_perm, int T, int k,
+                                    int H, int is_f32, pxl_stream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (k <= 0 || H <= 0) return PXL_ERR_INVALID_ARG;
+  const bool vec = !is_f32 && !((ldx | H) & 7) && !((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(x_perm)) & 15);
+  if (is_f32)
+    moe_scatter_rows_kernel<float, 1><<<T, 128, 0, stream>>>(static_cast<const float*>(x), ldx, pos_of, w,
+                                                             static_cast<float*>(x_perm), k, H);
+  else if (vec)
+    moe_scatter_rows_kernel<bf16, 8><<<T, 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, pos_of, w,
+                                                            static_cast<bf16*>(x_perm), k, H);
+  else
+    moe_scatter_rows_kernel<bf16, 1><<<T, 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, pos_of, w,
+                                                            static_cast<bf16*>(x_perm), k, H);
   return check_launch();
 }
 

@@ -29,6 +29,7 @@ typedef struct CUstream_st* pxl_stream_t;
 #define PXL_EPI_SPLITK_CN 8 // internal: mid-M path (operands not swapped), K ranges of a tile reduce inside a cluster
 #define PXL_EPI_GATE 9      // internal: C = (A W^T) * sigmoid(gate)      bf16 out (pxl_gemm_bf16_heads)
 #define PXL_EPI_GLU 11      // act(gate) * up (* sigmoid(row gate)), arranged alike (pxl_gemm_bf16_act_glu)
+#define PXL_EPI_ACT 12      // act(A W^T) (* table[ids[row], column])       bf16 out (pxl_gemm_bf16_act)
 #define PXL_EPI_CLIP_GLU 10 // clipped GLU of gate / up groups arranged as for PXL_EPI_SILU_MUL (pxl_gemm_bf16_glu)
 
 #define PXL_NORM_LAYER 0    // (x - mean) / sqrt(variance + eps)
@@ -57,6 +58,10 @@ int pxl_gemm_bf16_small_m(const void* A, const void* W, void* C, const void* res
 // W rows in groups of 128 (64 gate rows, the 64 up rows of the same outputs); C has N / 2 columns.
 int pxl_gemm_bf16_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, float limit,
                       int bn, int* status, pxl_stream_t stream);
+// C = act(A W^T), times table[ids[row] * ld_table + column] if table is given (bf16). act 2 = gelu (tanh form), 3 = square
+// of relu.
+int pxl_gemm_bf16_act(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
+                      const void* table, int64_t ld_table, const int* ids, int64_t num_ids, int* status, pxl_stream_t stream);
 // Gated activation in the epilogue: C = act(g) u, act 0 = silu, 2 = gelu (tanh form); with row_gate (fp32) row m times
 // sigmoid(row_gate[m * ld_row_gate]). W and C as above.
 int pxl_gemm_bf16_act_glu(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldw, int ldc, int act,
@@ -135,13 +140,13 @@ int pxl_add_inplace(void* y, const void* x, int64_t n, pxl_stream_t stream);
 // ---- attention_decode.cu -----------------------------------------------------
 // Single-query GQA attention over the paged cache [blocks, Hkv, page, D] (D = 64 or 128).
 // q [B, Hq, D] with row stride q_stride elements; out [B, Hq, D]; block_tables [B, max_blocks]; ctx_lens [B].
-// window <= 0: full attention. sinks: optional fp32 [Hq] logits added to the
+// window <= 0: full attention; with a window the sequence's first keep_first keys stay visible. sinks: optional fp32 [Hq] logits added to the
 // softmax denominator. workspace: fp32, >= B*Hq*num_splits*(D+2) floats when
 // num_splits > 1. num_splits = 0 picks automatically (see pxl_attn_decode_splits).
 int pxl_attn_decode(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
                     const int* block_tables, const int* ctx_lens, void* out, float* workspace,
                     const float* sinks, int B, int Hq, int Hkv, int D, int page_size,
-                    int max_blocks, int64_t num_blocks, float scale, int window, int num_splits,
+                    int max_blocks, int64_t num_blocks, float scale, int window, int keep_first, int num_splits,
                     int max_ctx, int* status, pxl_stream_t stream);
 int pxl_attn_decode_splits(int B, int Hkv, int max_ctx);
 
@@ -154,7 +159,7 @@ int pxl_attn_prefill(const void* q, int64_t q_stride, const void* k_cache, const
                      const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                      int64_t out_stride, const float* sinks, int B, int max_q_len, int Hq, int Hkv,
                      int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                     int window, int* status, pxl_stream_t stream);
+                     int window, int keep_first, int* status, pxl_stream_t stream);
 
 // ---- attention_prefill_tc.cu ------------------------------------------------------
 // Same contract on the tcgen05 tensor cores (D = 128, page 16 / 32 / 64). total_q = rows of q / out.
@@ -162,7 +167,7 @@ int pxl_attn_prefill_tc(const void* q, int64_t q_stride, const void* k_cache, co
                         const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                         int64_t out_stride, const float* sinks, int B, int max_q_len, int total_q, int Hq,
                         int Hkv, int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                        int window, int* status, pxl_stream_t stream);
+                        int window, int keep_first, int* status, pxl_stream_t stream);
 
 // ---- sampler.cu ----------------------------------------------------------------
 // Greedy arg-max over logits [B, V] (bf16 if logits_bf16 else fp32, row stride ld).
@@ -190,6 +195,9 @@ int pxl_moe_align(const int* ids, int T, int k, int E, int e_lo, int e_hi, int* 
                   int* num_mt, int max_mt, int* pos_of, int* src_tok, pxl_stream_t stream);
 int pxl_moe_gather(const void* x, const int* src_tok, const int* n_rows, void* x_perm,
                    int max_rows, int H, pxl_stream_t stream);
+// x_perm[pos_of[t, j]] = w[t, j] * x[t] (pos_of < 0: no row); any width, bf16 or fp32
+int pxl_moe_scatter_rows(const void* x, int64_t ldx, const int* pos_of, const float* w, void* x_perm, int T, int k, int H,
+                         int is_f32, pxl_stream_t stream);
 int pxl_moe_combine(const void* y_perm, const int* pos_of, const float* w, const void* base,
                     void* out, int T, int k, int H, pxl_stream_t stream);
 // Grouped GEMM over experts (see gemm_tcgen05.cu).
@@ -367,17 +375,18 @@ int pxl_conv_qkv_prep(const void* proj, int64_t ld, int q_off, int k_off, int v_
                       const int* seq_slots, int prefill_seqs, int prefill_tokens, int T, const int64_t* slots,
                       int64_t num_slots, int page, void* k_cache, void* v_cache, void* q_out, float eps, int is_f32,
                       int* status, pxl_stream_t stream);
-// out[t, h * dv + d] = x[t, h, d] (, RMS-normed over all heads * norm_w) * sigmoid(gate[t, h * dv + d]); columns up to
-// out_cols are zeroed. x [T, heads, x_cols].
+// Without convolution and norm weights (all null) q and k are only rotated.
+// out[t, h * dv + d] = x[t, h, d] (, RMS-normed over all heads, or per head, * norm_w) * sigmoid(gate[t, h * dv + d]) * scale;
+// columns up to out_cols are zeroed. x [T, heads, x_cols].
 int pxl_gated_rows(const void* x, int heads, int x_cols, int dv, const void* gate, int64_t ldg, const float* norm_w, float eps,
-                   void* out, int64_t ldo, int out_cols, int T, int is_f32, pxl_stream_t stream);
+                   int per_head, float scale, void* out, int64_t ldo, int out_cols, int T, int is_f32, pxl_stream_t stream);
 
 // ---- attention_any.cu: paged attention of any head size, bf16 or fp32, on the FMA pipes ------------------
 // Arguments as pxl_attn_prefill; cu_q null: token i is the only query of sequence i.
 int pxl_attn_any(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const int* block_tables,
                  const int* cu_q, const int* ctx_lens, void* out, int64_t out_stride, const float* sinks, int B, int max_q,
-                 int Hq, int Hkv, int D, int page, int max_blocks, int64_t num_blocks, float scale, int window, int is_f32,
-                 int* status, pxl_stream_t stream);
+                 int Hq, int Hkv, int D, int page, int max_blocks, int64_t num_blocks, float scale, int window, int keep_first,
+                 int is_f32, int* status, pxl_stream_t stream);
 
 // ---- lightning_attn.cu: linear attention with a fixed decay per head ------------------------------------
 // q, k [T, H x dk] and v [T, H x dv] are columns of proj, all passed through silu here. state [slots, H, dk, dv] fp32,
@@ -395,6 +404,15 @@ int pxl_latent_prep(const void* proj, int64_t ld, int kv_off, int heads, int q_w
                     const float* cos_sin, const int* positions, int max_pos, const int64_t* slots, void* cache,
                     int64_t num_slots, void* q_cat, int T, int L, int R, int rot, float eps, int is_f32, int* status,
                     pxl_stream_t stream);
+// The same for queries that go through a latent of their own: pxl_latent_rows writes the cache rows and
+// c_q[t] = RMSnorm(proj[t, q_off : q_off + q_rank]) * q_norm, pxl_latent_queries the rotated parts of q [T, ldq].
+int pxl_latent_rows(const void* proj, int64_t ld, int q_off, int q_rank, const float* q_norm, void* c_q, int kv_off,
+                    const float* norm_w, const float* cos_sin, const int* positions, int max_pos, const int64_t* slots,
+                    void* cache, int64_t num_slots, int T, int L, int R, int rot, float eps, int is_f32, int* status,
+                    pxl_stream_t stream);
+int pxl_latent_queries(const void* q, int64_t ldq, int heads, int q_width, int q_rot_off, const float* cos_sin,
+                       const int* positions, int max_pos, void* q_cat, int T, int L, int R, int rot, int is_f32, int* status,
+                       pxl_stream_t stream);
 // out[t, h, :L] = attention of q[t, h, :L+R] over the cached rows of t's sequence (cu_q null: token t is the only
 // query of sequence t). The queries are the last tokens of ctx_lens[b]. window <= 0: no window; sinks may be null.
 int pxl_latent_attn(const void* q, const void* cache, const int* block_tables, const int* cu_q, const int* ctx_lens,
@@ -405,6 +423,31 @@ int pxl_latent_attn_tc_supported(int L, int R, int page, float scale);
 int pxl_latent_attn_tc(const void* q, const void* cache, const int* block_tables, const int* cu_q, const int* ctx_lens,
                        void* out, const float* sinks, int B, int max_q, int total_q, int H, int L, int R, int page,
                        int max_blocks, int64_t num_blocks, float scale, int window, int* status, pxl_stream_t stream);
+
+// ---- matrix_memory.cu: mLSTM ------------------------------------------------------------------------------
+// q, k [T, H x dk] and v [T, H x dv] are columns of proj; gates [T, ldg] fp32: H input gates | H forget gates before
+// bias [2 H] and the soft cap. state [slots, H, words] fp32, words >= dk * dv + ceil(dv / 32) * (dk + 1): S, then per 32
+// columns of v a copy of the normaliser, then as many copies of the running maximum. out [T, ldo]: heads side by side.
+// Sequences as for pxl_conv_qkv_prep.
+int pxl_matrix_memory(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int H, int dk, int dv, const float* gates,
+                      int64_t ldg, const float* bias, float cap, float* state, int64_t words, int num_slots, const int* seq_cu,
+                      const int* seq_slots, const int* positions, void* out, int64_t ldo, int prefill_seqs, int decode_seqs,
+                      int is_f32, int* status, pxl_stream_t stream);
+
+// ---- tanh_norm.cu: the fp32 residual between two products --------------------------------------------------
+// In place: x += norm(y + sum_j weights[t, j] * rows[pos_of[t, j]]) (post 1: tanh(alpha z) w + b, 2: z / rms(z) * w),
+// x += table[ids[t]], x += step; then low = x (pre 2) or tanh(pre_alpha x) pre_w + pre_b (pre 1). Null or 0: left out;
+// null weights count as 1. y, rows, table and low are bf16, or fp32 when is_f32.
+int pxl_residual_step(float* x, const void* y, int64_t ldy, const void* rows, int64_t ldr, int64_t num_rows, const int* pos_of,
+                      const float* weights, int k, int post, const float* post_w, const float* post_b, float post_alpha, float eps,
+                      const void* table, const int* ids, int64_t num_ids, const float* step, int pre, const float* pre_w,
+                      const float* pre_b, float pre_alpha, void* low, int T, int W, int is_f32, int* status, pxl_stream_t stream);
+// out[t] = tanh(alpha x[rows ? rows[t] : t]) w + b
+int pxl_tanh_norm(const float* x, const float* w, const float* b, float alpha, const int* rows, int64_t num_rows, void* out,
+                  int T, int W, int out_f32, int* status, pxl_stream_t stream);
+// out[t, c] = act(x[t, c]) (* table[ids[t] * ldt + col + c]); act 2 = gelu (tanh form), 3 = square of relu
+int pxl_act_rows(const void* x, int64_t ldx, int x_f32, int act, const void* table, int64_t ldt, int col, const int* ids,
+                 int64_t num_ids, void* out, int64_t ldo, int out_f32, int T, int N, int* status, pxl_stream_t stream);
 
 // ---- stage_exec.cu: all layers of a dense GQA stage for one step behind one call --------------
 // The descriptor structs are defined in stage_exec.cu (mirrored by parallax_b200/engine/native_stage.py).

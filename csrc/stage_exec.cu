@@ -134,18 +134,18 @@ PXL_EXPORT int pxl_stage_forward_dense(const PxlStageDesc* st, const PxlStepDesc
       if (prefill_tc) {
         PXL_TRY(pxl_attn_prefill_tc(qkv, qkv_n, L.k_cache, L.v_cache, sp->p_bt, sp->p_cu_q, sp->p_ctx, attn,
                                     static_cast<int64_t>(Hq) * D, L.sinks, sp->Bp, sp->p_max_q, sp->Tp, Hq, Hkv, D,
-                                    st->page, sp->p_max_blocks, st->num_blocks, st->scale, L.window, status, stream));
+                                    st->page, sp->p_max_blocks, st->num_blocks, st->scale, L.window, 0, status, stream));
       } else {
         PXL_TRY(pxl_attn_prefill(qkv, qkv_n, L.k_cache, L.v_cache, sp->p_bt, sp->p_cu_q, sp->p_ctx, attn,
                                  static_cast<int64_t>(Hq) * D, L.sinks, sp->Bp, sp->p_max_q, Hq, Hkv, D, st->page,
-                                 sp->p_max_blocks, st->num_blocks, st->scale, L.window, status, stream));
+                                 sp->p_max_blocks, st->num_blocks, st->scale, L.window, 0, status, stream));
       }
       ++n;
     }
     if (sp->Bd > 0) {
       PXL_TRY(pxl_attn_decode(qkv + static_cast<size_t>(sp->Tp) * qkv_n, qkv_n, L.k_cache, L.v_cache, sp->d_bt,
                               sp->d_ctx, attn + static_cast<size_t>(sp->Tp) * Hq * D, ws->decode, L.sinks, sp->Bd, Hq,
-                              Hkv, D, st->page, sp->d_max_blocks, st->num_blocks, st->scale, L.window, splits,
+                              Hkv, D, st->page, sp->d_max_blocks, st->num_blocks, st->scale, L.window, 0, splits,
                               sp->d_max_ctx, status, stream));
       n += splits > 1 ? 2 : 1;
     }

@@ -35,6 +35,14 @@ NVCC_FLAGS = [
 ]
 
 
+# Sources whose elementary functions must be accurate in fp32 (arithmetic of a recurrence, tanh norms)
+ACCURATE = ("matrix_memory", "tanh_norm")
+
+
+def _flags(src: Path) -> list[str]:
+    return [f for f in NVCC_FLAGS if f != "--use_fast_math" or src.stem not in ACCURATE]
+
+
 def _nvcc() -> str:
     cand = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not os.path.exists(cand):
@@ -46,6 +54,8 @@ def _nvcc() -> str:
 # that only runs this family compiles these into a library of their own.
 FAMILY_SOURCES = {
     "latent": ["elementwise", "gemm_simt", "gemm_tcgen05", "latent_attn", "latent_attn_tc", "residual", "sampler"],
+    "looped": ["attention", "attention_any", "attention_prefill_tc", "attn_prep", "elementwise", "gemm_simt", "gemm_tcgen05",
+               "latent_attn", "latent_attn_tc", "matrix_memory", "moe", "residual", "sampler", "tanh_norm"],
     "parallel_block": ["attention", "attention_any", "attention_prefill_tc", "attn_prep", "elementwise", "gemm_simt",
                        "gemm_tcgen05", "lightning_attn", "moe", "residual", "sampler"],
 }
@@ -66,7 +76,7 @@ def _digest(paths: list[Path]) -> str:
     for p in sorted(paths):
         h.update(p.name.encode())
         h.update(p.read_bytes())
-    h.update(" ".join(NVCC_FLAGS).encode())
+    h.update(" ".join(NVCC_FLAGS).encode() + " ".join(ACCURATE).encode())
     return h.hexdigest()
 
 
@@ -122,7 +132,7 @@ def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool =
         want = _digest([src]) + hdr_digest
         if not force and obj.exists() and tag.exists() and tag.read_text() == want:
             return obj
-        cmd = [nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+        cmd = [nvcc, *_flags(src), "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
         if ptxas_info:
             cmd[1:1] = ["-Xptxas", "-v"]
         res = subprocess.run(cmd, capture_output=True, text=True)

@@ -14,13 +14,17 @@ hybrid cache, ``src/parallax/server/cache_manager.py:188-259``):
 Any layer may keep per-request slots beside its pages (``ModelConfig.slot_dims``), e.g. the window of a short
 convolution in front of softmax attention.
 
+A layer that runs several times for a token (``ModelConfig.layer_passes``) has one cache object per pass; block tables
+and slots are the same for all of them.
+
 Layouts are chosen for the sm_100a kernels (whole pages of one head are contiguous), not
 for compatibility with the reference's Metal layouts.
 """
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+import math
+from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
@@ -39,6 +43,13 @@ class LayerCache:
     # e4m3 K / V caches hold value / scale; the attention kernels multiply by the scale again
     k_scale: float = 1.0
     v_scale: float = 1.0
+    # a layer that runs several times for a token: the caches of its later passes
+    later: list = field(default_factory=list)
+
+    @property
+    def passes(self) -> list:
+        """The caches of the layer's passes, in order."""
+        return [self, *self.later]
 
     @property
     def kv_scale(self) -> tuple:
@@ -75,14 +86,14 @@ def bytes_per_block(cfg: ModelConfig, start: int, end: int, page: int, elem: int
     total = 0
     kv_elem = kv_elem or elem
     for li in range(start, end):
-        kind = cfg.layer_kind(li)
+        kind, passes = cfg.layer_kind(li), cfg.layer_passes(li)
         if kind in (ATTENTION, MSA_ATTENTION):
             heads, cols = cfg.kv_dims(li) or (0, 0)
-            total += 2 * (heads and max(1, heads // tp)) * page * cols * kv_elem
+            total += passes * 2 * (heads and max(1, heads // tp)) * page * cols * kv_elem
             if kind == MSA_ATTENTION:
                 total += page * int(cfg.raw.get("index_head_dim") or 0) * elem
         elif kind in (MLA_ATTENTION, DSA_ATTENTION):
-            total += page * sum(cfg.latent_dims(li)) * elem
+            total += passes * page * sum(cfg.latent_dims(li)) * elem
             if kind == DSA_ATTENTION:
                 total += page * cfg.index_head_dim * elem
     return total
@@ -92,7 +103,7 @@ def bytes_per_linear_slot(cfg: ModelConfig, start: int, end: int, elem: int = 2,
     total = 0
     for li in range(start, end):
         conv, rec = slot_dims(cfg, li, tp)
-        total += (conv[0] * conv[1] * elem if conv else 0) + (rec[0] * rec[1] * rec[2] * 4 if rec else 0)
+        total += cfg.layer_passes(li) * ((math.prod(conv) * elem if conv else 0) + (math.prod(rec) * 4 if rec else 0))
     return total
 
 
@@ -112,31 +123,41 @@ class KVPool:
         self.dtype = dtype
         self.layers: list[LayerCache] = []
         for li in range(start_layer, end_layer):
-            kind = cfg.layer_kind(li)
-            lc = LayerCache(kind)
-            if kind in (ATTENTION, MSA_ATTENTION):
-                dims = cfg.kv_dims(li)
-                if dims is not None:
-                    shape = (num_blocks, max(1, dims[0] // tp), page_size, dims[1])
-                    lc.k = torch.zeros(shape, device=self.device, dtype=kv_dt)
-                    lc.v = torch.zeros(shape, device=self.device, dtype=kv_dt)
-                if kv_dt == torch.float8_e4m3fn:
-                    lc.k_scale, lc.v_scale = float(kv_scale[0]), float(kv_scale[1])
-                if kind == MSA_ATTENTION:
-                    lc.index_k = torch.zeros((num_blocks, 1, page_size, int(cfg.raw.get("index_head_dim") or 0)),
-                                             device=self.device, dtype=dtype)
-            elif kind in (MLA_ATTENTION, DSA_ATTENTION):
-                lc.k = torch.zeros((num_blocks, 1, page_size, sum(cfg.latent_dims(li))),
-                                   device=self.device, dtype=dtype)
-                if kind == DSA_ATTENTION:
-                    lc.index_k = torch.zeros((num_blocks, 1, page_size, cfg.index_head_dim),
-                                             device=self.device, dtype=dtype)
-            conv, rec = slot_dims(cfg, li, tp)
-            if conv is not None:
-                lc.conv_state = torch.zeros((num_linear_slots, *conv), device=self.device, dtype=dtype)
-            if rec is not None:
-                lc.rec_state = torch.zeros((num_linear_slots, *rec), device=self.device, dtype=torch.float32)
-            self.layers.append(lc)
+            first, *rest = [self._layer_cache(li, kv_dt, tp, num_linear_slots, kv_scale) for _ in range(cfg.layer_passes(li))]
+            first.later = rest
+            self.layers.append(first)
+
+    def _layer_cache(self, li: int, kv_dt, tp: int, num_linear_slots: int, kv_scale: tuple) -> LayerCache:
+        cfg, num_blocks, page_size, dtype = self.cfg, self.num_blocks, self.page_size, self.dtype
+        kind = cfg.layer_kind(li)
+        lc = LayerCache(kind)
+        if kind in (ATTENTION, MSA_ATTENTION):
+            dims = cfg.kv_dims(li)
+            if dims is not None:
+                shape = (num_blocks, max(1, dims[0] // tp), page_size, dims[1])
+                lc.k = torch.zeros(shape, device=self.device, dtype=kv_dt)
+                lc.v = torch.zeros(shape, device=self.device, dtype=kv_dt)
+            if kv_dt == torch.float8_e4m3fn:
+                lc.k_scale, lc.v_scale = float(kv_scale[0]), float(kv_scale[1])
+            if kind == MSA_ATTENTION:
+                lc.index_k = torch.zeros((num_blocks, 1, page_size, int(cfg.raw.get("index_head_dim") or 0)),
+                                         device=self.device, dtype=dtype)
+        elif kind in (MLA_ATTENTION, DSA_ATTENTION):
+            lc.k = torch.zeros((num_blocks, 1, page_size, sum(cfg.latent_dims(li))),
+                               device=self.device, dtype=dtype)
+            if kind == DSA_ATTENTION:
+                lc.index_k = torch.zeros((num_blocks, 1, page_size, cfg.index_head_dim),
+                                         device=self.device, dtype=dtype)
+        conv, rec = slot_dims(cfg, li, tp)
+        if conv is not None:
+            lc.conv_state = torch.zeros((num_linear_slots, *conv), device=self.device, dtype=dtype)
+        if rec is not None:
+            lc.rec_state = torch.zeros((num_linear_slots, *rec), device=self.device, dtype=torch.float32)
+        return lc
+
+    def caches(self):
+        """Every cache object of the stage: one per layer and pass."""
+        return [c for lc in self.layers for c in lc.passes]
 
     def zero_slot(self, slot: int) -> None:
         for t in self._slot_tensors():
@@ -147,11 +168,11 @@ class KVPool:
             t[dst].copy_(t[src])
 
     def _slot_tensors(self):
-        return [t for lc in self.layers for t in (lc.conv_state, lc.rec_state) if t is not None]
+        return [t for lc in self.caches() for t in (lc.conv_state, lc.rec_state) if t is not None]
 
     def nbytes(self) -> int:
         n = 0
-        for lc in self.layers:
+        for lc in self.caches():
             for t in (lc.k, lc.v, lc.index_k, lc.conv_state, lc.rec_state):
                 if t is not None:
                     n += t.numel() * t.element_size()

@@ -20,7 +20,7 @@ class ForwardBatch:
     num_prefill_tokens: int = 0
     num_prefill_seqs: int = 0
     num_decode: int = 0
-    input_ids: Optional[torch.Tensor] = None      # int32 [T] (first stage only)
+    input_ids: Optional[torch.Tensor] = None      # int32 [T] (first stage; every stage if layers read the ids)
     prev_ids: Optional[torch.Tensor] = None       # int32 [T] token before each token, -1 = none (first stage, if needed)
     positions: Optional[torch.Tensor] = None      # int32 [T]
     slot_mapping: Optional[torch.Tensor] = None   # int64 [T]

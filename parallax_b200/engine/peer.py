@@ -141,7 +141,7 @@ class PeerExecutor:
             if on_gpu:
                 _cuda.status_copy_async(self.device)
             return arrays, out
-        fb = self.builder.build(arrays["ids"] if self.is_first else None, arrays["pos"], arrays["slots"],
+        fb = self.builder.build(arrays["ids"] if self.is_first or self.cfg.needs_ids_everywhere else None, arrays["pos"], arrays["slots"],
                                 arrays["p_q"], arrays["p_ctx"], arrays["p_tables"], arrays["d_ctx"],
                                 arrays["d_tables"], arrays["logit_rows"], arrays["seq_rows"], extra=extra,
                                 prev_ids=arrays["prev_ids"])

@@ -18,9 +18,11 @@ from typing import Iterable, Optional
 
 _LM_PREFIXES = ("model.language_model.", "language_model.")
 _LAYER_RE = re.compile(r"(?:^|\.)layers\.(\d+)\.|^l(\d+)\.")
-# flat naming of layer-list checkpoints: embed, bigram, l<i>.*, final.norm, head
+# flat naming of layer-list checkpoints: embed, bigram, l<i>.*, final.norm, head; the tables that layers read by token
+# id or by pass go to every stage
 _FLAT_FIRST = ("embed", "bigram")
 _FLAT_LAST = ("final.norm", "head")
+_FLAT_EVERY = ("side.embed", "loop.step")
 
 
 def normalize_weight_key(key: str) -> str:
@@ -44,8 +46,10 @@ def should_include_weight_key(key: str, start_layer: int, end_layer: int, is_fir
                               is_last_shard: bool, tie_word_embeddings: bool = False) -> bool:
     if key in _FLAT_FIRST:
         return is_first_shard
-    if key in _FLAT_LAST:
+    if key in _FLAT_LAST or key.startswith("final.norm."):
         return is_last_shard
+    if key in _FLAT_EVERY:
+        return True
     if key.startswith("model.") and "embed_tokens" in key:
         if is_first_shard:
             return True

@@ -88,6 +88,8 @@ class ModelConfig:
     embedding_scale: float = 1.0
     bigram: Optional[object] = None      # BigramSpec: hashed (previous token, token) embedding
     residual_mult: float = 1.0           # factor of every sublayer's contribution to the residual
+    loop: Optional[object] = None        # LoopSpec: layers that run several times, every pass with its own cache
+    token_side_dim: int = 0              # width of the per-layer input that a token's row of a side table gives
     raw: dict = field(default_factory=dict, repr=False)
 
     # ------------------------------------------------------------------ derived
@@ -95,6 +97,15 @@ class ModelConfig:
     def needs_prev_token(self) -> bool:
         """Whether the embedding of a token also depends on the token before it in its sequence."""
         return self.bigram is not None
+
+    @property
+    def needs_ids_everywhere(self) -> bool:
+        """Whether layers read the token ids themselves, so that every pipeline stage needs them."""
+        return self.token_side_dim > 0
+
+    def layer_passes(self, layer_idx: int) -> int:
+        """How often a layer runs for a token; it keeps pages and state once per pass."""
+        return self.loop.times if self.loop is not None and self.loop.start <= layer_idx < self.loop.stop else 1
 
     def latent_dims(self, layer_idx: int) -> tuple[int, int]:
         """(latent width, rotated key width) of a latent-attention layer's cache row."""
@@ -123,8 +134,12 @@ class ModelConfig:
 
     @property
     def linked_layers(self) -> list[tuple[int, int]]:
-        """Pairs (layer that owns keys and values, later layer that reads them): both belong in one pipeline stage."""
-        return [(s.mixer.kv_from, i) for i, s in enumerate(self.layer_specs) if s.mixer.kv_from is not None]
+        """Pairs of layers that belong in one pipeline stage: one that owns keys and values and a later one that reads
+        them; everything up to the end of a loop, whose later passes start from the embedding again."""
+        pairs = [(s.mixer.kv_from, i) for i, s in enumerate(self.layer_specs) if s.mixer.kv_from is not None]
+        if self.loop is not None and self.loop.times > 1:
+            pairs.append((0, self.loop.stop - 1))
+        return pairs
 
     @property
     def is_moe(self) -> bool:
@@ -195,10 +210,10 @@ class ModelConfig:
             rows = 0
             for i in range(self.num_hidden_layers):
                 if self.layer_kind(i) == MLA_ATTENTION:
-                    rows += sum(self.latent_dims(i))
+                    rows += sum(self.latent_dims(i)) * self.layer_passes(i)
                 elif self.kv_dims(i) is not None:
                     heads, cols = self.kv_dims(i)
-                    rows += 2 * heads * cols
+                    rows += 2 * heads * cols * self.layer_passes(i)
             return -(-rows * elem_bytes // self.num_hidden_layers)
         if self.is_mla:
             return (self.kv_lora_rank + self.qk_rope_head_dim) * elem_bytes
@@ -229,7 +244,7 @@ def config_from_layer_list(cfg: dict) -> ModelConfig:
     """Config whose ``layers`` entry describes every layer by itself (see ``models/layer_spec.py``). The scalar
     sizes of :class:`ModelConfig` hold the largest value of any layer: capacity estimates use them, the model
     itself reads ``layer_specs``."""
-    from parallax_b200.models.layer_spec import parse_bigram, parse_layers
+    from parallax_b200.models.layer_spec import parse_bigram, parse_layers, parse_loop
 
     specs = parse_layers(cfg["architecture"], cfg["layers"])
     if not specs:
@@ -249,12 +264,13 @@ def config_from_layer_list(cfg: dict) -> ModelConfig:
         vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]),
         rope_theta=next((m.rot.base for m in mixers if hasattr(m, "rot")), 1e4),
         max_position_embeddings=int(cfg.get("max_position_embeddings") or 32768),
-        kv_lora_rank=top(latent, "kv_rank"), qk_nope_head_dim=top(latent, "dim"),
+        q_lora_rank=top(latent, "q_rank"), kv_lora_rank=top(latent, "kv_rank"), qk_nope_head_dim=top(latent, "dim"),
         qk_rope_head_dim=top(latent, "rot_dim"), v_head_dim=top(mixers, "vdim"),
         num_experts=top(routed, "experts"), num_experts_per_tok=top(routed, "top"), moe_intermediate_size=top(routed, "ff"),
         shared_expert_intermediate_size=top([m.shared for m in routed], "ff"),
         layer_specs=specs, embedding_scale=float(emb.get("scale", 1.0)), bigram=parse_bigram(emb),
-        residual_mult=float(cfg.get("residual_mult", 1.0)), raw=cfg)
+        residual_mult=float(cfg.get("residual_mult", 1.0)), loop=parse_loop(cfg.get("loop"), len(specs)),
+        token_side_dim=int((cfg.get("token_side") or {}).get("dim") or 0), raw=cfg)
 
 
 def config_from_hf(cfg: dict) -> ModelConfig:
@@ -462,6 +478,35 @@ def named_config(name: str) -> ModelConfig:
                                         router=dict(experts=ex, identity=ident, top=top,
                                                     groups=dict(count=groups[0], keep=groups[1])))))
         return config_from_hf(dict(architecture="Zudepel", vocab=vocab, width=w, norm=dict(eps=1e-6), layers=layers))
+    if n in {"tiny-zasalix", "small-zasalix", "zasalix-1b", "zasalix-8b"}:
+        # layer list: l = latent attention, p = attention beside a matrix memory, m = matrix memory; d / e behind it: dense or
+        # routed feed-forward. (layers, width, latent (heads, dim, rot, vdim, kv rank, q rank), attention (heads, kv heads, dim,
+        # vdim, window, kept), memory (heads, dim, vdim), ff, (experts, top, expert ff), side, loop, vocab)
+        pattern, w, lat, att, mem, ff, (ex, top, eff), side, loop, vocab = {
+            "tiny-zasalix": ("ldpemeld", 64, (4, 16, 8, 24, 40, 32), (4, 2, 16, 24, 20, 5), (2, 16, 32), 96, (6, 2, 32), 16,
+                             (0, 2, 2), 260),
+            "small-zasalix": ("ldpemdpele", 512, (8, 64, 32, 64, 192, 256), (8, 2, 64, 64, 100, 16), (4, 64, 96), 1024,
+                              (12, 3, 256), 64, (1, 3, 3), 1024),
+            "zasalix-1b": ("ld" + "pemepele" * 3, 2048, (16, 128, 64, 128, 512, 768), (16, 4, 128, 128, 1024, 64), (8, 128, 256),
+                           5632, (32, 4, 768), 256, (0, 2, 3), 32768),
+            "zasalix-8b": ("ldld" + "pemepele" * 7, 4096, (32, 128, 64, 128, 512, 1536), (32, 8, 128, 128, 2048, 64),
+                           (16, 128, 256), 12288, (64, 4, 1536), 256, (0, 3, 3), 131072)}[n]
+        layers = []
+        for kind, mlp in zip(pattern[::2], pattern[1::2]):
+            memory = dict(heads=mem[0], dim=mem[1], vdim=mem[2], gate_cap=15.0)
+            if kind == "l":
+                t, m = "latent_attention", dict(heads=lat[0], dim=lat[1], rot_dim=lat[2], vdim=lat[3], kv_rank=lat[4], q_rank=lat[5],
+                                                scale=(lat[1] + lat[2]) ** -0.5, rot=dict(base=1e4, dims=lat[2]))
+            elif kind == "p":
+                left = dict(heads=att[0], kv_heads=att[1], dim=att[2], vdim=att[3], scale=att[2] ** -0.5,
+                            rot=dict(base=1e4, dims=att[2] // 2), mask=dict(size=att[4], keep_first=att[5]))
+                t, m = "parallel", dict(left=left, right=memory, left_scale=0.5, right_scale=0.5)
+            else:
+                t, m = "mlstm", memory
+            layers.append(dict(type=t, mixer=m, mlp=dict(kind="dense", ff=ff) if mlp == "d" else dict(
+                kind="moe", expert=dict(ff=eff), shared=dict(ff=eff), router=dict(experts=ex, top=top))))
+        return config_from_hf(dict(architecture="Zasalix", vocab=vocab, width=w, norm=dict(eps=1e-6), layers=layers,
+                                   loop=dict(zip(("start", "stop", "times"), loop)), token_side=dict(dim=side)))
     if n == "tiny":
         return config_from_hf(dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", hidden_size=256,
                                    num_hidden_layers=4, num_attention_heads=4, num_key_value_heads=2,

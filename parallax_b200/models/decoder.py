@@ -226,6 +226,7 @@ class DecoderStage(ExpertParallelMixin):
     _LAYER_KEY = re.compile(r"(?:^|\.)layers\.(\d+)\.")
     _GLOBAL_KEYS = ("embed_tokens.weight", ".norm.weight", "lm_head.weight")
     _GLOBAL_TENSORS = ("embed", "norm_w", "lm_head")
+    _TABLES_EVERYWHERE = False      # whether a stage in the middle of a pipeline has tensors outside its layers, too
 
     @classmethod
     def _layer_of_key(cls, key: str) -> Optional[int]:
@@ -270,7 +271,7 @@ class DecoderStage(ExpertParallelMixin):
             built.append((gi, shadow))
         glob = None
         wants_embed = self.is_first or (self.is_last and self.cfg.tie_word_embeddings)
-        if n_global and (wants_embed or self.is_last):
+        if n_global and (wants_embed or self.is_last or self._TABLES_EVERYWHERE):
             glob = copy.copy(self)
             glob.start_layer = glob.end_layer = self.start_layer
             glob.layers, glob.kv_caches, glob._native, glob.lora = [], [], False, None

@@ -83,6 +83,17 @@ class LayerListStage(DecoderStage):
         lw.cos_sin = self._tables[rot]
 
     # ------------------------------------------------------------------ weights
+    def global_shapes(self) -> dict[str, tuple]:
+        """Checkpoint tensors outside the layers that this stage holds (name -> shape)."""
+        cfg, W, sh = self.cfg, self.cfg.hidden_size, {}
+        if self.is_first:
+            sh["embed"] = (cfg.vocab_size, W)
+            if cfg.bigram is not None:
+                sh["bigram"] = (cfg.bigram.buckets + 1, W)
+        if self.is_last:
+            sh.update({"final.norm": (W,), "head": (cfg.vocab_size, W)})
+        return sh
+
     def weight_shapes(self, gi: int) -> dict[str, tuple]:
         """Checkpoint tensors of layer ``gi`` (name -> shape)."""
         raise NotImplementedError
@@ -98,19 +109,16 @@ class LayerListStage(DecoderStage):
             g.manual_seed(seed * 1000003 + k)
             return (torch.randn(*shape, generator=g, device=dev, dtype=torch.float32) * std).to(torch.bfloat16)
 
-        W = cfg.hidden_size
-        tensors = {}
-        if self.is_first:
-            tensors["embed"] = rnd((cfg.vocab_size, W), 900001)
-            if cfg.bigram is not None:
-                tensors["bigram"] = rnd((cfg.bigram.buckets + 1, W), 900003)
-        if self.is_last:
-            tensors["final.norm"], tensors["head"] = torch.ones(W, device=dev), rnd((cfg.vocab_size, W), 900002)
-        self._load_globals(tensors)
+        seeds = {"embed": 900001, "head": 900002, "bigram": 900003, "side.embed": 900004, "loop.step": 900005}
+        self._load_globals({name: self._random(name, shape, lambda s, k=seeds.get(name): rnd(s, k))     # (alike on every stage)
+                            for name, shape in self.global_shapes().items()})
         for gi, lw in enumerate(self.layers, self.start_layer):      # layer by layer: one raw copy at a time
-            layer = {name: (torch.ones(shape, device=dev) if "norm" in name else rnd(shape, gi * 4096 + i))
+            layer = {name: self._random(name, shape, lambda s, i=i: rnd(s, gi * 4096 + i))
                      for i, (name, shape) in enumerate(self.weight_shapes(gi).items())}
             self._load_layer(lw, gi, layer)
+
+    def _random(self, name: str, shape: tuple, rnd) -> torch.Tensor:
+        return torch.ones(shape, device=self.device) if "norm" in name else rnd(shape)
 
     def load_weights(self, tensors: dict[str, torch.Tensor]) -> None:
         self._load_globals(tensors)
@@ -135,26 +143,33 @@ class LayerListStage(DecoderStage):
 
         return get
 
+    def _global_getter(self, tensors):
+        """``get(name)``: checked tensor outside the layers on the stage's device."""
+        shapes = self.global_shapes()
+
+        def get(name, dtype=self.dtype):
+            return self._take(tensors, name, shapes[name]).to(device=self.device, dtype=dtype).contiguous()
+
+        return get
+
     def _load_globals(self, tensors) -> None:
-        cfg, W = self.cfg, self.cfg.hidden_size
-
-        def get(name, shape, dtype=self.dtype):
-            return self._take(tensors, name, shape).to(device=self.device, dtype=dtype).contiguous()
-
+        get = self._global_getter(tensors)
         if self.is_first:
-            self.embed = get("embed", (cfg.vocab_size, W))
-            if cfg.bigram is not None:
-                self.bigram = get("bigram", (cfg.bigram.buckets + 1, W))
+            self.embed = get("embed")
+            if self.cfg.bigram is not None:
+                self.bigram = get("bigram")
         if self.is_last:
-            self.norm_w = get("final.norm", (W,), torch.float32)
-            self.lm_head = pad_rows(get("head", (cfg.vocab_size, W)), 8)
+            self.norm_w = get("final.norm", torch.float32)
+            self.lm_head = pad_rows(get("head"), 8)
 
     def update_weights(self, tensors) -> int:
         """Online refit: layers named in ``tensors`` are rebuilt by the loader and moved into the live weights."""
         return self.reload_layers(tensors)
 
     def weight_bytes(self) -> int:
-        ts = [t for t in (self.embed, self.bigram, self.norm_w, self.lm_head) if t is not None]
+        ts = []
+        for t in (getattr(self, name) for name in self._GLOBAL_TENSORS):
+            ts += t.tensors() if hasattr(t, "tensors") else [] if t is None else [t]
         ts += [t for lw in self.layers for t in lw.tensors()]
         return sum(t.numel() * t.element_size() for t in ts)
 

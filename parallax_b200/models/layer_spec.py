@@ -10,18 +10,21 @@ Config layout (``config_from_layer_list``)::
 
     architecture, vocab, width, norm.eps, residual_mult,
     embedding: {scale, bigram: {buckets, mul_prev, mul_cur} | null},
+    loop: {start, stop, times} | null, token_side: {dim} | null,
     layers: [{type, mixer: {...}, mlp: {...} | null}, ...]
 
 Every mixer says what the cache keeps for it: pages (``kv_dims``, one row per token) and / or a slot per
-request (``slot_dims``: the last inputs of a short convolution, a recurrent state).
+request (``slot_dims``: the last inputs of a short convolution, a recurrent state). A layer inside a loop keeps all of
+that once per pass.
 """
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Optional
 
-ACT_SILU, ACT_CLIPPED, ACT_GELU_TANH = 0, 1, 2      # the modes of ops.act_mul / ops.glu_linear
+# the modes of ops.act_mul / ops.glu_linear / ops.act_linear (the square of relu: act_linear only)
+ACT_SILU, ACT_CLIPPED, ACT_GELU_TANH, ACT_RELU_SQUARED = 0, 1, 2, 3
 
 
 @dataclass(frozen=True)
@@ -45,6 +48,8 @@ class LatentAttentionSpec:
     scale: float        # factor of the attention scores
     rot: RotarySpec
     window: int = 0     # keys a query sees, itself included (0: all before it)
+    q_rank: int = 0     # width of the normed latent that queries go through (0: projected directly)
+    gated: bool = True  # whether the heads are multiplied by sigmoid(W_g x)
 
     kind = "mla_attention"
     kv_from = None
@@ -66,8 +71,9 @@ class LatentAttentionSpec:
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """Softmax attention with grouped heads: a short causal convolution on q, k and v, RMS norm over the whole q and
-    k projections, half-split rotation, sinks, an output gate."""
+    """Softmax attention with grouped heads: optionally a short causal convolution on q, k and v and RMS norm over the
+    whole q and k projections; half-split rotation, an output gate. With a ``window`` a query sees that many keys, itself
+    included, and the sequence's first ``keep_first`` ones."""
 
     heads: int
     kv_heads: int
@@ -78,6 +84,7 @@ class AttentionSpec:
     conv: int = 0       # taps of the convolution (0: none)
     kv_from: Optional[int] = None    # layer whose cached keys and values this layer reads instead of its own
     window: int = 0
+    keep_first: int = 0
 
     kind = "attention"
 
@@ -155,6 +162,79 @@ class LightningSpec:
 
 
 @dataclass(frozen=True)
+class MatrixMemorySpec:
+    """mLSTM: linear attention whose decay and input weight are gates of the token (exponential, soft-capped logarithms
+    kept stable by a running maximum), with a normaliser beside the state."""
+
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    kind = "linear"
+    kv_from = None
+    kv_dims = None
+    window = 0
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads
+
+    @property
+    def q_rows(self) -> int:
+        return self.heads * self.dim
+
+    k_rows = q_rows
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    v_rows = out_width
+
+    @property
+    def slot_dims(self) -> tuple:
+        return None, (self.heads, memory_words(self.dim, self.vdim))
+
+    q_width = property(lambda self: self.dim)
+
+
+MEMORY_SLICE = 32    # value columns that share one copy of a matrix memory's normaliser and maximum
+
+
+def memory_words(dim: int, vdim: int) -> int:
+    """fp32 words of one head's matrix memory in a state slot: the matrix ``[dim, vdim]``, then for every slice of
+    :data:`MEMORY_SLICE` value columns a copy of the normaliser ``[dim]``, then their maxima; padded to 16 bytes. (Every
+    thread block owns whole slices with their copies, so the blocks of a head never wait for one another.)"""
+    slices = -(-vdim // MEMORY_SLICE)
+    n = dim * vdim + slices * (dim + 1)
+    return n + -n % 4
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same input: attention with pages beside a recurrent memory with a slot, added with fixed
+    factors."""
+
+    left: AttentionSpec
+    right: MatrixMemorySpec
+    left_scale: float
+    right_scale: float
+
+    kind = "attention"
+    kv_from = None
+
+    heads = property(lambda self: self.left.heads)
+    kv_heads = property(lambda self: self.left.kv_heads)
+    vdim = property(lambda self: max(self.left.vdim, self.right.vdim))
+    rot = property(lambda self: self.left.rot)
+    window = property(lambda self: self.left.window)
+    kv_dims = property(lambda self: self.left.kv_dims)
+    slot_dims = property(lambda self: self.right.slot_dims)
+    q_width = property(lambda self: self.left.q_width)
+
+
+@dataclass(frozen=True)
 class ClippedGLUSpec:
     """``down((up' + 1) * g' * sigmoid(alpha g'))``, ``g' = min(gate, limit)``, ``up' = clamp(up, -limit, limit)``."""
 
@@ -171,10 +251,19 @@ class GLUSpec:
 
 
 @dataclass(frozen=True)
+class DenseSpec:
+    """``down(act(up))``."""
+
+    ff: int
+    act: int
+
+
+@dataclass(frozen=True)
 class RoutedSpec:
-    """Mixture of gated experts. The router's softmax covers ``experts`` experts with weights and ``identity`` ones
-    that return their input; ``top`` of them are chosen by score + correction, out of the ``groups_keep`` best of
-    ``groups`` groups of neighbours (a group counts as its best expert), and weighted by their scores, normalised."""
+    """Mixture of gated experts. The router's scores (softmax or sigmoid) cover ``experts`` experts with weights and
+    ``identity`` ones that return their input; ``top`` of them are chosen by score (+ correction), out of the
+    ``groups_keep`` best of ``groups`` groups of neighbours (a group counts as its best expert), and weighted by their
+    scores, normalised or not. The weight multiplies an expert's output, or its input."""
 
     experts: int
     identity: int
@@ -182,7 +271,12 @@ class RoutedSpec:
     expert: GLUSpec
     groups: int = 1
     groups_keep: int = 1
-    shared: Optional[GLUSpec] = None    # runs for every token, times a sigmoid gate per token
+    shared: Optional[GLUSpec] = None    # runs for every token
+    shared_gate: bool = True            # times a sigmoid gate per token
+    sigmoid: bool = False               # scores: sigmoid instead of softmax
+    correction: bool = True             # a learned number per expert takes part in the choice
+    normalised: bool = True
+    weighted_input: bool = False
 
     @property
     def outputs(self) -> int:
@@ -205,6 +299,16 @@ class BigramSpec:
 
 
 @dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights, each pass with a cache and state of
+    its own."""
+
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     mixer: object
     mlp: Optional[object]
@@ -224,10 +328,16 @@ def _latent_attention(m: dict) -> LatentAttentionSpec:
                                window=int(mask.get("size") or 0))
 
 
+def _query_latent_attention(m: dict) -> LatentAttentionSpec:
+    return replace(_latent_attention(m), q_rank=int(m["q_rank"]), gated=False)
+
+
 def _attention(m: dict) -> AttentionSpec:
+    mask = m.get("mask") or {}
     spec = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                          scale=float(m["scale"]), rot=_rotary(m, int(m["dim"])), conv=int(m.get("conv") or 0),
-                         kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
+                         kv_from=None if m.get("kv_from") is None else int(m["kv_from"]),
+                         window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0))
     if spec.heads % spec.kv_heads:
         raise ValueError(f"{spec.heads} query heads cannot share {spec.kv_heads} key / value heads evenly")
     return spec
@@ -241,12 +351,28 @@ def _lightning(m: dict) -> LightningSpec:
     return spec
 
 
+def _memory(m: dict) -> MatrixMemorySpec:
+    spec = MatrixMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+    if spec.gate_cap <= 0:
+        raise ValueError(f"a gate cap of {spec.gate_cap} closes every gate")
+    return spec
+
+
+def _parallel(m: dict) -> ParallelSpec:
+    return ParallelSpec(left=_attention(m["left"]), right=_memory(m["right"]), left_scale=float(m["left_scale"]),
+                        right_scale=float(m["right_scale"]))
+
+
 def _clipped_glu(m: dict) -> ClippedGLUSpec:
     return ClippedGLUSpec(ff=int(m["ff"]), limit=float(m["limit"]))
 
 
 def _gelu_glu(m: dict) -> GLUSpec:
     return GLUSpec(ff=int(m["ff"]), act=ACT_GELU_TANH)
+
+
+def _relu_squared(m: dict) -> DenseSpec:
+    return DenseSpec(ff=int(m["ff"]), act=ACT_RELU_SQUARED)
 
 
 def _routed(m: dict) -> RoutedSpec:
@@ -263,10 +389,16 @@ def _routed(m: dict) -> RoutedSpec:
     return spec
 
 
+def _sigmoid_routed(m: dict) -> RoutedSpec:
+    return replace(_routed(m), sigmoid=True, correction=False, normalised=False, shared_gate=False, weighted_input=True)
+
+
 # per architecture: layer types and feed-forward kinds its configs may name
 _DESIGNS = {
     "Piburax": ({"latent_attention": _latent_attention}, {"dense": _clipped_glu}),
     "Zudepel": ({"attention": _attention, "lightning": _lightning}, {"dense": _gelu_glu, "moe": _routed}),
+    "Zasalix": ({"latent_attention": _query_latent_attention, "parallel": _parallel, "mlstm": _memory},
+                {"dense": _relu_squared, "moe": _sigmoid_routed}),
 }
 
 
@@ -302,3 +434,12 @@ def _check_shared_kv(before: list, i: int, m: AttentionSpec) -> None:
 def parse_bigram(emb: dict) -> Optional[BigramSpec]:
     b = emb.get("bigram")
     return None if b is None else BigramSpec(int(b["buckets"]), int(b["mul_prev"]), int(b["mul_cur"]))
+
+
+def parse_loop(loop: Optional[dict], layers: int) -> Optional[LoopSpec]:
+    if not loop:
+        return None
+    spec = LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+    if not 0 <= spec.start < spec.stop <= layers or spec.times < 1:
+        raise ValueError(f"layers {spec.start} to {spec.stop - 1}, {spec.times} times, is no loop over {layers} layers")
+    return spec

@@ -275,15 +275,16 @@ class MoEWeights:
 
 
 class RoutedExperts:
-    """Routed feed-forward of a layer-list model (:class:`parallax_b200.models.layer_spec.RoutedSpec`): softmax scores
-    over experts and identity experts, choice by score + correction within the best groups. The experts' rows are left
-    in expert order; :func:`ops.residual_add` weights and adds them (an identity expert adds the layer's input). The
-    gate of a shared expert is one more row of the router product, whose logits are fp32."""
+    """Routed feed-forward of a layer-list model (:class:`parallax_b200.models.layer_spec.RoutedSpec`): softmax or sigmoid
+    scores over experts and identity experts, choice by score (+ correction) within the best groups. The experts' rows are
+    left in expert order; :func:`ops.residual_add` weights and adds them (an identity expert adds the layer's input), or
+    :func:`ops.residual_step` adds them when the weights have gone into the experts' input. The gate of a shared expert is
+    one more row of the router product, whose logits are fp32."""
 
-    def __init__(self, spec, router: torch.Tensor, correction: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor):
+    def __init__(self, spec, router: torch.Tensor, correction: Optional[torch.Tensor], w1: torch.Tensor, w2: torch.Tensor):
         self.spec = spec
         self.router = router            # [outputs (+ shared gate), padded to 8, W]
-        self.correction = correction    # [outputs] fp32
+        self.correction = correction    # [outputs] fp32, or None
         self.w1, self.w2 = w1, w2       # [E * 2 ff, W] gate / up interleaved per expert, [E * W padded to 64, ff]
         self.ep = None                  # (expert parallelism is not available for these models)
         self.capture = None             # callable(ids [T, k]) when the engine records the routed experts
@@ -292,7 +293,7 @@ class RoutedExperts:
     def build(cls, spec, get, device) -> "RoutedExperts":
         """``get(name)``: checkpoint tensor of this feed-forward. Sizes are padded with zero rows / columns to what the
         grouped tensor-core product takes (expert width to 64, model width to 64)."""
-        rows = [get("router")] + ([get("shared.sg")] if spec.shared else [])
+        rows = [get("router")] + ([get("shared.sg")] if spec.shared and spec.shared_gate else [])
         router = torch.cat(rows, 0)
         router = torch.nn.functional.pad(router, (0, 0, 0, -router.shape[0] % 8)).contiguous()
         W, ff, E = router.shape[1], spec.expert.ff, spec.experts
@@ -304,17 +305,19 @@ class RoutedExperts:
             for i, name in enumerate(("gate", "up")):
                 w1[e, :, i] = pad(get(f"e{e}.{name}"), (0, 0, 0, ffp - ff)).view(ffp // 64, 64, W)
             w2[e, :W, :ff] = get(f"e{e}.down")
-        return cls(spec, router, get("correction", torch.float32), w1.view(-1, W), w2.view(-1, ffp))
+        correction = get("correction", torch.float32) if spec.correction else None
+        return cls(spec, router, correction, w1.view(-1, W), w2.view(-1, ffp))
 
     def tensors(self):
-        return [self.router, self.correction, self.w1, self.w2]
+        return [t for t in (self.router, self.correction, self.w1, self.w2) if t is not None]
 
     def forward(self, h: torch.Tensor):
         """(expert rows for :func:`ops.residual_add`, logits of the shared expert's gate ``[T]`` or None)."""
         s = self.spec
         logits = ops.linear(h, self.router, epi=ops.EPI_F32)
-        ids, w = ops.moe_route(logits[:, :s.outputs], self.correction, s.top, 0, True, s.groups, s.groups_keep, group_top=1)
+        ids, w = ops.moe_route(logits[:, :s.outputs], self.correction, s.top, int(s.sigmoid), s.normalised, s.groups,
+                               s.groups_keep, group_top=1)
         if self.capture is not None:
             self.capture(ids)
-        gate = logits[:, s.outputs] if s.shared else None
-        return ops.routed_ffn(h, ids, w, self.w1, self.w2, s.experts), gate
+        gate = logits[:, s.outputs] if s.shared and s.shared_gate else None
+        return ops.routed_ffn(h, ids, w, self.w1, self.w2, s.experts, s.weighted_input), gate

@@ -35,9 +35,14 @@ _REGISTRY: dict[str, str] = {
     "Piburax": "latent",
     # layer-list configs: attention / lightning layers beside (not before) their feed-forward
     "Zudepel": "parallel_block",
+    # layer-list configs: looped layers, norms on both sides of a sublayer, matrix memories beside or instead of attention
+    "Zasalix": "looped",
     # block-sparse (MSA)
     "MiniMaxM3SparseForCausalLM": "msa",
 }
+
+
+_LISTED = ("latent", "looped", "parallel_block")      # families of layer-list configs
 
 
 def supported_architectures() -> list[str]:
@@ -53,7 +58,7 @@ def family_of(arch: str) -> str:
 
 def runs_in_float32(arch: str) -> bool:
     """Whether the family's GPU stages also run in 32-bit throughout (``dtype=torch.float32``)."""
-    return family_of(arch) in ("latent", "parallel_block")
+    return family_of(arch) in _LISTED
 
 
 def build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype, max_positions=None,
@@ -73,13 +78,14 @@ def build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtyp
 def _build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dtype, max_positions, tp_rank, tp_size,
                  tp_group, comm):
     fam = family_of(cfg.architecture)
-    if fam in ("latent", "parallel_block"):
+    if fam in _LISTED:
         from parallax_b200.models.latent import LatentStage
+        from parallax_b200.models.looped import LoopedStage
         from parallax_b200.models.parallel_block import ParallelBlockStage
 
         if tp_size > 1:
             raise ValueError(f"tensor parallelism is not available for {cfg.architecture}; use pipeline stages")
-        cls = LatentStage if fam == "latent" else ParallelBlockStage
+        cls = {"latent": LatentStage, "looped": LoopedStage, "parallel_block": ParallelBlockStage}[fam]
         return cls(cfg, start_layer, end_layer, device, dtype, max_positions=max_positions)
     if tp_size > 1 and fam != "decoder":
         from parallax_b200.models import tp_families

@@ -20,6 +20,7 @@ _NAMES = [
     "quant_fp8_rows", "linear_fp8", "moe_ffn_fp8", "causal_conv1d_silu", "gated_delta_rule", "sigmoid_gate_mul", "gate_mul_grouped", "row_dot", "msa_block_scores", "msa_select",
     "embed_rows", "to_low", "residual_norm", "row_norm", "latent_prep", "head_linear", "latent_attn",
     "glu_linear", "routed_ffn", "residual_add", "conv_qkv_prep", "gated_rows", "lightning_attn",
+    "latent_rows", "latent_queries", "act_linear", "tanh_norm", "residual_step", "matrix_memory",
 ]
 
 

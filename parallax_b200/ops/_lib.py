@@ -78,12 +78,12 @@ _SIGS = {
     "pxl_selftest_bounded_wait": [_P, c_uint32, _P, _P, _P],
     "pxl_patch_i32": [_P, _P, _P, _P, c_int, c_int, c_int, _P, _P],
     "pxl_attn_decode": [_P, c_int64, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
-                        c_int64, c_float, c_int, c_int, c_int, _P, _P],
+                        c_int64, c_float, c_int, c_int, c_int, c_int, _P, _P],
     "pxl_attn_decode_splits": [c_int, c_int, c_int],
     "pxl_attn_prefill": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int,
-                         c_int, c_int, c_int, c_int, c_int64, c_float, c_int, _P, _P],
+                         c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_int, _P, _P],
     "pxl_attn_prefill_tc": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int, c_int,
-                            c_int, c_int, c_int, c_int, c_int64, c_float, c_int, _P, _P],
+                            c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_int, _P, _P],
     "pxl_moe_route": [_P, c_int64, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, _P],
     "pxl_moe_align": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, _P],
     "pxl_moe_gather": [_P, _P, _P, _P, c_int, c_int, _P],
@@ -132,9 +132,20 @@ _SIGS = {
     "pxl_glu_act": [_P, _P, c_int64, _P, c_int64, c_int, c_int, c_int, c_int, _P],
     "pxl_conv_qkv_prep": [_P, c_int64] + [c_int] * 10 + [_P, _P, c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P,
                           c_int64, c_int, _P, _P, _P, c_float, c_int, _P, _P],
-    "pxl_gated_rows": [_P, c_int, c_int, c_int, _P, c_int64, _P, c_float, _P, c_int64, c_int, c_int, c_int, _P],
+    "pxl_gated_rows": [_P, c_int, c_int, c_int, _P, c_int64, _P, c_float, c_int, c_float, _P, c_int64, c_int, c_int, c_int, _P],
     "pxl_attn_any": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64,
-                     c_float, c_int, c_int, _P, _P],
+                     c_float, c_int, c_int, c_int, _P, _P],
+    "pxl_latent_rows": [_P, c_int64, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, _P, _P, c_int64, c_int, c_int, c_int, c_int,
+                        c_float, c_int, _P, _P],
+    "pxl_latent_queries": [_P, c_int64, c_int, c_int, c_int, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, _P],
+    "pxl_matrix_memory": [_P, c_int64] + [c_int] * 6 + [_P, c_int64, _P, c_float, _P, c_int64, c_int, _P, _P, _P, _P, c_int64,
+                          c_int, c_int, c_int, _P, _P],
+    "pxl_residual_step": [_P, _P, c_int64, _P, c_int64, c_int64, _P, _P, c_int, c_int, _P, _P, c_float, c_float, _P, _P, c_int64,
+                          _P, c_int, _P, _P, c_float, _P, c_int, c_int, c_int, _P, _P],
+    "pxl_tanh_norm": [_P, _P, _P, c_float, _P, c_int64, _P, c_int, c_int, c_int, _P, _P],
+    "pxl_act_rows": [_P, c_int64, c_int, c_int, _P, c_int64, c_int, _P, c_int64, _P, c_int64, c_int, c_int, c_int, _P, _P],
+    "pxl_gemm_bf16_act": [_P, _P, _P] + [c_int] * 7 + [_P, c_int64, _P, c_int64, _P, _P],
+    "pxl_moe_scatter_rows": [_P, c_int64, _P, _P, _P, c_int, c_int, c_int, c_int, _P],
     "pxl_lightning_attn": [_P, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, c_int, _P, _P, _P, _P, c_int64,
                            c_int, c_int, c_int, _P, _P],
     "pxl_rmsnorm_strided": [_P, c_int64, _P, _P, c_int64, c_int, c_int, c_float, c_float, _P],

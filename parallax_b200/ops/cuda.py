@@ -410,7 +410,7 @@ def add_inplace(y: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------ attention
-def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, window, sinks, out):
+def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, window, sinks, out, keep_first):
     """FMA-pipe form: fp32, any head size, any number of query heads per key head."""
     T, Hq, D = q.shape
     Hkv, page = k_cache.shape[1], k_cache.shape[2]
@@ -418,7 +418,7 @@ def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, w
     check(_lib.lib().pxl_attn_any(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
                                   _ptr(cu_q), ctx_lens.data_ptr(), out.data_ptr(), out.stride(0), _ptr(sinks),
                                   ctx_lens.numel(), max_q, Hq, Hkv, D, page, block_tables.shape[1], k_cache.shape[0],
-                                  float(scale), window, int(q.dtype == torch.float32), status_tensor(q.device).data_ptr(),
+                                  float(scale), window, keep_first, int(q.dtype == torch.float32), status_tensor(q.device).data_ptr(),
                                   _stream(q.device)), "pxl_attn_any")
     _count()
     return out
@@ -441,24 +441,28 @@ def attn_decode(
     num_splits: int = 0,
     out: Optional[torch.Tensor] = None,
     kv_scale: tuple = (1.0, 1.0),
+    keep_first: int = 0,
 ) -> torch.Tensor:
     """q ``[B, Hq, D]`` (may be a strided view into a packed qkv buffer) vs the paged cache (bf16, or e4m3
-    with ``kv_scale``)."""
+    with ``kv_scale``). With a ``window`` the first ``keep_first`` keys of a sequence stay visible."""
     B, Hq, D = q.shape
     assert q.stride(2) == 1 and q.stride(1) == D
     Hkv, page = k_cache.shape[1], k_cache.shape[2]
     if out is None:
         out = torch.empty((B, Hq, D), dtype=q.dtype, device=q.device)
     if not _is_fp8_cache(k_cache) and not _attn_on_tensor_cores(q, k_cache, scale, 16):
-        return _attn_any(q, k_cache, v_cache, block_tables, None, ctx_lens, 1, scale, window, sinks, out)
+        return _attn_any(q, k_cache, v_cache, block_tables, None, ctx_lens, 1, scale, window, sinks, out, keep_first)
     if max_ctx <= 0:
         max_ctx = block_tables.shape[1] * page
     if num_splits <= 0:
-        num_splits = _lib.lib().pxl_attn_decode_splits(B, Hkv, max_ctx)
+        # keys a query reads: whole tiles of 64 of the window and of the kept ones
+        span = min(max_ctx, window + keep_first + 128) if window > 0 else max_ctx
+        num_splits = _lib.lib().pxl_attn_decode_splits(B, Hkv, span)
     ws = None
     if num_splits > 1:
         ws = workspace(q.device, "attn_decode", B * Hq * num_splits * (D + 2) * 4)
     if _is_fp8_cache(k_cache):
+        assert keep_first == 0
         check(
             _lib.lib().pxl_attn_decode_fp8(
                 q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
@@ -474,7 +478,7 @@ def attn_decode(
             q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
             block_tables.data_ptr(), ctx_lens.data_ptr(), out.data_ptr(), _ptr(ws), _ptr(sinks),
             B, Hq, Hkv, D, page,
-            block_tables.shape[1], k_cache.shape[0], scale, window, num_splits, max_ctx,
+            block_tables.shape[1], k_cache.shape[0], scale, window, keep_first, num_splits, max_ctx,
             status_tensor(q.device).data_ptr(), _stream(q.device)),
         "pxl_attn_decode",
     )
@@ -495,6 +499,7 @@ def attn_prefill(
     sinks: Optional[torch.Tensor] = None,
     out: Optional[torch.Tensor] = None,
     kv_scale: tuple = (1.0, 1.0),
+    keep_first: int = 0,
 ) -> torch.Tensor:
     """q ``[T, Hq, D]`` (may be a strided view into a packed qkv buffer)."""
     T, Hq, D = q.shape
@@ -506,8 +511,9 @@ def attn_prefill(
     if T == 0 or B == 0:
         return out
     if not _is_fp8_cache(k_cache) and not _attn_on_tensor_cores(q, k_cache, scale, 64):
-        return _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window, sinks, out)
+        return _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window, sinks, out, keep_first)
     if _is_fp8_cache(k_cache):
+        assert keep_first == 0
         check(
             _lib.lib().pxl_attn_prefill_fp8(
                 q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
@@ -527,7 +533,7 @@ def attn_prefill(
                 q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
                 block_tables.data_ptr(), cu_q.data_ptr(), ctx_lens.data_ptr(), out.data_ptr(),
                 out.stride(0), _ptr(sinks), B, max_q_len, T, Hq, Hkv, D, page, block_tables.shape[1],
-                k_cache.shape[0], scale, window, status_tensor(q.device).data_ptr(),
+                k_cache.shape[0], scale, window, keep_first, status_tensor(q.device).data_ptr(),
                 _stream(q.device)),
             "pxl_attn_prefill_tc",
         )
@@ -538,7 +544,7 @@ def attn_prefill(
             q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
             block_tables.data_ptr(), cu_q.data_ptr(), ctx_lens.data_ptr(), out.data_ptr(),
             out.stride(0), _ptr(sinks), B, max_q_len, Hq, Hkv, D, page, block_tables.shape[1],
-            k_cache.shape[0], scale, window, status_tensor(q.device).data_ptr(),
+            k_cache.shape[0], scale, window, keep_first, status_tensor(q.device).data_ptr(),
             _stream(q.device)),
         "pxl_attn_prefill",
     )
@@ -705,18 +711,32 @@ def moe_ffn(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w1: torch
     return moe_combine(y, plan, weights, base, x.shape[0])
 
 
-def routed_ffn(x, ids, weights, w1, w2, num_experts: int):
+def moe_scatter_rows(x, plan: MoEPlan, weights) -> torch.Tensor:
+    """Rows in expert order, each times its routing weight (bf16 or fp32, any width)."""
+    T, H = x.shape
+    assert x.stride(1) == 1 and weights.is_contiguous() and weights.dtype == torch.float32
+    xp = torch.empty((plan.max_rows + 128, H), dtype=x.dtype, device=x.device)      # (a padding tile as in moe_gather)
+    check(_lib.lib().pxl_moe_scatter_rows(x.data_ptr(), x.stride(0), plan.pos_of.data_ptr(), weights.data_ptr(), xp.data_ptr(), T,
+                                          weights.shape[1], H, int(x.dtype == torch.float32), _stream(x.device)),
+          "pxl_moe_scatter_rows")
+    _count()
+    return xp
+
+
+def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool = False):
     """Gated (SiLU) experts; rows stay in expert order for :func:`residual_add` to pick up. ``w1 [E * 2 I, W]`` gate / up
-    rows interleaved per expert, ``w2 [E * N, I]`` (N >= W: padded outputs). Ids >= ``num_experts`` are identity experts."""
+    rows interleaved per expert, ``w2 [E * N, I]`` (N >= W: padded outputs). Ids >= ``num_experts`` are identity experts.
+    ``weighted_input``: the weights multiply the experts' input rows."""
     plan = moe_align(ids, num_experts)
+    xp = moe_scatter_rows(x, plan, weights) if weighted_input else None
     if x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
         n = w2.shape[0] // num_experts
-        act = grouped_linear(moe_gather(x, plan), w1, plan, num_experts, epi=EPI_SILU_MUL)
+        act = grouped_linear(moe_gather(x, plan) if xp is None else xp, w1, plan, num_experts, epi=EPI_SILU_MUL)
         y = grouped_linear(act, w2, plan, num_experts, bn=0 if n % 128 == 0 else 64)
     else:
-        act = _glu_act(_grouped_simt(x, w1, plan, num_experts, plan.src_tok), 0)
-        y = _grouped_simt(act, w2, plan, num_experts, None)
-    return y, plan.pos_of, weights
+        gu = _grouped_simt(x, w1, plan, num_experts, plan.src_tok) if xp is None else _grouped_simt(xp, w1, plan, num_experts, None)
+        y = _grouped_simt(_glu_act(gu, 0), w2, plan, num_experts, None)
+    return y, plan.pos_of, None if weighted_input else weights
 
 
 def _grouped_simt(x, w, plan, num_experts: int, a_rows):
@@ -757,6 +777,35 @@ def glu_linear(x, w_gu, act: int = 0, row_gate=None, out=None):
                                            w_gu.stride(0), out.stride(0), act, _ptr(row_gate),
                                            row_gate.stride(0) if row_gate is not None else 0, 0,
                                            status_tensor(x.device).data_ptr(), _stream(x.device)), "pxl_gemm_bf16_act_glu")
+    _count()
+    return out
+
+
+def act_linear(x, w, act: int, table=None, ids=None, col: int = 0, out=None):
+    T, N = x.shape[0], w.shape[0]
+    if out is None:
+        out = torch.empty((T, N), dtype=x.dtype, device=x.device)
+    if T == 0:
+        return out
+    assert out.stride(1) == 1 and (table is None or (table.is_contiguous() and table.dtype == x.dtype and ids.dtype == torch.int32
+                                                     and ids.numel() == T and col + N <= table.shape[1]))
+    ldt, num = (table.shape[1], table.shape[0]) if table is not None else (0, 0)
+    dev = x.device
+    # enough output tiles for half of the SMs: the activation rides in the product's epilogue; few: split-K product, then rows
+    tiles = -(-T // 128) * -(-N // 64)
+    if x.dtype == torch.bfloat16 and _tma_ok(x, w) and tiles >= 74 and not (out.stride(0) | ldt | col) & 7 \
+            and not (out.data_ptr() | (table.data_ptr() if table is not None else 0)) & 15:
+        check(_lib.lib().pxl_gemm_bf16_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), T, N, x.shape[1], x.stride(0), w.stride(0),
+                                           out.stride(0), act, None if table is None else table.data_ptr() + 2 * col, ldt,
+                                           _ptr(ids if table is not None else None), num, status_tensor(dev).data_ptr(),
+                                           _stream(dev)), "pxl_gemm_bf16_act")
+        _count()
+        return out
+    y = linear(x, w, epi=EPI_F32)
+    check(_lib.lib().pxl_act_rows(y.data_ptr(), y.stride(0), int(y.dtype == torch.float32), act, _ptr(table), ldt, col,
+                                  _ptr(ids if table is not None else None), num, out.data_ptr(), out.stride(0),
+                                  int(out.dtype == torch.float32), T, N, status_tensor(dev).data_ptr(), _stream(dev)),
+          "pxl_act_rows")
     _count()
     return out
 
@@ -1194,7 +1243,7 @@ def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, co
         assert k_cache.shape[1] == kv_heads and k_cache.shape[3] == v_cache.shape[3] == cols
     check(_lib.lib().pxl_conv_qkv_prep(
         proj.data_ptr(), proj.stride(0), *offs, heads, kv_heads if own else 0, dim, vdim, cols, rot, taps, _ptr(conv_w),
-        _ptr(state), state.shape[0] if state is not None else 0, q_norm.data_ptr(), _ptr(k_norm), cos_sin.data_ptr(),
+        _ptr(state), state.shape[0] if state is not None else 0, _ptr(q_norm), _ptr(k_norm), cos_sin.data_ptr(),
         positions.data_ptr(), cos_sin.shape[0], seq_cu.data_ptr(), seq_slots.data_ptr(), prefill_seqs, prefill_tokens, T,
         slot_mapping.data_ptr(), k_cache.shape[0] * k_cache.shape[2] if own else 0, k_cache.shape[2] if own else 1,
         _ptr(k_cache), _ptr(v_cache), q_out.data_ptr(), eps, int(proj.dtype == torch.float32),
@@ -1202,11 +1251,11 @@ def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, co
     _count(2 if taps > 1 and prefill_seqs else 1)
 
 
-def gated_rows(x, vdim: int, gate, out, norm_w=None, eps: float = 0.0):
+def gated_rows(x, vdim: int, gate, out, norm_w=None, eps: float = 0.0, per_head: bool = False, scale: float = 1.0):
     T, heads, cols = x.shape
     assert x.is_contiguous() and gate.stride(1) == 1 and out.stride(1) == 1 and x.dtype == gate.dtype == out.dtype
     check(_lib.lib().pxl_gated_rows(x.data_ptr(), heads, cols, vdim, gate.data_ptr(), gate.stride(0), _ptr(norm_w), eps,
-                                    out.data_ptr(), out.stride(0), out.shape[1], T, int(x.dtype == torch.float32),
+                                    int(per_head), scale, out.data_ptr(), out.stride(0), out.shape[1], T, int(x.dtype == torch.float32),
                                     _stream(x.device)), "pxl_gated_rows")
     _count()
     return out
@@ -1225,5 +1274,95 @@ def lightning_attn(proj, offs, heads: int, dim: int, vdim: int, decay_pow, state
                                         seq_slots.data_ptr(), positions.data_ptr(), out.data_ptr(), heads * vdim, prefill_seqs,
                                         n - prefill_seqs, int(proj.dtype == torch.float32),
                                         status_tensor(proj.device).data_ptr(), _stream(proj.device)), "pxl_lightning_attn")
+    _count((prefill_seqs > 0) + (n > prefill_seqs))
+    return out
+
+
+# ---------------------------------------------------------------------------- query latents, tanh norms, matrix memory
+def latent_rows(proj, q_off: int, q_norm, c_q, kv_off: int, norm_w, cos_sin, positions, slot_mapping, cache, eps: float,
+                latent: int, rot_dim: int, rot: int):
+    T, rank = c_q.shape
+    assert proj.stride(1) == 1 and proj.dtype == cache.dtype == c_q.dtype and cos_sin.shape[1] == rot
+    assert cache.is_contiguous() and cache.shape[-1] == latent + rot_dim and c_q.is_contiguous() and q_norm.numel() == rank
+    check(_lib.lib().pxl_latent_rows(proj.data_ptr(), proj.stride(0), q_off, rank, q_norm.data_ptr(), c_q.data_ptr(), kv_off,
+                                     norm_w.data_ptr(), cos_sin.data_ptr(), positions.data_ptr(), cos_sin.shape[0],
+                                     slot_mapping.data_ptr(), cache.data_ptr(), cache.numel() // cache.shape[-1], T, latent,
+                                     rot_dim, rot, eps, int(proj.dtype == torch.float32), status_tensor(proj.device).data_ptr(),
+                                     _stream(proj.device)), "pxl_latent_rows")
+    _count()
+
+
+def latent_queries(q, heads: int, q_width: int, q_rot_off: int, cos_sin, positions, q_cat, latent: int, rot_dim: int, rot: int):
+    T = q.shape[0]
+    assert q.stride(1) == 1 and q.dtype == q_cat.dtype and cos_sin.shape[1] == rot
+    assert q_cat.is_contiguous() and q_cat.shape == (T, heads, latent + rot_dim)
+    check(_lib.lib().pxl_latent_queries(q.data_ptr(), q.stride(0), heads, q_width, q_rot_off, cos_sin.data_ptr(),
+                                        positions.data_ptr(), cos_sin.shape[0], q_cat.data_ptr(), T, latent, rot_dim, rot,
+                                        int(q.dtype == torch.float32), status_tensor(q.device).data_ptr(), _stream(q.device)),
+          "pxl_latent_queries")
+    _count()
+
+
+def tanh_norm(x, w, b, alpha: float, rows=None, dtype=None):
+    W = x.shape[1]
+    T = x.shape[0] if rows is None else rows.numel()
+    assert x.dtype == w.dtype == b.dtype == torch.float32 and x.is_contiguous() and w.numel() == b.numel() == W
+    assert rows is None or rows.dtype == torch.int32
+    out = torch.empty((T, W), dtype=dtype or torch.float32, device=x.device)
+    check(_lib.lib().pxl_tanh_norm(x.data_ptr(), w.data_ptr(), b.data_ptr(), alpha, _ptr(rows), x.shape[0], out.data_ptr(), T, W,
+                                   int(out.dtype == torch.float32), status_tensor(x.device).data_ptr(), _stream(x.device)),
+          "pxl_tanh_norm")
+    _count()
+    return out
+
+
+def residual_step(x, y=None, post=None, routed=None, table=None, ids=None, step=None, pre=None, dtype=None, eps: float = 0.0):
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    rows, pos_of, weights = routed or (None, None, None)
+    assert (post is None) == (y is None and rows is None)
+    if pre is not None:
+        f32 = dtype == torch.float32
+    else:
+        f32 = next((t.dtype for t in (y, rows, table) if t is not None), torch.float32) == torch.float32
+    dt = torch.float32 if f32 else torch.bfloat16
+    assert y is None or (y.shape == x.shape and y.stride(1) == 1 and y.dtype == dt)
+    assert rows is None or (rows.stride(1) == 1 and rows.shape[1] >= W and rows.dtype == dt)
+    assert table is None or (table.is_contiguous() and table.shape[1] == W and table.dtype == dt and ids.dtype == torch.int32)
+    assert step is None or (step.dtype == torch.float32 and step.stride(0) == 1)
+    mode, low = 0, None
+    if pre is not None:
+        mode = 1 if pre else 2
+        if mode == 2 and f32:       # the operand is the residual itself
+            mode, low = 0, x
+        else:
+            low = torch.empty((T, W), dtype=dt, device=x.device)
+    pw, pb, pa = (tuple(post or ()) + (None, None, None))[:3]
+    nw, nb, na = (tuple(pre or ()) + (None, None, None))[:3]
+    check(_lib.lib().pxl_residual_step(
+        x.data_ptr(), _ptr(y), y.stride(0) if y is not None else 0, _ptr(rows), rows.stride(0) if rows is not None else 0,
+        rows.shape[0] if rows is not None else 0, _ptr(pos_of), _ptr(weights), pos_of.numel() // T if pos_of is not None else 0,
+        0 if post is None else 1 if len(post) == 3 else 2, _ptr(pw), _ptr(pb), pa or 0.0, eps, _ptr(table),
+        _ptr(ids if table is not None else None), table.shape[0] if table is not None else 0, _ptr(step), mode, _ptr(nw), _ptr(nb),
+        na or 0.0, _ptr(low) if mode else None, T, W, int(f32), status_tensor(x.device).data_ptr(), _stream(x.device)),
+        "pxl_residual_step")
+    _count()
+    return low
+
+
+def matrix_memory(proj, offs, heads: int, dim: int, vdim: int, gates, gate_bias, cap: float, state, positions, seq_cu, seq_slots,
+                  prefill_seqs: int, slice_cols: int = 32, out=None):
+    T = proj.shape[0]
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=proj.dtype, device=proj.device)
+    assert slice_cols == 32 and proj.stride(1) == 1 and out.is_contiguous() and out.dtype == proj.dtype
+    assert gates.dtype == gate_bias.dtype == torch.float32 and gates.stride(1) == 1 and gates.shape[1] >= 2 * heads
+    assert gate_bias.numel() == 2 * heads and state.is_contiguous() and state.dtype == torch.float32 and state.shape[1] == heads
+    n = seq_slots.numel()
+    check(_lib.lib().pxl_matrix_memory(proj.data_ptr(), proj.stride(0), *offs, heads, dim, vdim, gates.data_ptr(), gates.stride(0),
+                                       gate_bias.data_ptr(), cap, state.data_ptr(), state.shape[2], state.shape[0],
+                                       seq_cu.data_ptr(), seq_slots.data_ptr(), positions.data_ptr(), out.data_ptr(), heads * vdim,
+                                       prefill_seqs, n - prefill_seqs, int(proj.dtype == torch.float32),
+                                       status_tensor(proj.device).data_ptr(), _stream(proj.device)), "pxl_matrix_memory")
     _count((prefill_seqs > 0) + (n > prefill_seqs))
     return out

@@ -181,7 +181,7 @@ def _gather_kv(cache, block_table, n, scale: float = 1.0):
     return blocks.permute(1, 0, 2, 3).reshape(cache.shape[1], nb * page, cache.shape[3])[:, :n]
 
 
-def _attend(q, k, v, scale, q_pos, window, sinks):
+def _attend(q, k, v, scale, q_pos, window, sinks, keep_first=0):
     # q [Lq, Hq, D]; k, v [Hkv, Lk, D]; q_pos [Lq] absolute positions of the queries
     Lq, Hq, D = q.shape
     Hkv, Lk, _ = k.shape
@@ -193,7 +193,7 @@ def _attend(q, k, v, scale, q_pos, window, sinks):
     kpos = torch.arange(Lk, device=q.device)[None, :]
     mask = kpos <= q_pos[:, None]
     if window and window > 0:
-        mask = mask & (kpos > q_pos[:, None] - window)
+        mask = mask & ((kpos > q_pos[:, None] - window) | (kpos < keep_first))
     s = s.masked_fill(~mask[None], float("-inf"))
     if sinks is not None:
         s = torch.cat([s, sinks.float()[:, None, None].expand(Hq, Lq, 1)], dim=-1)
@@ -206,7 +206,9 @@ def _attend(q, k, v, scale, q_pos, window, sinks):
 
 
 def attn_decode(q, k_cache, v_cache, block_tables, ctx_lens, scale, window=0, sinks=None,
-                max_ctx=0, num_splits=0, out=None, kv_scale=(1.0, 1.0)):
+                max_ctx=0, num_splits=0, out=None, kv_scale=(1.0, 1.0), keep_first=0):
+    """One query per sequence over the paged cache; ``window`` keys per query (0: all) and the sequence's first
+    ``keep_first``."""
     B = q.shape[0]
     res = torch.zeros_like(q) if out is None else out
     for b in range(B):
@@ -217,12 +219,12 @@ def attn_decode(q, k_cache, v_cache, block_tables, ctx_lens, scale, window=0, si
         k = _gather_kv(k_cache, block_tables[b], n, kv_scale[0])
         v = _gather_kv(v_cache, block_tables[b], n, kv_scale[1])
         pos = torch.tensor([n - 1], device=q.device)
-        res[b] = _attend(q[b:b + 1], k, v, scale, pos, window, sinks)[0]
+        res[b] = _attend(q[b:b + 1], k, v, scale, pos, window, sinks, keep_first)[0]
     return res
 
 
 def attn_prefill(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window=0,
-                 sinks=None, out=None, kv_scale=(1.0, 1.0)):
+                 sinks=None, out=None, kv_scale=(1.0, 1.0), keep_first=0):
     T, Hq, D = q.shape
     res = torch.zeros((T, Hq, D), dtype=q.dtype, device=q.device) if out is None else out
     B = ctx_lens.numel()
@@ -235,7 +237,7 @@ def attn_prefill(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, s
         k = _gather_kv(k_cache, block_tables[b], n, kv_scale[0])
         v = _gather_kv(v_cache, block_tables[b], n, kv_scale[1])
         pos = prefix + torch.arange(e - s, device=q.device)
-        res[s:e] = _attend(q[s:e], k, v, scale, pos, window, sinks)
+        res[s:e] = _attend(q[s:e], k, v, scale, pos, window, sinks, keep_first)
     return res
 
 
@@ -700,15 +702,31 @@ def latent_prep(proj, kv_off: int, q_heads: int, q_width: int, q_rot_off: int, n
     """One step's latent-attention inputs out of the packed projection ``proj`` (columns: ``q_heads`` heads of
     ``q_width``, and at ``kv_off`` the raw latent | rotated key part): RMS-normed latent and rotated key go to
     the cache rows ``slot_mapping``, the rotated query parts to ``q_cat[:, :, latent:]``."""
-    T = proj.shape[0]
+    _store_latent_rows(proj, kv_off, norm_w, cos_sin, positions, slot_mapping, cache, eps, latent, rot_dim, rot)
+    latent_queries(proj, q_heads, q_width, q_rot_off, cos_sin, positions, q_cat, latent, rot_dim, rot)
+
+
+def _store_latent_rows(proj, kv_off, norm_w, cos_sin, positions, slot_mapping, cache, eps, latent, rot_dim, rot):
     kv = proj[:, kv_off:kv_off + latent + rot_dim].float()
     c = _normalised(kv[:, :latent], eps, NORM_RMS) * norm_w.float()
     k = _rotate_pairs(kv[:, latent:], cos_sin, positions, rot)
     flat = cache.view(-1, latent + rot_dim)
     ok = slot_mapping >= 0
     flat[slot_mapping[ok]] = torch.cat([c, k], -1)[ok].to(cache.dtype)
-    q = proj[:, :q_heads * q_width].reshape(T, q_heads, q_width)[..., q_rot_off:q_rot_off + rot_dim].float()
-    q_cat[:, :, latent:] = _rotate_pairs(q, cos_sin, positions, rot).to(q_cat.dtype)
+
+
+def latent_rows(proj, q_off: int, q_norm, c_q, kv_off: int, norm_w, cos_sin, positions, slot_mapping, cache, eps: float,
+                latent: int, rot_dim: int, rot: int):
+    """Key half of :func:`latent_prep` for queries that go through a latent of their own: cache rows from column
+    ``kv_off`` of ``proj``, and ``c_q = rmsnorm(proj[:, q_off:]) * q_norm``."""
+    c_q.copy_((_normalised(proj[:, q_off:q_off + q_norm.numel()], eps, NORM_RMS) * q_norm.float()).to(c_q.dtype))
+    _store_latent_rows(proj, kv_off, norm_w, cos_sin, positions, slot_mapping, cache, eps, latent, rot_dim, rot)
+
+
+def latent_queries(q, heads: int, q_width: int, q_rot_off: int, cos_sin, positions, q_cat, latent: int, rot_dim: int, rot: int):
+    """Query half of :func:`latent_prep`: the rotated parts of ``q [T, heads * q_width]`` into ``q_cat[:, :, latent:]``."""
+    part = q[:, :heads * q_width].reshape(q.shape[0], heads, q_width)[..., q_rot_off:q_rot_off + rot_dim].float()
+    q_cat[:, :, latent:] = _rotate_pairs(part, cos_sin, positions, rot).to(q_cat.dtype)
 
 
 def head_linear(x, x_head_stride: int, w, heads: int, out, gate=None):
@@ -768,10 +786,23 @@ def glu_linear(x, w_gu, act: int = 0, row_gate=None, out=None):
     return out
 
 
-def routed_ffn(x, ids, weights, w1, w2, num_experts: int):
+def act_linear(x, w, act: int, table=None, ids=None, col: int = 0, out=None):
+    """``act(x @ w^T)`` (2: GELU, tanh form; 3: square of relu), times ``table[ids, col : col + N]`` if given."""
+    y = x.float() @ w.float().t()
+    y = torch.nn.functional.gelu(y, approximate="tanh") if act == 2 else y.clamp_min(0) ** 2
+    if table is not None:
+        y = y * table[ids.long(), col:col + w.shape[0]].float()
+    if out is None:
+        return y.to(x.dtype)
+    out.copy_(y)
+    return out
+
+
+def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool = False):
     """Outputs of the chosen gated (SiLU) experts for :func:`residual_add`: ``(rows, pos_of, weights)``, where
     ``rows[pos_of[t, j]]`` is expert ``ids[t, j]``'s output. ``w1 [E * 2 I, W]`` gate / up rows interleaved per expert,
-    ``w2 [E * N, I]``. Ids >= ``num_experts`` are identity experts: position -1."""
+    ``w2 [E * N, I]``. Ids >= ``num_experts`` are identity experts: position -1. ``weighted_input``: the weights multiply
+    the experts' input rows, and None comes back for them."""
     T, k = ids.shape
     n1, n2 = w1.shape[0] // num_experts, w2.shape[0] // num_experts
     rows = torch.zeros((T * k, n2), dtype=x.dtype, device=x.device)
@@ -779,9 +810,10 @@ def routed_ffn(x, ids, weights, w1, w2, num_experts: int):
     for e in range(num_experts):
         tok, slot = (ids == e).nonzero(as_tuple=True)
         if tok.numel():
-            act = glu_linear(x[tok], w1[e * n1:(e + 1) * n1])
+            xe = (x[tok].float() * weights[tok, slot].float()[:, None]).to(x.dtype) if weighted_input else x[tok]
+            act = glu_linear(xe, w1[e * n1:(e + 1) * n1])
             rows[tok * k + slot] = linear(act, w2[e * n2:(e + 1) * n2])
-    return rows, torch.where(ids < num_experts, pos, torch.full_like(pos, -1)).to(torch.int32), weights
+    return rows, torch.where(ids < num_experts, pos, torch.full_like(pos, -1)).to(torch.int32), None if weighted_input else weights
 
 
 def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None):
@@ -802,7 +834,7 @@ def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, co
     """Queries and cache rows of one step out of the packed projection: q, k, v start at columns ``offs`` of ``proj``.
     Causal convolution per channel (``conv_w [taps, channels]`` over q | k | v, or None) with the state slots
     ``conv_state [slots, taps - 1, channels]``, RMS norm over the whole q and k rows, half-split rotation
-    (``cos_sin [positions, dims]``). ``q_out [T, heads, cols]`` and the pages ``[blocks, kv_heads, page, cols]`` get heads
+    (``cos_sin [positions, dims]``); norm weights None: no norm. ``q_out [T, heads, cols]`` and the pages ``[blocks, kv_heads, page, cols]`` get heads
     padded with zeros; without caches only q is made."""
     T, cols, rot = proj.shape[0], q_out.shape[2], cos_sin.shape[1]
     own = k_cache is not None
@@ -831,7 +863,7 @@ def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, co
     c, s = cs[..., :rot // 2], cs[..., rot // 2:]
 
     def rotate(x, norm_w, n):
-        x = (_normalised(x, eps, NORM_RMS) * norm_w.float()).view(T, n, dim)
+        x = (x if norm_w is None else _normalised(x, eps, NORM_RMS) * norm_w.float()).view(T, n, dim)
         a, b = x[..., :rot // 2], x[..., rot // 2:rot]
         return torch.cat([a * c - b * s, b * c + a * s, x[..., rot:]], -1)
 
@@ -843,14 +875,17 @@ def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, co
         reshape_and_cache(pad(k, (0, cols - dim)), pad(v, (0, cols - vdim)), slot_mapping, k_cache, v_cache)
 
 
-def gated_rows(x, vdim: int, gate, out, norm_w=None, eps: float = 0.0):
-    """``out[:, :heads * vdim] = heads side by side (, rmsnorm over them all * norm_w) * sigmoid(gate)``, zeros behind;
-    ``x [T, heads, cols]``, of which the first ``vdim`` columns count."""
-    y = x[:, :, :vdim].reshape(x.shape[0], -1).float()
+def gated_rows(x, vdim: int, gate, out, norm_w=None, eps: float = 0.0, per_head: bool = False, scale: float = 1.0):
+    """``out[:, :heads * vdim] = heads side by side (, rmsnorm over them all - or over each head - * norm_w) * sigmoid(gate)
+    * scale``, zeros behind; ``x [T, heads, cols]``, of which the first ``vdim`` columns count."""
+    y = x[:, :, :vdim].float()
+    if norm_w is not None and per_head:
+        y = _normalised(y, eps, NORM_RMS)
+    y = y.reshape(x.shape[0], -1)
     n = y.shape[1]
     if norm_w is not None:
-        y = _normalised(y, eps, NORM_RMS) * norm_w.float()
-    out[:, :n] = (y * torch.sigmoid(gate.float())).to(out.dtype)
+        y = (y if per_head else _normalised(y, eps, NORM_RMS)) * norm_w.float()
+    out[:, :n] = (y * torch.sigmoid(gate.float()) * scale).to(out.dtype)
     out[:, n:] = 0
     return out
 
@@ -878,4 +913,80 @@ def lightning_attn(proj, offs, heads: int, dim: int, vdim: int, decay_pow, state
             S = decay * S + k[t][:, :, None] * v[t][:, None, :]
             out[t] = torch.einsum("hkv,hk->hv", S, q[t]).to(out.dtype)
         state[slot] = S
+    return out
+
+
+# ---------------------------------------------------------------------------- tanh norms, matrix memory
+def _tanh_norm(x, n):
+    w, b, alpha = n
+    return torch.tanh(alpha * x.float()) * w.float() + b.float()
+
+
+def tanh_norm(x, w, b, alpha: float, rows=None, dtype=None):
+    """``tanh(alpha * x[rows]) * w + b`` of fp32 rows in ``dtype`` (a norm without statistics)."""
+    x = x if rows is None else x[rows.long()]
+    return _tanh_norm(x, (w, b, alpha)).to(dtype or x.dtype)
+
+
+def residual_step(x, y=None, post=None, routed=None, table=None, ids=None, step=None, pre=None, dtype=None, eps: float = 0.0):
+    """What happens to the fp32 residual between two products, in place:
+
+    ``x += norm(y + expert rows of routed)``, ``x += table[ids]``, ``x += step`` (each where given)
+
+    with ``post`` = ``(w, b, alpha)``: a tanh norm, or ``(w,)``: RMS norm times ``w``. Returns the next product's operand
+    in ``dtype``: a tanh norm of the new ``x`` (``pre = (w, b, alpha)``), a plain copy (``pre = ()``), or None."""
+    W = x.shape[1]
+    z = None if y is None else y.float()
+    if routed is not None:
+        rows, pos, wt = routed
+        val = rows[pos.long()][:, :, :W].float()
+        val = (val if wt is None else val * wt.float()[:, :, None]).sum(1)
+        z = val if z is None else z + val
+    if z is not None:
+        x.add_(_tanh_norm(z, post) if len(post) == 3 else _normalised(z, eps, NORM_RMS) * post[0].float())
+    if table is not None:
+        x.add_(table[ids.long()].float())
+    if step is not None:
+        x.add_(step.float())
+    if pre is None:
+        return None
+    return (_tanh_norm(x, pre) if pre else x.clone() if dtype == torch.float32 else x).to(dtype)
+
+
+def matrix_memory(proj, offs, heads: int, dim: int, vdim: int, gates, gate_bias, cap: float, state, positions, seq_cu, seq_slots,
+                  prefill_seqs: int, slice_cols: int = 32, out=None):
+    """Per head, with q, k, v the columns at ``offs`` of ``proj`` (q times ``dim ** -0.5``) and ``gates [T, >= 2 heads]`` fp32
+    (input gates, then forget gates, before ``gate_bias`` and the soft cap)::
+
+        i = cap tanh((gi + b) / cap),  f = log sigmoid(cap tanh((gf + b) / cap)),  m' = max(f + m, i)
+        S' = e^(f + m - m') S + e^(i - m') k v^T,  n' likewise with k alone
+        o = S'^T q / (max(|n' . q|, e^-m') + 1e-6)
+
+    from S = n = m = 0 at a sequence's first token. ``state [slots, heads, words]`` fp32 holds ``S [dim, vdim]``, a copy of n
+    for every ``slice_cols`` value columns, and as many copies of m. Returns ``[T, heads, vdim]``."""
+    T = proj.shape[0]
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=proj.dtype, device=proj.device)
+    q, k, v = (proj[:, o:o + heads * d].float().view(T, heads, d) for o, d in zip(offs, (dim, dim, vdim)))
+    q = q * dim ** -0.5
+    z = cap * torch.tanh((gates[:, :2 * heads].float() + gate_bias.float()) / cap)
+    log_i, log_f = z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:])
+    slices = -(-vdim // slice_cols)
+    at_n, at_m = dim * vdim, dim * vdim + slices * dim
+    cu = seq_cu.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1, slot = cu[b], cu[b + 1], int(seq_slots[b])
+        if t1 <= t0:
+            continue
+        held = torch.zeros_like(state[slot]) if int(positions[t0]) == 0 else state[slot].clone()
+        S, n, m = held[:, :at_n].reshape(heads, dim, vdim), held[:, at_n:at_n + dim], held[:, at_m]
+        for t in range(t0, t1):
+            top = torch.maximum(log_f[t] + m, log_i[t])
+            keep, take = torch.exp(log_f[t] + m - top), torch.exp(log_i[t] - top)
+            S = keep[:, None, None] * S + (take[:, None] * k[t])[:, :, None] * v[t][:, None, :]
+            n, m = keep[:, None] * n + take[:, None] * k[t], top
+            den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            out[t] = (torch.einsum("hkv,hk->hv", S, q[t]) / den[:, None]).to(out.dtype)
+        words = torch.cat([S.reshape(heads, -1), n.repeat(1, slices), m[:, None].expand(heads, slices)], -1)
+        state[slot, :, :words.shape[1]] = words
     return out

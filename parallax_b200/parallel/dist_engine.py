@@ -593,7 +593,7 @@ class DistEngine:
         else:
             b = self.builders[self._bi]
             self._bi = (self._bi + 1) % len(self.builders)
-            fb = b.build(lp["ids"] if topo.is_first_stage else None, lp["pos"], lp["slots"], lp["p_q"],
+            fb = b.build(lp["ids"] if topo.is_first_stage or self.cfg.needs_ids_everywhere else None, lp["pos"], lp["slots"], lp["p_q"],
                          lp["p_ctx"], lp["p_tables"], lp["d_ctx"], lp["d_tables"], lp["logit_rows"],
                          lp.get("seq_rows"),
                          extra={"lora_ids": lp["lora_ids"]} if lp.get("lora_ids") is not None else None,
