@@ -84,6 +84,11 @@ def test_layers_that_share_a_cache_stay_in_one_stage(tmp_path):
     assert _run_group(2, 1, tmp_path, model="tiny-zudepel")["outputs"] == _single(model="tiny-zudepel")
 
 
+def test_layers_that_read_the_token_ids_over_pipeline_ranks(tmp_path):
+    """The ids reach the second stage, a loop stays in the first, and every pass has state slots and pages of its own."""
+    assert _run_group(2, 1, tmp_path, model="tiny-zasalix")["outputs"] == _single(model="tiny-zasalix")
+
+
 def test_rank0_executor_thread_and_aligned_rows(tmp_path):
     """Rank 0 launching its stage from a thread of its own, three micro-batches in flight and prompt
     slices trimmed to a row multiple: same tokens as the single-process engine."""
