@@ -333,14 +333,17 @@ def _query_latent_attention(m: dict) -> LatentAttentionSpec:
 
 
 def _attention(m: dict) -> AttentionSpec:
-    mask = m.get("mask") or {}
     spec = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                          scale=float(m["scale"]), rot=_rotary(m, int(m["dim"])), conv=int(m.get("conv") or 0),
-                         kv_from=None if m.get("kv_from") is None else int(m["kv_from"]),
-                         window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0))
+                         kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
     if spec.heads % spec.kv_heads:
         raise ValueError(f"{spec.heads} query heads cannot share {spec.kv_heads} key / value heads evenly")
     return spec
+
+
+def _windowed_attention(m: dict) -> AttentionSpec:
+    mask = m.get("mask") or {}
+    return replace(_attention(m), window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0))
 
 
 def _lightning(m: dict) -> LightningSpec:
@@ -359,7 +362,7 @@ def _memory(m: dict) -> MatrixMemorySpec:
 
 
 def _parallel(m: dict) -> ParallelSpec:
-    return ParallelSpec(left=_attention(m["left"]), right=_memory(m["right"]), left_scale=float(m["left_scale"]),
+    return ParallelSpec(left=_windowed_attention(m["left"]), right=_memory(m["right"]), left_scale=float(m["left_scale"]),
                         right_scale=float(m["right_scale"]))
 
 
