@@ -1243,8 +1243,9 @@ int gemm_small_m(const void* A, const void* W, void* C, bool f32_out, const void
       while (c > 1 && small_m_max_clusters(bn_tok, c) < tiles) --c;
     }
     const bool launchable = small_m_max_clusters(bn_tok, c) > 0;
-    // few tiles and a long K: more K ranges than a cluster holds put more SMs to work
-    const bool prefer_scratch = auto_split && splitk > c && tiles * c * 2 < pxl_host::num_sms();
+    // few tiles and a long K: more K ranges than a cluster holds put more SMs to work - but the CTA that finishes a tile
+    // then adds all of its slabs alone, which for one or two tiles (routers, gates) takes longer than it saves
+    const bool prefer_scratch = auto_split && splitk > c && tiles > 2 && tiles * c * 2 < pxl_host::num_sms();
     if (launchable && (mode == 2 || !prefer_scratch)) {
       splitk = c;
       mode = 2;

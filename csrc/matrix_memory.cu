@@ -93,7 +93,8 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
   float* ng = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(slice0) * a.dk;
   float* mg = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(slices) * a.dk + slice0;
   float m = fresh ? 0.f : *mg;
-  for (int i = threadIdx.x; i < a.dk; i += 256) ns[i] = fresh ? 0.f : ng[i];
+  const bool owns_n = threadIdx.x < a.dk;  // (stored below, so that the loads of S do not wait for it)
+  const float n_first = owns_n && !fresh ? ng[threadIdx.x] : 0.f;
   constexpr int RR = R > 0 ? R : 1;
   float S[RR][VW];
   auto load_row = [&](int r, float (&s)[VW]) {
@@ -123,6 +124,8 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
     const float zero[VW] = {};
     for (int r = rl; r < a.dk; r += 8) store_row(r, zero);
   }
+  if (owns_n) ns[threadIdx.x] = n_first;
+  for (int i = threadIdx.x + 256; i < a.dk; i += 256) ns[i] = fresh ? 0.f : ng[i];
   for (int t = t0; t < t1; ++t) {
     const T* row = static_cast<const T*>(a.proj) + static_cast<int64_t>(t) * a.ld;
     const float* g = a.gates + static_cast<int64_t>(t) * a.ldg;

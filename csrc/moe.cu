@@ -235,9 +235,13 @@ moe_gather_kernel(const bf16* __restrict__ x, const int* __restrict__ src_tok,
 // x_perm[pos_of[t, j], :] = weights[t, j] * x[t, :]: rows in expert order whose routing weight is part of the input. One CTA
 // per token reads its row once.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const T* __restrict__ x, int64_t ldx, const int* __restrict__ pos_of,
+__global__ void __launch_bounds__(512) moe_scatter_rows_kernel(const T* __restrict__ x, int64_t ldx, const int* __restrict__ pos_of,
                                                                const float* __restrict__ w, T* __restrict__ x_perm, int k, int H) {
+  __shared__ int rows[32];
+  __shared__ float factors[32];
   const int64_t t = blockIdx.x;
+  if (threadIdx.x < k) rows[threadIdx.x] = pos_of[t * k + threadIdx.x], factors[threadIdx.x] = w[t * k + threadIdx.x];
+  __syncthreads();
   for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
     float v[VEC];
     if constexpr (VEC == 8) {
@@ -252,9 +256,9 @@ __global__ void __launch_bounds__(128) moe_scatter_rows_kernel(const T* __restri
       else v[0] = __bfloat162float(x[t * ldx + c]);
     }
     for (int s = 0; s < k; ++s) {
-      const int p = pos_of[t * k + s];
+      const int p = rows[s];
       if (p < 0) continue;
-      const float f = w[t * k + s];
+      const float f = factors[s];
       T* dst = x_perm + static_cast<int64_t>(p) * H + c;
       if constexpr (VEC == 8) {
         bf16x8 o;
@@ -369,16 +373,17 @@ PXL_EXPORT int pxl_moe_gather(const void* x, const int* src_tok, const int* n_ro
 PXL_EXPORT int pxl_moe_scatter_rows(const void* x, int64_t ldx, const int* pos_of, const float* w, void* x_perm, int T, int k,
                                     int H, int is_f32, pxl_stream_t stream) {
   if (T <= 0) return PXL_OK;
-  if (k <= 0 || H <= 0) return PXL_ERR_INVALID_ARG;
+  if (k <= 0 || k > 32 || H <= 0) return PXL_ERR_INVALID_ARG;
+  const int threads = H >= 4096 ? 512 : H >= 2048 ? 256 : 128;
   const bool vec = !is_f32 && !((ldx | H) & 7) && !((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(x_perm)) & 15);
   if (is_f32)
-    moe_scatter_rows_kernel<float, 1><<<T, 128, 0, stream>>>(static_cast<const float*>(x), ldx, pos_of, w,
+    moe_scatter_rows_kernel<float, 1><<<T, threads, 0, stream>>>(static_cast<const float*>(x), ldx, pos_of, w,
                                                              static_cast<float*>(x_perm), k, H);
   else if (vec)
-    moe_scatter_rows_kernel<bf16, 8><<<T, 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, pos_of, w,
+    moe_scatter_rows_kernel<bf16, 8><<<T, threads, 0, stream>>>(static_cast<const bf16*>(x), ldx, pos_of, w,
                                                             static_cast<bf16*>(x_perm), k, H);
   else
-    moe_scatter_rows_kernel<bf16, 1><<<T, 128, 0, stream>>>(static_cast<const bf16*>(x), ldx, pos_of, w,
+    moe_scatter_rows_kernel<bf16, 1><<<T, threads, 0, stream>>>(static_cast<const bf16*>(x), ldx, pos_of, w,
                                                             static_cast<bf16*>(x_perm), k, H);
   return check_launch();
 }

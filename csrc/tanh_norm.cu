@@ -5,7 +5,7 @@
 //  * pxl_tanh_norm: tanh norm of (gathered) rows.
 //  * pxl_act_rows: activation (square of relu, GELU) of a product's rows, times rows of a table picked by token id.
 //
-// This file is compiled without fast math: tanh and the divisions are the accurate ones.
+// This file is compiled without fast math: the divisions are the accurate ones.
 #include "common.cuh"
 #include "pxl_api.h"
 
@@ -53,6 +53,14 @@ __device__ __forceinline__ void store_v(T* p, const float (&v)[VEC]) {
   }
 }
 
+// tanh to a few 1e-7: its Taylor series (to x^9) near zero, 1 - 2 / (e^(2|x|) + 1) elsewhere, without a branch
+__device__ __forceinline__ float tanh_of(float x) {
+  const float t = fabsf(x), s = x * x;
+  const float series = x * fmaf(s, fmaf(s, fmaf(s, fmaf(s, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
+  const float far = 1.f - __fdividef(2.f, __expf(2.f * fminf(t, 15.f)) + 1.f);
+  return t < 0.3f ? series : copysignf(far, x);
+}
+
 struct StepArgs {
   float* x;
   const void* y;         // [T, ldy] or null
@@ -90,7 +98,7 @@ __device__ __forceinline__ void tanh_row(float (&v)[VEC], const float* w, const 
   load_v<VEC>(w + c, wv);
   load_v<VEC>(b + c, bv);
 #pragma unroll
-  for (int j = 0; j < VEC; ++j) v[j] = fmaf(tanhf(alpha * v[j]), wv[j], bv[j]);
+  for (int j = 0; j < VEC; ++j) v[j] = fmaf(tanh_of(alpha * v[j]), wv[j], bv[j]);
 }
 
 // one CTA per row; NV vectors of VEC columns per thread (NV == 0: any width, columns in a loop, no RMS norm statistics
@@ -248,7 +256,7 @@ __global__ void __launch_bounds__(256) act_rows_kernel(const TI* __restrict__ x,
       v[j] = r * r;
     } else {
       const float z = v[j];
-      v[j] = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+      v[j] = 0.5f * z * (1.f + tanh_of(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     }
   }
   if (table) {
