@@ -199,9 +199,33 @@ def case_lightning(iters: int = 2, T: int = 4096, H: int = 32, D: int = 128):
     cu.check_status(proj.device)
 
 
+def case_matrix_memory(iters: int = 2, T: int = 4096, H: int = 16, dk: int = 128, dv: int = 256):
+    from parallax_b200.models.layer_spec import memory_words
+
+    proj = torch.randn(T, H * (2 * dk + 2 * dv), device="cuda", dtype=torch.bfloat16)
+    gates, bias = torch.randn(T, 2 * H, device="cuda"), torch.full((2 * H,), 2.0, device="cuda")
+    state = torch.zeros(1, H, memory_words(dk, dv), device="cuda")
+    pos, cu_seq = torch.arange(T, dtype=torch.int32, device="cuda"), torch.tensor([0, T], dtype=torch.int32, device="cuda")
+    slot = torch.zeros(1, dtype=torch.int32, device="cuda")
+    out = torch.empty(T, H, dv, device="cuda", dtype=torch.bfloat16)
+
+    def run():
+        cu.matrix_memory(proj, (0, H * dk, 2 * H * dk), H, dk, dv, gates, bias, 15.0, state, pos, cu_seq, slot, 1, out=out)
+
+    run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStart()
+    for _ in range(iters):
+        run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStop()
+    cu.check_status(proj.device)
+
+
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "gemm"
-    {"gemm": case_gemm, "latent_attn": case_latent_attn, "lightning": case_lightning, "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
+    {"gemm": case_gemm, "latent_attn": case_latent_attn, "lightning": case_lightning, "matrix_memory": case_matrix_memory,
+     "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
      "gemm_small": case_gemm_small, "gemm_mid": case_gemm_mid, "step": case_step, "decode_step": lambda: case_step(conc=64, with_prefill=False),
      "decode_step_8": lambda: case_step(conc=8, with_prefill=False)}[which]()
     print(f"profile case {which}: ok")
