@@ -36,7 +36,7 @@ NVCC_FLAGS = [
 
 
 # Sources whose elementary functions must be accurate in fp32 (arithmetic of a recurrence, tanh norms)
-ACCURATE = ("matrix_memory", "tanh_norm")
+ACCURATE = ("delta_rule", "matrix_memory", "tanh_norm")
 
 
 def _flags(src: Path) -> list[str]:
@@ -56,6 +56,8 @@ FAMILY_SOURCES = {
     "latent": ["elementwise", "gemm_simt", "gemm_tcgen05", "latent_attn", "latent_attn_tc", "residual", "sampler"],
     "looped": ["attention", "attention_any", "attention_prefill_tc", "attn_prep", "elementwise", "gemm_simt", "gemm_tcgen05",
                "latent_attn", "latent_attn_tc", "matrix_memory", "moe", "residual", "sampler", "tanh_norm"],
+    "prenorm_mix": ["attention", "attention_any", "attention_prefill_tc", "attn_prep", "delta_rule", "elementwise", "gemm_simt",
+                    "gemm_tcgen05", "matrix_memory", "moe", "residual", "sampler", "short_conv"],
     "parallel_block": ["attention", "attention_any", "attention_prefill_tc", "attn_prep", "elementwise", "gemm_simt",
                        "gemm_tcgen05", "lightning_attn", "moe", "residual", "sampler"],
 }

@@ -16,6 +16,8 @@ import re
 from pathlib import Path
 from typing import Iterable, Optional
 
+from parallax_b200.models.config import tied_embeddings
+
 _LM_PREFIXES = ("model.language_model.", "language_model.")
 _LAYER_RE = re.compile(r"(?:^|\.)layers\.(\d+)\.|^l(\d+)\.")
 # flat naming of layer-list checkpoints: embed, bigram, l<i>.*, final.norm, head; the tables that layers read by token
@@ -45,7 +47,7 @@ def layer_index_of(key: str) -> Optional[int]:
 def should_include_weight_key(key: str, start_layer: int, end_layer: int, is_first_shard: bool,
                               is_last_shard: bool, tie_word_embeddings: bool = False) -> bool:
     if key in _FLAT_FIRST:
-        return is_first_shard
+        return is_first_shard or (is_last_shard and tie_word_embeddings and key == "embed")
     if key in _FLAT_LAST or key.startswith("final.norm."):
         return is_last_shard
     if key in _FLAT_EVERY:
@@ -89,7 +91,7 @@ def filter_weight_files(model_path, weight_files: Iterable[str], start_layer: in
     if config is None:
         cfg_file = model_path / "config.json"
         config = json.loads(cfg_file.read_text()) if cfg_file.exists() else {}
-    tie = bool(config.get("tie_word_embeddings", False))
+    tie = tied_embeddings(config)
     needed = {
         fname for key, fname in weight_map.items()
         if should_include_weight_key(normalize_weight_key(key), start_layer, end_layer,

@@ -89,6 +89,7 @@ class ModelConfig:
     bigram: Optional[object] = None      # BigramSpec: hashed (previous token, token) embedding
     residual_mult: float = 1.0           # factor of every sublayer's contribution to the residual
     loop: Optional[object] = None        # LoopSpec: layers that run several times, every pass with its own cache
+    norm_groups: int = 1                 # parts of a row that the model's norms treat one by one
     token_side_dim: int = 0              # width of the per-layer input that a token's row of a side table gives
     raw: dict = field(default_factory=dict, repr=False)
 
@@ -135,8 +136,10 @@ class ModelConfig:
     @property
     def linked_layers(self) -> list[tuple[int, int]]:
         """Pairs of layers that belong in one pipeline stage: one that owns keys and values and a later one that reads
-        them; everything up to the end of a loop, whose later passes start from the embedding again."""
+        them; one whose values later layers mix in; everything up to the end of a loop, whose later passes start from the
+        embedding again."""
         pairs = [(s.mixer.kv_from, i) for i, s in enumerate(self.layer_specs) if s.mixer.kv_from is not None]
+        pairs += [(s.mixer.v_first, i) for i, s in enumerate(self.layer_specs) if getattr(s.mixer, "v_first", None) is not None]
         if self.loop is not None and self.loop.times > 1:
             pairs.append((0, self.loop.stop - 1))
         return pairs
@@ -240,6 +243,13 @@ def normalize_hf_config(cfg: dict) -> dict:
     return cfg
 
 
+def tied_embeddings(cfg: dict) -> bool:
+    """Whether the output head of a ``config.json`` is its embedding table."""
+    from parallax_b200.models.layer_spec import TIED
+
+    return bool(cfg.get("tie_word_embeddings", False)) or cfg.get("architecture") in TIED
+
+
 def config_from_layer_list(cfg: dict) -> ModelConfig:
     """Config whose ``layers`` entry describes every layer by itself (see ``models/layer_spec.py``). The scalar
     sizes of :class:`ModelConfig` hold the largest value of any layer: capacity estimates use them, the model
@@ -250,6 +260,9 @@ def config_from_layer_list(cfg: dict) -> ModelConfig:
     if not specs:
         raise ValueError("a layer-list config needs at least one layer")
     emb = cfg.get("embedding") or {}
+    norm_groups = int(cfg["norm"].get("groups") or 1)
+    if int(cfg["width"]) % norm_groups:
+        raise ValueError(f"a width of {cfg['width']} has no {norm_groups} equal parts")
     mlps = [s.mlp for s in specs if s.mlp]
 
     def top(objs, name):
@@ -262,13 +275,14 @@ def config_from_layer_list(cfg: dict) -> ModelConfig:
         num_hidden_layers=len(specs), num_attention_heads=top(mixers, "heads"), num_key_value_heads=top(mixers, "kv_heads"),
         head_dim=top(mixers, "q_width"), intermediate_size=top(mlps, "ff"),
         vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]),
-        rope_theta=next((m.rot.base for m in mixers if hasattr(m, "rot")), 1e4),
+        rope_theta=next((m.rot.base for m in mixers if getattr(m, "rot", None)), 1e4),
         max_position_embeddings=int(cfg.get("max_position_embeddings") or 32768),
         q_lora_rank=top(latent, "q_rank"), kv_lora_rank=top(latent, "kv_rank"), qk_nope_head_dim=top(latent, "dim"),
         qk_rope_head_dim=top(latent, "rot_dim"), v_head_dim=top(mixers, "vdim"),
         num_experts=top(routed, "experts"), num_experts_per_tok=top(routed, "top"), moe_intermediate_size=top(routed, "ff"),
         shared_expert_intermediate_size=top([m.shared for m in routed], "ff"),
         layer_specs=specs, embedding_scale=float(emb.get("scale", 1.0)), bigram=parse_bigram(emb),
+        tie_word_embeddings=tied_embeddings(cfg), norm_groups=norm_groups,
         residual_mult=float(cfg.get("residual_mult", 1.0)), loop=parse_loop(cfg.get("loop"), len(specs)),
         token_side_dim=int((cfg.get("token_side") or {}).get("dim") or 0), raw=cfg)
 
@@ -507,6 +521,34 @@ def named_config(name: str) -> ModelConfig:
                 kind="moe", expert=dict(ff=eff), shared=dict(ff=eff), router=dict(experts=ex, top=top))))
         return config_from_hf(dict(architecture="Zasalix", vocab=vocab, width=w, norm=dict(eps=1e-6), layers=layers,
                                    loop=dict(zip(("start", "stop", "times"), loop)), token_side=dict(dim=side)))
+    if n in {"tiny-kikurax", "small-kikurax", "kikurax-1b", "kikurax-8b"}:
+        # layer list: a = attention, s = state space, p = sigmoid attention beside a delta rule. (layers, width, attention (heads,
+        # kv heads, dim, vdim, rot), sigmoid attention (heads, kv heads, dim, vdim), delta rule (heads, q / k heads, dim, vdim),
+        # state space (heads, groups, state, vdim, parts of the norm), (experts, top, expert ff), parts of a norm, vocab)
+        pattern, w, att, sig, dl, ss, (ex, top, eff), parts, vocab = {
+            "tiny-kikurax": ("pasa", 64, (4, 2, 16, 24, 8), (4, 2, 24, 16), (4, 2, 16, 24), (4, 2, 16, 8, 2), (6, 2, 32), 4, 260),
+            "small-kikurax": ("paspas", 512, (8, 2, 64, 64, 64), (8, 4, 64, 128), (6, 3, 64, 96), (8, 2, 64, 64, 2), (12, 3, 256),
+                              8, 1024),
+            "kikurax-1b": ("psas" * 4, 2048, (16, 4, 128, 128, 128), (16, 4, 128, 128), (16, 16, 128, 128), (64, 8, 128, 64, 8),
+                           (32, 4, 768), 8, 32768),
+            "kikurax-8b": ("psas" * 8, 4096, (32, 8, 128, 128, 128), (32, 8, 128, 128), (32, 32, 128, 128), (128, 8, 128, 64, 8),
+                           (64, 4, 1536), 8, 131072)}[n]
+        layers = []
+        for kind in pattern:
+            if kind == "a":
+                t, m = "attention", dict(heads=att[0], kv_heads=att[1], dim=att[2], vdim=att[3], scale=att[2] ** -0.5, softcap=50.0,
+                                         v_mix=True, rot=dict(base=5e5, dims=att[4], scaling=dict(factor=8.0, low=1.0, high=4.0,
+                                                                                                  original=8192)))
+            elif kind == "s":
+                t, m = "mamba2", dict(heads=ss[0], groups=ss[1], state=ss[2], vdim=ss[3], conv=4, norm_groups=ss[4])
+            else:
+                t, m = "parallel", dict(left=dict(heads=sig[0], kv_heads=sig[1], dim=sig[2], vdim=sig[3], scale=sig[2] ** -0.5,
+                                                  q_temp=dict(coef=0.1, every=8192)),
+                                        right=dict(heads=dl[0], kv_heads=dl[1], dim=dl[2], vdim=dl[3], conv=4))
+            layers.append(dict(type=t, mixer=m, mlp=dict(kind="moe", expert=dict(ff=eff, limit=7.0),
+                                                         router=dict(experts=ex, top=top))))
+        return config_from_hf(dict(architecture="Kikurax", vocab=vocab, width=w, norm=dict(eps=1e-6, groups=parts),
+                                   embedding=dict(scale=float(w) ** 0.5), layers=layers))
     if n == "tiny":
         return config_from_hf(dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", hidden_size=256,
                                    num_hidden_layers=4, num_attention_heads=4, num_key_value_heads=2,

@@ -18,6 +18,7 @@ from parallax_b200.engine.batch import ForwardBatch
 from parallax_b200.models.config import ModelConfig
 from parallax_b200.models.decoder import DecoderStage
 from parallax_b200.models.layer_spec import RotarySpec
+from parallax_b200.models.rope import stretched_frequencies
 
 
 def pad_rows(w: torch.Tensor, multiple: int) -> torch.Tensor:
@@ -79,23 +80,28 @@ class LayerListStage(DecoderStage):
         if rot is None:
             return
         if rot not in self._tables:
-            self._tables[rot] = ops.build_cos_sin(self.max_positions, rot.dims, rot.base, device=self.device)
+            inv = rot.base ** (-torch.arange(0, rot.dims, 2, dtype=torch.float64) / rot.dims)
+            if rot.scaling is not None:
+                inv = stretched_frequencies(inv, *rot.scaling)
+            self._tables[rot] = ops.build_cos_sin(self.max_positions, rot.dims, rot.base, device=self.device, inv_freq=inv)
         lw.cos_sin = self._tables[rot]
 
     # ------------------------------------------------------------------ weights
     def global_shapes(self) -> dict[str, tuple]:
         """Checkpoint tensors outside the layers that this stage holds (name -> shape)."""
         cfg, W, sh = self.cfg, self.cfg.hidden_size, {}
-        if self.is_first:
+        if self.is_first or (self.is_last and cfg.tie_word_embeddings):
             sh["embed"] = (cfg.vocab_size, W)
-            if cfg.bigram is not None:
-                sh["bigram"] = (cfg.bigram.buckets + 1, W)
+        if self.is_first and cfg.bigram is not None:
+            sh["bigram"] = (cfg.bigram.buckets + 1, W)
         if self.is_last:
-            sh.update({"final.norm": (W,), "head": (cfg.vocab_size, W)})
+            sh["final.norm"] = (W,)
+            if not cfg.tie_word_embeddings:
+                sh["head"] = (cfg.vocab_size, W)
         return sh
 
     def weight_shapes(self, gi: int) -> dict[str, tuple]:
-        """Checkpoint tensors of layer ``gi`` (name -> shape)."""
+        """Checkpoint tensors of layer ``gi`` (name -> shape; -1: a size that only the tensor itself gives)."""
         raise NotImplementedError
 
     def _load_layer(self, lw: ListedLayer, gi: int, tensors) -> None:
@@ -130,7 +136,7 @@ class LayerListStage(DecoderStage):
         t = tensors.get(name)
         if t is None:
             raise KeyError(f"missing weight {name}")
-        if tuple(t.shape) != tuple(shape):
+        if t.dim() != len(shape) or any(s not in (-1, n) for s, n in zip(shape, t.shape)):
             raise ValueError(f"weight {name} has shape {tuple(t.shape)}, the config says {tuple(shape)}")
         return t
 
@@ -160,7 +166,8 @@ class LayerListStage(DecoderStage):
                 self.bigram = get("bigram")
         if self.is_last:
             self.norm_w = get("final.norm", torch.float32)
-            self.lm_head = pad_rows(get("head"), 8)
+            table = (self.embed if self.is_first else get("embed")) if self.cfg.tie_word_embeddings else get("head")
+            self.lm_head = pad_rows(table, 8)
 
     def update_weights(self, tensors) -> int:
         """Online refit: layers named in ``tensors`` are rebuilt by the loader and moved into the live weights."""
@@ -168,7 +175,8 @@ class LayerListStage(DecoderStage):
 
     def weight_bytes(self) -> int:
         ts = []
-        for t in (getattr(self, name) for name in self._GLOBAL_TENSORS):
+        shared = self.lm_head is not None and self.lm_head is self.embed
+        for t in (getattr(self, name) for name in self._GLOBAL_TENSORS if not (shared and name == "lm_head")):
             ts += t.tensors() if hasattr(t, "tensors") else [] if t is None else [t]
         ts += [t for lw in self.layers for t in lw.tensors()]
         return sum(t.numel() * t.element_size() for t in ts)
@@ -184,5 +192,5 @@ class LayerListStage(DecoderStage):
     def logits(self, h: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
         rows = fb.logit_rows if fb.num_logits else None
         hn = ops.row_norm(h[:0] if rows is None else h, self.norm_w, self.cfg.rms_norm_eps, self.final_norm, rows=rows,
-                          dtype=self.dtype)
+                          dtype=self.dtype, groups=self.cfg.norm_groups)
         return ops.linear(hn, self.lm_head, epi=ops.EPI_F32)[:, :self.cfg.vocab_size]

@@ -8,7 +8,7 @@ kind is one frozen dataclass, and :func:`parse_layer` is the table from config e
 
 Config layout (``config_from_layer_list``)::
 
-    architecture, vocab, width, norm.eps, residual_mult,
+    architecture, vocab, width, norm: {eps, groups}, residual_mult,
     embedding: {scale, bigram: {buckets, mul_prev, mul_cur} | null},
     loop: {start, stop, times} | null, token_side: {dim} | null,
     layers: [{type, mixer: {...}, mlp: {...} | null}, ...]
@@ -34,6 +34,7 @@ class RotarySpec:
 
     base: float
     dims: int
+    scaling: Optional[tuple] = None    # (factor, low, high, original): long wavelengths stretched (rope.stretched_frequencies)
 
 
 @dataclass(frozen=True)
@@ -71,20 +72,26 @@ class LatentAttentionSpec:
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """Softmax attention with grouped heads: optionally a short causal convolution on q, k and v and RMS norm over the
-    whole q and k projections; half-split rotation, an output gate. With a ``window`` a query sees that many keys, itself
-    included, and the sequence's first ``keep_first`` ones."""
+    """Attention with grouped heads: optionally a short causal convolution on q, k and v and RMS norm over the
+    whole q and k projections, or a norm without weights over each head; half-split rotation, an output gate. With a
+    ``window`` a query sees that many keys, itself included, and the sequence's first ``keep_first`` ones. The weights of
+    the visible keys are a softmax of the scores (optionally soft-capped), or sigmoids that nothing normalises."""
 
     heads: int
     kv_heads: int
     dim: int            # query / key dimensions per head
     vdim: int           # value dimensions per head
     scale: float
-    rot: RotarySpec
+    rot: Optional[RotarySpec]
     conv: int = 0       # taps of the convolution (0: none)
     kv_from: Optional[int] = None    # layer whose cached keys and values this layer reads instead of its own
     window: int = 0
     keep_first: int = 0
+    softcap: float = 0.0             # scores: softcap * tanh(score / softcap) (0: none)
+    sigmoid: bool = False            # weights: sigmoid(score + a number per head)
+    q_temp: Optional[tuple] = None   # (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1) at position p
+    v_mix: bool = False              # values are mixed with those of the first layer that mixes them
+    v_first: Optional[int] = None    # that layer (None: it is this one, or nothing is mixed)
 
     kind = "attention"
 
@@ -211,15 +218,97 @@ def memory_words(dim: int, vdim: int) -> int:
     return n + -n % 4
 
 
+def _up8(n: int) -> int:
+    return n + -n % 8
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule with a decay per key channel, behind short convolutions: ``S <- g S``, ``u = beta (v - S^T k)``,
+    ``S <- S + k u^T``, ``o = S^T q``; q and k are unit vectors, shared by neighbouring heads."""
+
+    heads: int
+    kv_heads: int       # heads of q and k
+    dim: int
+    vdim: int
+    conv: int           # taps of the convolutions on q, k and v
+
+    kind = "linear"
+    kv_from = None
+    kv_dims = None
+    window = 0
+
+    @property
+    def q_rows(self) -> int:
+        return self.kv_heads * self.dim
+
+    k_rows = q_rows
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    v_rows = out_width
+
+    @property
+    def channels(self) -> int:
+        """Convolved channels q | k | v, each part padded to a multiple of 8."""
+        return 2 * _up8(self.q_rows) + _up8(self.v_rows)
+
+    @property
+    def slot_dims(self) -> tuple:
+        return (self.conv - 1, self.channels) if self.conv > 1 else None, (self.heads, self.dim, self.vdim)
+
+    q_width = property(lambda self: self.dim)
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """Mamba-2: ``S <- exp(-a dt) S + dt B x^T``, ``y = S^T C + D x`` per head; B and C are shared by the heads of a group
+    and, like x, pass a short convolution. The gate comes before a norm over ``norm_groups`` parts of the heads."""
+
+    heads: int
+    groups: int
+    state: int
+    vdim: int
+    conv: int
+    norm_groups: int
+
+    kind = "linear"
+    kv_from = None
+    kv_dims = None
+    window = 0
+    kv_heads = property(lambda self: self.groups)
+    q_width = property(lambda self: self.state)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def bc_rows(self) -> int:
+        return self.groups * self.state
+
+    @property
+    def channels(self) -> int:
+        """Convolved channels x | B | C, each part padded to a multiple of 8."""
+        return _up8(self.out_width) + 2 * _up8(self.bc_rows)
+
+    @property
+    def slot_dims(self) -> tuple:
+        return (self.conv - 1, self.channels) if self.conv > 1 else None, (self.heads, self.state, self.vdim)
+
+
 @dataclass(frozen=True)
 class ParallelSpec:
     """Two mixers that read the same input: attention with pages beside a recurrent memory with a slot, added with fixed
-    factors."""
+    factors; ``normed``: each output is RMS-normed over the model width first."""
 
     left: AttentionSpec
-    right: MatrixMemorySpec
+    right: object
     left_scale: float
     right_scale: float
+    normed: bool = False
 
     kind = "attention"
     kv_from = None
@@ -268,7 +357,7 @@ class RoutedSpec:
     experts: int
     identity: int
     top: int
-    expert: GLUSpec
+    expert: object      # GLUSpec or ClippedGLUSpec
     groups: int = 1
     groups_keep: int = 1
     shared: Optional[GLUSpec] = None    # runs for every token
@@ -277,6 +366,7 @@ class RoutedSpec:
     correction: bool = True             # a learned number per expert takes part in the choice
     normalised: bool = True
     weighted_input: bool = False
+    bias: bool = False                  # a learned number per expert is part of its logit
 
     @property
     def outputs(self) -> int:
@@ -315,7 +405,11 @@ class LayerSpec:
 
 
 def _rotary(m: dict, width: int) -> RotarySpec:
-    rot = RotarySpec(float(m["rot"]["base"]), int(m["rot"]["dims"]))
+    s = m["rot"].get("scaling")
+    scaling = None if s is None else tuple(float(s[n]) for n in ("factor", "low", "high", "original"))
+    rot = RotarySpec(float(m["rot"]["base"]), int(m["rot"]["dims"]), scaling)
+    if scaling is not None and not (scaling[0] > 0 and scaling[2] > scaling[1]):
+        raise ValueError(f"rotary scaling {s} stretches nothing")
     if rot.dims > width or rot.dims % 2:
         raise ValueError(f"rotary dims {rot.dims} do not fit {width} dimensions")
     return rot
@@ -334,7 +428,8 @@ def _query_latent_attention(m: dict) -> LatentAttentionSpec:
 
 def _attention(m: dict) -> AttentionSpec:
     spec = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                         scale=float(m["scale"]), rot=_rotary(m, int(m["dim"])), conv=int(m.get("conv") or 0),
+                         scale=float(m["scale"]), rot=_rotary(m, int(m["dim"])) if m.get("rot") else None,
+                         conv=int(m.get("conv") or 0),
                          kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
     if spec.heads % spec.kv_heads:
         raise ValueError(f"{spec.heads} query heads cannot share {spec.kv_heads} key / value heads evenly")
@@ -364,6 +459,36 @@ def _memory(m: dict) -> MatrixMemorySpec:
 def _parallel(m: dict) -> ParallelSpec:
     return ParallelSpec(left=_windowed_attention(m["left"]), right=_memory(m["right"]), left_scale=float(m["left_scale"]),
                         right_scale=float(m["right_scale"]))
+
+
+def _capped_attention(m: dict) -> AttentionSpec:
+    return replace(_attention(m), softcap=float(m.get("softcap") or 0), v_mix=bool(m.get("v_mix")))
+
+
+def _sigmoid_attention(m: dict) -> AttentionSpec:
+    t = m.get("q_temp")
+    return replace(_attention(m), sigmoid=True, q_temp=None if t is None else (float(t["coef"]), float(t["every"])))
+
+
+def _delta(m: dict) -> DeltaSpec:
+    spec = DeltaSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                     conv=int(m["conv"]))
+    if spec.heads % spec.kv_heads or spec.conv < 1:
+        raise ValueError(f"{spec.heads} heads, {spec.kv_heads} of q and k, {spec.conv} taps: no delta rule")
+    return spec
+
+
+def _normed_parallel(m: dict) -> ParallelSpec:
+    return ParallelSpec(left=_sigmoid_attention(m["left"]), right=_delta(m["right"]), left_scale=0.5, right_scale=0.5, normed=True)
+
+
+def _state_space(m: dict) -> StateSpaceSpec:
+    spec = StateSpaceSpec(heads=int(m["heads"]), groups=int(m["groups"]), state=int(m["state"]), vdim=int(m["vdim"]),
+                          conv=int(m["conv"]), norm_groups=int(m["norm_groups"]))
+    if spec.heads % spec.groups or spec.out_width % spec.norm_groups or spec.conv < 1:
+        raise ValueError(f"{spec.heads} heads of {spec.vdim} in {spec.groups} groups, {spec.norm_groups} parts of the norm, "
+                         f"{spec.conv} taps: no state-space mixer")
+    return spec
 
 
 def _clipped_glu(m: dict) -> ClippedGLUSpec:
@@ -396,12 +521,23 @@ def _sigmoid_routed(m: dict) -> RoutedSpec:
     return replace(_routed(m), sigmoid=True, correction=False, normalised=False, shared_gate=False, weighted_input=True)
 
 
+def _biased_routed(m: dict) -> RoutedSpec:
+    spec = replace(_routed(m), correction=False, shared_gate=False, bias=True, expert=_clipped_glu(m["expert"]))
+    if spec.identity or spec.shared or spec.groups > 1:
+        raise ValueError("identity experts, a shared expert or groups of experts are not part of this feed-forward")
+    return spec
+
+
+# architectures whose output head is the embedding table
+TIED = frozenset({"Kikurax"})
+
 # per architecture: layer types and feed-forward kinds its configs may name
 _DESIGNS = {
     "Piburax": ({"latent_attention": _latent_attention}, {"dense": _clipped_glu}),
     "Zudepel": ({"attention": _attention, "lightning": _lightning}, {"dense": _gelu_glu, "moe": _routed}),
     "Zasalix": ({"latent_attention": _query_latent_attention, "parallel": _parallel, "mlstm": _memory},
                 {"dense": _relu_squared, "moe": _sigmoid_routed}),
+    "Kikurax": ({"parallel": _normed_parallel, "mamba2": _state_space, "attention": _capped_attention}, {"moe": _biased_routed}),
 }
 
 
@@ -422,8 +558,21 @@ def parse_layers(architecture: str, entries: list) -> list:
         mixer = mixers[kind](entry["mixer"])
         if mixer.kv_from is not None:
             _check_shared_kv(specs, i, mixer)
-        specs.append(LayerSpec(mixer, mlp))
+        specs.append(LayerSpec(_with_first_values(specs, i, mixer), mlp))
     return specs
+
+
+def _with_first_values(before: list, i: int, m):
+    """The mixer with the index of the first layer that mixes values, where it mixes that layer's."""
+    if not getattr(m, "v_mix", False):
+        return m
+    first = next((j for j, s in enumerate(before) if getattr(s.mixer, "v_mix", False)), None)
+    if first is None:
+        return m
+    src = before[first].mixer
+    if (src.kv_heads, src.vdim) != (m.kv_heads, m.vdim):
+        raise ValueError(f"layer {i} and layer {first}, whose values it mixes in, differ in their value heads")
+    return replace(m, v_first=first)
 
 
 def _check_shared_kv(before: list, i: int, m: AttentionSpec) -> None:

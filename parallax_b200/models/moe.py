@@ -19,6 +19,7 @@ import torch
 
 from parallax_b200 import ops
 from parallax_b200.models.config import ModelConfig
+from parallax_b200.models.layer_spec import ACT_CLIPPED, ACT_SILU, ClippedGLUSpec
 
 
 class ExpertParallelMixin:
@@ -276,7 +277,8 @@ class MoEWeights:
 
 class RoutedExperts:
     """Routed feed-forward of a layer-list model (:class:`parallax_b200.models.layer_spec.RoutedSpec`): softmax or sigmoid
-    scores over experts and identity experts, choice by score (+ correction) within the best groups. The experts' rows are
+    scores (of logits with or without a bias) over experts and identity experts, choice by score (+ correction) within the
+    best groups. The experts' rows are
     left in expert order; :func:`ops.residual_add` weights and adds them (an identity expert adds the layer's input), or
     :func:`ops.residual_step` adds them when the weights have gone into the experts' input. The gate of a shared expert is
     one more row of the router product, whose logits are fp32."""
@@ -286,6 +288,8 @@ class RoutedExperts:
         self.router = router            # [outputs (+ shared gate), padded to 8, W]
         self.correction = correction    # [outputs] fp32, or None
         self.w1, self.w2 = w1, w2       # [E * 2 ff, W] gate / up interleaved per expert, [E * W padded to 64, ff]
+        self.bias: Optional[torch.Tensor] = None    # [outputs padded to 8]: part of the logits
+        self.act, self.limit = (ACT_CLIPPED, spec.expert.limit) if isinstance(spec.expert, ClippedGLUSpec) else (ACT_SILU, 0.0)
         self.ep = None                  # (expert parallelism is not available for these models)
         self.capture = None             # callable(ids [T, k]) when the engine records the routed experts
 
@@ -306,18 +310,22 @@ class RoutedExperts:
                 w1[e, :, i] = pad(get(f"e{e}.{name}"), (0, 0, 0, ffp - ff)).view(ffp // 64, 64, W)
             w2[e, :W, :ff] = get(f"e{e}.down")
         correction = get("correction", torch.float32) if spec.correction else None
-        return cls(spec, router, correction, w1.view(-1, W), w2.view(-1, ffp))
+        experts = cls(spec, router, correction, w1.view(-1, W), w2.view(-1, ffp))
+        if spec.bias:
+            b = get("router.b")
+            experts.bias = torch.nn.functional.pad(b, (0, router.shape[0] - b.shape[0])).contiguous()
+        return experts
 
     def tensors(self):
-        return [t for t in (self.router, self.correction, self.w1, self.w2) if t is not None]
+        return [t for t in (self.router, self.correction, self.bias, self.w1, self.w2) if t is not None]
 
     def forward(self, h: torch.Tensor):
         """(expert rows for :func:`ops.residual_add`, logits of the shared expert's gate ``[T]`` or None)."""
         s = self.spec
-        logits = ops.linear(h, self.router, epi=ops.EPI_F32)
+        logits = ops.linear(h, self.router, bias=self.bias, epi=ops.EPI_F32)
         ids, w = ops.moe_route(logits[:, :s.outputs], self.correction, s.top, int(s.sigmoid), s.normalised, s.groups,
                                s.groups_keep, group_top=1)
         if self.capture is not None:
             self.capture(ids)
         gate = logits[:, s.outputs] if s.shared and s.shared_gate else None
-        return ops.routed_ffn(h, ids, w, self.w1, self.w2, s.experts, s.weighted_input), gate
+        return ops.routed_ffn(h, ids, w, self.w1, self.w2, s.experts, s.weighted_input, self.act, self.limit), gate

@@ -37,12 +37,15 @@ _REGISTRY: dict[str, str] = {
     "Zudepel": "parallel_block",
     # layer-list configs: looped layers, norms on both sides of a sublayer, matrix memories beside or instead of attention
     "Zasalix": "looped",
+    # layer-list configs: grouped norms, attention with sinks and mixed values, state-space layers, sigmoid attention beside a
+    # gated delta rule
+    "Kikurax": "prenorm_mix",
     # block-sparse (MSA)
     "MiniMaxM3SparseForCausalLM": "msa",
 }
 
 
-_LISTED = ("latent", "looped", "parallel_block")      # families of layer-list configs
+_LISTED = ("latent", "looped", "parallel_block", "prenorm_mix")      # families of layer-list configs
 
 
 def supported_architectures() -> list[str]:
@@ -82,10 +85,11 @@ def _build_stage(cfg: ModelConfig, start_layer: int, end_layer: int, device, dty
         from parallax_b200.models.latent import LatentStage
         from parallax_b200.models.looped import LoopedStage
         from parallax_b200.models.parallel_block import ParallelBlockStage
+        from parallax_b200.models.prenorm_mix import PreNormStage
 
         if tp_size > 1:
             raise ValueError(f"tensor parallelism is not available for {cfg.architecture}; use pipeline stages")
-        cls = {"latent": LatentStage, "looped": LoopedStage, "parallel_block": ParallelBlockStage}[fam]
+        cls = {"latent": LatentStage, "looped": LoopedStage, "parallel_block": ParallelBlockStage, "prenorm_mix": PreNormStage}[fam]
         return cls(cfg, start_layer, end_layer, device, dtype, max_positions=max_positions)
     if tp_size > 1 and fam != "decoder":
         from parallax_b200.models import tp_families

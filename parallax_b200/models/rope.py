@@ -14,6 +14,17 @@ def _yarn_find_dim(num_rot: float, dim: int, base: float, max_pos: int) -> float
     return (dim * math.log(max_pos / (num_rot * 2 * math.pi))) / (2 * math.log(base))
 
 
+def stretched_frequencies(inv: torch.Tensor, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """The Llama 3.1 rule: frequencies whose wavelength exceeds ``original / low`` are divided by ``factor``, those below
+    ``original / high`` stay, with a linear blend (in original / wavelength) in between."""
+    wavelen = 2 * math.pi / inv
+    smooth = (original / wavelen - low) / (high - low)
+    scaled = torch.where(wavelen > original / low, inv / factor, inv)
+    mid = (1 - smooth) * inv / factor + smooth * inv
+    is_mid = (wavelen <= original / low) & (wavelen >= original / high)
+    return torch.where(is_mid, mid, scaled)
+
+
 def rope_inv_freq(cfg: ModelConfig) -> tuple[torch.Tensor, float]:
     """Returns (inv_freq [rot_dim/2] float64, attention scaling factor for cos/sin)."""
     rot = cfg.rot_dim
@@ -30,12 +41,7 @@ def rope_inv_freq(cfg: ModelConfig) -> tuple[torch.Tensor, float]:
         low = float(sc.get("low_freq_factor", 1.0))
         high = float(sc.get("high_freq_factor", 4.0))
         old = float(sc.get("original_max_position_embeddings", 8192))
-        wavelen = 2 * math.pi / inv
-        smooth = (old / wavelen - low) / (high - low)
-        scaled = torch.where(wavelen > old / low, inv / factor, inv)
-        mid = (1 - smooth) * inv / factor + smooth * inv
-        is_mid = (wavelen <= old / low) & (wavelen >= old / high)
-        return torch.where(is_mid, mid, scaled), 1.0
+        return stretched_frequencies(inv, factor, low, high, old), 1.0
     if kind == "yarn":
         old = float(sc.get("original_max_position_embeddings", cfg.max_position_embeddings))
         beta_fast = float(sc.get("beta_fast", 32))

@@ -21,6 +21,7 @@ _NAMES = [
     "embed_rows", "to_low", "residual_norm", "row_norm", "latent_prep", "head_linear", "latent_attn",
     "glu_linear", "routed_ffn", "residual_add", "conv_qkv_prep", "gated_rows", "lightning_attn",
     "latent_rows", "latent_queries", "act_linear", "tanh_norm", "residual_step", "matrix_memory",
+    "head_qkv_prep", "short_conv", "delta_rule", "state_space", "gated_norm_rows",
 ]
 
 

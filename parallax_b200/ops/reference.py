@@ -181,7 +181,7 @@ def _gather_kv(cache, block_table, n, scale: float = 1.0):
     return blocks.permute(1, 0, 2, 3).reshape(cache.shape[1], nb * page, cache.shape[3])[:, :n]
 
 
-def _attend(q, k, v, scale, q_pos, window, sinks, keep_first=0):
+def _attend(q, k, v, scale, q_pos, window, sinks, keep_first=0, softcap=0.0, sigmoid_bias=None):
     # q [Lq, Hq, D]; k, v [Hkv, Lk, D]; q_pos [Lq] absolute positions of the queries
     Lq, Hq, D = q.shape
     Hkv, Lk, _ = k.shape
@@ -190,10 +190,15 @@ def _attend(q, k, v, scale, q_pos, window, sinks, keep_first=0):
     kf = k.float().repeat_interleave(G, dim=0)
     vf = v.float().repeat_interleave(G, dim=0)
     s = torch.einsum("hqd,hkd->hqk", qf, kf) * scale
+    if softcap:
+        s = softcap * torch.tanh(s / softcap)
     kpos = torch.arange(Lk, device=q.device)[None, :]
     mask = kpos <= q_pos[:, None]
     if window and window > 0:
         mask = mask & ((kpos > q_pos[:, None] - window) | (kpos < keep_first))
+    if sigmoid_bias is not None:
+        p = torch.sigmoid(s + sigmoid_bias.float()[:, None, None]) * mask[None]
+        return torch.einsum("hqk,hkd->hqd", p, vf).permute(1, 0, 2).to(q.dtype)
     s = s.masked_fill(~mask[None], float("-inf"))
     if sinks is not None:
         s = torch.cat([s, sinks.float()[:, None, None].expand(Hq, Lq, 1)], dim=-1)
@@ -206,9 +211,10 @@ def _attend(q, k, v, scale, q_pos, window, sinks, keep_first=0):
 
 
 def attn_decode(q, k_cache, v_cache, block_tables, ctx_lens, scale, window=0, sinks=None,
-                max_ctx=0, num_splits=0, out=None, kv_scale=(1.0, 1.0), keep_first=0):
+                max_ctx=0, num_splits=0, out=None, kv_scale=(1.0, 1.0), keep_first=0, softcap=0.0, sigmoid_bias=None):
     """One query per sequence over the paged cache; ``window`` keys per query (0: all) and the sequence's first
-    ``keep_first``."""
+    ``keep_first``. ``softcap``: scores become ``softcap * tanh(score / softcap)``. ``sigmoid_bias [Hq]``: the weight of a
+    key is ``sigmoid(score + bias)``, not a softmax, and nothing normalises the weights."""
     B = q.shape[0]
     res = torch.zeros_like(q) if out is None else out
     for b in range(B):
@@ -219,12 +225,12 @@ def attn_decode(q, k_cache, v_cache, block_tables, ctx_lens, scale, window=0, si
         k = _gather_kv(k_cache, block_tables[b], n, kv_scale[0])
         v = _gather_kv(v_cache, block_tables[b], n, kv_scale[1])
         pos = torch.tensor([n - 1], device=q.device)
-        res[b] = _attend(q[b:b + 1], k, v, scale, pos, window, sinks, keep_first)[0]
+        res[b] = _attend(q[b:b + 1], k, v, scale, pos, window, sinks, keep_first, softcap, sigmoid_bias)[0]
     return res
 
 
 def attn_prefill(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window=0,
-                 sinks=None, out=None, kv_scale=(1.0, 1.0), keep_first=0):
+                 sinks=None, out=None, kv_scale=(1.0, 1.0), keep_first=0, softcap=0.0, sigmoid_bias=None):
     T, Hq, D = q.shape
     res = torch.zeros((T, Hq, D), dtype=q.dtype, device=q.device) if out is None else out
     B = ctx_lens.numel()
@@ -237,7 +243,7 @@ def attn_prefill(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, s
         k = _gather_kv(k_cache, block_tables[b], n, kv_scale[0])
         v = _gather_kv(v_cache, block_tables[b], n, kv_scale[1])
         pos = prefix + torch.arange(e - s, device=q.device)
-        res[s:e] = _attend(q[s:e], k, v, scale, pos, window, sinks, keep_first)
+        res[s:e] = _attend(q[s:e], k, v, scale, pos, window, sinks, keep_first, softcap, sigmoid_bias)
     return res
 
 
@@ -679,10 +685,15 @@ def residual_norm(x, y, w, eps: float, mult: float = 1.0, kind: int = NORM_LAYER
     return to_low(x, y.dtype)
 
 
-def row_norm(x, w, eps: float, kind: int = NORM_LAYER, rows=None, dtype=None):
-    """``norm(x[rows]) * w`` of fp32 rows in ``dtype``."""
+def _in_groups(x, eps, kind: int, groups: int):
+    return _normalised(x.reshape(*x.shape[:-1], groups, x.shape[-1] // groups), eps, kind).reshape(x.shape)
+
+
+def row_norm(x, w, eps: float, kind: int = NORM_LAYER, rows=None, dtype=None, groups: int = 1):
+    """``norm(x[rows]) * w`` of fp32 rows in ``dtype``; the statistics are those of each of ``groups`` equal parts of the
+    row (more than one: RMS norm)."""
     x = x if rows is None else x[rows.long()]
-    return (_normalised(x, eps, kind) * w.float()).to(dtype or x.dtype)
+    return (_in_groups(x, eps, kind, groups) * w.float()).to(dtype or x.dtype)
 
 
 def _rotate_pairs(x, cos_sin, positions, dims: int):
@@ -798,8 +809,8 @@ def act_linear(x, w, act: int, table=None, ids=None, col: int = 0, out=None):
     return out
 
 
-def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool = False):
-    """Outputs of the chosen gated (SiLU) experts for :func:`residual_add`: ``(rows, pos_of, weights)``, where
+def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool = False, act: int = 0, limit: float = 0.0):
+    """Outputs of the chosen gated experts (``act`` 0: SiLU, 1: clipped GLU with ``limit``) for :func:`residual_add`: ``(rows, pos_of, weights)``, where
     ``rows[pos_of[t, j]]`` is expert ``ids[t, j]``'s output. ``w1 [E * 2 I, W]`` gate / up rows interleaved per expert,
     ``w2 [E * N, I]``. Ids >= ``num_experts`` are identity experts: position -1. ``weighted_input``: the weights multiply
     the experts' input rows, and None comes back for them."""
@@ -811,21 +822,28 @@ def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool =
         tok, slot = (ids == e).nonzero(as_tuple=True)
         if tok.numel():
             xe = (x[tok].float() * weights[tok, slot].float()[:, None]).to(x.dtype) if weighted_input else x[tok]
-            act = glu_linear(xe, w1[e * n1:(e + 1) * n1])
-            rows[tok * k + slot] = linear(act, w2[e * n2:(e + 1) * n2])
+            w1e = w1[e * n1:(e + 1) * n1]
+            y = linear(xe, w1e, epi=EPI_CLIP_GLU, limit=limit) if act == 1 else glu_linear(xe, w1e)
+            rows[tok * k + slot] = linear(y, w2[e * n2:(e + 1) * n2])
     return rows, torch.where(ids < num_experts, pos, torch.full_like(pos, -1)).to(torch.int32), None if weighted_input else weights
 
 
-def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None):
-    """In place on the fp32 residual: ``x += y`` plus the weighted expert rows of :func:`routed_ffn` (an identity
-    expert's row is ``h[t]``). With a norm weight returns ``rmsnorm(x) * w`` in ``y``'s dtype."""
+def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None, groups: int = 1, branches=None):
+    """In place on the fp32 residual: ``x += y`` (None: nothing) plus the weighted expert rows of :func:`routed_ffn` (an
+    identity expert's row is ``h[t]``). ``branches = (factor, (y1, w1), (y2, w2))`` instead of ``y``: ``x += factor *
+    (rmsnorm(y1) * w1 + rmsnorm(y2) * w2)``. With a norm weight returns ``rmsnorm(x) * w``, the statistics those of each of
+    ``groups`` equal parts, in the updates' dtype."""
     W = x.shape[1]
-    x.add_(y.float())
+    low = next(t for t in (y, branches and branches[1][0], routed and routed[0]) if t is not None).dtype
+    if y is not None:
+        x.add_(y.float())
+    if branches is not None:
+        x.add_(sum(_normalised(b, eps, NORM_RMS) * bw.float() for b, bw in branches[1:]) * branches[0])
     if routed is not None:
         rows, pos, wt = routed
         val = torch.where(pos[:, :, None] < 0, h[:, None, :].float(), rows[pos.clamp_min(0).long()][:, :, :W].float())
         x.add_((val * wt.float()[:, :, None]).sum(1))
-    return None if w is None else (_normalised(x, eps, NORM_RMS) * w.float()).to(y.dtype)
+    return None if w is None else (_in_groups(x, eps, NORM_RMS, groups) * w.float()).to(low)
 
 
 def conv_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, conv_w, conv_state, q_norm, k_norm, cos_sin,
@@ -989,4 +1007,133 @@ def matrix_memory(proj, offs, heads: int, dim: int, vdim: int, gates, gate_bias,
             out[t] = (torch.einsum("hkv,hk->hv", S, q[t]) / den[:, None]).to(out.dtype)
         words = torch.cat([S.reshape(heads, -1), n.repeat(1, slices), m[:, None].expand(heads, slices)], -1)
         state[slot, :, :words.shape[1]] = words
+    return out
+
+
+# ---------------------------------------------------------------------------- heads without norm weights, delta rule, state space
+def head_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, eps: float, cos_sin, positions, slot_mapping, k_cache,
+                  v_cache, q_out, head_scale=None, pos_scale=None, v_first=None, v_mix: float = 0.0):
+    """Queries and cache rows of one step out of the packed projection (q, k, v start at columns ``offs``): half-split
+    rotation (``cos_sin [positions, dims]`` or None), every head of q and k over its root mean square, queries times
+    ``head_scale [heads]`` and ``pos_scale [positions]``, values ``(1 - v_mix) v + v_mix v_first`` (``v_first [T, kv_heads *
+    vdim]`` or None). Heads are padded with zeros to the columns of ``q_out [T, heads, cols]`` and of the pages."""
+    T, cols = proj.shape[0], q_out.shape[2]
+
+    def part(o, n, d):
+        return proj[:, o:o + n * d].float().view(T, n, d)
+
+    def rotated(x):
+        if cos_sin is None:
+            return x
+        rot = cos_sin.shape[1]
+        cs = cos_sin[positions.long()].float()[:, None]
+        c, s, a, b = cs[..., :rot // 2], cs[..., rot // 2:], x[..., :rot // 2], x[..., rot // 2:rot]
+        return torch.cat([a * c - b * s, b * c + a * s, x[..., rot:]], -1)
+
+    q = _normalised(rotated(part(offs[0], heads, dim)), eps, NORM_RMS)
+    k = _normalised(rotated(part(offs[1], kv_heads, dim)), eps, NORM_RMS)
+    v = part(offs[2], kv_heads, vdim)
+    if head_scale is not None:
+        q = q * head_scale.float()[:, None]
+    if pos_scale is not None:
+        q = q * pos_scale[positions.long()].float()[:, None, None]
+    if v_first is not None:
+        v = (1 - v_mix) * v + v_mix * v_first.float().view(T, kv_heads, vdim)
+    pad = torch.nn.functional.pad
+    q_out.copy_(pad(q, (0, cols - dim)))
+    reshape_and_cache(pad(k, (0, cols - dim)), pad(v, (0, cols - vdim)), slot_mapping, k_cache, v_cache)
+
+
+def short_conv(x, w, bias, state, positions, seq_cu, seq_slots, prefill_seqs: int, prefill_tokens: int):
+    """``silu`` of the causal convolution per channel: ``x [T, C]`` (columns of a projection), taps ``w [taps, C]``, the last
+    one the token's own, ``bias [C]`` or None; the last ``taps - 1`` inputs are kept in ``state [slots, taps - 1, C]``."""
+    taps, u, wf = w.shape[0], x.float(), w.float()
+    y, cu = torch.empty_like(u), seq_cu.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1, slot = cu[b], cu[b + 1], int(seq_slots[b])
+        if t1 <= t0:
+            continue
+        hist = u.new_zeros((0, u.shape[1]))
+        if taps > 1:
+            hist = state[slot].float().clone()
+            start = int(positions[t0])
+            if start < taps - 1:       # zeros before the sequence
+                hist[:taps - 1 - start] = 0
+        full = torch.cat([hist, u[t0:t1]], 0)
+        y[t0:t1] = sum(wf[j] * full[j:j + t1 - t0] for j in range(taps))
+        if taps > 1:
+            state[slot] = full[-(taps - 1):].to(state.dtype)
+    return torch.nn.functional.silu(y if bias is None else y + bias.float()).to(x.dtype)
+
+
+def delta_rule(x, offs, heads: int, kv_heads: int, dim: int, vdim: int, decay, dt_bias, A_log, beta, state, positions, seq_cu,
+               seq_slots, prefill_seqs: int, prefill_tokens: int = 0, out=None):
+    """Gated delta rule with a decay per head and key channel; q, k, v are the columns of ``x`` at ``offs``, ``decay [T, >=
+    heads * dim]`` and ``beta [T, >= heads]`` fp32 logits::
+
+        g = exp(-exp(A_log) softplus(decay + dt_bias)),  b = sigmoid(beta),  q, k over sqrt(sum of squares + 1e-6), q times dim^-1/2
+        S <- g S,  u = b (v - S^T k),  S <- S + k u^T,  o = S^T q
+
+    from S = 0 at a sequence's first token; ``state [slots, heads, dim, vdim]`` fp32. Returns ``[T, heads, vdim]``."""
+    T, rep = x.shape[0], heads // kv_heads
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=x.dtype, device=x.device)
+
+    def unit(o):
+        y = x[:, o:o + kv_heads * dim].float().view(T, kv_heads, dim)
+        return (y * torch.rsqrt(y.pow(2).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(rep, 1)
+
+    q, k = unit(offs[0]) * dim ** -0.5, unit(offs[1])
+    v = x[:, offs[2]:offs[2] + heads * vdim].float().view(T, heads, vdim)
+    dt = torch.nn.functional.softplus(decay[:, :heads * dim].float() + dt_bias.float(), threshold=80.0).view(T, heads, dim)
+    g = torch.exp(-torch.exp(A_log.float())[:, None] * dt)
+    b_ = torch.sigmoid(beta[:, :heads].float())
+    cu = seq_cu.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1, slot = cu[b], cu[b + 1], int(seq_slots[b])
+        if t1 <= t0:
+            continue
+        S = torch.zeros_like(state[slot]) if int(positions[t0]) == 0 else state[slot].clone()
+        for t in range(t0, t1):
+            S = g[t][:, :, None] * S
+            u = b_[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+            S = S + k[t][:, :, None] * u[:, None, :]
+            out[t] = torch.einsum("hkv,hk->hv", S, q[t]).to(out.dtype)
+        state[slot] = S
+    return out
+
+
+def state_space(x, offs, heads: int, groups: int, dim: int, vdim: int, dt, dt_bias, A_log, D, state, positions, seq_cu, seq_slots,
+                prefill_seqs: int, out=None):
+    """``S <- exp(-exp(A_log) d) S + d B x^T``, ``y = S^T C + D x`` per head with ``d = softplus(dt + dt_bias)`` (``dt [T, >=
+    heads]`` fp32); x (heads x vdim), B and C (groups x dim) are the columns of ``x`` at ``offs``; ``state [slots, heads, dim,
+    vdim]`` fp32, zero at a sequence's first token. Returns ``[T, heads, vdim]``."""
+    T, rep = x.shape[0], heads // groups
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=x.dtype, device=x.device)
+    xs = x[:, offs[0]:offs[0] + heads * vdim].float().view(T, heads, vdim)
+    B, C = (x[:, o:o + groups * dim].float().view(T, groups, dim).repeat_interleave(rep, 1) for o in offs[1:])
+    d = torch.nn.functional.softplus(dt[:, :heads].float() + dt_bias.float(), threshold=80.0)
+    keep = torch.exp(-torch.exp(A_log.float()) * d)
+    cu = seq_cu.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1, slot = cu[b], cu[b + 1], int(seq_slots[b])
+        if t1 <= t0:
+            continue
+        S = torch.zeros_like(state[slot]) if int(positions[t0]) == 0 else state[slot].clone()
+        for t in range(t0, t1):
+            S = keep[t][:, None, None] * S + (d[t][:, None] * B[t])[:, :, None] * xs[t][:, None, :]
+            out[t] = (torch.einsum("hkv,hk->hv", S, C[t]) + D.float()[:, None] * xs[t]).to(out.dtype)
+        state[slot] = S
+    return out
+
+
+def gated_norm_rows(x, gate, w, groups: int, eps: float, out):
+    """``out = rmsnorm(x * silu(gate)) * w``, the statistics those of each of ``groups`` equal parts of a row; ``x [T, heads,
+    vdim]``; zeros in the columns of ``out`` behind the row."""
+    T = x.shape[0]
+    y = x.reshape(T, -1).float() * torch.nn.functional.silu(gate.float())
+    n = y.shape[1]
+    out[:, :n] = (_in_groups(y, eps, NORM_RMS, groups) * w.float()).to(out.dtype)
+    out[:, n:] = 0
     return out

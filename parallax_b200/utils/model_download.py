@@ -63,6 +63,8 @@ def _snapshot(repo: str, patterns: list[str], local_files_only: bool) -> Path:
 
 def selective_model_download(model: str, start_layer: Optional[int] = None, end_layer: Optional[int] = None,
                              local_files_only: bool = False) -> Path:
+    from parallax_b200.models.config import tied_embeddings
+
     p = Path(model)
     if p.is_dir():
         return p
@@ -73,6 +75,6 @@ def selective_model_download(model: str, start_layer: Optional[int] = None, end_
     if start_layer is None or end_layer is None or not index_file.exists():
         return _snapshot(model, METADATA_PATTERNS + ["*.safetensors"], local_files_only)
     files = needed_weight_files(json.loads(index_file.read_text()), start_layer, end_layer, n,
-                                bool(cfg.get("tie_word_embeddings", False)))
+                                tied_embeddings(cfg))
     logger.info("stage [%s, %s): downloading %d weight file(s)", start_layer, end_layer, len(files))
     return _snapshot(model, METADATA_PATTERNS + files, local_files_only)

@@ -89,6 +89,11 @@ def test_layers_that_read_the_token_ids_over_pipeline_ranks(tmp_path):
     assert _run_group(2, 1, tmp_path, model="tiny-zasalix")["outputs"] == _single(model="tiny-zasalix")
 
 
+def test_mixed_values_over_pipeline_ranks(tmp_path):
+    """Layers that mix in an earlier layer's values stay in its stage; the last stage has the embedding table as its head."""
+    assert _run_group(2, 1, tmp_path, model="tiny-kikurax")["outputs"] == _single(model="tiny-kikurax")
+
+
 def test_rank0_executor_thread_and_aligned_rows(tmp_path):
     """Rank 0 launching its stage from a thread of its own, three micro-batches in flight and prompt
     slices trimmed to a row multiple: same tokens as the single-process engine."""

@@ -48,8 +48,8 @@ def _run_pipeline(cfg, spans, prompts, max_new, **kw):
 
 
 @pytest.mark.parametrize("name,layers", [("tiny-piburax", [(0, 1), (1, 2), (2, 3)]), ("tiny-zudepel", [(0, 2), (2, 3), (3, 4)]),
-                                         ("tiny-zasalix", [(0, 2), (2, 3), (3, 4)])])
-def test_three_peers_of_a_layer_list_model(name, layers):
+                                         ("tiny-zasalix", [(0, 2), (2, 3), (3, 4)]), ("tiny-kikurax", [(0, 1), (1, 4)])])
+def test_peers_of_a_layer_list_model(name, layers):
     cfg = named_config(name)
     prompts = _prompts(3, 41, cfg.vocab_size, seed=4)
     want = Engine(cfg, device="cpu", num_blocks=128, max_batch_size=8).generate(
