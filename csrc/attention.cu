@@ -16,6 +16,7 @@
 
 #include <atomic>
 
+#include "attention_score.cuh"
 #include "common.cuh"
 #include "pxl_api.h"
 #include "pxl_noalloc.h"
@@ -172,14 +173,14 @@ __device__ __forceinline__ float quad_sum(float v) {
 }
 
 // =============================================================================== decode
-template <int D, bool FP8 = false>
+template <int D, bool FP8 = false, int SM = kPlain>
 __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __restrict__ k_cache,
                    const void* __restrict__ v_cache, const int* __restrict__ block_tables,
                    const int* __restrict__ ctx_lens, bf16* __restrict__ out,
                    float* __restrict__ workspace, const float* __restrict__ sinks, int Hq, int Hkv,
                    int page_size, int max_blocks, int64_t num_blocks, float scale_log2, int window,
-                   int keep, int num_splits, float v_scale, int* status) {
+                   int keep, int num_splits, float v_scale, const ScoreArgs sa, int* status) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int TILE_BYTES = TILE * D * 2;
   const uint32_t k_smem0 = smem_u32(smem);
@@ -215,6 +216,14 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
     }
   }
 
+  float bias2[2] = {0.f, 0.f};  // of this thread's two rows
+  if constexpr (SM == kSigmoid) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = (lane >> 2) + h * 8;
+      if (r < G) bias2[h] = sa.bias[kvh * G + r] * kLog2e;
+    }
+  }
   float o[D / 8][4];
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -246,10 +255,15 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
         for (int e = 0; e < 4; ++e) {
           const int tok = tok_base + j * 8 + 2 * (lane & 3) + (e & 1);
           const bool valid = tok < hi && (tok >= lo || tok < keep);
-          s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
-          mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+          if constexpr (SM == kSigmoid) {
+            s[j][e] = valid ? sigmoid_weight(s[j][e], scale_log2, bias2[e >> 1]) : 0.f;
+          } else {
+            s[j][e] = valid ? score_log2<SM>(s[j][e], scale_log2, sa) : -INFINITY;
+            mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+          }
         }
       }
+      if constexpr (SM != kSigmoid) {
       float corr[2], m_use[2];
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
@@ -275,6 +289,7 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
         o[i][1] *= corr[0];
         o[i][2] *= corr[1];
         o[i][3] *= corr[1];
+      }
       }
       uint32_t pf[4];
       pf[0] = pack_bf16x2(s[0][0], s[0][1]);
@@ -315,10 +330,18 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
   __syncthreads();
   for (int idx = threadIdx.x; idx < G * D; idx += 128) {
     const int r = idx / D, d = idx % D;
+    const int head = kvh * G + r;
+    if constexpr (SM == kSigmoid) {  // weights as they are: sums of the warps, of the splits
+      float acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) acc += o_sm[(w * 16 + r) * D + d];
+      if (num_splits == 1) out[(static_cast<size_t>(b) * Hq + head) * D + d] = __float2bfloat16(acc);
+      else workspace[((static_cast<size_t>(b) * Hq + head) * num_splits + split) * D + d] = acc;
+      continue;
+    }
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) M = fmaxf(M, m_sm[w * 16 + r]);
-    const int head = kvh * G + r;
     const float sink = (sinks && num_splits == 1) ? sinks[head] * kLog2e : -INFINITY;
     const float Mx = fmaxf(M, sink);
     const float Mu = (Mx == -INFINITY) ? 0.f : Mx;
@@ -356,12 +379,14 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
 constexpr int kDecStages = 3;
 constexpr int kDecThreads = 160;  // 4 consumer warps + 1 producer warp
 
+template <int SM>
 __global__ void __launch_bounds__(kDecThreads, 2)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                        const bf16* __restrict__ q, int64_t q_stride, const int* __restrict__ block_tables,
                        const int* __restrict__ ctx_lens, bf16* __restrict__ out, float* __restrict__ workspace,
                        const float* __restrict__ sinks, int Hq, int Hkv, int page_size, int max_blocks,
-                       int64_t num_blocks, float scale_log2, int window, int keep, int num_splits, int* status) {
+                       int64_t num_blocks, float scale_log2, int window, int keep, int num_splits, const ScoreArgs sa,
+                       int* status) {
   constexpr int D = 128;
   constexpr int TILE_BYTES = TILE * D * 2;
   extern __shared__ uint8_t smem_raw[];
@@ -456,6 +481,14 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       qf[ks][3] = r_hi < G ? *reinterpret_cast<const uint32_t*>(q_hi + c + 8) : 0u;
     }
   }
+  float bias2[2] = {0.f, 0.f};  // of this thread's two rows
+  if constexpr (SM == kSigmoid) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = (lane >> 2) + h * 8;
+      if (r < G) bias2[h] = sa.bias[kvh * G + r] * kLog2e;
+    }
+  }
   float o[D / 8][4];
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -483,10 +516,15 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         for (int e = 0; e < 4; ++e) {
           const int tok = tok_base + j * 8 + 2 * (lane & 3) + (e & 1);
           const bool valid = tok < hi && (tok >= lo || tok < keep);
-          s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
-          mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+          if constexpr (SM == kSigmoid) {
+            s[j][e] = valid ? sigmoid_weight(s[j][e], scale_log2, bias2[e >> 1]) : 0.f;
+          } else {
+            s[j][e] = valid ? score_log2<SM>(s[j][e], scale_log2, sa) : -INFINITY;
+            mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+          }
         }
       }
+      if constexpr (SM != kSigmoid) {
       float corr[2], m_use[2];
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
@@ -512,6 +550,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         o[i][1] *= corr[0];
         o[i][2] *= corr[1];
         o[i][3] *= corr[1];
+      }
       }
       uint32_t pf[4];
       pf[0] = pack_bf16x2(s[0][0], s[0][1]);
@@ -556,10 +595,18 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   __syncthreads();
   for (int idx = threadIdx.x; warp < 4 && idx < G * D; idx += 128) {
     const int r = idx / D, d = idx % D;
+    const int head = kvh * G + r;
+    if constexpr (SM == kSigmoid) {  // weights as they are: sums of the warps, of the splits
+      float acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) acc += o_sm[(w * 16 + r) * D + d];
+      if (num_splits == 1) out[(static_cast<size_t>(b) * Hq + head) * D + d] = __float2bfloat16(acc);
+      else workspace[((static_cast<size_t>(b) * Hq + head) * num_splits + split) * D + d] = acc;
+      continue;
+    }
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) M = fmaxf(M, m_sm[w * 16 + r]);
-    const int head = kvh * G + r;
     const float sink = (sinks && num_splits == 1) ? sinks[head] * kLog2e : -INFINITY;
     const float Mx = fmaxf(M, sink);
     const float Mu = (Mx == -INFINITY) ? 0.f : Mx;
@@ -583,7 +630,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   }
 }
 
-template <int D>
+template <int D, int SM = kPlain>
 __global__ void __launch_bounds__(D)
 attn_decode_reduce_kernel(const float* __restrict__ workspace, const float* __restrict__ sinks,
                           bf16* __restrict__ out, int Hq, int num_splits) {
@@ -593,6 +640,12 @@ attn_decode_reduce_kernel(const float* __restrict__ workspace, const float* __re
   const float* po = workspace;
   const float* plse = workspace + static_cast<size_t>(gridDim.y) * Hq * num_splits * D;
   const size_t row0 = (static_cast<size_t>(b) * Hq + head) * num_splits;
+  if constexpr (SM == kSigmoid) {
+    float sum = 0.f;
+    for (int s = 0; s < num_splits; ++s) sum += po[(row0 + s) * D + d];
+    out[(static_cast<size_t>(b) * Hq + head) * D + d] = __float2bfloat16(sum);
+    return;
+  }
   const float sink = sinks ? sinks[head] * kLog2e : -INFINITY;
   float M = sink;
   for (int s = 0; s < num_splits; ++s) M = fmaxf(M, plse[row0 + s]);
@@ -608,14 +661,14 @@ attn_decode_reduce_kernel(const float* __restrict__ workspace, const float* __re
 }
 
 // ============================================================================== prefill
-template <int D, bool FP8 = false>
+template <int D, bool FP8 = false, int SM = kPlain>
 __global__ void __launch_bounds__(128)
 attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __restrict__ k_cache,
                     const void* __restrict__ v_cache, const int* __restrict__ block_tables,
                     const int* __restrict__ cu_q, const int* __restrict__ ctx_lens,
                     bf16* __restrict__ out, int64_t out_stride, const float* __restrict__ sinks,
                     int Hq, int Hkv, int page_size, int max_blocks, int64_t num_blocks,
-                    float scale_log2, int window, int keep, float v_scale, int* status) {
+                    float scale_log2, int window, int keep, float v_scale, const ScoreArgs sa, int* status) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int TILE_BYTES = TILE * D * 2;
   const uint32_t k_smem0 = smem_u32(smem);
@@ -678,6 +731,12 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
   KVTileArgs ka{k_cache, v_cache, block_tables + static_cast<size_t>(b) * max_blocks, max_blocks,
                 num_blocks, Hkv, kvh, page_size};
 
+  float bias2[2] = {0.f, 0.f};
+  if constexpr (SM == kSigmoid) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+      if (rvalid[h]) bias2[h] = sa.bias[rhead[h]] * kLog2e;
+  }
   float o[D / 8][4];
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -713,9 +772,14 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
           const int h = e >> 1;
           const int tok = tok0 + j * 8 + 2 * (lane & 3) + (e & 1);
           const bool valid = tok <= rpos[h] && (tok >= rlo[h] || tok < keep);
-          s[j][e] = valid ? s[j][e] * scale_log2 : -INFINITY;
-          mx[h] = fmaxf(mx[h], s[j][e]);
+          if constexpr (SM == kSigmoid) {
+            s[j][e] = valid ? sigmoid_weight(s[j][e], scale_log2, bias2[h]) : 0.f;
+          } else {
+            s[j][e] = valid ? score_log2<SM>(s[j][e], scale_log2, sa) : -INFINITY;
+            mx[h] = fmaxf(mx[h], s[j][e]);
+          }
         }
+      if constexpr (SM != kSigmoid) {
       float corr[2], m_use[2];
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
@@ -742,6 +806,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
         o[i][2] *= corr[1];
         o[i][3] *= corr[1];
       }
+      }
 #pragma unroll
       for (int g = 0; g < 4; ++g) {
         uint32_t pf[4];
@@ -766,7 +831,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
     const float Mu = (Mx == -INFINITY) ? 0.f : Mx;
     const float f = exp2f(M - Mu);
     const float denom = L * f + exp2f(sink - Mu);
-    const float inv = denom > 0.f ? f / denom * v_scale : 0.f;
+    const float inv = SM == kSigmoid ? 1.f : denom > 0.f ? f / denom * v_scale : 0.f;
     bf16* dst = out + static_cast<size_t>(q0 + rtok[h]) * out_stride + rhead[h] * D;
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) {
@@ -805,8 +870,12 @@ int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache, const
                      const int* block_tables, const int* ctx_lens, void* out, float* workspace,
                      const float* sinks, int B, int Hq, int Hkv, int D, int page_size, int max_blocks,
                      int64_t num_blocks, float scale, int window, int keep_first, int num_splits, int max_ctx,
-                     bool cache_fp8, float k_scale, float v_scale, int* status, pxl_stream_t stream) {
+                     bool cache_fp8, float k_scale, float v_scale, float softcap, const float* sig_bias, int* status,
+                     pxl_stream_t stream) {
   if (B <= 0) return PXL_OK;
+  const int mode = score_mode(softcap, sig_bias);
+  const ScoreArgs sa = score_args(scale, softcap, sig_bias);
+  if (cache_fp8 && mode != kPlain) return PXL_ERR_INVALID_ARG;
   if (Hkv <= 0 || Hq % Hkv || Hq / Hkv > 16 || page_size <= 0) return PXL_ERR_INVALID_ARG;
   if (num_splits <= 0) num_splits = pxl_attn_decode_splits(B, Hkv, max_ctx);
   if (num_splits > 1 && workspace == nullptr) return PXL_ERR_INVALID_ARG;
@@ -821,46 +890,58 @@ int attn_decode_impl(const void* q, int64_t q_stride, const void* k_cache, const
         !pxl_host::make_tmap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, v_cache, rows, 128, 128, page_size, 64))
       return PXL_ERR_TENSORMAP;
     constexpr int SMEM = 1024 + kDecStages * 2 * TILE * 128 * 2 + 128;
-    static bool done[64] = {false};      // function attributes are per device
-    const int dev = pxl_host::current_device_slot();
-    if (!done[dev]) {
-      if (set_smem(attn_decode_tma_kernel, SMEM)) return PXL_ERR_CUDA;
-      done[dev] = true;
-    }
-    pxl_host::launch(attn_decode_tma_kernel, grid, kDecThreads, SMEM, stream,
-        tk, tv, static_cast<const bf16*>(q), q_stride, block_tables, ctx_lens, static_cast<bf16*>(out), workspace,
-        sinks, Hq, Hkv, page_size, max_blocks, num_blocks, scale_log2, window, keep_first, num_splits, status);
-    if (num_splits > 1)
-      pxl_host::launch(attn_decode_reduce_kernel<128>, dim3(Hq, B), 128, 0, stream, workspace, sinks,
-                       static_cast<bf16*>(out), Hq, num_splits);
+#define PXL_DEC_TMA(M)                                                                                                  \
+  {                                                                                                                     \
+    static bool done[64] = {false}; /* function attributes are per device */                                            \
+    const int dev = pxl_host::current_device_slot();                                                                    \
+    if (!done[dev]) {                                                                                                   \
+      if (set_smem(attn_decode_tma_kernel<M>, SMEM)) return PXL_ERR_CUDA;                                               \
+      done[dev] = true;                                                                                                 \
+    }                                                                                                                   \
+    pxl_host::launch(attn_decode_tma_kernel<M>, grid, kDecThreads, SMEM, stream, tk, tv, static_cast<const bf16*>(q),   \
+                     q_stride, block_tables, ctx_lens, static_cast<bf16*>(out), workspace, sinks, Hq, Hkv, page_size,   \
+                     max_blocks, num_blocks, scale_log2, window, keep_first, num_splits, sa, status);                   \
+    if (num_splits > 1)                                                                                                 \
+      pxl_host::launch(attn_decode_reduce_kernel<128, M>, dim3(Hq, B), 128, 0, stream, workspace, sinks,                \
+                       static_cast<bf16*>(out), Hq, num_splits);                                                        \
+  }
+    if (mode == kSigmoid) PXL_DEC_TMA(kSigmoid)
+    else if (mode == kCapped) PXL_DEC_TMA(kCapped)
+    else PXL_DEC_TMA(kPlain)
+#undef PXL_DEC_TMA
     return check_launch();
   }
-#define PXL_DEC(DD, F8)                                                                          \
+#define PXL_DEC(DD, F8, M)                                                                       \
   {                                                                                              \
     constexpr int SMEM = 4 * TILE * DD * 2 > (4 * 16 * DD + 128) * 4 ? 4 * TILE * DD * 2         \
                                                                      : (4 * 16 * DD + 128) * 4;  \
     static bool done[64] = {false};                                                              \
     const int dev = pxl_host::current_device_slot();                                                       \
     if (!done[dev]) {                                                                            \
-      if (set_smem(attn_decode_kernel<DD, F8>, SMEM)) return PXL_ERR_CUDA;                       \
+      if (set_smem(attn_decode_kernel<DD, F8, M>, SMEM)) return PXL_ERR_CUDA;                       \
       done[dev] = true;                                                                          \
     }                                                                                            \
-    attn_decode_kernel<DD, F8><<<grid, 128, SMEM, stream>>>(                                     \
+    attn_decode_kernel<DD, F8, M><<<grid, 128, SMEM, stream>>>(                                  \
         static_cast<const bf16*>(q), q_stride, k_cache, v_cache, block_tables, ctx_lens,         \
         static_cast<bf16*>(out), workspace, sinks, Hq, Hkv, page_size, max_blocks, num_blocks,   \
-        scale_log2 * k_scale, window, keep_first, num_splits, v_scale, status);                  \
+        scale_log2 * k_scale, window, keep_first, num_splits, v_scale, sa, status);              \
     if (num_splits > 1)                                                                          \
-      attn_decode_reduce_kernel<DD><<<dim3(Hq, B), DD, 0, stream>>>(                             \
+      attn_decode_reduce_kernel<DD, M><<<dim3(Hq, B), DD, 0, stream>>>(                          \
           workspace, sinks, static_cast<bf16*>(out), Hq, num_splits);                            \
   }
+  if (D != 64 && D != 128) return PXL_ERR_INVALID_ARG;
   if (cache_fp8) {
-    if (D == 128) PXL_DEC(128, true)
-    else if (D == 64) PXL_DEC(64, true)
-    else return PXL_ERR_INVALID_ARG;
+    if (D == 128) PXL_DEC(128, true, kPlain)
+    else PXL_DEC(64, true, kPlain)
+  } else if (mode == kSigmoid) {
+    if (D == 128) PXL_DEC(128, false, kSigmoid)
+    else PXL_DEC(64, false, kSigmoid)
+  } else if (mode == kCapped) {
+    if (D == 128) PXL_DEC(128, false, kCapped)
+    else PXL_DEC(64, false, kCapped)
   } else {
-    if (D == 128) PXL_DEC(128, false)
-    else if (D == 64) PXL_DEC(64, false)
-    else return PXL_ERR_INVALID_ARG;
+    if (D == 128) PXL_DEC(128, false, kPlain)
+    else PXL_DEC(64, false, kPlain)
   }
 #undef PXL_DEC
   return check_launch();
@@ -872,11 +953,11 @@ PXL_EXPORT int pxl_attn_decode(const void* q, int64_t q_stride, const void* k_ca
                                const int* block_tables, const int* ctx_lens, void* out,
                                float* workspace, const float* sinks, int B, int Hq, int Hkv, int D,
                                int page_size, int max_blocks, int64_t num_blocks, float scale,
-                               int window, int keep_first, int num_splits, int max_ctx, int* status,
-                               pxl_stream_t stream) {
+                               int window, int keep_first, int num_splits, int max_ctx, float softcap,
+                               const float* sig_bias, int* status, pxl_stream_t stream) {
   return attn_decode_impl(q, q_stride, k_cache, v_cache, block_tables, ctx_lens, out, workspace, sinks,
                           B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, keep_first, num_splits,
-                          max_ctx, false, 1.f, 1.f, status, stream);
+                          max_ctx, false, 1.f, 1.f, softcap, sig_bias, status, stream);
 }
 
 // Decode attention over e4m3 caches written by pxl_qk_norm_rope_cache_fp8 / pxl_reshape_and_cache_fp8
@@ -892,7 +973,7 @@ PXL_EXPORT int pxl_attn_decode_fp8(const void* q, int64_t q_stride, const void* 
   if (!(k_scale > 0.f) || !(v_scale > 0.f)) return PXL_ERR_INVALID_ARG;
   return attn_decode_impl(q, q_stride, k_cache, v_cache, block_tables, ctx_lens, out, workspace, sinks,
                           B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, 0, num_splits,
-                          max_ctx, true, k_scale, v_scale, status, stream);
+                          max_ctx, true, k_scale, v_scale, 0.f, nullptr, status, stream);
 }
 
 namespace {
@@ -900,36 +981,44 @@ int attn_prefill_impl(const void* q, int64_t q_stride, const void* k_cache, cons
                       const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                       int64_t out_stride, const float* sinks, int B, int max_q_len, int Hq, int Hkv,
                       int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                      int window, int keep_first, bool cache_fp8, float k_scale, float v_scale, int* status,
-                      pxl_stream_t stream) {
+                      int window, int keep_first, bool cache_fp8, float k_scale, float v_scale, float softcap,
+                      const float* sig_bias, int* status, pxl_stream_t stream) {
   if (B <= 0 || max_q_len <= 0) return PXL_OK;
+  const int mode = score_mode(softcap, sig_bias);
+  const ScoreArgs sa = score_args(scale, softcap, sig_bias);
+  if (cache_fp8 && mode != kPlain) return PXL_ERR_INVALID_ARG;
   if (Hkv <= 0 || Hq % Hkv || Hq / Hkv > 64 || page_size <= 0) return PXL_ERR_INVALID_ARG;
   const int G = Hq / Hkv;
   const int TQ = 64 / G;
   const float scale_log2 = scale * kLog2e;
   dim3 grid(pxl::ceil_div(max_q_len, TQ), Hkv, B);
-#define PXL_PRE(DD, F8)                                                                          \
+#define PXL_PRE(DD, F8, M)                                                                       \
   {                                                                                              \
     constexpr int SMEM = 4 * TILE * DD * 2;                                                      \
     static bool done[64] = {false};                                                              \
     const int dev = pxl_host::current_device_slot();                                             \
     if (!done[dev]) {                                                                            \
-      if (set_smem(attn_prefill_kernel<DD, F8>, SMEM)) return PXL_ERR_CUDA;                      \
+      if (set_smem(attn_prefill_kernel<DD, F8, M>, SMEM)) return PXL_ERR_CUDA;                      \
       done[dev] = true;                                                                          \
     }                                                                                            \
-    attn_prefill_kernel<DD, F8><<<grid, 128, SMEM, stream>>>(                                    \
+    attn_prefill_kernel<DD, F8, M><<<grid, 128, SMEM, stream>>>(                                 \
         static_cast<const bf16*>(q), q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens,   \
         static_cast<bf16*>(out), out_stride, sinks, Hq, Hkv, page_size, max_blocks, num_blocks,  \
-        scale_log2 * k_scale, window, keep_first, v_scale, status);                              \
+        scale_log2 * k_scale, window, keep_first, v_scale, sa, status);                          \
   }
+  if (D != 64 && D != 128) return PXL_ERR_INVALID_ARG;
   if (cache_fp8) {
-    if (D == 128) PXL_PRE(128, true)
-    else if (D == 64) PXL_PRE(64, true)
-    else return PXL_ERR_INVALID_ARG;
+    if (D == 128) PXL_PRE(128, true, kPlain)
+    else PXL_PRE(64, true, kPlain)
+  } else if (mode == kSigmoid) {
+    if (D == 128) PXL_PRE(128, false, kSigmoid)
+    else PXL_PRE(64, false, kSigmoid)
+  } else if (mode == kCapped) {
+    if (D == 128) PXL_PRE(128, false, kCapped)
+    else PXL_PRE(64, false, kCapped)
   } else {
-    if (D == 128) PXL_PRE(128, false)
-    else if (D == 64) PXL_PRE(64, false)
-    else return PXL_ERR_INVALID_ARG;
+    if (D == 128) PXL_PRE(128, false, kPlain)
+    else PXL_PRE(64, false, kPlain)
   }
 #undef PXL_PRE
   return check_launch();
@@ -941,10 +1030,11 @@ PXL_EXPORT int pxl_attn_prefill(const void* q, int64_t q_stride, const void* k_c
                                 const int* ctx_lens, void* out, int64_t out_stride,
                                 const float* sinks, int B, int max_q_len, int Hq, int Hkv, int D,
                                 int page_size, int max_blocks, int64_t num_blocks, float scale,
-                                int window, int keep_first, int* status, pxl_stream_t stream) {
+                                int window, int keep_first, float softcap, const float* sig_bias, int* status,
+                                pxl_stream_t stream) {
   return attn_prefill_impl(q, q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens, out, out_stride,
                            sinks, B, max_q_len, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale,
-                           window, keep_first, false, 1.f, 1.f, status, stream);
+                           window, keep_first, false, 1.f, 1.f, softcap, sig_bias, status, stream);
 }
 
 // Prefix-aware prefill over e4m3 caches (see pxl_attn_decode_fp8).
@@ -958,7 +1048,7 @@ PXL_EXPORT int pxl_attn_prefill_fp8(const void* q, int64_t q_stride, const void*
   if (!(k_scale > 0.f) || !(v_scale > 0.f)) return PXL_ERR_INVALID_ARG;
   return attn_prefill_impl(q, q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens, out, out_stride,
                            sinks, B, max_q_len, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale,
-                           window, 0, true, k_scale, v_scale, status, stream);
+                           window, 0, true, k_scale, v_scale, 0.f, nullptr, status, stream);
 }
 
 // ----------------------------------------------------------------------------------------
@@ -1012,5 +1102,5 @@ PXL_EXPORT int pxl_attn_decode_static_scratch(const void* q, int64_t q_stride, c
   // kernel of this same call, so the array needs no clearing between calls.
   return pxl_attn_decode(q, q_stride, k_cache, v_cache, block_tables, ctx_lens, out, scratch, sinks,
                          B, Hq, Hkv, D, page_size, max_blocks, num_blocks, scale, window, 0, num_splits,
-                         0, status, stream);
+                         0, 0.f, nullptr, status, stream);
 }

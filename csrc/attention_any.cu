@@ -1,7 +1,7 @@
 // Paged attention with grouped heads on the FMA pipes, bf16 or fp32, any head size: what the tensor-core kernels
 // (attention.cu, attention_prefill_tc.cu) do not take - fp32 models, head sizes other than 64 and 128, many query
 // heads per key head. Causal, optional sliding window (which may keep a sequence's first keys), optional sink per head (exp(sink) in the softmax
-// denominator, no key, no value, not scaled). Cache layout as in attention.cu: K, V = [blocks, Hkv, page, D].
+// denominator, no key, no value, not scaled), optional soft cap of the scores, or sigmoid weights. Cache layout as in attention.cu: K, V = [blocks, Hkv, page, D].
 //
 // One CTA per (query token, up to four query heads of one key head); keys stream through shared memory in small
 // tiles with an online softmax, all in fp32.
@@ -34,6 +34,8 @@ struct AnyArgs {
   int Hq, Hkv, D, page, max_blocks, window, keep;
   int64_t num_blocks;
   float scale;
+  float softcap;          // scores: softcap * tanh(score / softcap) (0: none)
+  const float* sig_bias;  // [Hq]: weights sigmoid(score + bias), not normalised (null: softmax)
   int* status;
 };
 
@@ -91,10 +93,16 @@ __global__ void __launch_bounds__(kThreads) attn_any_kernel(const AnyArgs a) {
       float d = 0.f;
       for (int i = lane; i < D; i += 32) d = fmaf(q[h * D + i], ks[k * D + i], d);
       d = warp_reduce_sum(d);
-      if (lane == 0) s[h * kTile + k] = d * a.scale;
+      if (lane == 0) {
+        float x = d * a.scale;
+        if (a.softcap > 0.f) x = a.softcap * tanhf(x / a.softcap);
+        s[h * kTile + k] = a.sig_bias ? 1.f / (1.f + expf(-(x + a.sig_bias[h0 + h]))) : x;
+      }
     }
     __syncthreads();
-    if (threadIdx.x < nh) {
+    if (threadIdx.x < nh && a.sig_bias) {
+      st[2 * kHG + threadIdx.x] = 1.f;
+    } else if (threadIdx.x < nh) {
       const int h = threadIdx.x;
       float m = st[h];
       for (int k = 0; k < n; ++k) m = fmaxf(m, s[h * kTile + k]);
@@ -122,7 +130,9 @@ __global__ void __launch_bounds__(kThreads) attn_any_kernel(const AnyArgs a) {
   for (int i = threadIdx.x; i < nh * D; i += kThreads) {
     const int h = i / D;
     float m = st[h], l = st[kHG + h], f = 1.f;
-    if (a.sinks) {
+    if (a.sig_bias) {
+      l = 1.f;
+    } else if (a.sinks) {
       const float sink = a.sinks[h0 + h], mm = fmaxf(m, sink);
       f = expf(m - mm);
       l = l * f + expf(sink - mm);
@@ -147,10 +157,11 @@ int launch_any(const AnyArgs& a, int B, int max_q, cudaStream_t stream) {
 PXL_EXPORT int pxl_attn_any(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const int* block_tables,
                             const int* cu_q, const int* ctx_lens, void* out, int64_t out_stride, const float* sinks, int B,
                             int max_q, int Hq, int Hkv, int D, int page, int max_blocks, int64_t num_blocks, float scale,
-                            int window, int keep_first, int is_f32, int* status, cudaStream_t stream) {
+                            int window, int keep_first, float softcap, const float* sig_bias, int is_f32, int* status,
+                            cudaStream_t stream) {
   if (B <= 0 || max_q <= 0) return PXL_OK;
   if (Hkv <= 0 || Hq % Hkv || D <= 0 || page <= 0 || B > 65535) return PXL_ERR_INVALID_ARG;
   AnyArgs a{q, q_stride, k_cache, v_cache, block_tables, cu_q, ctx_lens, out, out_stride, sinks, Hq, Hkv, D, page, max_blocks,
-            window, keep_first, num_blocks, scale, status};
+            window, keep_first, num_blocks, scale, softcap, sig_bias, status};
   return is_f32 ? launch_any<float>(a, B, max_q, stream) : launch_any<pxl::bf16>(a, B, max_q, stream);
 }

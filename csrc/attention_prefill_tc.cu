@@ -21,6 +21,7 @@
 //
 // Reference counterpart: the MLX SDPA call with a gathered KV prefix
 // (src/parallax/server/cache/prefix_cache_utils.py:11-91, src/parallax/models/qwen3.py:84-120).
+#include "attention_score.cuh"
 #include "common.cuh"
 #include "pxl_api.h"
 
@@ -66,12 +67,14 @@ __device__ __forceinline__ float fast_exp2(float x) {  // 2^x, -inf -> 0
 constexpr uint32_t kIdescS = umma_idesc(kQ, kT, 1, 1);
 constexpr uint32_t kIdescPV = umma_idesc(kQ, 64, 1, 1) | (1u << 16);  // B (V) is MN-major
 
+template <int SM>
 __global__ void __launch_bounds__(kThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                        const __grid_constant__ CUtensorMap tm_v, const int* __restrict__ block_tables,
                        const int* __restrict__ cu_q, const int* __restrict__ ctx_lens, bf16* __restrict__ out,
                        int64_t out_stride, const float* __restrict__ sinks, int Hq, int Hkv, int page_size,
-                       int max_blocks, int64_t num_blocks, float scale_log2, int window, int keep, int* status) {
+                       int max_blocks, int64_t num_blocks, float scale_log2, int window, int keep, const ScoreArgs sa,
+                       int* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sm0 = smem_u32(smem);
@@ -231,7 +234,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const uint32_t p_row = sm0 + kOffP + hc * kHalf + r * 128;  // this thread's 64 keys = one swizzled 128-byte row
     float* mx_sm = reinterpret_cast<float*>(smem + kOffXchg);    // [tile parity][half][row]
     float* l_sm = mx_sm + 2 * 2 * 128;                           // [half][row]
-    float m_run = -INFINITY, l_run = 0.f;
+    float m_run = SM == kSigmoid ? 0.f : -INFINITY, l_run = 0.f;
+    const float bias2 = SM == kSigmoid ? sa.bias[head] * kLog2eF : 0.f;
     // 1 after a wait ran out; agreed among the 256 softmax threads at the barrier of every tile, so
     // that they all leave the loop at the same place
     int failed = 0;
@@ -266,6 +270,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         tmem_ld_32x32b_x32(t_s, *reinterpret_cast<uint32_t(*)[32]>(&sc[0]));
         tmem_ld_32x32b_x32(t_s + 32, *reinterpret_cast<uint32_t(*)[32]>(&sc[32]));
         tmem_ld_wait();
+        if constexpr (SM == kCapped) {
+#pragma unroll
+          for (int j = 0; j < 64; ++j) sc[j] = __float_as_uint(score_log2<SM>(__uint_as_float(sc[j]), 0.f, sa));
+        }
         if (!interior) {
           // keys this thread's row may see among its 64 columns: [a, e), and those before f
           const int key0 = tile_key0 + hc * 64;
@@ -274,25 +282,29 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
           for (int j = 0; j < 64; ++j)
             if ((j < a && j >= f) || j >= e) sc[j] = 0xff800000u;  // -inf
         }
-        float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        if constexpr (SM != kSigmoid) {
+          float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-        for (int j = 0; j < 64; j += 4) {
+          for (int j = 0; j < 64; j += 4) {
 #pragma unroll
-          for (int k = 0; k < 4; ++k) m4[k] = fmaxf(m4[k], __uint_as_float(sc[j + k]));
+            for (int k = 0; k < 4; ++k) m4[k] = fmaxf(m4[k], __uint_as_float(sc[j + k]));
+          }
+          mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
         }
-        mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
       }
-      mx_sm[((it & 1) * 2 + hc) * 128 + r] = mx;
+      if constexpr (SM != kSigmoid) mx_sm[((it & 1) * 2 + hc) * 128 + r] = mx;
       failed = agree(failed);
       if (failed) break;
-      mx = fmaxf(mx, mx_sm[((it & 1) * 2 + (hc ^ 1)) * 128 + r]) * scale_log2;  // scale > 0
+      // (sigmoid weights need no reference maximum: O is never rescaled; capped scores are exponents already)
+      if constexpr (SM != kSigmoid)
+        mx = fmaxf(mx, mx_sm[((it & 1) * 2 + (hc ^ 1)) * 128 + r]) * (SM == kCapped ? 1.f : scale_log2);  // scale > 0
       const float m_new = fmaxf(m_run, mx);
       // The output accumulates in TMEM across tiles, relative to the reference maximum m_run. The
       // reference only moves (and O is rescaled) when some row of this lane quarter grew by more
       // than 2^8: until then the stale reference keeps every probability below 256, which bf16 and
       // the fp32 sums hold without trouble. Both warps of a lane quarter see the same 32 rows and
       // the same maxima, so they take the same decision.
-      const bool grow = __any_sync(0xffffffffu, m_new > m_run + 8.f);
+      const bool grow = SM != kSigmoid && __any_sync(0xffffffffu, m_new > m_run + 8.f);
       // P of the previous tile must have been consumed (and O be complete) before either is touched
       if (it > 0) failed = mbar_wait_bounded(o_full, (it - 1) & 1, abort_flag, status, PXL_DEV_TIMEOUT_TMEM_FULL) ? 0 : 1;
       failed = __any_sync(0xffffffffu, failed);
@@ -322,8 +334,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         uint32_t pk[4];
 #pragma unroll
         for (int j = 0; j < 8; j += 2) {
-          const float p0 = fast_exp2(fmaf(__uint_as_float(sc[c + j]), scale_log2, -m_use));
-          const float p1 = fast_exp2(fmaf(__uint_as_float(sc[c + j + 1]), scale_log2, -m_use));
+          const float s0 = __uint_as_float(sc[c + j]), s1 = __uint_as_float(sc[c + j + 1]);
+          float p0, p1;
+          if constexpr (SM == kSigmoid) {
+            p0 = sigmoid_weight(s0, scale_log2, bias2);  // (a masked score, -inf, gives 0)
+            p1 = sigmoid_weight(s1, scale_log2, bias2);
+          } else if constexpr (SM == kCapped) {
+            p0 = fast_exp2(s0 - m_use);
+            p1 = fast_exp2(s1 - m_use);
+          } else {
+            p0 = fast_exp2(fmaf(s0, scale_log2, -m_use));
+            p1 = fast_exp2(fmaf(s1, scale_log2, -m_use));
+          }
           sum2[0] += p0;
           sum2[1] += p1;
           pk[j >> 1] = pack_bf16x2(p0, p1);
@@ -354,7 +376,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         f = exp2f(m_run - M);
         denom = denom * f + exp2f(sink - M);
       }
-      const float inv = denom > 0.f ? f / denom : 0.f;
+      const float inv = SM == kSigmoid ? 1.f : denom > 0.f ? f / denom : 0.f;
       bf16* dst = out + static_cast<size_t>(q_begin + q0 + r) * out_stride + head * kD + hc * 64;
       tc_fence_after_sync();
 #pragma unroll
@@ -384,6 +406,25 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
   if (warp == kMmaWarp) tmem_dealloc(tmem_base, 512);
 }
 
+template <int SM>
+int launch_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const int* block_tables, const int* cu_q,
+              const int* ctx_lens, void* out, int64_t out_stride, const float* sinks, int B, int max_q_len, int Hq, int Hkv,
+              int page_size, int max_blocks, int64_t num_blocks, float scale, int window, int keep_first, const ScoreArgs& sa,
+              int* status, cudaStream_t stream) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev >= 0 && dev < 64 && !configured[dev]) {
+    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<SM>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) != cudaSuccess)
+      return PXL_ERR_CUDA;
+    configured[dev] = true;
+  }
+  pxl_host::launch(attn_prefill_tc_kernel<SM>, dim3(ceil_div(max_q_len, kQ), Hq, B), kThreads, kSmemBytes, stream, tq, tk, tv,
+                   block_tables, cu_q, ctx_lens, static_cast<bf16*>(out), out_stride, sinks, Hq, Hkv, page_size, max_blocks,
+                   num_blocks, scale * kLog2eF, window, keep_first, sa, status);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
 }  // namespace
 
 // Same contract as pxl_attn_prefill plus total_q = rows of q / out (sum of the new lengths): the
@@ -392,7 +433,8 @@ PXL_EXPORT int pxl_attn_prefill_tc(const void* q, int64_t q_stride, const void* 
                                    const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                                    int64_t out_stride, const float* sinks, int B, int max_q_len, int total_q, int Hq,
                                    int Hkv, int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                                   int window, int keep_first, int* status, cudaStream_t stream) {
+                                   int window, int keep_first, float softcap, const float* sig_bias, int* status,
+                                   cudaStream_t stream) {
   if (B <= 0 || max_q_len <= 0 || total_q <= 0) return PXL_OK;
   if (D != kD || Hkv <= 0 || Hq % Hkv) return PXL_ERR_INVALID_ARG;
   if (page_size != 16 && page_size != 32 && page_size != 64) return PXL_ERR_INVALID_ARG;
@@ -406,18 +448,14 @@ PXL_EXPORT int pxl_attn_prefill_tc(const void* q, int64_t q_stride, const void* 
       !pxl_host::make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, k_cache, rows, 128, 128, page_size, 64) ||
       !pxl_host::make_tmap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, v_cache, rows, 128, 128, page_size, 64))
     return PXL_ERR_TENSORMAP;
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes) !=
-        cudaSuccess)
-      return PXL_ERR_CUDA;
-    configured[dev] = true;
+  const ScoreArgs sa = score_args(scale, softcap, sig_bias);
+  auto go = [&](auto launch) {
+    return launch(tq, tk, tv, block_tables, cu_q, ctx_lens, out, out_stride, sinks, B, max_q_len, Hq, Hkv, page_size, max_blocks,
+                  num_blocks, scale, window, keep_first, sa, status, stream);
+  };
+  switch (score_mode(softcap, sig_bias)) {
+    case kSigmoid: return go(launch_tc<kSigmoid>);
+    case kCapped: return go(launch_tc<kCapped>);
+    default: return go(launch_tc<kPlain>);
   }
-  dim3 grid(pxl::ceil_div(max_q_len, kQ), Hq, B);
-  pxl_host::launch(attn_prefill_tc_kernel, grid, kThreads, kSmemBytes, stream,
-      tq, tk, tv, block_tables, cu_q, ctx_lens, static_cast<pxl::bf16*>(out), out_stride, sinks, Hq, Hkv, page_size,
-      max_blocks, num_blocks, scale * kLog2eF, window, keep_first, status);
-  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }

@@ -8,6 +8,10 @@
 //  * pxl_conv_state_update: the last taps - 1 projected rows of every prompt slice become the state of its slot
 //    (a launch of its own: the first tokens of the slice read the state that its last tokens replace; a decoded
 //    token reads and replaces it in pxl_conv_qkv_prep itself).
+//  * pxl_head_qkv_prep: the same hand-over for heads that are normed one by one without weights: half-split rotation (or
+//    none), every head of q and k over its root mean square, factors of the queries per head and per position, values mixed
+//    with those of another layer, scatter. A few lanes per head, no barrier.
+//  * pxl_gated_norm_rows: concatenated heads times silu(gate), then RMS norm over equal parts of the row.
 //  * pxl_gated_rows: concatenated heads, optionally RMS-normed together or one by one, times sigmoid(gate) and a factor,
 //    into the columns of the output product's operand.
 //
@@ -445,6 +449,175 @@ __global__ void __launch_bounds__(256) conv_state_update_kernel(const PrepArgs a
   }
 }
 
+struct HeadPrepArgs {
+  const void* proj;  // [T, ld]
+  int64_t ld;
+  int q_off, k_off, v_off, H, G, dk, dv, cols, rot;
+  float eps;
+  const float* cos_sin;     // [max_pos, rot], or null
+  const float* pos_scale;   // [max_pos], or null
+  const float* head_scale;  // [H], or null
+  const int* positions;
+  int max_pos;
+  const void* v_first;      // [T, ldf], or null
+  int64_t ldf;
+  float v_mix;
+  const int64_t* slots;
+  int64_t num_slots;
+  int page;
+  void* k_cache;  // [blocks, G, page, cols]
+  void* v_cache;
+  void* q_out;    // [T, H, cols]
+  int* status;
+};
+
+// LANES neighbouring threads make one head of one token (query heads, key heads, value heads)
+template <typename T, int VEC, int LANES>
+__global__ void __launch_bounds__(256) head_prep_kernel(const HeadPrepArgs a, int64_t items) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x % LANES;
+  int64_t i = static_cast<int64_t>(blockIdx.x) * (256 / LANES) + threadIdx.x / LANES;
+  const bool live = i < items;
+  if (!live) i = items - 1;  // (takes part in the shuffles)
+  const int heads = a.H + 2 * a.G, h = static_cast<int>(i % heads);
+  const int64_t t = i / heads;
+  const bool query = h < a.H, value = h >= a.H + a.G;
+  const int g = value ? h - a.H - a.G : h - a.H;
+  const T* row = static_cast<const T*>(a.proj) + t * a.ld;
+  const T* src = query ? row + a.q_off + h * a.dk : value ? row + a.v_off + g * a.dv : row + a.k_off + g * a.dk;
+  const int width = value ? a.dv : a.dk, half = a.rot / 2;
+  float factor = 1.f;
+  int pos = a.positions[t];
+  if (!value) {
+    float sq = 0.f;
+    for (int d0 = lane * VEC; d0 < width; d0 += LANES * VEC) {
+      float v[VEC];
+      load_v<VEC>(src + d0, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) sq = fmaf(v[j], v[j], sq);
+    }
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    factor = 1.f / sqrtf(sq / width + a.eps);  // (a rotation leaves the norm alone)
+    if ((a.cos_sin || a.pos_scale) && (pos < 0 || pos >= a.max_pos)) {
+      if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_POSITION);
+      pos = 0;
+    }
+    if (query && a.head_scale) factor *= a.head_scale[h];
+    if (query && a.pos_scale) factor *= a.pos_scale[pos];
+  }
+  T* dst = nullptr;
+  if (query) {
+    dst = static_cast<T*>(a.q_out) + (t * a.H + h) * a.cols;
+  } else {
+    const int64_t slot = a.slots[t];
+    if (slot >= a.num_slots) {
+      if (a.status) atomicCAS(a.status, 0, PXL_DEV_BAD_SLOT);
+    } else if (slot >= 0) {
+      const uint32_t us = static_cast<uint32_t>(slot), page = static_cast<uint32_t>(a.page);
+      dst = static_cast<T*>(value ? a.v_cache : a.k_cache) +
+            ((static_cast<int64_t>(us / page) * a.G + g) * a.page + us % page) * a.cols;
+    }
+  }
+  if (!live || dst == nullptr) return;
+  const T* first = value && a.v_first ? static_cast<const T*>(a.v_first) + t * a.ldf + g * a.dv : nullptr;
+  const float* cs = a.cos_sin ? a.cos_sin + static_cast<int64_t>(pos) * a.rot : nullptr;
+  for (int d0 = lane * VEC; d0 < a.cols; d0 += LANES * VEC) {
+    float o[VEC];
+    if (d0 >= width) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+    } else {
+      load_v<VEC>(src + d0, o);
+      if (first) {
+        float f[VEC];
+        load_v<VEC>(first + d0, f);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) o[j] = fmaf(a.v_mix, f[j], (1.f - a.v_mix) * o[j]);
+      } else if (!value) {
+        if (d0 < a.rot) {
+          const bool lower = d0 < half;
+          const int f = lower ? d0 : d0 - half;
+          float c[VEC], sn[VEC], x[VEC];
+          load_v<VEC>(cs + f, c);
+          load_v<VEC>(cs + half + f, sn);
+          load_v<VEC>(src + (lower ? d0 + half : f), x);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) o[j] = lower ? o[j] * c[j] - x[j] * sn[j] : o[j] * c[j] + x[j] * sn[j];
+        }
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) o[j] *= factor;
+      }
+    }
+    store_v<VEC>(dst + d0, o);
+  }
+}
+
+// x [T, n] (the heads of a token) times silu(gate), RMS norm over `groups` equal parts, times w
+struct GatedNormArgs {
+  const void* x;
+  const void* gate;  // [T, ldg]
+  int64_t ldg;
+  const float* w;
+  int n, groups;
+  float eps;
+  void* out;  // [T, ldo], out_cols columns: n, then zeros
+  int64_t ldo;
+  int out_cols;
+};
+
+template <typename T, int VEC>
+__device__ __forceinline__ void gated_vector(const T* x, const T* g, float (&v)[VEC]) {
+  float z[VEC];
+  load_v<VEC>(x, v);
+  load_v<VEC>(g, z);
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) v[j] *= z[j] / (1.f + expf(-z[j]));
+}
+
+// eight warps: several per part, or several parts one after the other for a warp
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) gated_norm_rows_kernel(const GatedNormArgs a) {
+  __shared__ float sums[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const T* x = static_cast<const T*>(a.x) + t * a.n;
+  const T* gate = static_cast<const T*>(a.gate) + t * a.ldg;
+  T* out = static_cast<T*>(a.out) + t * a.ldo;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int share = a.groups >= 8 ? 1 : a.groups >= 4 ? 2 : a.groups >= 2 ? 4 : 8;  // warps per part
+  const int per = a.n / a.groups, sub = warp % share;
+  for (int g0 = 0; g0 < a.groups; g0 += 8 / share) {
+    const int g = g0 + warp / share;
+    const bool mine = g < a.groups;
+    float sq = 0.f;
+    for (int c = (sub * 32 + lane) * VEC; mine && c < per; c += share * 32 * VEC) {
+      float v[VEC];
+      gated_vector<T, VEC>(x + g * per + c, gate + g * per + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) sq = fmaf(v[j], v[j], sq);
+    }
+    sq = warp_reduce_sum(sq);
+    if (lane == 0) sums[warp] = sq;
+    __syncthreads();
+    float sum = 0.f;
+    for (int i = 0; i < share; ++i) sum += sums[warp / share * share + i];
+    __syncthreads();
+    const float inv = 1.f / sqrtf(sum / per + a.eps);
+    for (int c = (sub * 32 + lane) * VEC; mine && c < per; c += share * 32 * VEC) {
+      float v[VEC], w[VEC];
+      gated_vector<T, VEC>(x + g * per + c, gate + g * per + c, v);
+      load_v<VEC>(a.w + g * per + c, w);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] *= inv * w[j];
+      store_v<VEC>(out + g * per + c, v);
+    }
+  }
+  for (int c = a.n + threadIdx.x; c < a.out_cols; c += blockDim.x) put(out + c, 0.f);
+}
+
 struct GateArgs {
   const void* x;        // [T, heads, x_cols]
   int heads, x_cols, dv;
@@ -588,6 +761,17 @@ int dispatch_prep(const PrepArgs& a, bool update, cudaStream_t stream) {
   return vec ? launch_prep<T, 8>(a, update, stream) : launch_prep<T, 1>(a, update, stream);
 }
 
+template <typename T, int VEC>
+int launch_head_prep(const HeadPrepArgs& a, int T_, cudaStream_t stream) {
+  const int64_t items = static_cast<int64_t>(T_) * (a.H + 2 * a.G);
+  const int vecs = a.cols / VEC;
+  auto grid = [&](int lanes) { return dim3(static_cast<unsigned>((items + 256 / lanes - 1) / (256 / lanes))); };
+  if (vecs <= 8) pxl_host::launch(head_prep_kernel<T, VEC, 8>, grid(8), dim3(256), 0, stream, a, items);
+  else if (vecs <= 16) pxl_host::launch(head_prep_kernel<T, VEC, 16>, grid(16), dim3(256), 0, stream, a, items);
+  else pxl_host::launch(head_prep_kernel<T, VEC, 32>, grid(32), dim3(256), 0, stream, a, items);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
 inline bool bad_prep(const PrepArgs& a) {
   return a.H <= 0 || a.G < 0 || a.dk <= 0 || (a.G && a.dv <= 0) || a.cols < a.dk || (a.G && a.cols < a.dv) || a.rot < 0 ||
          a.rot > a.dk || (a.rot & 1) || a.taps < 1 || a.page <= 0 || a.num_slots >= (1ll << 31) || (a.q_norm == nullptr && a.conv_w) ||
@@ -628,6 +812,41 @@ PXL_EXPORT int pxl_gated_rows(const void* x, int heads, int x_cols, int dv, cons
   } else {
     if (vec) pxl_host::launch(gated_rows_kernel<pxl::bf16, 8>, dim3(T), dim3(256), smem, stream, a);
     else pxl_host::launch(gated_rows_kernel<pxl::bf16, 1>, dim3(T), dim3(256), smem, stream, a);
+  }
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
+
+PXL_EXPORT int pxl_head_qkv_prep(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int H, int G, int dk, int dv,
+                                 int cols, int rot, float eps, const float* cos_sin, const float* pos_scale,
+                                 const float* head_scale, const int* positions, int max_pos, const void* v_first, int64_t ldf,
+                                 float v_mix, const int64_t* slots, int64_t num_slots, int page, void* k_cache, void* v_cache,
+                                 void* q_out, int T, int is_f32, int* status, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || cols < dk || cols < dv || rot < 0 || rot > dk || (rot & 1) || page <= 0 ||
+      num_slots >= (1ll << 31) || (rot && !cos_sin))
+    return PXL_ERR_INVALID_ARG;
+  const HeadPrepArgs a{proj, ld, q_off, k_off, v_off, H, G, dk, dv, cols, rot, eps, rot ? cos_sin : nullptr, pos_scale, head_scale,
+                       positions, max_pos, v_first, ldf, v_mix, slots, num_slots, page, k_cache, v_cache, q_out, status};
+  const bool vec = !((q_off | k_off | v_off | dk | dv | cols | (rot / 2) | static_cast<int>(ld) | static_cast<int>(ldf)) & 7) &&
+                   aligned16(proj) && aligned16(v_first) && aligned16(k_cache) && aligned16(v_cache) && aligned16(q_out) &&
+                   aligned16(cos_sin);
+  if (is_f32) return vec ? launch_head_prep<float, 8>(a, T, stream) : launch_head_prep<float, 1>(a, T, stream);
+  return vec ? launch_head_prep<pxl::bf16, 8>(a, T, stream) : launch_head_prep<pxl::bf16, 1>(a, T, stream);
+}
+
+PXL_EXPORT int pxl_gated_norm_rows(const void* x, int n, const void* gate, int64_t ldg, const float* w, int groups, float eps,
+                                   void* out, int64_t ldo, int out_cols, int T, int is_f32, cudaStream_t stream) {
+  if (T <= 0) return PXL_OK;
+  if (n <= 0 || groups <= 0 || n % groups || out_cols < n) return PXL_ERR_INVALID_ARG;
+  const GatedNormArgs a{x, gate, ldg, w, n, groups, eps, out, ldo, out_cols};
+  const bool vec = !((n | (n / groups) | static_cast<int>(ldg) | static_cast<int>(ldo)) & 7) && aligned16(x) && aligned16(gate) &&
+                   aligned16(out) && aligned16(w);
+  if (is_f32) {
+    if (vec) pxl_host::launch(gated_norm_rows_kernel<float, 8>, dim3(T), dim3(256), 0, stream, a);
+    else pxl_host::launch(gated_norm_rows_kernel<float, 1>, dim3(T), dim3(256), 0, stream, a);
+  } else {
+    if (vec) pxl_host::launch(gated_norm_rows_kernel<pxl::bf16, 8>, dim3(T), dim3(256), 0, stream, a);
+    else pxl_host::launch(gated_norm_rows_kernel<pxl::bf16, 1>, dim3(T), dim3(256), 0, stream, a);
   }
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }

@@ -1085,6 +1085,7 @@ int dispatch_epi(int epi, const CUtensorMap& ta, const CUtensorMap& tb, const Ge
     PXL_GEMM_CASE(PXL_EPI_NONE);
     PXL_GEMM_CASE(PXL_EPI_RESIDUAL);
     PXL_GEMM_CASE(PXL_EPI_SILU_MUL);
+    PXL_GEMM_CASE(PXL_EPI_CLIP_GLU);
     PXL_GEMM_CASE(PXL_EPI_F32);
     PXL_GEMM_CASE(PXL_EPI_RS);
     PXL_GEMM_CASE(PXL_EPI_SCATTER);
@@ -1585,15 +1586,17 @@ PXL_EXPORT int pxl_gemm_bf16_heads(const void* A, const void* W, void* C, const 
 // Grouped GEMM over experts: for every m-tile i listed on the device,
 //   C[rows of tile i, :] = A[rows of tile i, :] * W[expert_i]^T
 // A: [P, K] activations permuted so that each expert's tokens are contiguous; W: [E*N, K]
-// (expert matrices stacked); C: [P, N] (N/2 columns with PXL_EPI_SILU_MUL); bias: optional [E*N].
+// (expert matrices stacked); C: [P, N] (N/2 columns with PXL_EPI_SILU_MUL and PXL_EPI_CLIP_GLU, whose clip is `limit`);
+// bias: optional [E*N].
 // max_m_tiles bounds the device-side count and sizes the grid.
 PXL_EXPORT int pxl_gemm_bf16_grouped(const void* A, const void* W, void* C, const void* bias, int P, int E,
                                      int N, int K, int lda, int ldw, int ldc, const int* mt_expert,
                                      const int* mt_row0, const int* mt_row_end, const int* num_mt,
-                                     int max_m_tiles, int epi, int bn, int* status,
+                                     int max_m_tiles, int epi, float limit, int bn, int* status,
                                      cudaStream_t stream) {
   if (P <= 0 || E <= 0 || N <= 0 || K <= 0 || max_m_tiles <= 0) return PXL_ERR_INVALID_ARG;
   if ((K % 8) || (lda % 8) || (ldw % 8) || (ldc % 8) || (N % 8)) return PXL_ERR_INVALID_ARG;
+  if (epi == PXL_EPI_CLIP_GLU && !(limit > 0.f)) return PXL_ERR_INVALID_ARG;
   if (epi == PXL_EPI_RESIDUAL) return PXL_ERR_INVALID_ARG;
   if (bn == 0) bn = (N % 256 == 0 && N >= 1024) ? 256 : 128;
   if (N % bn) return PXL_ERR_INVALID_ARG;  // a tile must not straddle two experts' rows of W
@@ -1609,6 +1612,7 @@ PXL_EXPORT int pxl_gemm_bf16_grouped(const void* A, const void* W, void* C, cons
   ep.residual = nullptr;
   ep.bias = static_cast<const pxl::bf16*>(bias);  // optional [E * N], applied with PXL_EPI_NONE / F32
   ep.ldc = ldc;
+  ep.act_limit = limit;
   GemmGroupArgs grp{mt_expert, mt_row0, mt_row_end, num_mt, N, 0, 0, 0};
   const int max_tiles = max_m_tiles * pxl::ceil_div(N, bn);
   switch (bn) {

@@ -1,10 +1,19 @@
-// Matrix memory (mLSTM): linear attention whose decay and input weight are gates of the token. Per head, in fp32,
+// Linear attention over a matrix state whose decay and input weight are gates of the token, in two forms.
+//
+// Matrix memory (mLSTM), per head, in fp32,
 //
 //   i = cap tanh((gi + bi) / cap)   f = log sigmoid(cap tanh((gf + bf) / cap))   (logarithms)
 //   m' = max(f + m, i)              S' = e^(f + m - m') S + e^(i - m') k v^T     n' = e^(f + m - m') n + e^(i - m') k
 //   o  = S'^T q / (max(|n' . q|, e^-m') + 1e-6),                                 q scaled by dk^-1/2
 //
-// State slots [slots, H, words] fp32: S [dk, dv], then for every slice of 32 columns of v a copy of n [dk], then the
+// State space (Mamba-2, kSpace), with q = C and k = B shared by the heads of a group,
+//
+//   d = softplus(dt + bias)   S' = e^(-a d) S + d k v^T   o = S'^T q + D v,      a = e^A_log
+//
+// whose state slot is S [dk, dv] alone. In the chunked kernel it is the case m_0 = 0, M_t = -F_t with F_t = -a times the sum
+// of d, a_j = ln d_j - F_j, without a normaliser.
+//
+// State slots of the matrix memory [slots, H, words] fp32: S [dk, dv], then for every slice of 32 columns of v a copy of n [dk], then the
 // slices' copies of m (all equal). A CTA owns whole slices with their copies, so the CTAs of a head never wait for one
 // another and none reads what another one writes. A sequence whose first token of this step sits at position 0 starts
 // from zero (m too). Two kernels share the state:
@@ -53,8 +62,12 @@ struct MemoryArgs {
   void* out;  // [T, ldo]: heads side by side
   int64_t ldo;
   int* status;
+  int rep = 1;                  // heads that share q and k
+  const float* A_log = nullptr;  // kSpace: [H]
+  const float* D = nullptr;      // kSpace: [H]
 };
 
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
@@ -71,7 +84,7 @@ __device__ __forceinline__ float* state_of(const MemoryArgs& a, int seq, int h) 
 // ---- recurrent ---------------------------------------------------------------------------------------------
 // 256 threads = 8 row lanes x 32 column lanes of VW columns; R rows of S per thread in registers (R == 0: the state
 // stays in global memory, any dk).
-template <typename T, int VW, int R>
+template <typename T, int VW, int R, bool kSpace>
 __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs a, int seq0) {
   extern __shared__ float sm[];
   pdl_wait();
@@ -92,8 +105,8 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
   const int slices = ceil_div(a.dv, kSlice), slice0 = blockIdx.y * VW, own = min(VW, slices - slice0);
   float* ng = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(slice0) * a.dk;
   float* mg = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(slices) * a.dk + slice0;
-  float m = fresh ? 0.f : *mg;
-  const bool owns_n = threadIdx.x < a.dk;  // (stored below, so that the loads of S do not wait for it)
+  float m = fresh || kSpace ? 0.f : *mg;
+  const bool owns_n = !kSpace && threadIdx.x < a.dk;  // (stored below, so that the loads of S do not wait for it)
   const float n_first = owns_n && !fresh ? ng[threadIdx.x] : 0.f;
   constexpr int RR = R > 0 ? R : 1;
   float S[RR][VW];
@@ -125,23 +138,39 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
     for (int r = rl; r < a.dk; r += 8) store_row(r, zero);
   }
   if (owns_n) ns[threadIdx.x] = n_first;
-  for (int i = threadIdx.x + 256; i < a.dk; i += 256) ns[i] = fresh ? 0.f : ng[i];
+  if constexpr (!kSpace)
+    for (int i = threadIdx.x + 256; i < a.dk; i += 256) ns[i] = fresh ? 0.f : ng[i];
+  const int hq = h / a.rep;
+  float rate = 0.f, skip = 0.f;
+  if constexpr (kSpace) rate = expf(a.A_log[h]), skip = a.D[h];
   for (int t = t0; t < t1; ++t) {
     const T* row = static_cast<const T*>(a.proj) + static_cast<int64_t>(t) * a.ld;
     const float* g = a.gates + static_cast<int64_t>(t) * a.ldg;
-    const float li = soft_cap(g[h] + a.bias[h], a.cap);
-    const float lf = log_sigmoid(soft_cap(g[a.H + h] + a.bias[a.H + h], a.cap));
-    const float top = fmaxf(lf + m, li), keep = expf(lf + m - top), take = expf(li - top);
-    m = top;
+    float keep, take;
+    if constexpr (kSpace) {
+      take = softplus(g[h] + a.bias[h]);
+      keep = expf(-rate * take);
+    } else {
+      const float li = soft_cap(g[h] + a.bias[h], a.cap);
+      const float lf = log_sigmoid(soft_cap(g[a.H + h] + a.bias[a.H + h], a.cap));
+      const float top = fmaxf(lf + m, li);
+      keep = expf(lf + m - top), take = expf(li - top);
+      m = top;
+    }
     float dot = 0.f;
     for (int i = threadIdx.x; i < a.dk; i += 256) {
-      const float q = to_f(row[a.q_off + h * a.dk + i]) * a.scale, k = to_f(row[a.k_off + h * a.dk + i]) * take;
-      const float n = fmaf(keep, ns[i], k);
-      qs[i] = q, ks[i] = k, ns[i] = n;
-      dot = fmaf(n, q, dot);
+      const float q = to_f(row[a.q_off + hq * a.dk + i]) * a.scale, k = to_f(row[a.k_off + hq * a.dk + i]) * take;
+      qs[i] = q, ks[i] = k;
+      if constexpr (!kSpace) {
+        const float n = fmaf(keep, ns[i], k);
+        ns[i] = n;
+        dot = fmaf(n, q, dot);
+      }
     }
-    dot = warp_reduce_sum(dot);
-    if (cl == 0) dens[rl] = dot;
+    if constexpr (!kSpace) {
+      dot = warp_reduce_sum(dot);
+      if (cl == 0) dens[rl] = dot;
+    }
     float v[VW], o[VW];
 #pragma unroll
     for (int c = 0; c < VW; ++c) {
@@ -150,8 +179,10 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
     }
     __syncthreads();
     float den = 0.f;
+    if constexpr (!kSpace) {
 #pragma unroll
-    for (int w = 0; w < 8; ++w) den += dens[w];
+      for (int w = 0; w < 8; ++w) den += dens[w];
+    }
     if constexpr (R > 0) {
 #pragma unroll
       for (int i = 0; i < R; ++i) {
@@ -181,13 +212,14 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
 #pragma unroll
     for (int c = 0; c < VW; ++c) red[(rl * VW + c) * 32 + cl] = o[c];
     __syncthreads();
-    const float inv = 1.f / (fmaxf(fabsf(den), expf(-m)) + kTiny);
+    const float inv = kSpace ? 1.f : 1.f / (fmaxf(fabsf(den), expf(-m)) + kTiny);
     for (int i = threadIdx.x; i < 32 * VW; i += 256) {  // column i of this CTA's slices
       const int col = blockIdx.y * 32 * VW + i;
       if (col < a.dv) {
         float sum = 0.f;
 #pragma unroll
         for (int r = 0; r < 8; ++r) sum += red[(r * VW + i % VW) * 32 + i / VW];
+        if constexpr (kSpace) sum = fmaf(skip, to_f(row[a.v_off + h * a.dv + col]), sum);
         put(static_cast<T*>(a.out) + static_cast<int64_t>(t) * a.ldo + h * a.dv + col, sum * inv);
       }
     }
@@ -199,27 +231,29 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
       if (live && r < a.dk) store_row(r, S[i]);
     }
   }
-  for (int i = threadIdx.x; i < a.dk; i += 256)
-    for (int s = 0; s < own; ++s) ng[static_cast<int64_t>(s) * a.dk + i] = ns[i];
-  if (threadIdx.x < own) mg[threadIdx.x] = m;  // (every thread has read m before the first barrier)
+  if constexpr (!kSpace) {
+    for (int i = threadIdx.x; i < a.dk; i += 256)
+      for (int s = 0; s < own; ++s) ng[static_cast<int64_t>(s) * a.dk + i] = ns[i];
+    if (threadIdx.x < own) mg[threadIdx.x] = m;  // (every thread has read m before the first barrier)
+  }
 }
 
-template <typename T, int VW>
+template <bool kSpace, typename T, int VW>
 int launch_recurrent(const MemoryArgs& a, int seq0, int n, cudaStream_t stream) {
   const dim3 grid(a.H, ceil_div(a.dv, 32 * VW), n);
   const size_t smem = sizeof(float) * (3 * a.dk + 8 + 8 * 32 * VW);
   if (smem > 48 * 1024 || n > 65535) return PXL_ERR_TOO_LARGE;
-  if (a.dk <= 32) pxl_host::launch(memory_recurrent_kernel<T, VW, 4>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 64) pxl_host::launch(memory_recurrent_kernel<T, VW, 8>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 128) pxl_host::launch(memory_recurrent_kernel<T, VW, 16>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 256) pxl_host::launch(memory_recurrent_kernel<T, VW, 32>, grid, dim3(256), smem, stream, a, seq0);
-  else pxl_host::launch(memory_recurrent_kernel<T, VW, 0>, grid, dim3(256), smem, stream, a, seq0);
+  if (a.dk <= 32) pxl_host::launch(memory_recurrent_kernel<T, VW, 4, kSpace>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 64) pxl_host::launch(memory_recurrent_kernel<T, VW, 8, kSpace>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 128) pxl_host::launch(memory_recurrent_kernel<T, VW, 16, kSpace>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 256) pxl_host::launch(memory_recurrent_kernel<T, VW, 32, kSpace>, grid, dim3(256), smem, stream, a, seq0);
+  else pxl_host::launch(memory_recurrent_kernel<T, VW, 0, kSpace>, grid, dim3(256), smem, stream, a, seq0);
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }
-template <typename T>
+template <bool kSpace, typename T>
 int launch_recurrent(const MemoryArgs& a, int seq0, int n, cudaStream_t stream) {
   const bool vec = !((a.dv | static_cast<int>(a.words)) & 3) && (reinterpret_cast<uintptr_t>(a.state) & 15) == 0;
-  return vec ? launch_recurrent<T, 4>(a, seq0, n, stream) : launch_recurrent<T, 1>(a, seq0, n, stream);
+  return vec ? launch_recurrent<kSpace, T, 4>(a, seq0, n, stream) : launch_recurrent<kSpace, T, 1>(a, seq0, n, stream);
 }
 
 // ---- chunked -----------------------------------------------------------------------------------------------
@@ -262,7 +296,7 @@ struct ChunkSmem {
 };
 
 // grid (slices of v, heads, sequences). Per chunk: stage q, k, v | scores and S_0^T q | P v, new state.
-template <int DK>
+template <int DK, bool kSpace>
 __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryArgs a) {
   extern __shared__ __align__(16) uint8_t raw[];
   using Sm = ChunkSmem<DK>;
@@ -276,7 +310,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
   if (Sg == nullptr) return;
   float* ng = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(blockIdx.x) * a.dk;
   float* mg = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(ceil_div(a.dv, kSlice)) * a.dk + blockIdx.x;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, hq = h / a.rep;
   const int mi = lane >> 3, r8 = lane & 7;
   const bool fresh = a.positions[t0] == 0;
 
@@ -294,7 +328,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
         const int r = m0 + (lane >> 2) + (e >> 1) * 8, c = v0 + n0 + j * 8 + (lane & 3) * 2 + (e & 1);
         S[i][j][e] = (!fresh && tile < kTiles && r < a.dk && c < a.dv) ? Sg[static_cast<int64_t>(r) * a.dv + c] : 0.f;
       }
-    if (i < NN) {
+    if (!kSpace && i < NN) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = m0 + (lane >> 2) + (e >> 1) * 8;
@@ -317,7 +351,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
           *reinterpret_cast<uint32_t*>(&s.s_hi[r][c]) = hi;
           *reinterpret_cast<uint32_t*>(&s.s_lo[r][c]) = lo;
         }
-      if (i < NN && tile < kTilesK) {
+      if (!kSpace && i < NN && tile < kTilesK) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int r = m0 + (lane >> 2) + e * 8, c = kSlice + (lane & 3) * 2;
@@ -332,25 +366,32 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
   publish_state();
 
   // gates of a chunk, by one warp: two neighbouring tokens per lane, prefix sums and maxima across the lanes
-  float m = fresh ? 0.f : *mg;   // running maximum (natural units) after the chunks prepared so far; used by the gate warp
+  float m = fresh || kSpace ? 0.f : *mg;   // running maximum (natural units) after the chunks prepared so far; used by the gate warp
   float raw_i[2], raw_f[2];      // gates of the chunk that is prepared next
+  float rate = 0.f, skip = 0.f;
+  if constexpr (kSpace) rate = expf(a.A_log[h]), skip = a.D[h];
   auto fetch_gates = [&](int c0) {
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
       const int t = c0 + lane * 2 + u;
       const float* g = a.gates + static_cast<int64_t>(t0 + t) * a.ldg;
       raw_i[u] = t < n_all ? g[h] : 0.f;
-      raw_f[u] = t < n_all ? g[a.H + h] : 0.f;
+      if constexpr (!kSpace) raw_f[u] = t < n_all ? g[a.H + h] : 0.f;
     }
   };
   auto prepare_gates = [&](int c0, ChunkGates& g) {
-    const float bi = a.bias[h], bf = a.bias[a.H + h];
     float F[2], A[2], M[2];
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
       const bool in = c0 + lane * 2 + u < n_all;
-      F[u] = in ? log_sigmoid(soft_cap(raw_f[u] + bf, a.cap)) : 0.f;
-      A[u] = in ? soft_cap(raw_i[u] + bi, a.cap) : -INFINITY;
+      if constexpr (kSpace) {
+        const float d = softplus(raw_i[u] + a.bias[h]);
+        F[u] = in ? -rate * d : 0.f;
+        A[u] = in ? logf(d) : -INFINITY;
+      } else {
+        F[u] = in ? log_sigmoid(soft_cap(raw_f[u] + a.bias[a.H + h], a.cap)) : 0.f;
+        A[u] = in ? soft_cap(raw_i[u] + a.bias[h], a.cap) : -INFINITY;
+      }
     }
     F[1] += F[0];
     float sum = F[1];
@@ -371,8 +412,8 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
     }
     float prev = __shfl_up_sync(0xffffffffu, top, 1);
     if (lane == 0) prev = -INFINITY;
-    M[0] = fmaxf(fmaxf(m, prev), A[0]);
-    M[1] = fmaxf(M[0], A[1]);
+    M[0] = kSpace ? -F[0] : fmaxf(fmaxf(m, prev), A[0]);
+    M[1] = kSpace ? -F[1] : fmaxf(M[0], A[1]);
     const float last_M = __shfl_sync(0xffffffffu, M[1], 31), last_F = __shfl_sync(0xffffffffu, F[1], 31);
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -384,7 +425,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
       g.floor[j] = expf(-(F[u] + M[u]));
     }
     if (lane == 0) g.all = expf(m - last_M);
-    m = last_F + last_M;
+    m = kSpace ? 0.f : last_F + last_M;
   };
 
   // rows of the next chunk travel through registers while this one is computed
@@ -397,7 +438,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
     for (int i = 0; i < kVecQ; ++i) {
       const int x = i * kWarps * 32 + tid, r = x / (DK / 8), d = x % (DK / 8) * 8;
       const bool in = c0 + r < n_all && d < a.dk;
-      const bf16* p = base + static_cast<int64_t>(c0 + r) * a.ld + h * a.dk + d;
+      const bf16* p = base + static_cast<int64_t>(c0 + r) * a.ld + hq * a.dk + d;
       rq[i] = in ? ld_bf16x8(p + a.q_off) : zero8;
       rk[i] = in ? ld_bf16x8(p + a.k_off) : zero8;
     }
@@ -471,10 +512,12 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
         ldmatrix_x4_trans(b, smem_u32(&s.s_lo[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
         mma2(o[0], qa, b[0], b[1]);
         mma2(o[1], qa, b[2], b[3]);
+        if constexpr (!kSpace) {
         const bf16* nrow = mi < 2 ? &s.s_hi[kk * 16 + (mi & 1) * 8 + r8][kSlice] : &s.s_lo[kk * 16 + (mi & 1) * 8 + r8][kSlice];
         ldmatrix_x4_trans(b, smem_u32(nrow));
         mma2(o[2], qa, b[0], b[1]);
         mma2(o[2], qa, b[2], b[3]);
+        }
       }
       if (needed) {
         const float M[2] = {g.M[r_lo], g.M[r_lo + 8]};
@@ -515,15 +558,15 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
       ldmatrix_x4(pa, smem_u32(&s.p_hi[rg * 16 + (mi & 1) * 8 + r8][kk * 16 + (mi >> 1) * 8]));
       mma2(o[0], pa, b[0], b[1]);
       mma2(o[1], pa, b[2], b[3]);
-      mma2(o[2], pa, ones, ones);
+      if constexpr (!kSpace) mma2(o[2], pa, ones, ones);
       ldmatrix_x4(pa, smem_u32(&s.p_lo[rg * 16 + (mi & 1) * 8 + r8][kk * 16 + (mi >> 1) * 8]));
       mma2(o[0], pa, b[0], b[1]);
       mma2(o[1], pa, b[2], b[3]);
-      mma2(o[2], pa, ones, ones);
+      if constexpr (!kSpace) mma2(o[2], pa, ones, ones);
     }
-    float inv[2];
+    float inv[2] = {1.f, 1.f};
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
+    for (int e = 0; e < 2 && !kSpace; ++e) {
       const float den = __shfl_sync(0xffffffffu, o[2][2 * e], lane & ~3);
       inv[e] = 1.f / (fmaxf(fabsf(den), g.floor[r_lo + e * 8]) + kTiny);
     }
@@ -532,6 +575,11 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = r_lo + e * 8, c = v0 + ch * 16 + j * 8 + (lane & 3) * 2;
+        if constexpr (kSpace) {
+          const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(&s.v[r][c - v0]));
+          o[j][2 * e] = fmaf(skip, v.x, o[j][2 * e]);
+          o[j][2 * e + 1] = fmaf(skip, v.y, o[j][2 * e + 1]);
+        }
         if (r < n && c < a.dv)
           *reinterpret_cast<uint32_t*>(static_cast<bf16*>(a.out) + static_cast<int64_t>(t0 + c0 + r) * a.ldo + h * a.dv + c) =
               pack_bf16x2(o[j][2 * e] * inv[e], o[j][2 * e + 1] * inv[e]);
@@ -541,7 +589,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
     for (int i = 0; i < NT; ++i) {
       const int tile = warp + i * kWarps, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
       if (tile >= kTiles) continue;
-      const bool with_n = i < NN && tile < kTilesK;
+      const bool with_n = !kSpace && i < NN && tile < kTilesK;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -587,7 +635,7 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
         const int r = m0 + (lane >> 2) + (e >> 1) * 8, c = v0 + n0 + j * 8 + (lane & 3) * 2 + (e & 1);
         if (tile < kTiles && r < a.dk && c < a.dv) Sg[static_cast<int64_t>(r) * a.dv + c] = S[i][j][e];
       }
-    if (i < NN && tile < kTilesK && (lane & 3) == 0) {
+    if (!kSpace && i < NN && tile < kTilesK && (lane & 3) == 0) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = m0 + (lane >> 2) + e * 8;
@@ -595,27 +643,45 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
       }
     }
   }
-  if (warp == kGateWarp && lane == 0) *mg = m;
+  if (!kSpace && warp == kGateWarp && lane == 0) *mg = m;
 }
 
-template <int DK>
+template <bool kSpace, int DK>
 int launch_chunk(const MemoryArgs& a, int n, cudaStream_t stream) {
   constexpr int smem = sizeof(ChunkSmem<DK>);
   static bool done[64] = {false};
   const int dev = pxl_host::current_device_slot();
   if (!done[dev]) {
-    if (cudaFuncSetAttribute(memory_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(memory_chunk_kernel<DK, kSpace>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
       return PXL_ERR_CUDA;
     done[dev] = true;
   }
   if (n > 65535) return PXL_ERR_TOO_LARGE;
-  pxl_host::launch(memory_chunk_kernel<DK>, dim3(ceil_div(a.dv, kSlice), a.H, n), dim3(kWarps * 32), smem, stream, a);
+  pxl_host::launch(memory_chunk_kernel<DK, kSpace>, dim3(ceil_div(a.dv, kSlice), a.H, n), dim3(kWarps * 32), smem, stream, a);
   return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
 }
 
 inline bool chunkable(const MemoryArgs& a) {
   return a.dk <= 256 && !((a.q_off | a.k_off | a.v_off | a.dk | a.dv | static_cast<int>(a.ld) | static_cast<int>(a.ldo)) & 7) &&
          ((reinterpret_cast<uintptr_t>(a.proj) | reinterpret_cast<uintptr_t>(a.out)) & 15) == 0;
+}
+
+template <bool kSpace>
+int run(const MemoryArgs& a, int prefill_seqs, int decode_seqs, int is_f32, cudaStream_t stream) {
+  int code = PXL_OK;
+  if (prefill_seqs > 0) {
+    if (is_f32) code = launch_recurrent<kSpace, float>(a, 0, prefill_seqs, stream);
+    else if (!chunkable(a)) code = launch_recurrent<kSpace, bf16>(a, 0, prefill_seqs, stream);
+    else if (a.dk <= 32) code = launch_chunk<kSpace, 32>(a, prefill_seqs, stream);
+    else if (a.dk <= 64) code = launch_chunk<kSpace, 64>(a, prefill_seqs, stream);
+    else if (a.dk <= 96) code = launch_chunk<kSpace, 96>(a, prefill_seqs, stream);
+    else if (a.dk <= 128) code = launch_chunk<kSpace, 128>(a, prefill_seqs, stream);
+    else code = launch_chunk<kSpace, 256>(a, prefill_seqs, stream);
+  }
+  if (code == PXL_OK && decode_seqs > 0)
+    code = is_f32 ? launch_recurrent<kSpace, float>(a, prefill_seqs, decode_seqs, stream)
+                  : launch_recurrent<kSpace, bf16>(a, prefill_seqs, decode_seqs, stream);
+  return code;
 }
 }  // namespace
 
@@ -627,18 +693,15 @@ PXL_EXPORT int pxl_matrix_memory(const void* proj, int64_t ld, int q_off, int k_
   if (words < static_cast<int64_t>(dk) * dv + static_cast<int64_t>(pxl::ceil_div(dv, kSlice)) * (dk + 1)) return PXL_ERR_INVALID_ARG;
   const MemoryArgs a{proj, ld, q_off, k_off, v_off, H, dk, dv, gates, ldg, bias, cap, 1.f / sqrtf(static_cast<float>(dk)), state,
                      words, num_slots, seq_cu, seq_slots, positions, out, ldo, status};
-  int code = PXL_OK;
-  if (prefill_seqs > 0) {
-    if (is_f32) code = launch_recurrent<float>(a, 0, prefill_seqs, stream);
-    else if (!chunkable(a)) code = launch_recurrent<pxl::bf16>(a, 0, prefill_seqs, stream);
-    else if (dk <= 32) code = launch_chunk<32>(a, prefill_seqs, stream);
-    else if (dk <= 64) code = launch_chunk<64>(a, prefill_seqs, stream);
-    else if (dk <= 96) code = launch_chunk<96>(a, prefill_seqs, stream);
-    else if (dk <= 128) code = launch_chunk<128>(a, prefill_seqs, stream);
-    else code = launch_chunk<256>(a, prefill_seqs, stream);
-  }
-  if (code == PXL_OK && decode_seqs > 0)
-    code = is_f32 ? launch_recurrent<float>(a, prefill_seqs, decode_seqs, stream)
-                  : launch_recurrent<pxl::bf16>(a, prefill_seqs, decode_seqs, stream);
-  return code;
+  return run<false>(a, prefill_seqs, decode_seqs, is_f32, stream);
+}
+
+PXL_EXPORT int pxl_state_space(const void* x, int64_t ld, int x_off, int b_off, int c_off, int H, int groups, int n, int dv,
+                               const float* dt, int64_t ldt, const float* dt_bias, const float* A_log, const float* D, float* state,
+                               int num_slots, const int* seq_cu, const int* seq_slots, const int* positions, void* out, int64_t ldo,
+                               int prefill_seqs, int decode_seqs, int is_f32, int* status, cudaStream_t stream) {
+  if (H <= 0 || groups <= 0 || H % groups || n <= 0 || dv <= 0) return PXL_ERR_INVALID_ARG;
+  const MemoryArgs a{x, ld, c_off, b_off, x_off, H, n, dv, dt, ldt, dt_bias, 1.f, 1.f, state, static_cast<int64_t>(n) * dv,
+                     num_slots, seq_cu, seq_slots, positions, out, ldo, status, H / groups, A_log, D};
+  return run<true>(a, prefill_seqs, decode_seqs, is_f32, stream);
 }

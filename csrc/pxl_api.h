@@ -147,8 +147,11 @@ int pxl_attn_decode(const void* q, int64_t q_stride, const void* k_cache, const 
                     const int* block_tables, const int* ctx_lens, void* out, float* workspace,
                     const float* sinks, int B, int Hq, int Hkv, int D, int page_size,
                     int max_blocks, int64_t num_blocks, float scale, int window, int keep_first, int num_splits,
-                    int max_ctx, int* status, pxl_stream_t stream);
+                    int max_ctx, float softcap, const float* sig_bias, int* status, pxl_stream_t stream);
 int pxl_attn_decode_splits(int B, int Hkv, int max_ctx);
+
+// softcap > 0: scores become softcap * tanh(score / softcap). sig_bias [Hq]: the weight of a key is sigmoid(score + bias) and
+// nothing normalises the weights (sinks do not count then). The same in the prefill entry points.
 
 // ---- attention_prefill.cu ----------------------------------------------------
 // Ragged causal attention of new query tokens against the paged cache, which must
@@ -159,7 +162,7 @@ int pxl_attn_prefill(const void* q, int64_t q_stride, const void* k_cache, const
                      const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                      int64_t out_stride, const float* sinks, int B, int max_q_len, int Hq, int Hkv,
                      int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                     int window, int keep_first, int* status, pxl_stream_t stream);
+                     int window, int keep_first, float softcap, const float* sig_bias, int* status, pxl_stream_t stream);
 
 // ---- attention_prefill_tc.cu ------------------------------------------------------
 // Same contract on the tcgen05 tensor cores (D = 128, page 16 / 32 / 64). total_q = rows of q / out.
@@ -167,7 +170,7 @@ int pxl_attn_prefill_tc(const void* q, int64_t q_stride, const void* k_cache, co
                         const int* block_tables, const int* cu_q, const int* ctx_lens, void* out,
                         int64_t out_stride, const float* sinks, int B, int max_q_len, int total_q, int Hq,
                         int Hkv, int D, int page_size, int max_blocks, int64_t num_blocks, float scale,
-                        int window, int keep_first, int* status, pxl_stream_t stream);
+                        int window, int keep_first, float softcap, const float* sig_bias, int* status, pxl_stream_t stream);
 
 // ---- sampler.cu ----------------------------------------------------------------
 // Greedy arg-max over logits [B, V] (bf16 if logits_bf16 else fp32, row stride ld).
@@ -203,7 +206,7 @@ int pxl_moe_combine(const void* y_perm, const int* pos_of, const float* w, const
 // Grouped GEMM over experts (see gemm_tcgen05.cu).
 int pxl_gemm_bf16_grouped(const void* A, const void* W, void* C, const void* bias, int P, int E, int N, int K,
                           int lda, int ldw, int ldc, const int* mt_expert, const int* mt_row0,
-                          const int* mt_row_end, const int* num_mt, int max_m_tiles, int epi,
+                          const int* mt_row_end, const int* num_mt, int max_m_tiles, int epi, float limit,
                           int bn, int* status, pxl_stream_t stream);
 
 // Fused tensor-parallel collectives (see gemm_tcgen05.cu for the buffer contracts).
@@ -347,21 +350,23 @@ int pxl_f32_to_bf16(const float* x, void* out, int64_t n, pxl_stream_t stream);
 // x += mult * norm(y) * w in place; low (bf16) receives the sum when y is bf16. kind: PXL_NORM_*.
 int pxl_residual_norm(float* x, const void* y, const float* w, void* low, int T, int W, float eps, float mult, int kind,
                       int y_f32, pxl_stream_t stream);
-// out[t] = norm(x[rows ? rows[t] : t]) * w
+// out[t] = norm(x[rows ? rows[t] : t]) * w; groups > 1 (RMS): statistics of each of that many equal parts of the row
 int pxl_row_norm(const float* x, const float* w, const int* rows, int64_t num_rows, void* out, int T, int W, float eps,
-                 int kind, int out_f32, int* status, pxl_stream_t stream);
+                 int kind, int groups, int out_f32, int* status, pxl_stream_t stream);
 // fp32 form of pxl_act_mul
 int pxl_act_mul_f32(const float* x, float* out, int T, int I, int mode, float limit, pxl_stream_t stream);
 
 // x += y (+ sum_j weights[t, j] * (pos_of[t, j] >= 0 ? rows[pos_of[t, j]] : h[t])) in place; with a norm weight w:
-// low = x / sqrt(mean(x^2) + eps) * w. y, rows, h and low are bf16, or fp32 when y_f32.
+// low = x / sqrt(mean(x^2) + eps) * w, the mean taken over each of `groups` equal parts of the row. y may be null. With y2:
+// x += mult * (y / rms(y) * yw + y2 / rms(y2) * y2w) instead of y. y, y2, rows, h and low are bf16, or fp32 when y_f32.
 int pxl_residual_add(float* x, const void* y, int64_t ldy, const void* rows, int64_t ldr, int64_t num_rows,
                      const int* pos_of, const float* weights, int k, const void* h, const float* w, void* low, int T, int W,
-                     float eps, int y_f32, int* status, pxl_stream_t stream);
+                     float eps, const float* yw, const void* y2, const float* y2w, float mult, int groups, int y_f32,
+                     int* status, pxl_stream_t stream);
 // out[t, c] = act(gate) * up (* sigmoid(row_gate[t * ldg])) of x [T, 2 I] with gate / up columns in alternating groups
-// of 64; mode 0 = silu, 2 = gelu (tanh form)
-int pxl_glu_act(const void* x, const float* row_gate, int64_t ldg, void* out, int64_t ldo, int T, int I, int mode, int is_f32,
-                pxl_stream_t stream);
+// of 64; mode 0 = silu, 1 = clipped GLU with `limit`, 2 = gelu (tanh form)
+int pxl_glu_act(const void* x, const float* row_gate, int64_t ldg, void* out, int64_t ldo, int T, int I, int mode, float limit,
+                int is_f32, pxl_stream_t stream);
 
 // ---- attn_prep.cu: in front of and behind softmax attention with grouped heads ---------------------------
 // proj [T, ld]: q (H x dk columns from q_off), k (G x dk), v (G x dv; G == 0: no keys and values). Convolution taps
@@ -381,12 +386,22 @@ int pxl_conv_qkv_prep(const void* proj, int64_t ld, int q_off, int k_off, int v_
 int pxl_gated_rows(const void* x, int heads, int x_cols, int dv, const void* gate, int64_t ldg, const float* norm_w, float eps,
                    int per_head, float scale, void* out, int64_t ldo, int out_cols, int T, int is_f32, pxl_stream_t stream);
 
+// Heads normed one by one without weights: rotation of the first `rot` dimensions (0: none), q and k over their root mean
+// square, queries times head_scale [H] and pos_scale [max_pos], values (1 - v_mix) v + v_mix v_first ([T, ldf]; null: v).
+int pxl_head_qkv_prep(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int H, int G, int dk, int dv, int cols, int rot,
+                      float eps, const float* cos_sin, const float* pos_scale, const float* head_scale, const int* positions,
+                      int max_pos, const void* v_first, int64_t ldf, float v_mix, const int64_t* slots, int64_t num_slots, int page,
+                      void* k_cache, void* v_cache, void* q_out, int T, int is_f32, int* status, pxl_stream_t stream);
+// out[t] = x[t] * silu(gate[t]) over the root mean square of each of `groups` equal parts, times w; zeros behind the row
+int pxl_gated_norm_rows(const void* x, int n, const void* gate, int64_t ldg, const float* w, int groups, float eps, void* out,
+                        int64_t ldo, int out_cols, int T, int is_f32, pxl_stream_t stream);
+
 // ---- attention_any.cu: paged attention of any head size, bf16 or fp32, on the FMA pipes ------------------
 // Arguments as pxl_attn_prefill; cu_q null: token i is the only query of sequence i.
 int pxl_attn_any(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const int* block_tables,
                  const int* cu_q, const int* ctx_lens, void* out, int64_t out_stride, const float* sinks, int B, int max_q,
                  int Hq, int Hkv, int D, int page, int max_blocks, int64_t num_blocks, float scale, int window, int keep_first,
-                 int is_f32, int* status, pxl_stream_t stream);
+                 float softcap, const float* sig_bias, int is_f32, int* status, pxl_stream_t stream);
 
 // ---- lightning_attn.cu: linear attention with a fixed decay per head ------------------------------------
 // q, k [T, H x dk] and v [T, H x dv] are columns of proj, all passed through silu here. state [slots, H, dk, dv] fp32,
@@ -433,6 +448,29 @@ int pxl_matrix_memory(const void* proj, int64_t ld, int q_off, int k_off, int v_
                       int64_t ldg, const float* bias, float cap, float* state, int64_t words, int num_slots, const int* seq_cu,
                       const int* seq_slots, const int* positions, void* out, int64_t ldo, int prefill_seqs, int decode_seqs,
                       int is_f32, int* status, pxl_stream_t stream);
+
+// Mamba-2 state space on the same kernels: x (H x dv), B and C (groups x n) are columns of x, dt [T, ldt] fp32 logits; S <-
+// exp(-exp(A_log) d) S + d B x^T, out = S^T C + D x with d = softplus(dt + dt_bias); state [slots, H, n, dv] fp32.
+int pxl_state_space(const void* x, int64_t ld, int x_off, int b_off, int c_off, int H, int groups, int n, int dv, const float* dt,
+                    int64_t ldt, const float* dt_bias, const float* A_log, const float* D, float* state, int num_slots,
+                    const int* seq_cu, const int* seq_slots, const int* positions, void* out, int64_t ldo, int prefill_seqs,
+                    int decode_seqs, int is_f32, int* status, pxl_stream_t stream);
+
+// ---- delta_rule.cu: gated delta rule with a decay per key channel ------------------------------------------
+// q, k [T, Hk x dk] and v [T, H x dv] are columns of x; decay [T, ldd] (H x dk) and beta [T, ldb] (H) fp32 logits, state
+// [slots, H, dk, dv] fp32. Prompt slices in bf16 need `work` (pxl_delta_rule_workspace bytes); without it they run token by token.
+int64_t pxl_delta_rule_workspace(int H, int dk, int dv, int prefill_seqs, int prefill_tokens);
+int pxl_delta_rule(const void* x, int64_t ld, int q_off, int k_off, int v_off, int H, int Hk, int dk, int dv, const float* decay,
+                   int64_t ldd, const float* dt_bias, const float* A_log, const float* beta, int64_t ldb, float* state,
+                   int num_slots, const int* seq_cu, const int* seq_slots, const int* positions, void* out, int64_t ldo,
+                   int prefill_seqs, int prefill_tokens, int decode_seqs, void* work, int64_t work_bytes, int is_f32, int* status,
+                   pxl_stream_t stream);
+
+// ---- short_conv.cu: causal convolution per channel + SiLU ---------------------------------------------------
+// x [T, ldx] (C channels), w [taps, C], bias [C] or null, state [slots, taps - 1, C] (the last inputs), out [T, C].
+int pxl_short_conv(const void* x, int64_t ldx, int C, int taps, const void* w, const void* bias, void* state, int num_slots,
+                   const int* positions, const int* seq_cu, const int* seq_slots, int prefill_seqs, int prefill_tokens, int T,
+                   void* out, int is_f32, int* status, pxl_stream_t stream);
 
 // ---- tanh_norm.cu: the fp32 residual between two products --------------------------------------------------
 // In place: x += norm(y + sum_j weights[t, j] * rows[pos_of[t, j]]) (post 1: tanh(alpha z) w + b, 2: z / rms(z) * w),

@@ -134,11 +134,12 @@ PXL_EXPORT int pxl_stage_forward_dense(const PxlStageDesc* st, const PxlStepDesc
       if (prefill_tc) {
         PXL_TRY(pxl_attn_prefill_tc(qkv, qkv_n, L.k_cache, L.v_cache, sp->p_bt, sp->p_cu_q, sp->p_ctx, attn,
                                     static_cast<int64_t>(Hq) * D, L.sinks, sp->Bp, sp->p_max_q, sp->Tp, Hq, Hkv, D,
-                                    st->page, sp->p_max_blocks, st->num_blocks, st->scale, L.window, 0, status, stream));
+                                    st->page, sp->p_max_blocks, st->num_blocks, st->scale, L.window, 0, 0.f, nullptr, status,
+                                    stream));
       } else {
         PXL_TRY(pxl_attn_prefill(qkv, qkv_n, L.k_cache, L.v_cache, sp->p_bt, sp->p_cu_q, sp->p_ctx, attn,
                                  static_cast<int64_t>(Hq) * D, L.sinks, sp->Bp, sp->p_max_q, Hq, Hkv, D, st->page,
-                                 sp->p_max_blocks, st->num_blocks, st->scale, L.window, 0, status, stream));
+                                 sp->p_max_blocks, st->num_blocks, st->scale, L.window, 0, 0.f, nullptr, status, stream));
       }
       ++n;
     }
@@ -146,7 +147,7 @@ PXL_EXPORT int pxl_stage_forward_dense(const PxlStageDesc* st, const PxlStepDesc
       PXL_TRY(pxl_attn_decode(qkv + static_cast<size_t>(sp->Tp) * qkv_n, qkv_n, L.k_cache, L.v_cache, sp->d_bt,
                               sp->d_ctx, attn + static_cast<size_t>(sp->Tp) * Hq * D, ws->decode, L.sinks, sp->Bd, Hq,
                               Hkv, D, st->page, sp->d_max_blocks, st->num_blocks, st->scale, L.window, 0, splits,
-                              sp->d_max_ctx, status, stream));
+                              sp->d_max_ctx, 0.f, nullptr, status, stream));
       n += splits > 1 ? 2 : 1;
     }
     PXL_TRY(pxl_gemm_bf16(attn, L.w_o, h_mid, h, L.b_o, T, H, Hq * D, Hq * D, Hq * D, H, PXL_EPI_RESIDUAL, 0, status,

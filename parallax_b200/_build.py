@@ -35,8 +35,8 @@ NVCC_FLAGS = [
 ]
 
 
-# Sources whose elementary functions must be accurate in fp32 (arithmetic of a recurrence, tanh norms)
-ACCURATE = ("delta_rule", "matrix_memory", "tanh_norm")
+# Sources whose elementary functions must be accurate in fp32 (arithmetic of a recurrence, tanh norms, fp32 attention)
+ACCURATE = ("attention_any", "delta_rule", "matrix_memory", "tanh_norm")
 
 
 def _flags(src: Path) -> list[str]:

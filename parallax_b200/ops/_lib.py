@@ -78,18 +78,18 @@ _SIGS = {
     "pxl_selftest_bounded_wait": [_P, c_uint32, _P, _P, _P],
     "pxl_patch_i32": [_P, _P, _P, _P, c_int, c_int, c_int, _P, _P],
     "pxl_attn_decode": [_P, c_int64, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
-                        c_int64, c_float, c_int, c_int, c_int, c_int, _P, _P],
+                        c_int64, c_float, c_int, c_int, c_int, c_int, c_float, _P, _P, _P],
     "pxl_attn_decode_splits": [c_int, c_int, c_int],
     "pxl_attn_prefill": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int,
-                         c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_int, _P, _P],
+                         c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_int, c_float, _P, _P, _P],
     "pxl_attn_prefill_tc": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int, c_int,
-                            c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_int, _P, _P],
+                            c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_int, c_float, _P, _P, _P],
     "pxl_moe_route": [_P, c_int64, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, _P, _P],
     "pxl_moe_align": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P, _P],
     "pxl_moe_gather": [_P, _P, _P, _P, c_int, c_int, _P],
     "pxl_moe_combine": [_P, _P, _P, _P, _P, c_int, c_int, c_int, _P],
     "pxl_gemm_bf16_grouped": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P,
-                              c_int, c_int, c_int, _P, _P],
+                              c_int, c_int, c_float, c_int, _P, _P],
     "pxl_mla_kv_prep": [_P, c_int64, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int64, c_float, _P, _P],
     "pxl_mla_q_prep": [_P, c_int64, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
     "pxl_mla_attn": [_P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -117,7 +117,7 @@ _SIGS = {
     "pxl_embed_rows": [_P, _P, c_float, _P, _P, c_int64, c_int64, c_int64, _P, c_int, c_int, c_int64, c_int, _P, _P],
     "pxl_f32_to_bf16": [_P, _P, c_int64, _P],
     "pxl_residual_norm": [_P, _P, _P, _P, c_int, c_int, c_float, c_float, c_int, c_int, _P],
-    "pxl_row_norm": [_P, _P, _P, c_int64, _P, c_int, c_int, c_float, c_int, c_int, _P, _P],
+    "pxl_row_norm": [_P, _P, _P, c_int64, _P, c_int, c_int, c_float, c_int, c_int, c_int, _P, _P],
     "pxl_act_mul_f32": [_P, _P, c_int, c_int, c_int, c_float, _P],
     "pxl_latent_prep": [_P, c_int64, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, _P, _P, c_int64, _P, c_int, c_int, c_int,
                         c_int, c_float, c_int, _P, _P],
@@ -128,13 +128,23 @@ _SIGS = {
                            c_float, c_int, _P, _P],
     "pxl_gemm_bf16_act_glu": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int64, c_int, _P, _P],
     "pxl_gemm_simt_grouped": [_P, _P, _P, _P, c_int, c_int, c_int64, c_int64, c_int64, _P, _P, _P, _P, c_int, c_int, _P],
-    "pxl_residual_add": [_P, _P, c_int64, _P, c_int64, c_int64, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_float, c_int, _P, _P],
-    "pxl_glu_act": [_P, _P, c_int64, _P, c_int64, c_int, c_int, c_int, c_int, _P],
+    "pxl_residual_add": [_P, _P, c_int64, _P, c_int64, c_int64, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_float,
+                         _P, _P, _P, c_float, c_int, c_int, _P, _P],
+    "pxl_glu_act": [_P, _P, c_int64, _P, c_int64, c_int, c_int, c_int, c_float, c_int, _P],
     "pxl_conv_qkv_prep": [_P, c_int64] + [c_int] * 10 + [_P, _P, c_int, _P, _P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, _P,
                           c_int64, c_int, _P, _P, _P, c_float, c_int, _P, _P],
     "pxl_gated_rows": [_P, c_int, c_int, c_int, _P, c_int64, _P, c_float, c_int, c_float, _P, c_int64, c_int, c_int, c_int, _P],
     "pxl_attn_any": [_P, c_int64, _P, _P, _P, _P, _P, _P, c_int64, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int64,
-                     c_float, c_int, c_int, c_int, _P, _P],
+                     c_float, c_int, c_int, c_float, _P, c_int, _P, _P],
+    "pxl_head_qkv_prep": [_P, c_int64] + [c_int] * 9 + [c_float, _P, _P, _P, _P, c_int, _P, c_int64, c_float, _P, c_int64, c_int, _P,
+                          _P, _P, c_int, c_int, _P, _P],
+    "pxl_gated_norm_rows": [_P, c_int, _P, c_int64, _P, c_int, c_float, _P, c_int64, c_int, c_int, c_int, _P],
+    "pxl_short_conv": [_P, c_int64, c_int, c_int, _P, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, _P, c_int, _P, _P],
+    "pxl_state_space": [_P, c_int64] + [c_int] * 7 + [_P, c_int64, _P, _P, _P, _P, c_int, _P, _P, _P, _P, c_int64, c_int, c_int,
+                        c_int, _P, _P],
+    "pxl_delta_rule_workspace": [c_int] * 5,
+    "pxl_delta_rule": [_P, c_int64] + [c_int] * 7 + [_P, c_int64, _P, _P, _P, c_int64, _P, c_int, _P, _P, _P, _P, c_int64, c_int,
+                       c_int, c_int, _P, c_int64, c_int, _P, _P],
     "pxl_latent_rows": [_P, c_int64, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, _P, _P, c_int64, c_int, c_int, c_int, c_int,
                         c_float, c_int, _P, _P],
     "pxl_latent_queries": [_P, c_int64, c_int, c_int, c_int, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P, _P],
@@ -155,6 +165,9 @@ _SIGS = {
 }
 
 
+_SIZES = {"pxl_delta_rule_workspace"}      # functions that return a number of bytes
+
+
 @lru_cache(maxsize=1)
 def lib() -> ctypes.CDLL:
     path = _build.lib_path()
@@ -169,7 +182,7 @@ def lib() -> ctypes.CDLL:
         if fn is None:
             continue
         fn.argtypes = argtypes
-        fn.restype = c_int
+        fn.restype = c_int64 if name in _SIZES else c_int
     return handle
 
 

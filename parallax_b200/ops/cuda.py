@@ -410,7 +410,8 @@ def add_inplace(y: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------ attention
-def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, window, sinks, out, keep_first):
+def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, window, sinks, out, keep_first, softcap,
+              sigmoid_bias):
     """FMA-pipe form: fp32, any head size, any number of query heads per key head."""
     T, Hq, D = q.shape
     Hkv, page = k_cache.shape[1], k_cache.shape[2]
@@ -418,8 +419,8 @@ def _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q, scale, w
     check(_lib.lib().pxl_attn_any(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), block_tables.data_ptr(),
                                   _ptr(cu_q), ctx_lens.data_ptr(), out.data_ptr(), out.stride(0), _ptr(sinks),
                                   ctx_lens.numel(), max_q, Hq, Hkv, D, page, block_tables.shape[1], k_cache.shape[0],
-                                  float(scale), window, keep_first, int(q.dtype == torch.float32), status_tensor(q.device).data_ptr(),
-                                  _stream(q.device)), "pxl_attn_any")
+                                  float(scale), window, keep_first, softcap, _ptr(sigmoid_bias), int(q.dtype == torch.float32),
+                                  status_tensor(q.device).data_ptr(), _stream(q.device)), "pxl_attn_any")
     _count()
     return out
 
@@ -442,6 +443,8 @@ def attn_decode(
     out: Optional[torch.Tensor] = None,
     kv_scale: tuple = (1.0, 1.0),
     keep_first: int = 0,
+    softcap: float = 0.0,
+    sigmoid_bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """q ``[B, Hq, D]`` (may be a strided view into a packed qkv buffer) vs the paged cache (bf16, or e4m3
     with ``kv_scale``). With a ``window`` the first ``keep_first`` keys of a sequence stay visible."""
@@ -451,7 +454,8 @@ def attn_decode(
     if out is None:
         out = torch.empty((B, Hq, D), dtype=q.dtype, device=q.device)
     if not _is_fp8_cache(k_cache) and not _attn_on_tensor_cores(q, k_cache, scale, 16):
-        return _attn_any(q, k_cache, v_cache, block_tables, None, ctx_lens, 1, scale, window, sinks, out, keep_first)
+        return _attn_any(q, k_cache, v_cache, block_tables, None, ctx_lens, 1, scale, window, sinks, out, keep_first, softcap,
+                         sigmoid_bias)
     if max_ctx <= 0:
         max_ctx = block_tables.shape[1] * page
     if num_splits <= 0:
@@ -462,7 +466,7 @@ def attn_decode(
     if num_splits > 1:
         ws = workspace(q.device, "attn_decode", B * Hq * num_splits * (D + 2) * 4)
     if _is_fp8_cache(k_cache):
-        assert keep_first == 0
+        assert keep_first == 0 and softcap == 0 and sigmoid_bias is None
         check(
             _lib.lib().pxl_attn_decode_fp8(
                 q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
@@ -479,7 +483,7 @@ def attn_decode(
             block_tables.data_ptr(), ctx_lens.data_ptr(), out.data_ptr(), _ptr(ws), _ptr(sinks),
             B, Hq, Hkv, D, page,
             block_tables.shape[1], k_cache.shape[0], scale, window, keep_first, num_splits, max_ctx,
-            status_tensor(q.device).data_ptr(), _stream(q.device)),
+            softcap, _ptr(sigmoid_bias), status_tensor(q.device).data_ptr(), _stream(q.device)),
         "pxl_attn_decode",
     )
     _count(2 if num_splits > 1 else 1)
@@ -500,6 +504,8 @@ def attn_prefill(
     out: Optional[torch.Tensor] = None,
     kv_scale: tuple = (1.0, 1.0),
     keep_first: int = 0,
+    softcap: float = 0.0,
+    sigmoid_bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """q ``[T, Hq, D]`` (may be a strided view into a packed qkv buffer)."""
     T, Hq, D = q.shape
@@ -511,9 +517,10 @@ def attn_prefill(
     if T == 0 or B == 0:
         return out
     if not _is_fp8_cache(k_cache) and not _attn_on_tensor_cores(q, k_cache, scale, 64):
-        return _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window, sinks, out, keep_first)
+        return _attn_any(q, k_cache, v_cache, block_tables, cu_q, ctx_lens, max_q_len, scale, window, sinks, out, keep_first,
+                         softcap, sigmoid_bias)
     if _is_fp8_cache(k_cache):
-        assert keep_first == 0
+        assert keep_first == 0 and softcap == 0 and sigmoid_bias is None
         check(
             _lib.lib().pxl_attn_prefill_fp8(
                 q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
@@ -533,8 +540,8 @@ def attn_prefill(
                 q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
                 block_tables.data_ptr(), cu_q.data_ptr(), ctx_lens.data_ptr(), out.data_ptr(),
                 out.stride(0), _ptr(sinks), B, max_q_len, T, Hq, Hkv, D, page, block_tables.shape[1],
-                k_cache.shape[0], scale, window, keep_first, status_tensor(q.device).data_ptr(),
-                _stream(q.device)),
+                k_cache.shape[0], scale, window, keep_first, softcap, _ptr(sigmoid_bias),
+                status_tensor(q.device).data_ptr(), _stream(q.device)),
             "pxl_attn_prefill_tc",
         )
         _count()
@@ -544,8 +551,8 @@ def attn_prefill(
             q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
             block_tables.data_ptr(), cu_q.data_ptr(), ctx_lens.data_ptr(), out.data_ptr(),
             out.stride(0), _ptr(sinks), B, max_q_len, Hq, Hkv, D, page, block_tables.shape[1],
-            k_cache.shape[0], scale, window, keep_first, status_tensor(q.device).data_ptr(),
-            _stream(q.device)),
+            k_cache.shape[0], scale, window, keep_first, softcap, _ptr(sigmoid_bias),
+            status_tensor(q.device).data_ptr(), _stream(q.device)),
         "pxl_attn_prefill",
     )
     _count()
@@ -665,16 +672,16 @@ def moe_gather(x: torch.Tensor, plan: MoEPlan) -> torch.Tensor:
 
 
 def grouped_linear(a: torch.Tensor, w: torch.Tensor, plan: MoEPlan, num_local_experts: int,
-                   epi: int = EPI_NONE, bn: int = 0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   epi: int = EPI_NONE, bn: int = 0, bias: Optional[torch.Tensor] = None, limit: float = 0.0) -> torch.Tensor:
     """``a [P, K]`` (expert-sorted rows) times stacked expert weights ``w [E*N, K]``."""
     P, K = a.shape
     N = w.shape[0] // num_local_experts
-    n_out = N // 2 if epi == EPI_SILU_MUL else N
+    n_out = N // 2 if epi in (EPI_SILU_MUL, EPI_CLIP_GLU) else N
     out = torch.empty((P, n_out), dtype=a.dtype, device=a.device)
     check(_lib.lib().pxl_gemm_bf16_grouped(a.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(bias), P, num_local_experts, N, K,
                                            a.stride(0), w.stride(0), out.stride(0), plan.mt_expert.data_ptr(),
                                            plan.mt_row0.data_ptr(), plan.mt_row_end.data_ptr(),
-                                           plan.num_mt.data_ptr(), plan.max_mt, epi, bn,
+                                           plan.num_mt.data_ptr(), plan.max_mt, epi, limit, bn,
                                            status_tensor(a.device).data_ptr(), _stream(a.device)),
           "pxl_gemm_bf16_grouped")
     _count()
@@ -723,19 +730,20 @@ def moe_scatter_rows(x, plan: MoEPlan, weights) -> torch.Tensor:
     return xp
 
 
-def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool = False):
-    """Gated (SiLU) experts; rows stay in expert order for :func:`residual_add` to pick up. ``w1 [E * 2 I, W]`` gate / up
+def routed_ffn(x, ids, weights, w1, w2, num_experts: int, weighted_input: bool = False, act: int = 0, limit: float = 0.0):
+    """Gated experts (``act`` 0: SiLU, 1: clipped GLU with ``limit``); rows stay in expert order for :func:`residual_add` to pick up. ``w1 [E * 2 I, W]`` gate / up
     rows interleaved per expert, ``w2 [E * N, I]`` (N >= W: padded outputs). Ids >= ``num_experts`` are identity experts.
     ``weighted_input``: the weights multiply the experts' input rows."""
     plan = moe_align(ids, num_experts)
     xp = moe_scatter_rows(x, plan, weights) if weighted_input else None
     if x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
         n = w2.shape[0] // num_experts
-        act = grouped_linear(moe_gather(x, plan) if xp is None else xp, w1, plan, num_experts, epi=EPI_SILU_MUL)
-        y = grouped_linear(act, w2, plan, num_experts, bn=0 if n % 128 == 0 else 64)
+        y = grouped_linear(moe_gather(x, plan) if xp is None else xp, w1, plan, num_experts,
+                           epi=EPI_CLIP_GLU if act == 1 else EPI_SILU_MUL, limit=limit)
+        y = grouped_linear(y, w2, plan, num_experts, bn=0 if n % 128 == 0 else 64)
     else:
         gu = _grouped_simt(x, w1, plan, num_experts, plan.src_tok) if xp is None else _grouped_simt(xp, w1, plan, num_experts, None)
-        y = _grouped_simt(_glu_act(gu, 0), w2, plan, num_experts, None)
+        y = _grouped_simt(_glu_act(gu, act, limit=limit), w2, plan, num_experts, None)
     return y, plan.pos_of, None if weighted_input else weights
 
 
@@ -751,14 +759,14 @@ def _grouped_simt(x, w, plan, num_experts: int, a_rows):
     return out
 
 
-def _glu_act(x, act: int, row_gate=None, out=None):
+def _glu_act(x, act: int, row_gate=None, out=None, limit: float = 0.0):
     T, I = x.shape[0], x.shape[1] // 2
     assert x.is_contiguous()
     if out is None:
         out = torch.empty((T, I), dtype=x.dtype, device=x.device)
     assert out.stride(1) == 1 and out.dtype == x.dtype
     check(_lib.lib().pxl_glu_act(x.data_ptr(), _ptr(row_gate), row_gate.stride(0) if row_gate is not None else 0,
-                                 out.data_ptr(), out.stride(0), T, I, act, int(x.dtype == torch.float32), _stream(x.device)),
+                                 out.data_ptr(), out.stride(0), T, I, act, limit, int(x.dtype == torch.float32), _stream(x.device)),
           "pxl_glu_act")
     _count()
     return out
@@ -1133,13 +1141,13 @@ def residual_norm(x, y, w, eps: float, mult: float = 1.0, kind: int = 0):
     return low
 
 
-def row_norm(x, w, eps: float, kind: int = 0, rows=None, dtype=None):
+def row_norm(x, w, eps: float, kind: int = 0, rows=None, dtype=None, groups: int = 1):
     W = x.shape[1]
     T = x.shape[0] if rows is None else rows.numel()
     assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.is_contiguous() and w.numel() == W
     assert rows is None or rows.dtype == torch.int32
     out = torch.empty((T, W), dtype=dtype or torch.float32, device=x.device)
-    check(_lib.lib().pxl_row_norm(x.data_ptr(), w.data_ptr(), _ptr(rows), x.shape[0], out.data_ptr(), T, W, eps, kind,
+    check(_lib.lib().pxl_row_norm(x.data_ptr(), w.data_ptr(), _ptr(rows), x.shape[0], out.data_ptr(), T, W, eps, kind, groups,
                                   int(out.dtype == torch.float32), status_tensor(x.device).data_ptr(),
                                   _stream(x.device)), "pxl_row_norm")
     _count()
@@ -1210,18 +1218,21 @@ def latent_attn(q_cat, cache, block_tables, cu_q, ctx_lens, scale: float, latent
 
 
 # ---------------------------------------------------------------------------- convolved attention, lightning attention
-def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None):
+def residual_add(x, y, w=None, eps: float = 0.0, routed=None, h=None, groups: int = 1, branches=None):
     T, W = x.shape
-    assert x.dtype == torch.float32 and x.is_contiguous() and y.stride(1) == 1 and y.shape == x.shape
-    low = torch.empty((T, W), dtype=y.dtype, device=x.device) if w is not None else None
     rows, pos_of, weights = routed or (None, None, None)
+    mult, (y, yw), (y2, y2w) = branches or (1.0, (y, None), (None, None))
+    dt = (rows if y is None else y).dtype
+    assert x.dtype == torch.float32 and x.is_contiguous() and (y is None or (y.stride(1) == 1 and y.shape == x.shape))
+    assert y2 is None or (y2.stride() == y.stride() and y2.shape == y.shape and y2.dtype == dt)
+    low = torch.empty((T, W), dtype=dt, device=x.device) if w is not None else None
     if routed:
-        assert rows.dtype == h.dtype == y.dtype and h.is_contiguous() and weights.is_contiguous() and rows.shape[1] >= W
-    check(_lib.lib().pxl_residual_add(x.data_ptr(), y.data_ptr(), y.stride(0), _ptr(rows), rows.stride(0) if routed else 0,
+        assert rows.dtype == h.dtype == dt and h.is_contiguous() and weights.is_contiguous() and rows.shape[1] >= W
+    check(_lib.lib().pxl_residual_add(x.data_ptr(), _ptr(y), W if y is None else y.stride(0), _ptr(rows), rows.stride(0) if routed else 0,
                                       rows.shape[0] if routed else 0, _ptr(pos_of), _ptr(weights),
                                       weights.shape[1] if routed else 0, _ptr(h if routed else None), _ptr(w), _ptr(low), T, W,
-                                      eps, int(y.dtype == torch.float32), status_tensor(x.device).data_ptr(),
-                                      _stream(x.device)), "pxl_residual_add")
+                                      eps, _ptr(yw), _ptr(y2), _ptr(y2w), mult, groups, int(dt == torch.float32),
+                                      status_tensor(x.device).data_ptr(), _stream(x.device)), "pxl_residual_add")
     _count()
     return low
 
@@ -1365,4 +1376,92 @@ def matrix_memory(proj, offs, heads: int, dim: int, vdim: int, gates, gate_bias,
                                        prefill_seqs, n - prefill_seqs, int(proj.dtype == torch.float32),
                                        status_tensor(proj.device).data_ptr(), _stream(proj.device)), "pxl_matrix_memory")
     _count((prefill_seqs > 0) + (n > prefill_seqs))
+    return out
+
+
+# ---------------------------------------------------------------------------- heads without norm weights, delta rule, state space
+def head_qkv_prep(proj, offs, heads: int, kv_heads: int, dim: int, vdim: int, eps: float, cos_sin, positions, slot_mapping, k_cache,
+                  v_cache, q_out, head_scale=None, pos_scale=None, v_first=None, v_mix: float = 0.0):
+    T, cols = proj.shape[0], q_out.shape[2]
+    rot, tables = 0 if cos_sin is None else cos_sin.shape[1], [t.shape[0] for t in (cos_sin, pos_scale) if t is not None]
+    assert proj.stride(1) == 1 and q_out.is_contiguous() and q_out.dtype == k_cache.dtype == v_cache.dtype == proj.dtype
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[1] == kv_heads
+    assert k_cache.shape[3] == v_cache.shape[3] == cols and (head_scale is None or head_scale.numel() == heads)
+    assert v_first is None or (v_first.stride(1) == 1 and v_first.shape == (T, kv_heads * vdim) and v_first.dtype == proj.dtype)
+    check(_lib.lib().pxl_head_qkv_prep(
+        proj.data_ptr(), proj.stride(0), *offs, heads, kv_heads, dim, vdim, cols, rot, eps, _ptr(cos_sin), _ptr(pos_scale),
+        _ptr(head_scale), positions.data_ptr(), min(tables, default=0), _ptr(v_first), v_first.stride(0) if v_first is not None else 0,
+        v_mix, slot_mapping.data_ptr(), k_cache.shape[0] * k_cache.shape[2], k_cache.shape[2], k_cache.data_ptr(), v_cache.data_ptr(),
+        q_out.data_ptr(), T, int(proj.dtype == torch.float32), status_tensor(proj.device).data_ptr(), _stream(proj.device)),
+        "pxl_head_qkv_prep")
+    _count()
+
+
+def short_conv(x, w, bias, state, positions, seq_cu, seq_slots, prefill_seqs: int, prefill_tokens: int):
+    taps, C = w.shape
+    T = x.shape[0]
+    assert x.stride(1) == 1 and x.shape[1] == C and w.is_contiguous() and w.dtype == x.dtype
+    assert bias is None or (bias.numel() == C and bias.dtype == x.dtype)
+    if taps == 1:
+        state = None
+    assert taps == 1 or (state.is_contiguous() and state.dtype == x.dtype and state.shape[1:] == (taps - 1, C))
+    out = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    check(_lib.lib().pxl_short_conv(x.data_ptr(), x.stride(0), C, taps, w.data_ptr(), _ptr(bias), _ptr(state),
+                                    state.shape[0] if state is not None else 0, positions.data_ptr(), seq_cu.data_ptr(),
+                                    seq_slots.data_ptr(), prefill_seqs, prefill_tokens, T, out.data_ptr(),
+                                    int(x.dtype == torch.float32), status_tensor(x.device).data_ptr(), _stream(x.device)),
+          "pxl_short_conv")
+    _count((prefill_tokens > 0) + (T > prefill_tokens) + (taps > 1 and prefill_seqs > 0))
+    return out
+
+
+def delta_rule(x, offs, heads: int, kv_heads: int, dim: int, vdim: int, decay, dt_bias, A_log, beta, state, positions, seq_cu,
+               seq_slots, prefill_seqs: int, prefill_tokens: int = 0, out=None):
+    T, n = x.shape[0], seq_slots.numel()
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=x.dtype, device=x.device)
+    assert x.stride(1) == 1 and out.is_contiguous() and out.dtype == x.dtype and decay.dtype == beta.dtype == torch.float32
+    assert decay.stride(1) == beta.stride(1) == 1 and decay.shape[1] >= heads * dim and beta.shape[1] >= heads
+    assert dt_bias.dtype == A_log.dtype == torch.float32 and dt_bias.numel() == heads * dim and A_log.numel() == heads
+    assert state.is_contiguous() and state.dtype == torch.float32 and state.shape[1:] == (heads, dim, vdim)
+    ws, nbytes = None, 0
+    if prefill_seqs and x.dtype == torch.bfloat16:
+        nbytes = _lib.lib().pxl_delta_rule_workspace(heads, dim, vdim, prefill_seqs, prefill_tokens)
+        ws = workspace(x.device, "delta_rule", nbytes) if nbytes else None
+    check(_lib.lib().pxl_delta_rule(x.data_ptr(), x.stride(0), *offs, heads, kv_heads, dim, vdim, decay.data_ptr(), decay.stride(0),
+                                    dt_bias.data_ptr(), A_log.data_ptr(), beta.data_ptr(), beta.stride(0), state.data_ptr(),
+                                    state.shape[0], seq_cu.data_ptr(), seq_slots.data_ptr(), positions.data_ptr(), out.data_ptr(),
+                                    heads * vdim, prefill_seqs, prefill_tokens, n - prefill_seqs, _ptr(ws), nbytes,
+                                    int(x.dtype == torch.float32), status_tensor(x.device).data_ptr(), _stream(x.device)),
+          "pxl_delta_rule")
+    _count((2 if ws is not None else 1) * (prefill_seqs > 0) + (n > prefill_seqs))
+    return out
+
+
+def state_space(x, offs, heads: int, groups: int, dim: int, vdim: int, dt, dt_bias, A_log, D, state, positions, seq_cu, seq_slots,
+                prefill_seqs: int, out=None):
+    T, n = x.shape[0], seq_slots.numel()
+    if out is None:
+        out = torch.empty((T, heads, vdim), dtype=x.dtype, device=x.device)
+    assert x.stride(1) == 1 and out.is_contiguous() and out.dtype == x.dtype
+    assert dt.dtype == torch.float32 and dt.stride(1) == 1 and dt.shape[1] >= heads
+    assert all(t.dtype == torch.float32 and t.numel() == heads for t in (dt_bias, A_log, D))
+    assert state.is_contiguous() and state.dtype == torch.float32 and state.shape[1:] == (heads, dim, vdim)
+    check(_lib.lib().pxl_state_space(x.data_ptr(), x.stride(0), *offs, heads, groups, dim, vdim, dt.data_ptr(), dt.stride(0),
+                                     dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(), state.data_ptr(), state.shape[0],
+                                     seq_cu.data_ptr(), seq_slots.data_ptr(), positions.data_ptr(), out.data_ptr(), heads * vdim,
+                                     prefill_seqs, n - prefill_seqs, int(x.dtype == torch.float32),
+                                     status_tensor(x.device).data_ptr(), _stream(x.device)), "pxl_state_space")
+    _count((prefill_seqs > 0) + (n > prefill_seqs))
+    return out
+
+
+def gated_norm_rows(x, gate, w, groups: int, eps: float, out):
+    T, n = x.shape[0], x.shape[1] * x.shape[2]
+    assert x.is_contiguous() and gate.stride(1) == 1 and out.stride(1) == 1 and x.dtype == gate.dtype == out.dtype
+    assert w.dtype == torch.float32 and w.numel() == n
+    check(_lib.lib().pxl_gated_norm_rows(x.data_ptr(), n, gate.data_ptr(), gate.stride(0), w.data_ptr(), groups, eps, out.data_ptr(),
+                                         out.stride(0), out.shape[1], T, int(x.dtype == torch.float32), _stream(x.device)),
+          "pxl_gated_norm_rows")
+    _count()
     return out
