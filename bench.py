@@ -496,7 +496,7 @@ def main() -> None:
     ap.add_argument("--micro-batches", type=int, default=0, help="pipeline modes: micro-batches in flight")
     ap.add_argument("--parallelism", default="auto",
                     help="auto (the workload's layout on N GPUs) | dp | pp | pp<P>tp<T> | ep<E> | pp<P>ep<E>")
-    ap.add_argument("--design", default="", choices=["", "piburax", "zudepel", "zasalix"],
+    ap.add_argument("--design", default="", choices=["", "piburax", "zudepel", "zasalix", "kikurax"],
                     help="instead of the workload: layer throughput of this design beside the closest other model of equal "
                          "sizes, and its kernels against their rooflines (one GPU)")
     ap.add_argument("--design-sizes", default="1b,8b")
@@ -506,6 +506,8 @@ def main() -> None:
             from benchmarks.bench_latent import run as run_design
         elif args.design == "zasalix":
             from benchmarks.bench_looped import run as run_design
+        elif args.design == "kikurax":
+            from benchmarks.bench_prenorm import run as run_design
         else:
             from benchmarks.bench_parallel_block import run as run_design
 

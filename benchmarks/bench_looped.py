@@ -170,12 +170,15 @@ def zasalix_rows(r: Rows, keys: int, kv_tokens: int) -> None:
         routed, more = None, 0.0
     else:
         y2, plan, pairs, _ = routed_rows(r, lw, x)
-        r.gemm("shared: gate / up (+ activation)", x, lw.w_gu, lambda: cu.glu_linear(x, lw.w_gu, mlp.shared.act), True)
-        r.gemm("shared: down projection", r.rnd(T, lw.w_down.shape[1]), lw.w_down)
+        if mlp.shared:
+            r.gemm("shared: gate / up (+ activation)", x, lw.w_gu, lambda: cu.glu_linear(x, lw.w_gu, mlp.shared.act), True)
+            r.gemm("shared: down projection", r.rnd(T, lw.w_down.shape[1]), lw.w_down)
         routed, more = (y2, plan.pos_of, None), 2.0 * W * pairs
     name = "norm + residual" if routed is None else "experts' sum + norm + residual"
     r.add(name, lambda: cu.residual_step(h, y, lw.norm2b.args(), routed, pre=(), dtype=torch.bfloat16), 0,
           norm_bytes(T, W) + more)
+    if not r.stack.cfg.token_side_dim:
+        return
     r.gemm("token input: gate (+ activation, row)", x, lw.side_gate,
            lambda: cu.act_linear(x, lw.side_gate, ACT_GELU_TANH, st.side_table, fb.input_ids, 0))
     g = cu.act_linear(x, lw.side_gate, ACT_GELU_TANH, st.side_table, fb.input_ids, 0)
@@ -203,9 +206,10 @@ def lightning_rows(r: Rows) -> None:
                                                             cat[:, :m.out_width], lw.mix_norm, 1e-6), 0, 6.0 * T * m.out_width)
     y2, plan, pairs, wts = routed_rows(r, lw, x)
     gate = torch.zeros(T, device=x.device)
-    r.gemm("shared: gate / up (+ activation)", x, lw.w_gu, lambda: cu.glu_linear(x, lw.w_gu, mlp.shared.act, gate,
-                                                                                 cat[:, m.out_width:]), True)
-    r.gemm("output + shared down projection", cat, lw.w_out)
+    if mlp.shared:
+        r.gemm("shared: gate / up (+ activation)", x, lw.w_gu, lambda: cu.glu_linear(x, lw.w_gu, mlp.shared.act, gate,
+                                                                                     cat[:, m.out_width:]), True)
+    r.gemm("output + shared down projection" if mlp.shared else "output projection", cat, lw.w_out)
     h, y = torch.randn(T, W, device=r.stack.dev), r.rnd(T, W)
     r.add("experts' sum + residual + norm", lambda: cu.residual_add(h, y, lw.norm1, 1e-6, (y2, plan.pos_of, wts), x), 0,
           norm_bytes(T, W) + 2.0 * W * pairs)

@@ -72,16 +72,16 @@ class Rows:
         fn = fn or (lambda: cu.linear(x, w))
         self.add(name, fn, 2.0 * M * N * K, 2.0 * (M * K + N * K + M * N // (2 if halves else 1)))
 
-    def experts(self, x, ids, w1, w2, E):
+    def experts(self, x, ids, w1, w2, E, epi=cu.EPI_SILU_MUL, limit=0.0):
         plan = cu.moe_align(ids, E)
         pairs, n1, n2, K = int((plan.pos_of >= 0).sum()), w1.shape[0] // E, w2.shape[0] // E, w1.shape[1]
         used = int((torch.bincount(ids[ids < E].long().flatten(), minlength=E) > 0).sum())
         self.add("expert lists", lambda: cu.moe_align(ids, E), 0, 16.0 * ids.numel())
         self.add("rows in expert order", lambda: cu.moe_gather(x, plan), 0, 4.0 * pairs * K)
         xp = cu.moe_gather(x, plan)
-        self.add("experts: gate / up (+ SiLU)", lambda: cu.grouped_linear(xp, w1, plan, E, epi=cu.EPI_SILU_MUL),
+        self.add("experts: gate / up (+ SiLU)", lambda: cu.grouped_linear(xp, w1, plan, E, epi=epi, limit=limit),
                  2.0 * pairs * n1 * K, 2.0 * (pairs * (K + n1 / 2) + used * n1 * K))
-        act = cu.grouped_linear(xp, w1, plan, E, epi=cu.EPI_SILU_MUL)
+        act = cu.grouped_linear(xp, w1, plan, E, epi=epi, limit=limit)
         k2 = act.shape[1]
         self.add("experts: down", lambda: cu.grouped_linear(act, w2, plan, E), 2.0 * pairs * n2 * k2,
                  2.0 * (pairs * (k2 + n2) + used * n2 * k2))
@@ -150,9 +150,10 @@ def attention_rows(r: Rows, keys: int, kv_tokens: int) -> None:
     r.add("choice of experts", pick, 0, T * (4.0 * s.outputs + 8.0 * s.top))
     ids, wts = pick()
     y2, plan, pairs = r.experts(x, ids, moe.w1, moe.w2, s.experts)
-    r.gemm("shared: gate / up (+ activation)", x, lw.w_gu,
-           lambda: cu.glu_linear(x, lw.w_gu, 0, logits[:, s.outputs], cat[:, m.out_width:]), True)
-    r.gemm("output + shared down projection", cat, lw.w_out)
+    if s.shared:
+        r.gemm("shared: gate / up (+ activation)", x, lw.w_gu,
+               lambda: cu.glu_linear(x, lw.w_gu, 0, logits[:, s.outputs], cat[:, m.out_width:]), True)
+    r.gemm("output + shared down projection" if s.shared else "output projection", cat, lw.w_out)
     h, y = torch.randn(T, W, device=r.stack.dev), r.rnd(T, W)
     r.add("experts' sum + residual + norm", lambda: cu.residual_add(h, y, lw.norm1, 1e-6, (y2, plan.pos_of, wts), x), 0,
           T * W * 12.0 + 2.0 * W * (pairs + (T if pairs < T * s.top else 0)))
