@@ -7,6 +7,8 @@
     python benchmarks/profile_case.py attn_prefill # ragged prefill, 4 x 2048
     python benchmarks/profile_case.py latent_attn  # windowed latent attention, 4096-token prompt, 32 heads
     python benchmarks/profile_case.py lightning    # chunked lightning attention, 4096-token prompt, 32 heads
+    python benchmarks/profile_case.py delta_rule   # chunked gated delta rule, 4096-token prompt, 32 heads
+    python benchmarks/profile_case.py state_space  # chunked state space, 4096-token prompt, 128 heads in 8 groups
     python benchmarks/profile_case.py step         # 2 engine steps of a 4-layer Qwen3-8B-shaped
                                                    # model at 64 concurrent (launch list)
     python benchmarks/profile_case.py decode_step  # same, decode rows only (small-M GEMMs); decode_step_8: 8 rows
@@ -222,9 +224,41 @@ def case_matrix_memory(iters: int = 2, T: int = 4096, H: int = 16, dk: int = 128
     cu.check_status(proj.device)
 
 
+def _profiled(run, iters: int, dev):
+    run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStart()
+    for _ in range(iters):
+        run()
+    torch.cuda.synchronize()
+    torch.cuda.cudart().cudaProfilerStop()
+    cu.check_status(dev)
+
+
+def _one_prompt(T: int):
+    return (torch.arange(T, dtype=torch.int32, device="cuda"), torch.tensor([0, T], dtype=torch.int32, device="cuda"),
+            torch.zeros(1, dtype=torch.int32, device="cuda"))
+
+
+def case_delta_rule(iters: int = 2, T: int = 4096, H: int = 32, D: int = 128):
+    x = torch.randn(T, 3 * H * D, device="cuda", dtype=torch.bfloat16)
+    decay, beta = torch.randn(T, H * D, device="cuda"), torch.randn(T, H, device="cuda")
+    bias, A, state = torch.full((H * D,), -3.0, device="cuda"), torch.zeros(H, device="cuda"), torch.zeros(1, H, D, D, device="cuda")
+    _profiled(lambda: cu.delta_rule(x, (0, H * D, 2 * H * D), H, H, D, D, decay, bias, A, beta, state, *_one_prompt(T), 1, T), iters,
+              x.device)
+
+
+def case_state_space(iters: int = 2, T: int = 4096, H: int = 128, G: int = 8, N: int = 128, D: int = 64):
+    x, dt = torch.randn(T, H * D + 2 * G * N, device="cuda", dtype=torch.bfloat16), torch.randn(T, H, device="cuda")
+    one, state = torch.ones(H, device="cuda"), torch.zeros(1, H, N, D, device="cuda")
+    _profiled(lambda: cu.state_space(x, (0, H * D, H * D + G * N), H, G, N, D, dt, -3 * one, 0 * one, one, state, *_one_prompt(T), 1),
+              iters, x.device)
+
+
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "gemm"
     {"gemm": case_gemm, "latent_attn": case_latent_attn, "lightning": case_lightning, "matrix_memory": case_matrix_memory,
+     "delta_rule": case_delta_rule, "state_space": case_state_space,
      "attn_decode": case_attn_decode, "attn_prefill": case_attn_prefill,
      "gemm_small": case_gemm_small, "gemm_mid": case_gemm_mid, "step": case_step, "decode_step": lambda: case_step(conc=64, with_prefill=False),
      "decode_step_8": lambda: case_step(conc=8, with_prefill=False)}[which]()

@@ -71,22 +71,23 @@ __device__ __forceinline__ float* state_of(const DeltaArgs& a, int seq, int h) {
 }
 
 // ---- recurrent ---------------------------------------------------------------------------------------------
-// 256 threads = 8 row lanes (warps) x 32 column lanes of VW columns; R rows of S per thread in registers (R == 0: the
+// 256 threads = 256 / CL row lanes x CL column lanes of VW columns; R rows of S per thread in registers (R == 0: the
 // state stays in global memory, any dk).
-template <typename T, int VW, int R>
+template <typename T, int VW, int R, int CL>
 __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a, int seq0) {
   extern __shared__ float sm[];
   pdl_wait();
   pdl_launch_dependents();
   const int h = blockIdx.x, seq = seq0 + blockIdx.z, hq = h / a.rep;
-  const int cl = threadIdx.x & 31, rl = threadIdx.x >> 5;
-  const int c0 = (blockIdx.y * 32 + cl) * VW;
+  constexpr int RL = 256 / CL;
+  const int cl = threadIdx.x % CL, rl = threadIdx.x / CL;
+  const int c0 = (blockIdx.y * CL + cl) * VW;
   const int t0 = a.seq_cu[seq], t1 = a.seq_cu[seq + 1];
   if (t1 <= t0) return;
   float* Sg = state_of(a, seq, h);
   if (Sg == nullptr) return;
   const bool fresh = a.positions[t0] == 0, live = c0 < a.dv;
-  float* red = sm + 6 * a.dk;  // [2][8][VW][32], behind two sets of q, k, g
+  float* red = sm + 6 * a.dk;  // [2][RL][VW][CL], behind two sets of q, k, g
   constexpr int RR = R > 0 ? R : 1;
   float S[RR][VW];
   auto load_row = [&](int r, float (&s)[VW]) {
@@ -104,7 +105,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
   if constexpr (R > 0) {
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-      const int r = rl + 8 * i;
+      const int r = rl + RL * i;
       if (!fresh && live && r < a.dk) {
         load_row(r, S[i]);
       } else {
@@ -114,7 +115,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
     }
   } else if (fresh && live) {
     const float zero[VW] = {};
-    for (int r = rl; r < a.dk; r += 8) store_row(r, zero);
+    for (int r = rl; r < a.dk; r += RL) store_row(r, zero);
   }
   const float rate = expf(a.A_log[h]);
   for (int t = t0; t < t1; ++t) {
@@ -137,7 +138,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
     const float b = sigmoid(a.beta[static_cast<int64_t>(t) * a.ldb + h]);
     __syncthreads();
     float qq = 0.f, kk = 0.f, qk = 0.f;  // every warp for itself
-    for (int i = cl; i < a.dk; i += 32) {
+    for (int i = threadIdx.x & 31; i < a.dk; i += 32) {
       qq = fmaf(qs[i], qs[i], qq);
       kk = fmaf(ks[i], ks[i], kk);
       qk = fmaf(qs[i], ks[i], qk);
@@ -147,7 +148,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
     if constexpr (R > 0) {
 #pragma unroll
       for (int i = 0; i < R; ++i) {
-        const int r = rl + 8 * i;
+        const int r = rl + RL * i;
         if (r < a.dk) {
           const float k = ks[r], q = qs[r], g = gs[r];
 #pragma unroll
@@ -159,7 +160,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
         }
       }
     } else if (live) {
-      for (int r = rl; r < a.dk; r += 8) {
+      for (int r = rl; r < a.dk; r += RL) {
         float s[VW];
         load_row(r, s);
 #pragma unroll
@@ -172,8 +173,8 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
     }
 #pragma unroll
     for (int c = 0; c < VW; ++c) {
-      red[(rl * VW + c) * 32 + cl] = sk[c];
-      red[((8 + rl) * VW + c) * 32 + cl] = sq[c];
+      red[(rl * VW + c) * CL + cl] = sk[c];
+      red[((RL + rl) * VW + c) * CL + cl] = sq[c];
     }
     __syncthreads();
     float u[VW], o[VW];
@@ -181,9 +182,9 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
     for (int c = 0; c < VW; ++c) {
       float s1 = 0.f, s2 = 0.f;
 #pragma unroll
-      for (int w = 0; w < 8; ++w) {
-        s1 += red[(w * VW + c) * 32 + cl];
-        s2 += red[((8 + w) * VW + c) * 32 + cl];
+      for (int w = 0; w < RL; ++w) {
+        s1 += red[(w * VW + c) * CL + cl];
+        s2 += red[((RL + w) * VW + c) * CL + cl];
       }
       u[c] = b * (v[c] - s1 * ik);
       o[c] = fmaf(qk, u[c], s2 * iq);
@@ -192,7 +193,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
     if constexpr (R > 0) {
 #pragma unroll
       for (int i = 0; i < R; ++i) {
-        const int r = rl + 8 * i;
+        const int r = rl + RL * i;
         if (r < a.dk) {
           const float k = ks[r];
 #pragma unroll
@@ -200,7 +201,7 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
         }
       }
     } else if (live) {
-      for (int r = rl; r < a.dk; r += 8) {
+      for (int r = rl; r < a.dk; r += RL) {
         float s[VW];
         load_row(r, s);
 #pragma unroll
@@ -217,23 +218,28 @@ __global__ void __launch_bounds__(256) delta_recurrent_kernel(const DeltaArgs a,
   if constexpr (R > 0) {
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-      const int r = rl + 8 * i;
+      const int r = rl + RL * i;
       if (live && r < a.dk) store_row(r, S[i]);
     }
   }
 }
 
+template <typename T, int VW, int CL>
+int launch_recurrent(const DeltaArgs& a, int seq0, int n, cudaStream_t stream) {
+  constexpr int RL = 256 / CL;
+  const dim3 grid(a.H, ceil_div(a.dv, CL * VW), n);
+  const size_t smem = sizeof(float) * (6 * a.dk + 2 * 256 * VW);
+  if (smem > 48 * 1024 || n > 65535) return PXL_ERR_TOO_LARGE;
+  if (a.dk <= 4 * RL) pxl_host::launch(delta_recurrent_kernel<T, VW, 4, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 8 * RL) pxl_host::launch(delta_recurrent_kernel<T, VW, 8, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 16 * RL) pxl_host::launch(delta_recurrent_kernel<T, VW, 16, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 32 * RL) pxl_host::launch(delta_recurrent_kernel<T, VW, 32, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else pxl_host::launch(delta_recurrent_kernel<T, VW, 0, CL>, grid, dim3(256), smem, stream, a, seq0);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
 template <typename T, int VW>
 int launch_recurrent(const DeltaArgs& a, int seq0, int n, cudaStream_t stream) {
-  const dim3 grid(a.H, ceil_div(a.dv, 32 * VW), n);
-  const size_t smem = sizeof(float) * (6 * a.dk + 2 * 8 * 32 * VW);
-  if (smem > 48 * 1024 || n > 65535) return PXL_ERR_TOO_LARGE;
-  if (a.dk <= 32) pxl_host::launch(delta_recurrent_kernel<T, VW, 4>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 64) pxl_host::launch(delta_recurrent_kernel<T, VW, 8>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 128) pxl_host::launch(delta_recurrent_kernel<T, VW, 16>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 256) pxl_host::launch(delta_recurrent_kernel<T, VW, 32>, grid, dim3(256), smem, stream, a, seq0);
-  else pxl_host::launch(delta_recurrent_kernel<T, VW, 0>, grid, dim3(256), smem, stream, a, seq0);
-  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+  return a.dv <= 16 * VW ? launch_recurrent<T, VW, 16>(a, seq0, n, stream) : launch_recurrent<T, VW, 32>(a, seq0, n, stream);
 }
 template <typename T>
 int launch_recurrent(const DeltaArgs& a, int seq0, int n, cudaStream_t stream) {
@@ -574,13 +580,14 @@ struct WalkSmem {
   bf16 u_hi[kChunk][kV], u_lo[kChunk][kV];
 };
 
-constexpr int kWalkWarps = 8;
+// Warps 0 to 7 make u and keep the state, warps 8 to 15 make the outputs.
+constexpr int kHalf = 8, kWalkWarps = 2 * kHalf;
 
 __device__ __forceinline__ void copy16(void* dst, const void* src) { cp_async_16(smem_u32(dst), src, true); }
 
 // grid (slices of v, heads, sequences): the chunks [chunk0, chunk0 + chunks) of one sequence, in order
 template <int DK>
-__global__ void __launch_bounds__(kWalkWarps * 32) delta_walk_kernel(const DeltaArgs a, int chunk0, int chunks, int slices,
+__global__ void __launch_bounds__(kWalkWarps * 32, 1) delta_walk_kernel(const DeltaArgs a, int chunk0, int chunks, int slices,
                                                                     const uint32_t* __restrict__ work) {
   extern __shared__ __align__(16) uint8_t raw[];
   using Sm = WalkSmem<DK>;
@@ -620,13 +627,15 @@ __global__ void __launch_bounds__(kWalkWarps * 32) delta_walk_kernel(const Delta
   load_front(first);
   load_back(first);
 
-  // this warp's 16 x 16 tiles of the state, in the layout of the accumulators
-  constexpr int kTilesK = DK / 16, kTiles = kTilesK * 2, NT = (kTiles + kWalkWarps - 1) / kWalkWarps;
+  // 16 x 16 tiles of the state, in the layout of the accumulators (first half of the warps)
+  constexpr int kTilesK = DK / 16, kTiles = kTilesK * 2, NT = (kTiles + kHalf - 1) / kHalf;
+  const bool keeper = warp < kHalf;
+  const int w8 = warp % kHalf, rg = w8 & 3, ch = w8 >> 2;  // 16 tokens; half of the slice's columns
   float S[NT][2][4];
-  auto each = [&](auto f) {  // f(tile, half, element, row, column)
+  auto each = [&](auto f) {  // f(element, row, column)
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
-      const int tile = warp + i * kWalkWarps, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
+      const int tile = w8 + i * kHalf, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -634,13 +643,10 @@ __global__ void __launch_bounds__(kWalkWarps * 32) delta_walk_kernel(const Delta
           if (tile < kTiles) f(S[i][j][e], m0 + g8 + (e >> 1) * 8, n0 + j * 8 + t2 + (e & 1));
     }
   };
-  each([&](float& v, int r, int c) {
-    v = !fresh && r < a.dk && v0 + c < a.dv ? Sg[static_cast<int64_t>(r) * a.dv + v0 + c] : 0.f;
-  });
   auto publish = [&]() {
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
-      const int tile = warp + i * kWalkWarps, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
+      const int tile = w8 + i * kHalf, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
       if (tile >= kTiles) continue;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
@@ -653,95 +659,106 @@ __global__ void __launch_bounds__(kWalkWarps * 32) delta_walk_kernel(const Delta
         }
     }
   };
-  publish();
+  if (keeper) {
+    each([&](float& v, int r, int c) {
+      v = !fresh && r < a.dk && v0 + c < a.dv ? Sg[static_cast<int64_t>(r) * a.dv + v0 + c] : 0.f;
+    });
+    publish();
+  }
 
-  const int rg = warp & 3, ch = warp >> 2;  // 16 tokens; half of the slice's columns
   for (int i = first; i < last; ++i) {
     const int c0 = i * kChunk, n = n_all - c0 < kChunk ? n_all - c0 : kChunk;
     cp_async_wait<1>();  // front part (the back part may still be on its way)
     __syncthreads();
-    // ---- u = U - W S and (q e^G) S: 16 tokens x 16 columns
-    float u[2][4], o[2][4] = {};
-#pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) u[j][e] = 0.f;
+    // ---- W S and (q e^G) S: 16 tokens x 16 columns, the three products of the split operands side by side
+    float o[2][4] = {}, o1[2][4] = {}, o2[2][4] = {};
+    const auto& rows = keeper ? s.w : s.q;
 #pragma unroll
     for (int kk = 0; kk < kTilesK; ++kk) {
-      uint32_t wh[4], wl[4], qh[4], ql[4], sh[4], sl[4];
+      uint32_t ah[4], al[4], sh[4], sl[4];
 #pragma unroll
-      for (int x = 0; x < 4; ++x) {
-        const int r = rg * 16 + g8 + (x & 1) * 8, c = kk * 16 + t2 + (x >> 1) * 8;
-        join2(*reinterpret_cast<const uint2*>(&s.w[r][c]), wh[x], wl[x]);
-        join2(*reinterpret_cast<const uint2*>(&s.q[r][c]), qh[x], ql[x]);
-      }
+      for (int x = 0; x < 4; ++x)
+        join2(*reinterpret_cast<const uint2*>(&rows[rg * 16 + g8 + (x & 1) * 8][kk * 16 + t2 + (x >> 1) * 8]), ah[x], al[x]);
       ldmatrix_x4_trans(sh, smem_u32(&s.s_hi[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
       ldmatrix_x4_trans(sl, smem_u32(&s.s_lo[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
-        mma3(u[j], wh, wl, sh[2 * j], sh[2 * j + 1], sl[2 * j], sl[2 * j + 1]);
-        mma3(o[j], qh, ql, sh[2 * j], sh[2 * j + 1], sl[2 * j], sl[2 * j + 1]);
+        const uint32_t bh[2] = {sh[2 * j], sh[2 * j + 1]}, bl[2] = {sl[2 * j], sl[2 * j + 1]};
+        mma_m16n8k16_bf16(o[j], ah, bh);
+        mma_m16n8k16_bf16(o1[j], ah, bl);
+        mma_m16n8k16_bf16(o2[j], al, bh);
       }
     }
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int r = rg * 16 + g8 + e * 8, c = ch * 16 + j * 8 + t2;
-        const float2 u0 = *reinterpret_cast<const float2*>(&s.u0[r][c]);
-        uint32_t hi, lo;
-        split2(u0.x - u[j][2 * e], u0.y - u[j][2 * e + 1], hi, lo);
-        *reinterpret_cast<uint32_t*>(&s.u_hi[r][c]) = hi;
-        *reinterpret_cast<uint32_t*>(&s.u_lo[r][c]) = lo;
-      }
+      for (int e = 0; e < 4; ++e) o[j][e] += o1[j][e] + o2[j][e];
+    if (keeper) {  // u = U - W S
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int r = rg * 16 + g8 + e * 8, c = ch * 16 + j * 8 + t2;
+          const float2 u0 = *reinterpret_cast<const float2*>(&s.u0[r][c]);
+          uint32_t hi, lo;
+          split2(u0.x - o[j][2 * e], u0.y - o[j][2 * e + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(&s.u_hi[r][c]) = hi;
+          *reinterpret_cast<uint32_t*>(&s.u_lo[r][c]) = lo;
+        }
+    }
     cp_async_wait<0>();
     __syncthreads();
     if (i + 1 < last) load_front(i + 1);
 
-    // ---- o += P u (blocks up to this one); S = e^(G_n) S + (k e^(G_n - G))^T u
-    for (int kk = 0; kk <= rg; ++kk) {
-      uint32_t ph[4], pl[4], bh[4], bl[4];
+    if (!keeper) {
+      // ---- o += P u (blocks up to this one)
+      for (int kk = 0; kk <= rg; ++kk) {
+        uint32_t ph[4], pl[4], bh[4], bl[4];
 #pragma unroll
-      for (int x = 0; x < 4; ++x)
-        join2(*reinterpret_cast<const uint2*>(&s.p[rg * 16 + g8 + (x & 1) * 8][kk * 16 + t2 + (x >> 1) * 8]), ph[x], pl[x]);
-      ldmatrix_x4_trans(bh, smem_u32(&s.u_hi[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
-      ldmatrix_x4_trans(bl, smem_u32(&s.u_lo[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
+        for (int x = 0; x < 4; ++x)
+          join2(*reinterpret_cast<const uint2*>(&s.p[rg * 16 + g8 + (x & 1) * 8][kk * 16 + t2 + (x >> 1) * 8]), ph[x], pl[x]);
+        ldmatrix_x4_trans(bh, smem_u32(&s.u_hi[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
+        ldmatrix_x4_trans(bl, smem_u32(&s.u_lo[kk * 16 + (mi & 1) * 8 + r8][ch * 16 + (mi >> 1) * 8]));
 #pragma unroll
-      for (int j = 0; j < 2; ++j) mma3(o[j], ph, pl, bh[2 * j], bh[2 * j + 1], bl[2 * j], bl[2 * j + 1]);
-    }
-#pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int r = rg * 16 + g8 + e * 8, c = v0 + ch * 16 + j * 8 + t2;
-        if (r < n && c < a.dv)
-          *reinterpret_cast<uint32_t*>(static_cast<bf16*>(a.out) + static_cast<int64_t>(t0 + c0 + r) * a.ldo + h * a.dv + c) =
-              pack_bf16x2(o[j][2 * e], o[j][2 * e + 1]);
+        for (int j = 0; j < 2; ++j) mma3(o[j], ph, pl, bh[2 * j], bh[2 * j + 1], bl[2 * j], bl[2 * j + 1]);
       }
-    each([&](float& v, int r, int) { v *= s.g[r]; });
 #pragma unroll
-    for (int x = 0; x < NT; ++x) {
-      const int tile = warp + x * kWalkWarps, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
-      if (tile >= kTiles) continue;
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int r = rg * 16 + g8 + e * 8, c = v0 + ch * 16 + j * 8 + t2;
+          if (r < n && c < a.dv)
+            *reinterpret_cast<uint32_t*>(static_cast<bf16*>(a.out) + static_cast<int64_t>(t0 + c0 + r) * a.ldo + h * a.dv + c) =
+                pack_bf16x2(o[j][2 * e], o[j][2 * e + 1]);
+        }
+    } else {
+      // ---- S = e^(G_n) S + (k e^(G_n - G))^T u
+      each([&](float& v, int r, int) { v *= s.g[r]; });
 #pragma unroll
       for (int kk = 0; kk < kChunk / 16; ++kk) {
-        uint32_t kh[4], kl[4], bh[4], bl[4];
 #pragma unroll
-        for (int y = 0; y < 4; ++y)
-          join2(*reinterpret_cast<const uint2*>(&s.k[m0 + g8 + (y & 1) * 8][kk * 16 + t2 + (y >> 1) * 8]), kh[y], kl[y]);
-        ldmatrix_x4_trans(bh, smem_u32(&s.u_hi[kk * 16 + (mi & 1) * 8 + r8][n0 + (mi >> 1) * 8]));
-        ldmatrix_x4_trans(bl, smem_u32(&s.u_lo[kk * 16 + (mi & 1) * 8 + r8][n0 + (mi >> 1) * 8]));
+        for (int x = 0; x < NT; ++x) {
+          const int tile = w8 + x * kHalf, m0 = tile % kTilesK * 16, n0 = tile / kTilesK * 16;
+          if (tile >= kTiles) continue;
+          uint32_t kh[4], kl[4], bh[4], bl[4];
 #pragma unroll
-        for (int j = 0; j < 2; ++j) mma3(S[x][j], kh, kl, bh[2 * j], bh[2 * j + 1], bl[2 * j], bl[2 * j + 1]);
+          for (int y = 0; y < 4; ++y)
+            join2(*reinterpret_cast<const uint2*>(&s.k[m0 + g8 + (y & 1) * 8][kk * 16 + t2 + (y >> 1) * 8]), kh[y], kl[y]);
+          ldmatrix_x4_trans(bh, smem_u32(&s.u_hi[kk * 16 + (mi & 1) * 8 + r8][n0 + (mi >> 1) * 8]));
+          ldmatrix_x4_trans(bl, smem_u32(&s.u_lo[kk * 16 + (mi & 1) * 8 + r8][n0 + (mi >> 1) * 8]));
+#pragma unroll
+          for (int j = 0; j < 2; ++j) mma3(S[x][j], kh, kl, bh[2 * j], bh[2 * j + 1], bl[2 * j], bl[2 * j + 1]);
+        }
       }
+      publish();  // every read of the old state happened before the last barrier
     }
-    publish();  // every read of the old state happened before the last barrier
     __syncthreads();
     if (i + 1 < last) load_back(i + 1);
   }
-  each([&](float& v, int r, int c) {
-    if (r < a.dk && v0 + c < a.dv) Sg[static_cast<int64_t>(r) * a.dv + v0 + c] = v;
-  });
+  if (keeper)
+    each([&](float& v, int r, int c) {
+      if (r < a.dk && v0 + c < a.dv) Sg[static_cast<int64_t>(r) * a.dv + v0 + c] = v;
+    });
 }
 
 template <typename K>

@@ -82,16 +82,18 @@ __device__ __forceinline__ float* state_of(const MemoryArgs& a, int seq, int h) 
 }
 
 // ---- recurrent ---------------------------------------------------------------------------------------------
-// 256 threads = 8 row lanes x 32 column lanes of VW columns; R rows of S per thread in registers (R == 0: the state
-// stays in global memory, any dk).
-template <typename T, int VW, int R, bool kSpace>
+// 256 threads = 256 / CL row lanes x CL column lanes of VW columns (CL < 32: narrow states, kSpace only); R rows of S per
+// thread in registers (R == 0: the state stays in global memory, any dk).
+template <typename T, int VW, int R, bool kSpace, int CL = 32>
 __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs a, int seq0) {
   extern __shared__ float sm[];
   pdl_wait();
   pdl_launch_dependents();
   const int h = blockIdx.x, seq = seq0 + blockIdx.z;
-  const int cl = threadIdx.x & 31, rl = threadIdx.x >> 5;
-  const int c0 = (blockIdx.y * 32 + cl) * VW;
+  static_assert(CL == 32 || kSpace, "the normaliser is summed warp by warp");
+  constexpr int RL = 256 / CL;
+  const int cl = threadIdx.x % CL, rl = threadIdx.x / CL;
+  const int c0 = (blockIdx.y * CL + cl) * VW;
   const int t0 = a.seq_cu[seq], t1 = a.seq_cu[seq + 1];
   if (t1 <= t0) return;
   float* Sg = state_of(a, seq, h);
@@ -101,7 +103,7 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
   float* ks = qs + a.dk;       // [dk], times the input weight
   float* ns = ks + a.dk;       // [dk], every entry kept by one thread
   float* dens = ns + a.dk;     // [8] partial n . q
-  float* red = dens + 8;       // [8][32 * VW]
+  float* red = dens + 8;       // [RL][CL * VW]
   const int slices = ceil_div(a.dv, kSlice), slice0 = blockIdx.y * VW, own = min(VW, slices - slice0);
   float* ng = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(slice0) * a.dk;
   float* mg = Sg + static_cast<int64_t>(a.dk) * a.dv + static_cast<int64_t>(slices) * a.dk + slice0;
@@ -125,7 +127,7 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
   if constexpr (R > 0) {
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-      const int r = rl + 8 * i;
+      const int r = rl + RL * i;
       if (!fresh && live && r < a.dk) {
         load_row(r, S[i]);
       } else {
@@ -135,7 +137,7 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
     }
   } else if (fresh && live) {
     const float zero[VW] = {};
-    for (int r = rl; r < a.dk; r += 8) store_row(r, zero);
+    for (int r = rl; r < a.dk; r += RL) store_row(r, zero);
   }
   if (owns_n) ns[threadIdx.x] = n_first;
   if constexpr (!kSpace)
@@ -186,7 +188,7 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
     if constexpr (R > 0) {
 #pragma unroll
       for (int i = 0; i < R; ++i) {
-        const int r = rl + 8 * i;
+        const int r = rl + RL * i;
         if (r < a.dk) {
           const float k = ks[r], q = qs[r];
 #pragma unroll
@@ -197,7 +199,7 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
         }
       }
     } else if (live) {
-      for (int r = rl; r < a.dk; r += 8) {
+      for (int r = rl; r < a.dk; r += RL) {
         float s[VW];
         load_row(r, s);
         const float k = ks[r], q = qs[r];
@@ -210,15 +212,15 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
       }
     }
 #pragma unroll
-    for (int c = 0; c < VW; ++c) red[(rl * VW + c) * 32 + cl] = o[c];
+    for (int c = 0; c < VW; ++c) red[(rl * VW + c) * CL + cl] = o[c];
     __syncthreads();
     const float inv = kSpace ? 1.f : 1.f / (fmaxf(fabsf(den), expf(-m)) + kTiny);
-    for (int i = threadIdx.x; i < 32 * VW; i += 256) {  // column i of this CTA's slices
-      const int col = blockIdx.y * 32 * VW + i;
+    for (int i = threadIdx.x; i < CL * VW; i += 256) {  // column i of this CTA's slices
+      const int col = blockIdx.y * CL * VW + i;
       if (col < a.dv) {
         float sum = 0.f;
 #pragma unroll
-        for (int r = 0; r < 8; ++r) sum += red[(r * VW + i % VW) * 32 + i / VW];
+        for (int r = 0; r < RL; ++r) sum += red[(r * VW + i % VW) * CL + i / VW];
         if constexpr (kSpace) sum = fmaf(skip, to_f(row[a.v_off + h * a.dv + col]), sum);
         put(static_cast<T*>(a.out) + static_cast<int64_t>(t) * a.ldo + h * a.dv + col, sum * inv);
       }
@@ -227,7 +229,7 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
   if constexpr (R > 0) {
 #pragma unroll
     for (int i = 0; i < R; ++i) {
-      const int r = rl + 8 * i;
+      const int r = rl + RL * i;
       if (live && r < a.dk) store_row(r, S[i]);
     }
   }
@@ -238,17 +240,26 @@ __global__ void __launch_bounds__(256) memory_recurrent_kernel(const MemoryArgs 
   }
 }
 
+template <bool kSpace, typename T, int VW, int CL>
+int launch_recurrent(const MemoryArgs& a, int seq0, int n, cudaStream_t stream) {
+  constexpr int RL = 256 / CL;
+  const dim3 grid(a.H, ceil_div(a.dv, CL * VW), n);
+  const size_t smem = sizeof(float) * (3 * a.dk + 8 + 256 * VW);
+  if (smem > 48 * 1024 || n > 65535) return PXL_ERR_TOO_LARGE;
+  if (a.dk <= 4 * RL) pxl_host::launch(memory_recurrent_kernel<T, VW, 4, kSpace, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 8 * RL) pxl_host::launch(memory_recurrent_kernel<T, VW, 8, kSpace, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 16 * RL) pxl_host::launch(memory_recurrent_kernel<T, VW, 16, kSpace, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else if (a.dk <= 32 * RL) pxl_host::launch(memory_recurrent_kernel<T, VW, 32, kSpace, CL>, grid, dim3(256), smem, stream, a, seq0);
+  else pxl_host::launch(memory_recurrent_kernel<T, VW, 0, kSpace, CL>, grid, dim3(256), smem, stream, a, seq0);
+  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+}
 template <bool kSpace, typename T, int VW>
 int launch_recurrent(const MemoryArgs& a, int seq0, int n, cudaStream_t stream) {
-  const dim3 grid(a.H, ceil_div(a.dv, 32 * VW), n);
-  const size_t smem = sizeof(float) * (3 * a.dk + 8 + 8 * 32 * VW);
-  if (smem > 48 * 1024 || n > 65535) return PXL_ERR_TOO_LARGE;
-  if (a.dk <= 32) pxl_host::launch(memory_recurrent_kernel<T, VW, 4, kSpace>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 64) pxl_host::launch(memory_recurrent_kernel<T, VW, 8, kSpace>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 128) pxl_host::launch(memory_recurrent_kernel<T, VW, 16, kSpace>, grid, dim3(256), smem, stream, a, seq0);
-  else if (a.dk <= 256) pxl_host::launch(memory_recurrent_kernel<T, VW, 32, kSpace>, grid, dim3(256), smem, stream, a, seq0);
-  else pxl_host::launch(memory_recurrent_kernel<T, VW, 0, kSpace>, grid, dim3(256), smem, stream, a, seq0);
-  return cudaGetLastError() == cudaSuccess ? PXL_OK : PXL_ERR_CUDA;
+  if constexpr (kSpace) {
+    if (a.dv <= 8 * VW) return launch_recurrent<kSpace, T, VW, 8>(a, seq0, n, stream);
+    if (a.dv <= 16 * VW) return launch_recurrent<kSpace, T, VW, 16>(a, seq0, n, stream);
+  }
+  return launch_recurrent<kSpace, T, VW, 32>(a, seq0, n, stream);
 }
 template <bool kSpace, typename T>
 int launch_recurrent(const MemoryArgs& a, int seq0, int n, cudaStream_t stream) {

@@ -151,10 +151,18 @@ __global__ void __launch_bounds__(128) conv_run_kernel(const ConvArgs a, int run
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) wt[j] = ld_bf16x8(w + static_cast<int64_t>(j) * a.C);
   if (a.bias) load_v<8>(static_cast<const bf16*>(a.bias) + c, b0);
-  bf16x8 next = ld_bf16x8(cur);
-  for (int t = first; t < last; ++t, cur += a.ldx) {
-    while (a.seq_cu[seq + 1] <= t) ++seq;
-    const int li = t - a.seq_cu[seq];
+  constexpr int kAhead = 4;  // tokens whose inputs are on their way
+  bf16x8 ahead[kAhead];
+#pragma unroll
+  for (int i = 0; i < kAhead; ++i) ahead[i] = first + i < last ? ld_bf16x8(cur + static_cast<int64_t>(i) * a.ldx) : zero8;
+  int start = a.seq_cu[seq], end = a.seq_cu[seq + 1];
+  for (int t4 = first; t4 < last; t4 += kAhead)
+#pragma unroll
+  for (int i4 = 0; i4 < kAhead; ++i4, cur += a.ldx) {
+    const int t = t4 + i4;
+    if (t >= last) break;
+    while (end <= t) ++seq, start = end, end = a.seq_cu[seq + 1];
+    const int li = t - start;
     if (kBack > 0 && (t == first || li == 0)) {  // the inputs before this run, or of this sequence's earlier steps
       const int pos = a.positions[t];
       const bf16* state = li < kBack ? state_of<bf16>(a, seq) : nullptr;
@@ -167,8 +175,8 @@ __global__ void __launch_bounds__(128) conv_run_kernel(const ConvArgs a, int run
         else if (state) hist[j] = ld_bf16x8(state + static_cast<int64_t>(li + j) * a.C + c);
       }
     }
-    const bf16x8 here = next;
-    if (t + 1 < last) next = ld_bf16x8(cur + a.ldx);
+    const bf16x8 here = ahead[i4];
+    if (t + kAhead < last) ahead[i4] = ld_bf16x8(cur + kAhead * a.ldx);
     float y[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) y[e] = b0[e];

@@ -570,8 +570,8 @@ def _with_first_values(before: list, i: int, m):
     if first is None:
         return m
     src = before[first].mixer
-    if (src.kv_heads, src.vdim) != (m.kv_heads, m.vdim):
-        raise ValueError(f"layer {i} and layer {first}, whose values it mixes in, differ in their value heads")
+    if src.v_rows != m.v_rows:
+        raise ValueError(f"layer {i} and layer {first}, whose values it mixes in, differ in the width of their value heads")
     return replace(m, v_first=first)
 
 

@@ -403,7 +403,7 @@ def test_config_errors():
                               (("layers", 0, "mixer", "norm_groups"), 5, "no state-space"),
                               (("layers", 1, "mixer", "rot", "dims"), 25, "rotary"),
                               (("layers", 1, "mixer", "rot", "scaling", "high"), 1.0, "stretches"),
-                              (("layers", 3, "mixer", "vdim"), 24, "value heads"),
+                              (("layers", 3, "mixer", "vdim"), 24, "width of their value heads"),
                               (("norm", "groups"), 5, "equal parts"),
                               (("layers", 0, "mlp", "shared"), {"ff": 8}, "not part of"),
                               (("layers", 0, "mlp", "router", "top"), 7, "to choose from")):
