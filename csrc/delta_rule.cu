@@ -14,8 +14,8 @@
 //        U = (1 + A)^-1 (b v)    W = (1 + A)^-1 (b k e^G)     u = U - W S_0
 //        o = (q e^G) S_0 + P u                                S_end = e^(G_n) S_0 + (k e^(G_n - G))^T u
 //    The first kernel makes U, W, P, q e^G and k e^(G_n - G) of every chunk in parallel; the second walks the chunks of a
-//    (sequence, head, 32 columns of v) with S in registers. No exponent is ever positive: inside a block of 16 tokens
-//    A and P are summed with the exact differences G_t - G_j; between blocks the factors are split at the block borders
+//    (sequence, head, 32 columns of v) with S in registers. No exponent is ever positive: inside blocks of 8 tokens
+//    A and P are summed with the exact differences G_t - G_j; between blocks the factors are split at a border between them
 //    (e^(G_t - G_border) on the row, e^(G_border - G_j) on the column) and multiplied on the tensor cores. The triangular
 //    system is solved column by column in fp32. Products take operands as sums of two bf16 numbers (rounding 2^-17).
 //
@@ -279,6 +279,32 @@ __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], con
   mma_m16n8k16_bf16(d, al, bh);
 }
 
+// log2(e) * softplus(z) to a few 1e-6 of itself: log2(1 + e^-|z|) by its series where that is small
+__device__ __forceinline__ float softplus_log2(float z) {
+  const float w = z * kLog2E, e = ex2(-fabsf(w));
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + e));
+  const float series = e * kLog2E * fmaf(e, fmaf(e, fmaf(e, fmaf(e, 0.2f, -0.25f), 1.f / 3.f), -0.5f), 1.f);
+  return fmaxf(w, 0.f) + (e < 0.0625f ? series : y);
+}
+
+// two fp32 numbers in a register pair
+__device__ __forceinline__ uint64_t pair(float a, float b) {
+  uint64_t v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+  return v;
+}
+__device__ __forceinline__ float2 unpair(uint64_t v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+
 // What the first kernel hands to the second, per (chunk, head), in 32-bit words
 template <int DK>
 struct Record {
@@ -353,6 +379,24 @@ __global__ void __launch_bounds__(kMakeThreads, 2) delta_make_kernel(const Delta
   uint32_t* rec = work + (static_cast<int64_t>(blockIdx.x) * a.H + h) * Rec::words(slices);
   const bf16* x = static_cast<const bf16*>(a.x) + static_cast<int64_t>(t0) * a.ld;
   if (tid == 0) s.next = 0;
+  // logits of the decays (a channel and 16 tokens at a time) are on their way first, and v into L2
+  constexpr int kBlocks = kChunk / kBlock, kStride = kMakeThreads / DK, kMine = kBlocks > kStride ? kBlocks / kStride : 1;
+  const int chan = tid % DK, blk0 = tid / DK;
+  const bool has = chan < a.dk;
+  float z[kMine][kBlock];
+  {
+    const float* dec = a.decay + static_cast<int64_t>(t0) * a.ldd + h * a.dk + chan;
+#pragma unroll
+    for (int m = 0; m < kMine; ++m)
+#pragma unroll
+      for (int i = 0; i < kBlock; ++i) {
+        const int t = (blk0 + m * kStride) * kBlock + i;
+        z[m][i] = t < n && has ? dec[static_cast<int64_t>(t) * a.ldd] : 0.f;
+      }
+    const int lines = ceil_div(a.dv, 64);
+    for (int i = tid; i < n * lines; i += kMakeThreads)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(x + static_cast<int64_t>(i / lines) * a.ld + a.v_off + h * a.dv + i % lines * 64));
+  }
 
   // ---- q and k with the factors that make them unit vectors; the rate of every token's update
   {
@@ -387,35 +431,31 @@ __global__ void __launch_bounds__(kMakeThreads, 2) delta_make_kernel(const Delta
   }
   // ---- decays: sums of log2 g inside every block of 16 tokens
   {
-    const float rate = expf(a.A_log[h]) * kLog2E;
-    const int c = tid % DK;
-    const float bias = c < a.dk ? a.dt_bias[h * a.dk + c] : 0.f;
-    const float* dec = a.decay + static_cast<int64_t>(t0) * a.ldd + h * a.dk + c;
-    for (int blk = tid / DK; blk < kChunk / kBlock; blk += kMakeThreads / DK) {
-      float z[kBlock], sum = 0.f;
+    const float rate = expf(a.A_log[h]), bias = has ? a.dt_bias[h * a.dk + chan] : 0.f;
+#pragma unroll
+    for (int m = 0; m < kMine; ++m) {
+      const int blk = blk0 + m * kStride;
+      if (blk >= kBlocks) break;
+      float sum = 0.f;
 #pragma unroll
       for (int i = 0; i < kBlock; ++i) {
         const int t = blk * kBlock + i;
-        z[i] = t < n && c < a.dk ? dec[static_cast<int64_t>(t) * a.ldd] : 0.f;
+        if (t < n && has) sum -= rate * softplus_log2(z[m][i] + bias);
+        s.L[t][chan] = sum;
       }
-#pragma unroll
-      for (int i = 0; i < kBlock; ++i) {
-        const int t = blk * kBlock + i;
-        if (t < n && c < a.dk) sum -= rate * softplus(z[i] + bias);
-        s.L[t][c] = sum;
-      }
-      s.E[blk][c] = sum;
+      s.E[blk][chan] = sum;
     }
   }
   __syncthreads();
 
-  // ---- A and P: 6 pairs of different blocks (tensor cores), 64 rows of the diagonal blocks
+  // ---- A and P: 6 pairs of different blocks and the lower left quarters of 4 diagonal blocks (tensor cores), 64 rows of
+  // the 8 x 8 blocks on the diagonal
   const int g8 = lane >> 2, t2 = (lane & 3) * 2;
   for (;;) {
     int job = 0;
     if (lane == 0) job = atomicAdd(&s.next, 1);
     job = __shfl_sync(0xffffffffu, job, 0);
-    if (job >= 6 + kChunk) break;
+    if (job >= 10 + kChunk) break;
     if (job < 6) {
       const int ra = job < 1 ? 1 : job < 3 ? 2 : 3, cb = job - (ra * (ra - 1)) / 2;  // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
       const int r0 = ra * kBlock, j0 = cb * kBlock;
@@ -462,41 +502,71 @@ __global__ void __launch_bounds__(kMakeThreads, 2) delta_make_kernel(const Delta
           s.at[j][t] = da[u][e] * s.b[t] * s.ik[t] * s.ik[j];
           s.p[t][j] = dp[u][e] * s.iq[t] * s.ik[j];
         }
+    } else if (job < 10) {  // rows of k above rows of q: A and P in one product
+      const int j0 = (job - 6) * kBlock, t = j0 + 8 + g8, j = j0 + g8;
+      float d[4] = {};
+#pragma unroll 1
+      for (int kk = 0; kk < DK; kk += 16) {
+        uint32_t ah[4], al[4], bh[2], bl[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int c = kk + t2 + i * 8;
+          const float2 mid = *reinterpret_cast<const float2*>(&s.L[j0 + 7][c]);
+          const float2 Lt = *reinterpret_cast<const float2*>(&s.L[t][c]), Lj = *reinterpret_cast<const float2*>(&s.L[j][c]);
+          const float e0 = ex2(Lt.x - mid.x), e1 = ex2(Lt.y - mid.y);
+          const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(&s.k[t][c]));
+          const float2 q = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(&s.q[t][c]));
+          const float2 kj = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(&s.k[j][c]));
+          split2(k.x * e0, k.y * e1, ah[2 * i], al[2 * i]);
+          split2(q.x * e0, q.y * e1, ah[2 * i + 1], al[2 * i + 1]);
+          split2(kj.x * ex2(mid.x - Lj.x), kj.y * ex2(mid.y - Lj.y), bh[i], bl[i]);
+        }
+        mma3(d, ah, al, bh[0], bh[1], bl[0], bl[1]);
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int col = j0 + t2 + e;
+        s.at[col][t] = d[e] * s.b[t] * s.ik[t] * s.ik[col];
+        s.p[t][col] = d[2 + e] * s.iq[t] * s.ik[col];
+      }
     } else {
-      const int t = job - 6, j0 = t / kBlock * kBlock, last = t - j0;
+      const int t = job - 10, j0 = t & ~7, last = t - j0;
       constexpr int V = DK / 32;
-      float kt[V], qt[V], Lt[V], acc[32];
+      float kt[V], qt[V], Lt[V], acc[16];
 #pragma unroll
       for (int v = 0; v < V; ++v) {
         const int c = v * 32 + lane;
         kt[v] = __bfloat162float(s.k[t][c]), qt[v] = __bfloat162float(s.q[t][c]), Lt[v] = s.L[t][c];
       }
 #pragma unroll
-      for (int j = 0; j < kBlock; ++j) {
-        acc[j] = acc[16 + j] = 0.f;
-        if (j <= last && t < n) {
+      for (int j = 0; j < 8; ++j) {
+        acc[j] = acc[8 + j] = 0.f;
+        if (j <= last) {
 #pragma unroll
           for (int v = 0; v < V; ++v) {
             const int c = v * 32 + lane;
             const float w = __bfloat162float(s.k[j0 + j][c]) * ex2(Lt[v] - s.L[j0 + j][c]);
             acc[j] = fmaf(kt[v], w, acc[j]);
-            acc[16 + j] = fmaf(qt[v], w, acc[16 + j]);
+            acc[8 + j] = fmaf(qt[v], w, acc[8 + j]);
           }
         }
       }
-      // sum over the lanes; lane i ends with number i
+      // sums over the lanes; lanes 2 i and 2 i + 1 end with number i
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
+      for (int o = 16; o > 1; o >>= 1) {
 #pragma unroll
-        for (int i = 0; i < o; ++i) {
+        for (int i = 0; i < o / 2; ++i) {
           const bool up = lane & o;
-          const float give = up ? acc[i] : acc[i + o], keep = up ? acc[i + o] : acc[i];
+          const float give = up ? acc[i] : acc[i + o / 2], keep = up ? acc[i + o / 2] : acc[i];
           acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
         }
       }
-      const int j = j0 + (lane & 15);
-      if (lane < 16) s.at[j][t] = lane < last ? acc[0] * s.b[t] * s.ik[t] * s.ik[j] : 0.f;
-      else s.p[t][j] = lane - 16 <= last ? acc[0] * s.iq[t] * s.ik[j] : 0.f;
+      const float sum = acc[0] + __shfl_xor_sync(0xffffffffu, acc[0], 1);
+      const int i = lane >> 1, j = j0 + (i & 7);
+      if ((lane & 1) == 0) {
+        if (i < 8) s.at[j][t] = i < last ? sum * s.b[t] * s.ik[t] * s.ik[j] : 0.f;
+        else s.p[t][j] = sum * s.iq[t] * s.ik[j];
+      }
     }
   }
   __syncthreads();
@@ -511,38 +581,50 @@ __global__ void __launch_bounds__(kMakeThreads, 2) delta_make_kernel(const Delta
   for (int col = tid; col < DK + slices * kSlice; col += kMakeThreads) {
     const bool key = col < DK;
     const int c = key ? col : col - DK;
-    float y[kChunk];
+    uint64_t y[kChunk / 2];  // two tokens each
     if (key) {
       float base = 0.f;
 #pragma unroll
-      for (int t = 0; t < kChunk; ++t) {
+      for (int t = 0; t < kChunk; t += 2) {
         if (t % kBlock == 0 && t > 0) base += s.E[t / kBlock - 1][c];
-        y[t] = s.b[t] * s.ik[t] * __bfloat162float(s.k[t][c]) * ex2(base + s.L[t][c]);
+        y[t / 2] = pair(s.b[t] * s.ik[t] * __bfloat162float(s.k[t][c]) * ex2(base + s.L[t][c]),
+                        s.b[t + 1] * s.ik[t + 1] * __bfloat162float(s.k[t + 1][c]) * ex2(base + s.L[t + 1][c]));
       }
     } else {
       const bf16* v = x + a.v_off + h * a.dv + c;
+      auto value = [&](int t) { return t < n && c < a.dv ? s.b[t] * __bfloat162float(v[static_cast<int64_t>(t) * a.ld]) : 0.f; };
 #pragma unroll
-      for (int t = 0; t < kChunk; ++t) y[t] = t < n && c < a.dv ? s.b[t] * __bfloat162float(v[static_cast<int64_t>(t) * a.ld]) : 0.f;
+      for (int t = 0; t < kChunk; t += 2) y[t / 2] = pair(value(t), value(t + 1));
     }
 #pragma unroll
     for (int j = 0; j + 1 < kChunk; ++j) {
-      const float xj = y[j];
+      const float2 yj = unpair(y[j / 2]);
+      const float xj = j & 1 ? yj.y : yj.x;
+      const uint64_t xx = pair(-xj, -xj);
 #pragma unroll
       for (int t4 = (j + 1) / 4 * 4; t4 < kChunk; t4 += 4) {
-        const float4 w = *reinterpret_cast<const float4*>(&s.at[j][t4]);
-        if (t4 > j) y[t4] = fmaf(-w.x, xj, y[t4]);
-        if (t4 + 1 > j) y[t4 + 1] = fmaf(-w.y, xj, y[t4 + 1]);
-        if (t4 + 2 > j) y[t4 + 2] = fmaf(-w.z, xj, y[t4 + 2]);
-        if (t4 + 3 > j) y[t4 + 3] = fmaf(-w.w, xj, y[t4 + 3]);
+        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(&s.at[j][t4]);
+        if (t4 > j) y[t4 / 2] = fma2(w.x, xx, y[t4 / 2]);
+        else if (t4 == j) y[t4 / 2] = pair(yj.x, fmaf(-unpair(w.x).y, xj, yj.y));
+        if (t4 + 2 > j) y[t4 / 2 + 1] = fma2(w.y, xx, y[t4 / 2 + 1]);
+        else if (t4 + 2 == j) y[t4 / 2 + 1] = pair(yj.x, fmaf(-unpair(w.y).y, xj, yj.y));
       }
     }
     if (key) {
 #pragma unroll
-      for (int t = 0; t < kChunk; ++t) rec[Rec::W + t * DK + c] = split1(y[t]);
+      for (int t = 0; t < kChunk; t += 2) {
+        const float2 f = unpair(y[t / 2]);
+        rec[Rec::W + t * DK + c] = split1(f.x);
+        rec[Rec::W + (t + 1) * DK + c] = split1(f.y);
+      }
     } else {
       float* U = reinterpret_cast<float*>(rec) + Rec::U + static_cast<int64_t>(c / kSlice) * kChunk * kSlice + c % kSlice;
 #pragma unroll
-      for (int t = 0; t < kChunk; ++t) U[t * kSlice] = y[t];
+      for (int t = 0; t < kChunk; t += 2) {
+        const float2 f = unpair(y[t / 2]);
+        U[t * kSlice] = f.x;
+        U[(t + 1) * kSlice] = f.y;
+      }
     }
   }
   // ---- q e^G, k e^(G_n - G), e^(G_n): a channel and a part of the tokens per thread
@@ -565,7 +647,7 @@ __global__ void __launch_bounds__(kMakeThreads, 2) delta_make_kernel(const Delta
   }
   for (int i = tid; i < kChunk * kChunk; i += kMakeThreads) {
     const int t = i / kChunk, j = i % kChunk;
-    if (j / kBlock <= t / kBlock) rec[Rec::P + i] = t < n ? split1(s.p[t][j]) : 0u;
+    if (j / kBlock <= t / kBlock) rec[Rec::P + i] = t < n && j <= t ? split1(s.p[t][j]) : 0u;
   }
 }
 
