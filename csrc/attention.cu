@@ -264,32 +264,32 @@ attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __r
         }
       }
       if constexpr (SM != kSigmoid) {
-      float corr[2], m_use[2];
+        float corr[2], m_use[2];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        mx[h] = quad_max(mx[h]);
-        const float m_new = fmaxf(m_run[h], mx[h]);
-        m_use[h] = (m_new == -INFINITY) ? 0.f : m_new;
-        corr[h] = exp2f(m_run[h] - m_use[h]);
-        m_run[h] = m_new;
-      }
-      float ps[2] = {0.f, 0.f};
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          s[j][e] = exp2f(s[j][e] - m_use[e >> 1]);
-          ps[e >> 1] += s[j][e];
+        for (int h = 0; h < 2; ++h) {
+          mx[h] = quad_max(mx[h]);
+          const float m_new = fmaxf(m_run[h], mx[h]);
+          m_use[h] = (m_new == -INFINITY) ? 0.f : m_new;
+          corr[h] = exp2f(m_run[h] - m_use[h]);
+          m_run[h] = m_new;
         }
-      l_run[0] = l_run[0] * corr[0] + ps[0];
-      l_run[1] = l_run[1] * corr[1] + ps[1];
+        float ps[2] = {0.f, 0.f};
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) {
-        o[i][0] *= corr[0];
-        o[i][1] *= corr[0];
-        o[i][2] *= corr[1];
-        o[i][3] *= corr[1];
-      }
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            s[j][e] = exp2f(s[j][e] - m_use[e >> 1]);
+            ps[e >> 1] += s[j][e];
+          }
+        l_run[0] = l_run[0] * corr[0] + ps[0];
+        l_run[1] = l_run[1] * corr[1] + ps[1];
+#pragma unroll
+        for (int i = 0; i < D / 8; ++i) {
+          o[i][0] *= corr[0];
+          o[i][1] *= corr[0];
+          o[i][2] *= corr[1];
+          o[i][3] *= corr[1];
+        }
       }
       uint32_t pf[4];
       pf[0] = pack_bf16x2(s[0][0], s[0][1]);
@@ -525,32 +525,32 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         }
       }
       if constexpr (SM != kSigmoid) {
-      float corr[2], m_use[2];
+        float corr[2], m_use[2];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        mx[h] = quad_max(mx[h]);
-        const float m_new = fmaxf(m_run[h], mx[h]);
-        m_use[h] = (m_new == -INFINITY) ? 0.f : m_new;
-        corr[h] = exp2f(m_run[h] - m_use[h]);
-        m_run[h] = m_new;
-      }
-      float ps[2] = {0.f, 0.f};
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          s[j][e] = exp2f(s[j][e] - m_use[e >> 1]);
-          ps[e >> 1] += s[j][e];
+        for (int h = 0; h < 2; ++h) {
+          mx[h] = quad_max(mx[h]);
+          const float m_new = fmaxf(m_run[h], mx[h]);
+          m_use[h] = (m_new == -INFINITY) ? 0.f : m_new;
+          corr[h] = exp2f(m_run[h] - m_use[h]);
+          m_run[h] = m_new;
         }
-      l_run[0] = l_run[0] * corr[0] + ps[0];
-      l_run[1] = l_run[1] * corr[1] + ps[1];
+        float ps[2] = {0.f, 0.f};
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) {
-        o[i][0] *= corr[0];
-        o[i][1] *= corr[0];
-        o[i][2] *= corr[1];
-        o[i][3] *= corr[1];
-      }
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            s[j][e] = exp2f(s[j][e] - m_use[e >> 1]);
+            ps[e >> 1] += s[j][e];
+          }
+        l_run[0] = l_run[0] * corr[0] + ps[0];
+        l_run[1] = l_run[1] * corr[1] + ps[1];
+#pragma unroll
+        for (int i = 0; i < D / 8; ++i) {
+          o[i][0] *= corr[0];
+          o[i][1] *= corr[0];
+          o[i][2] *= corr[1];
+          o[i][3] *= corr[1];
+        }
       }
       uint32_t pf[4];
       pf[0] = pack_bf16x2(s[0][0], s[0][1]);
@@ -780,32 +780,32 @@ attn_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const void* __
           }
         }
       if constexpr (SM != kSigmoid) {
-      float corr[2], m_use[2];
+        float corr[2], m_use[2];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        mx[h] = quad_max(mx[h]);
-        const float m_new = fmaxf(m_run[h], mx[h]);
-        m_use[h] = (m_new == -INFINITY) ? 0.f : m_new;
-        corr[h] = exp2f(m_run[h] - m_use[h]);
-        m_run[h] = m_new;
-      }
-      float ps[2] = {0.f, 0.f};
-#pragma unroll
-      for (int j = 0; j < 8; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          s[j][e] = exp2f(s[j][e] - m_use[e >> 1]);
-          ps[e >> 1] += s[j][e];
+        for (int h = 0; h < 2; ++h) {
+          mx[h] = quad_max(mx[h]);
+          const float m_new = fmaxf(m_run[h], mx[h]);
+          m_use[h] = (m_new == -INFINITY) ? 0.f : m_new;
+          corr[h] = exp2f(m_run[h] - m_use[h]);
+          m_run[h] = m_new;
         }
-      l_run[0] = l_run[0] * corr[0] + ps[0];
-      l_run[1] = l_run[1] * corr[1] + ps[1];
+        float ps[2] = {0.f, 0.f};
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) {
-        o[i][0] *= corr[0];
-        o[i][1] *= corr[0];
-        o[i][2] *= corr[1];
-        o[i][3] *= corr[1];
-      }
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            s[j][e] = exp2f(s[j][e] - m_use[e >> 1]);
+            ps[e >> 1] += s[j][e];
+          }
+        l_run[0] = l_run[0] * corr[0] + ps[0];
+        l_run[1] = l_run[1] * corr[1] + ps[1];
+#pragma unroll
+        for (int i = 0; i < D / 8; ++i) {
+          o[i][0] *= corr[0];
+          o[i][1] *= corr[0];
+          o[i][2] *= corr[1];
+          o[i][3] *= corr[1];
+        }
       }
 #pragma unroll
       for (int g = 0; g < 4; ++g) {

@@ -13,10 +13,10 @@
 // whose state slot is S [dk, dv] alone. In the chunked kernel it is the case m_0 = 0, M_t = -F_t with F_t = -a times the sum
 // of d, a_j = ln d_j - F_j, without a normaliser.
 //
-// State slots of the matrix memory [slots, H, words] fp32: S [dk, dv], then for every slice of 32 columns of v a copy of n [dk], then the
-// slices' copies of m (all equal). A CTA owns whole slices with their copies, so the CTAs of a head never wait for one
-// another and none reads what another one writes. A sequence whose first token of this step sits at position 0 starts
-// from zero (m too). Two kernels share the state:
+// State slots of the matrix memory [slots, H, words] fp32: S [dk, dv], then for every slice of 32 columns of v a copy of n
+// [dk], then the slices' copies of m (all equal). A CTA owns whole slices with their copies, so the CTAs of a head never
+// wait for one another and none reads what another one writes. A sequence whose first token of this step sits at position 0
+// starts from zero (m too). Two kernels share the state:
 //
 //  * recurrent: one CTA per (head, 32 or 128 columns of v, sequence) keeps its part of S in registers and walks the
 //    sequence's tokens. Decoding (one pass over the state per token, memory bound), fp32, odd sizes.
@@ -524,10 +524,10 @@ __global__ void __launch_bounds__(kWarps * 32) memory_chunk_kernel(const MemoryA
         mma2(o[0], qa, b[0], b[1]);
         mma2(o[1], qa, b[2], b[3]);
         if constexpr (!kSpace) {
-        const bf16* nrow = mi < 2 ? &s.s_hi[kk * 16 + (mi & 1) * 8 + r8][kSlice] : &s.s_lo[kk * 16 + (mi & 1) * 8 + r8][kSlice];
-        ldmatrix_x4_trans(b, smem_u32(nrow));
-        mma2(o[2], qa, b[0], b[1]);
-        mma2(o[2], qa, b[2], b[3]);
+          const bf16* nrow = mi < 2 ? &s.s_hi[kk * 16 + (mi & 1) * 8 + r8][kSlice] : &s.s_lo[kk * 16 + (mi & 1) * 8 + r8][kSlice];
+          ldmatrix_x4_trans(b, smem_u32(nrow));
+          mma2(o[2], qa, b[0], b[1]);
+          mma2(o[2], qa, b[2], b[3]);
         }
       }
       if (needed) {

@@ -156,46 +156,47 @@ __global__ void __launch_bounds__(128) conv_run_kernel(const ConvArgs a, int run
 #pragma unroll
   for (int i = 0; i < kAhead; ++i) ahead[i] = first + i < last ? ld_bf16x8(cur + static_cast<int64_t>(i) * a.ldx) : zero8;
   int start = a.seq_cu[seq], end = a.seq_cu[seq + 1];
-  for (int t4 = first; t4 < last; t4 += kAhead)
+  for (int t4 = first; t4 < last; t4 += kAhead) {
 #pragma unroll
-  for (int i4 = 0; i4 < kAhead; ++i4, cur += a.ldx) {
-    const int t = t4 + i4;
-    if (t >= last) break;
-    while (end <= t) ++seq, start = end, end = a.seq_cu[seq + 1];
-    const int li = t - start;
-    if (kBack > 0 && (t == first || li == 0)) {  // the inputs before this run, or of this sequence's earlier steps
-      const int pos = a.positions[t];
-      const bf16* state = li < kBack ? state_of<bf16>(a, seq) : nullptr;
+    for (int i4 = 0; i4 < kAhead; ++i4, cur += a.ldx) {
+      const int t = t4 + i4;
+      if (t >= last) break;
+      while (end <= t) ++seq, start = end, end = a.seq_cu[seq + 1];
+      const int li = t - start;
+      if (kBack > 0 && (t == first || li == 0)) {  // the inputs before this run, or of this sequence's earlier steps
+        const int pos = a.positions[t];
+        const bf16* state = li < kBack ? state_of<bf16>(a, seq) : nullptr;
 #pragma unroll
-      for (int j = 0; j < kBack; ++j) {
-        const int b = kBack - j;
-        hist[j] = zero8;
-        if (pos - b < 0) continue;
-        if (b <= li) hist[j] = ld_bf16x8(cur - static_cast<int64_t>(b) * a.ldx);
-        else if (state) hist[j] = ld_bf16x8(state + static_cast<int64_t>(li + j) * a.C + c);
+        for (int j = 0; j < kBack; ++j) {
+          const int b = kBack - j;
+          hist[j] = zero8;
+          if (pos - b < 0) continue;
+          if (b <= li) hist[j] = ld_bf16x8(cur - static_cast<int64_t>(b) * a.ldx);
+          else if (state) hist[j] = ld_bf16x8(state + static_cast<int64_t>(li + j) * a.C + c);
+        }
       }
-    }
-    const bf16x8 here = ahead[i4];
-    if (t + kAhead < last) ahead[i4] = ld_bf16x8(cur + kAhead * a.ldx);
-    float y[8];
+      const bf16x8 here = ahead[i4];
+      if (t + kAhead < last) ahead[i4] = ld_bf16x8(cur + kAhead * a.ldx);
+      float y[8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) y[e] = b0[e];
+      for (int e = 0; e < 8; ++e) y[e] = b0[e];
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) {
-      const bf16x8& x = j < kBack ? hist[j < kBack ? j : 0] : here;
+      for (int j = 0; j < TAPS; ++j) {
+        const bf16x8& x = j < kBack ? hist[j < kBack ? j : 0] : here;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 xf = unpack_bf16x2(x.u[e]), wf = unpack_bf16x2(wt[j].u[e]);
-        y[2 * e] = fmaf(wf.x, xf.x, y[2 * e]);
-        y[2 * e + 1] = fmaf(wf.y, xf.y, y[2 * e + 1]);
+        for (int e = 0; e < 4; ++e) {
+          const float2 xf = unpack_bf16x2(x.u[e]), wf = unpack_bf16x2(wt[j].u[e]);
+          y[2 * e] = fmaf(wf.x, xf.x, y[2 * e]);
+          y[2 * e + 1] = fmaf(wf.y, xf.y, y[2 * e + 1]);
+        }
       }
+#pragma unroll
+      for (int j = 0; j + 1 < kBack; ++j) hist[j] = hist[j + 1];
+      if constexpr (kBack > 0) hist[kBack - 1] = here;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = silu(y[e]);
+      store_v<8>(static_cast<bf16*>(a.out) + static_cast<int64_t>(t) * a.C + c, y);
     }
-#pragma unroll
-    for (int j = 0; j + 1 < kBack; ++j) hist[j] = hist[j + 1];
-    if constexpr (kBack > 0) hist[kBack - 1] = here;
-#pragma unroll
-    for (int e = 0; e < 8; ++e) y[e] = silu(y[e]);
-    store_v<8>(static_cast<bf16*>(a.out) + static_cast<int64_t>(t) * a.C + c, y);
   }
 }
 
